@@ -7,13 +7,14 @@ modules here are its host-side mirror for tests and benchmarks:
   runtime    - prepared Model and Session (prefill / decode / verify / reset)
   checkpoint - admission of HF-style dense / AutoAWQ-GEMV checkpoints (names, layouts, metadata)
   model_bridge - the reference's Python binding surface (Model / Session / speculative session) over the above
+  trace      - replays a recorded trace of token portions through sessions (bin/trace_run)
   sharding   - session sharding over GPUs and the reductions of the benchmark
   synthetic  - seeded synthetic models, prompts and drafts
 The directory name is not an importable identifier; load it as `edge_infer_b200`
 (see __graft_entry__.load_package()).
 """
-from . import abi, checkpoint, model_bridge, operators, runtime, sharding, synthetic  # noqa: F401
-from .runtime import Model, Session, Shape  # noqa: F401
+from . import abi, checkpoint, model_bridge, operators, runtime, sharding, synthetic, trace  # noqa: F401
+from .runtime import LayeredShape, Model, Session, Shape  # noqa: F401
 
-__all__ = ["abi", "checkpoint", "model_bridge", "operators", "runtime", "sharding", "synthetic", "Model", "Session",
-           "Shape"]
+__all__ = ["abi", "checkpoint", "model_bridge", "operators", "runtime", "sharding", "synthetic", "trace", "LayeredShape",
+           "Model", "Session", "Shape"]

@@ -86,6 +86,21 @@ class ModelConfig(C.Structure):
                 ("qk_norm", C.c_int32)]
 
 
+class LayerSpec(C.Structure):
+    _fields_ = [("mixer", C.c_int32), ("mlp", C.c_int32), ("rnn_width", C.c_uint32), ("heads", C.c_uint32),
+                ("kv_heads", C.c_uint32), ("dim", C.c_uint32), ("vdim", C.c_uint32), ("rot_dims", C.c_uint32),
+                ("lin_heads", C.c_uint32), ("lin_dim", C.c_uint32), ("lin_vdim", C.c_uint32), ("ff", C.c_uint32),
+                ("rot_base", C.c_double), ("scale", C.c_double), ("left_scale", C.c_double),
+                ("right_scale", C.c_double), ("limit", C.c_double), ("decay", C.POINTER(C.c_double))]
+
+
+class LayeredConfig(C.Structure):
+    _fields_ = [("vocab_size", C.c_uint64), ("width", C.c_uint64), ("n_layers", C.c_uint64),
+                ("max_position_embeddings", C.c_uint64), ("loop_start", C.c_uint64), ("loop_stop", C.c_uint64),
+                ("loop_times", C.c_uint64), ("norm_eps", C.c_double), ("bos_token_id", C.c_uint32),
+                ("eos_token_id", C.c_uint32), ("true32", C.c_int32)]
+
+
 class NamedTensor(C.Structure):
     _fields_ = [("name", C.c_char_p), ("data", C.c_void_p), ("shape", C.c_uint64 * 2), ("rank", C.c_int32),
                 ("kind", C.c_int32)]
@@ -120,12 +135,15 @@ PROTOTYPES = {
     "ei_sample_greedy_bf16": (_S, [C.POINTER(Context), View2, View1, _P, _Z]),
     "ei_verify_accept": (_S, [C.POINTER(Context), _P, _P, _Z, _P, _P, _P]),
     "ei_model_create": (_S, [C.POINTER(ModelConfig), C.POINTER(NamedTensor), _Z, C.POINTER(_P)]),
+    "ei_model_create_layered": (_S, [C.POINTER(LayeredConfig), C.POINTER(LayerSpec), C.POINTER(NamedTensor), _Z,
+                                     C.POINTER(_P)]),
     "ei_model_destroy": (None, [_P]),
     "ei_model_config_of": (_S, [_P, C.POINTER(ModelConfig)]),
     "ei_model_weight_bytes": (_Z, [_P]),
     "ei_session_create": (_S, [_P, _Z, C.c_int, C.POINTER(_P)]),
     "ei_session_destroy": (None, [_P]),
     "ei_session_prefill": (_S, [_P, _P, _Z, C.POINTER(_P), _P]),
+    "ei_session_extend": (_S, [_P, _P, _Z, _P, _Z, _P]),
     "ei_session_decode": (_S, [_P, C.c_uint32, C.POINTER(_P)]),
     "ei_session_verify": (_S, [_P, _P, _Z, C.POINTER(VerifyResult), C.POINTER(_P)]),
     "ei_batch_create": (_S, [C.POINTER(_P), _Z, C.POINTER(_P)]),
@@ -148,6 +166,8 @@ PROTOTYPES = {
     "ei_session_stream": (_P, [_P]),
     "ei_session_read_kv": (_S, [_P, _Z, _P, _P]),
     "ei_session_read_logits": (_S, [_P, _Z, _P]),
+    "ei_session_read_logits_f32": (_S, [_P, _Z, _P]),
+    "ei_session_tap_residual": (_S, [_P, _P, _Z]),
     "ei_session_launches_per_step": (_Z, [_P, _Z]),
     "ei_session_write_kv": (_S, [_P, C.c_size_t, C.c_size_t, C.c_size_t, _P, _P]),
     "ei_session_adopt_history": (_S, [_P, C.c_size_t, C.c_uint32]),

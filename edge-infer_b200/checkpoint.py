@@ -24,11 +24,11 @@ from typing import Dict, List, Mapping, Optional, Tuple
 
 import numpy as np
 
-from .runtime import Shape
+from .runtime import Attention, Layer, LayeredShape, LinearAttention, Shape
 
 DENSE, QWEIGHT, SCALES, ZEROS = 0, 1, 2, 3
 
-MODEL_TYPES = ("qwen_bf16", "qwen_awq", "qwen3_bf16", "qwen3_awq")
+MODEL_TYPES = ("qwen_bf16", "qwen_awq", "qwen3_bf16", "qwen3_awq", "zofesun_bf16", "zofesun_f32")
 
 _PROJECTIONS = {
     "self_attn.q_proj": "wq", "self_attn.k_proj": "wk", "self_attn.v_proj": "wv", "self_attn.o_proj": "wo",
@@ -36,6 +36,145 @@ _PROJECTIONS = {
 }
 _FORMATS = {"weight": DENSE, "qweight": QWEIGHT, "scales": SCALES, "qzeros": ZEROS}
 _LAYER = re.compile(r"^model\.layers\.(0|[1-9][0-9]*)\.(.+)$")
+
+
+def model_type_of(config: Mapping, dtype: str = "bfloat16") -> str:
+    """The model type a config.json asks for: by `architecture` for designs that name themselves, by the Hugging Face
+    `model_type` and quantization settings otherwise. dtype float32 is there for the layered designs only."""
+    if dtype not in ("bfloat16", "float32"):
+        raise ValueError("dtype must be bfloat16 or float32")
+    if config.get("architecture") == "Zofesun":
+        return "zofesun_f32" if dtype == "float32" else "zofesun_bf16"
+    family = {"qwen2": "qwen", "qwen3": "qwen3"}.get(config.get("model_type"))
+    if family is None:
+        raise ValueError("Unsupported model architecture: %r" % (config.get("architecture") or config.get("model_type")))
+    if dtype != "bfloat16":
+        raise NotImplementedError("This model family runs in bfloat16 only")
+    return family + ("_awq" if "quantization_config" in config else "_bf16")
+
+
+# ---------------------------------------------------------------- layered designs
+def _size(section: Mapping, key: str, where: str, least: int = 1) -> int:
+    value = section.get(key)
+    if type(value) is not int or value < least:
+        raise ValueError(f"{where}.{key} must be an integer of at least {least}")
+    return value
+
+
+def _number(section: Mapping, key: str, where: str) -> float:
+    value = section.get(key)
+    if isinstance(value, bool) or not isinstance(value, (int, float)):
+        raise ValueError(f"{where}.{key} must be a number")
+    return float(value)
+
+
+def _section(parent: Mapping, key: str, where: str) -> Mapping:
+    value = parent.get(key)
+    if not isinstance(value, Mapping):
+        raise ValueError(f"{where}.{key} must be an object")
+    return value
+
+
+def _zofesun_layer(entry: Mapping, where: str) -> Layer:
+    mixer, layer = _section(entry, "mixer", where), Layer()
+    kind = entry.get("type")
+    if kind == "mingru":
+        layer.rnn_width = _size(mixer, "width", where + ".mixer")
+    elif kind == "parallel":
+        left, right = _section(mixer, "left", where + ".mixer"), _section(mixer, "right", where + ".mixer")
+        at = where + ".mixer.left"
+        rot = _section(left, "rot", at)
+        layer.attention = Attention(heads=_size(left, "heads", at), kv_heads=_size(left, "kv_heads", at),
+                                    dim=_size(left, "dim", at), vdim=_size(left, "vdim", at),
+                                    rot_dims=_size(rot, "dims", at + ".rot", 0), rot_base=_number(rot, "base", at + ".rot"),
+                                    scale=_number(left, "scale", at))
+        at = where + ".mixer.right"
+        decay = right.get("decay")
+        heads = _size(right, "heads", at)
+        if not isinstance(decay, (list, tuple)) or len(decay) != heads:
+            raise ValueError(at + ".decay must have one entry per head")
+        layer.linear = LinearAttention(heads=heads, dim=_size(right, "dim", at), vdim=_size(right, "vdim", at),
+                                       decay=[float(d) for d in decay])
+        layer.left_scale = _number(mixer, "left_scale", where + ".mixer")
+        layer.right_scale = _number(mixer, "right_scale", where + ".mixer")
+    else:
+        raise ValueError(f"{where}: unsupported mixer type {kind!r}")
+    mlp = entry.get("mlp")
+    if mlp is not None:
+        if not isinstance(mlp, Mapping) or mlp.get("kind") != "dense":
+            raise ValueError(where + ": unsupported feed-forward")
+        layer.ff, layer.limit = _size(mlp, "ff", where + ".mlp"), _number(mlp, "limit", where + ".mlp")
+    return layer
+
+
+def zofesun_shape(config: Mapping, true32: bool = False) -> LayeredShape:
+    """Decoder shape of a Zofesun config.json: every size and constant comes from it."""
+    entries = config.get("layers")
+    if not isinstance(entries, list) or not entries or not all(isinstance(e, Mapping) for e in entries):
+        raise ValueError("layers must be a nonempty list")
+    loop = config.get("loop")
+    if loop is not None:
+        loop = (_size(loop, "start", "loop", 0), _size(loop, "stop", "loop"), _size(loop, "times", "loop"))
+        if not loop[0] < loop[1] <= len(entries):
+            raise ValueError("loop must span existing layers")
+    return LayeredShape(vocab_size=_size(config, "vocab", "config"), hidden_size=_size(config, "width", "config"),
+                        layers=[_zofesun_layer(e, f"layers[{i}]") for i, e in enumerate(entries)],
+                        norm_eps=_number(_section(config, "norm", "config"), "eps", "norm"), loop=loop, true32=true32,
+                        max_position_embeddings=int(config.get("max_position_embeddings", 1 << 20)),
+                        bos_token_id=int(config.get("bos_token_id", 0) or 0),
+                        eos_token_id=_first_int(config.get("eos_token_id", 0xFFFFFFFF)))
+
+
+def layered_tensor_shapes(shape: LayeredShape) -> Dict[str, Tuple[int, ...]]:
+    """Every tensor a layered checkpoint must hold, with its shape ([out, in] for linears, () for scalars)."""
+    width = shape.hidden_size
+    shapes: Dict[str, Tuple[int, ...]] = {"embed": (shape.vocab_size, width), "head": (shape.vocab_size, width)}
+
+    def norm(name: str) -> None:
+        shapes.update({name: (width,), name + ".b": (width,), name + ".alpha": ()})
+
+    norm("final.norm")
+    if shape.loop is not None:
+        shapes["loop.step"] = (shape.loop[2], width)
+    for i, layer in enumerate(shape.layers):
+        p = f"l{i}."
+        norm(p + "norm1")
+        norm(p + "norm1b")
+        if layer.rnn_width is not None:
+            r = layer.rnn_width
+            shapes.update({p + "mix.z": (r, width), p + "mix.z.b": (r,), p + "mix.x": (r, width), p + "mix.x.b": (r,),
+                           p + "mix.g": (r, width), p + "mix.o": (width, r)})
+        else:
+            a, l = layer.attention, layer.linear
+            left, right = p + "mix.left.", p + "mix.right."
+            shapes.update({left + "q": (a.heads * a.dim, width), left + "k": (a.kv_heads * a.dim, width),
+                           left + "v": (a.kv_heads * a.vdim, width), left + "sink": (a.heads,),
+                           left + "o": (width, a.heads * a.vdim), right + "q": (l.heads * l.dim, width),
+                           right + "k": (l.heads * l.dim, width), right + "v": (l.heads * l.vdim, width),
+                           right + "g": (l.heads * l.vdim, width), right + "o": (width, l.heads * l.vdim),
+                           right + "norm": (l.heads * l.vdim,)})
+        if layer.ff is not None:
+            norm(p + "norm2")
+            norm(p + "norm2b")
+            shapes.update({p + "mlp.gate": (layer.ff, width), p + "mlp.up": (layer.ff, width),
+                           p + "mlp.down": (width, layer.ff)})
+    return shapes
+
+
+def _admit_layered(shape: LayeredShape, weights: Mapping):
+    expected = layered_tensor_shapes(shape)
+    missing, extra = sorted(set(expected) - set(weights)), sorted(set(weights) - set(expected))
+    if missing:
+        raise ValueError("Decoder checkpoint lacks " + missing[0])
+    if extra:
+        raise ValueError("Unsupported decoder weight key: " + extra[0])
+    tensors: Dict[str, List[Tuple[int, object]]] = {}
+    for name, dims in expected.items():
+        payload = _bits(weights[name], name, DENSE)
+        if tuple(int(d) for d in payload.shape) not in ((dims,) if dims else ((), (1,))):
+            raise ValueError("Decoder checkpoint weight shape mismatch: " + name)
+        tensors[name] = [(DENSE, payload)]
+    return shape, tensors
 
 
 def awq_group_size(config: Mapping) -> int:
@@ -109,10 +248,12 @@ def _projection(source: str, name: str, bias_name: str, fmt: str) -> Tuple[str, 
     raise ValueError("Unsupported decoder weight key: " + source)
 
 
-def shape_from_config(config: Mapping, model_type: str) -> Shape:
-    """Decoder shape from an HF config.json dictionary."""
+def shape_from_config(config: Mapping, model_type: str):
+    """Decoder shape from a config.json dictionary."""
     if model_type not in MODEL_TYPES:
         raise ValueError(f"Unsupported model type: {model_type}")
+    if model_type.startswith("zofesun"):
+        return zofesun_shape(config, true32=model_type.endswith("_f32"))
     heads = int(config["num_attention_heads"])
     head_dim = int(config.get("head_dim", int(config["hidden_size"]) // heads))
     awq = model_type.endswith("_awq")
@@ -159,6 +300,8 @@ def admit(config: Mapping, weights: Mapping, model_type: str):
     Validates names, ranks, AWQ completeness (packed weight, scales and zero points come together and never beside a
     dense weight of the same projection) and resolves a declared embedding tie."""
     shape = shape_from_config(config, model_type)
+    if isinstance(shape, LayeredShape):
+        return _admit_layered(shape, weights)
     tied = config.get("tie_word_embeddings", False)
     if not isinstance(tied, bool):
         raise ValueError("tie_word_embeddings must be a boolean")
@@ -227,10 +370,10 @@ def _checkpoint_file(root: Path, name) -> Path:
     return path
 
 
-def load_directory(model_path, model_type: str):
+def load_directory(model_path, model_type: Optional[str] = None):
     """(config, weights) of a local checkpoint directory: config.json plus model.safetensors or the shards its index
     names. Never fetches anything."""
-    if model_type not in MODEL_TYPES:
+    if model_type is not None and model_type not in MODEL_TYPES:
         raise ValueError(f"Unsupported model type: {model_type}")
     root = Path(model_path).resolve()
     config = json.loads((root / "config.json").read_text(encoding="utf-8"))

@@ -42,21 +42,6 @@ __device__ __forceinline__ int tile_offset(int token, int chunk) {
   return (chunk >> 3) * (kTile * 128) + token * 128 + (((chunk & 7) ^ (token & 7)) << 4);
 }
 
-__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3,
-                                                  const void* smem_ptr) {
-  const uint32_t address = static_cast<uint32_t>(__cvta_generic_to_shared(smem_ptr));
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3)
-               : "r"(address));
-}
-
-__device__ __forceinline__ void ldmatrix_x4(uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3, const void* smem_ptr) {
-  const uint32_t address = static_cast<uint32_t>(__cvta_generic_to_shared(smem_ptr));
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3)
-               : "r"(address));
-}
-
 // kDirect = false: the verify step. Block (split, kv head) covers one chunk of the sequence for all <= 16 query
 // rows and writes (o, m, l) partials for the merge kernel.
 // kDirect = true: a prompt of many rows. Block (query block, kv head) covers 16 consecutive query rows over their

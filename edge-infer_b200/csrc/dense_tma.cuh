@@ -195,7 +195,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
             up += __bfloat162float(p.bias[n]);
           }
           p.out[size_t(row) * p.out_stride + out_n] =
-              __float2bfloat16_rn(silu_multiply_value(round_bf16(gate), round_bf16(up)));
+              __float2bfloat16_rn(gated_pair_value(p.glu, p.glu_limit, gate, up));
         }
       } else if (p.epilogue == kEpiPartial) {
         p.partial[(size_t(slice) * p.M + row) * p.N + n] = sum;

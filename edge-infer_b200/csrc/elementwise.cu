@@ -123,29 +123,7 @@ __global__ void __launch_bounds__(kNormThreads) embed_norm_kernel(const EmbedPar
   grid_dependency_wait();
   const int row = blockIdx.x;
   if (threadIdx.x == 0) {
-    Control* control = p.control;
-    int local = row, step_rows = p.rows, capacity = p.capacity;
-    if (p.slots) {
-      const int session = row / p.rows_per_session;
-      local = row - session * p.rows_per_session;
-      step_rows = p.rows_per_session;
-      control = p.slots[session].control;
-      capacity = p.slots[session].capacity;
-    }
-    uint32_t token;
-    if (p.tokens) {
-      token = p.tokens[row];
-    } else if (local == 0) {
-      token = control->pending;
-    } else {
-      const DraftSource source = *p.source;
-      const long long index = (long long)control->context + local - source.base;
-      token = (source.drafts && index >= 0 && index < source.count) ? source.drafts[index] : 0u;
-    }
-    p.step_tokens[row] = token;
-    if (token >= uint32_t(p.vocab)) atomicOr(&control->status, 2);
-    if (local == 0 && control->context + step_rows > capacity) atomicOr(&control->status, 1);
-    token_shared = token;
+    token_shared = take_step_token(p, row);
   }
   __syncthreads();
   const uint32_t token = token_shared;

@@ -12,6 +12,7 @@ struct Control {
   int32_t context;    // committed KV rows; the step's first row goes to this position
   uint32_t pending;   // last emitted token = row 0 of the next step
   int32_t status;     // 0 ok; bit 0: step would exceed capacity (step skipped); bit 1: bad token id
+  int32_t state_base; // rows the recurrent state has absorbed; rows [state_base, context) are still pending behind it
   int32_t steps;      // verify steps executed since the last drain
   unsigned long long emitted_total;  // tokens emitted since the last drain
   ei_verify_result last;
@@ -72,6 +73,36 @@ struct EmbedParams {
 };
 // Token selection + embedding lookup + first RMSNorm, one block per row.
 void launch_embed_norm(const EmbedParams& p, cudaStream_t stream, bool pdl);
+
+#if defined(__CUDACC__)
+// The token of stacked row `row` of a step (given by the host, the pending token, or a draft), recorded in
+// step_tokens; raises the status bits for a bad id or a step that would pass the capacity. One thread per row.
+__device__ __forceinline__ uint32_t take_step_token(const EmbedParams& p, int row) {
+  Control* control = p.control;
+  int local = row, step_rows = p.rows, capacity = p.capacity;
+  if (p.slots) {
+    const int session = row / p.rows_per_session;
+    local = row - session * p.rows_per_session;
+    step_rows = p.rows_per_session;
+    control = p.slots[session].control;
+    capacity = p.slots[session].capacity;
+  }
+  uint32_t token;
+  if (p.tokens) {
+    token = p.tokens[row];
+  } else if (local == 0) {
+    token = control->pending;
+  } else {
+    const DraftSource source = *p.source;
+    const long long index = (long long)control->context + local - source.base;
+    token = (source.drafts && index >= 0 && index < source.count) ? source.drafts[index] : 0u;
+  }
+  p.step_tokens[row] = token;
+  if (token >= uint32_t(p.vocab)) atomicOr(&control->status, 2);
+  if (local == 0 && control->context + step_rows > capacity) atomicOr(&control->status, 1);
+  return token;
+}
+#endif
 
 struct QkvParams {
   bf16* qkv;                // [rows, (heads + 2 kv_heads) * 128] : q | k | v, q and k rotated in place
@@ -150,6 +181,8 @@ constexpr int kSampleMaxParts = 256;
 int sample_partial_blocks(size_t vocabulary, int multiprocessors);
 void launch_argmax_partials(const bf16* logits, size_t rows, size_t vocab, size_t row_stride,
                             float* best_value, int* best_index, int blocks, cudaStream_t stream, bool pdl);
+void launch_argmax_partials_f32(const float* logits, size_t rows, size_t vocab, size_t row_stride, float* best_value,
+                                int* best_index, int blocks, cudaStream_t stream, bool pdl);
 // Final argmax over `parts` partials per row; writes targets[rows]. With `control` non-null also
 // performs greedy acceptance against step_tokens and commits the context length.
 void launch_finalize(const float* best_value, const int* best_index, int parts, int rows,

@@ -1,0 +1,248 @@
+// Decoders described layer by layer: the operations their layers are made of, and the model and session parts that
+// hold their weights, caches and recurrent state.
+//
+// Head sizes and widths are free. Every head is stored with its size rounded up to a multiple of 16 and every
+// projection input to a multiple of 64, the padding zero in the weights, so that all shapes go through the same GEMMs,
+// copies and MMA tiles; the true sizes enter only where a mean is taken.
+//
+// Activations are BF16 or, for a model that runs in true 32-bit, FP32: the kernels are templates over the element
+// type. The residual stream, norms, angles, scores, softmax weights, gates and recurrent state are FP32 in both.
+#pragma once
+
+#include "session.cuh"
+
+namespace ei {
+
+constexpr int kPendingRows = 16;     // rows a step may leave pending behind the recurrent state
+constexpr int kRingRows = 32;        // ring of a recurrence's inputs: pending rows and the rows of the step
+constexpr int kLightningChunk = 128; // tokens of a prompt chunk of the decayed linear attention
+constexpr int kMaxHeadDim = 512;
+
+// tanh(alpha * x) * weight + bias; vectors padded with zeros to the row stride.
+struct DynamicTanh {
+  const bf16* weight = nullptr;
+  const bf16* bias = nullptr;
+  float alpha = 0.0f;
+};
+
+// What is added to the residual stream ahead of a layer: the embedding output of the row's token and / or a vector.
+struct Injection {
+  const uint32_t* tokens = nullptr;  // [rows]; with `table` set, table[token] is added
+  const bf16* table = nullptr;       // [vocab, stride of the residual]
+  const bf16* vector = nullptr;
+  int vocab = 0;
+};
+
+// x = embedding (+ injected vector); normed = norm(x). One block per row.
+struct LayeredEmbedParams {
+  EmbedParams token;        // token selection (its table, norm and output fields are not used)
+  const bf16* table;        // [vocab, residual_stride]
+  const bf16* vector;       // added to the stream ahead of the first layer, or null
+  DynamicTanh norm;
+  float* residual;          // [rows, residual_stride]
+  int residual_stride;
+  void* normed;             // [rows, normed_stride]
+  int normed_stride;
+};
+template <typename T>
+void launch_layered_embed(const LayeredEmbedParams& p, cudaStream_t stream, bool pdl);
+
+// The end of a sublayer and the start of the next: x += after(sum of partials); tap = x; x += injection;
+// normed = before(x).
+struct SublayerJoinParams {
+  const float* partial;     // [ksplit, rows, residual_stride]
+  int ksplit, rows;
+  DynamicTanh after, before;
+  float* residual;
+  int residual_stride;
+  float* tap;               // optional copy of the stream before the injection: [rows, tap_width]
+  int tap_width;
+  Injection inject;
+  void* normed;
+  int normed_stride;
+};
+template <typename T>
+void launch_sublayer_join(const SublayerJoinParams& p, cudaStream_t stream, bool pdl);
+
+// Per (row, head): rotation of q and k, value norm, KV append; SiLU of the linear attention's q, k, v, whose k and v
+// are also recorded in the ring when the step leaves its rows pending. In place in the fused projection output.
+struct MixerPrepareParams {
+  void* fused;              // [rows, stride]: q | k | v | linear q | k | v | gate
+  int rows, stride;
+  int heads, kv_heads, dim, vdim, dim_pad, vdim_pad, rot_dims;
+  float eps;
+  const float2* rotation;   // [capacity][rot_dims / 2] (cos, sin)
+  const Control* control;
+  int capacity;
+  void *k_cache, *v_cache;  // [capacity, kv_heads * dim_pad], [capacity, kv_heads * vdim_pad]
+  int lin_heads, lin_dim_pad, lin_vdim_pad;
+  void *ring_k, *ring_v;    // [kRingRows, lin_heads * pad] or null
+};
+template <typename T>
+void launch_mixer_prepare(const MixerPrepareParams& p, cudaStream_t stream, bool pdl);
+
+// ---- softmax attention with free head sizes, scale and per-head sink (sized_attention.cu) ----
+struct SizedAttentionParams {
+  const void* q;            // row r, head h at q + r * q_stride + h * dim_pad
+  int q_stride;
+  const void *k, *v;        // [capacity, kv_heads * pad]
+  int rows, heads, kv_heads, dim_pad, vdim_pad;
+  float scale, out_scale;   // out_scale multiplies the finished output
+  const float* sink;        // [heads]: exp(sink) joins the denominator; or null
+  const int32_t* device_offset;
+  int capacity;
+  int chunk, max_splits;    // step form
+  float* scratch;           // [max_splits][rows * heads][vdim_pad + 4]
+  void* out;                // row r, head h at out + r * out_stride + h * vdim_pad
+  int out_stride;
+  CUtensorMap k_map, v_map; // filled by the launch functions
+  int k_shift, v_shift;     // log2 of the 16-byte pieces in one row of a staged box
+  int* status;
+  uint32_t wait_limit, fault_tx;
+};
+// Head sizes the tiled kernels take (the others use launch_plain_attention).
+bool sized_attention_ok(int dim_pad, int vdim_pad);
+size_t sized_attention_scratch_bytes(size_t rows, size_t heads, size_t vdim_pad, size_t capacity);
+// Split form for at most 16 rows; leaves partials for launch_mixer_finish.
+void launch_sized_attention_step(const SizedAttentionParams& p, cudaStream_t stream, bool pdl);
+// Any number of rows, finished output.
+void launch_sized_attention_prompt(const SizedAttentionParams& p, cudaStream_t stream, bool pdl);
+// One block per (row, head), any head size up to kMaxHeadDim, FP32 or BF16 operands, finished output.
+template <typename T>
+void launch_plain_attention(const SizedAttentionParams& p, cudaStream_t stream, bool pdl);
+
+// ---- decayed linear attention (lightning.cu) ----
+struct LightningParams {
+  const void *q, *k, *v;    // row r at + r * stride, heads side by side
+  int stride, rows, heads, dim_pad, vdim_pad;
+  const void *ring_k, *ring_v;  // [kRingRows, heads * pad]
+  const float* powers;      // [heads][kLightningChunk + 1]: decay^n
+  float* state;             // [heads][vdim_pad / 16][dim_pad][16]: as of Control::state_base
+  float* chunk_states;      // prompt form: [chunks] of the same
+  const Control* control;
+  int capacity;
+  float* out;               // [rows, heads * vdim_pad]
+};
+// At most 16 rows: folds the pending rows into the state, reads it for the step's rows, leaves those pending.
+template <typename T>
+void launch_lightning_step(const LightningParams& p, cudaStream_t stream, bool pdl);
+// A prompt segment in chunks: pending rows and all rows of the segment end up in the state. BF16.
+bool lightning_prompt_ok(int dim_pad, int vdim_pad);
+void launch_lightning_prompt(const LightningParams& p, cudaStream_t stream, bool pdl, int* launches);
+
+// The mixer's activation row: merged attention splits in front, the normed and gated linear attention behind.
+struct MixerFinishParams {
+  SizedAttentionParams attention;  // merged if `merge`
+  int merge;
+  int rows, lin_heads, lin_vdim, lin_vdim_pad;
+  const float* lin_out;     // [rows, lin_heads * lin_vdim_pad]
+  const void* gate;         // row r at + r * gate_stride: pre-activation of the output gate
+  int gate_stride;
+  const bf16* norm;         // [lin_heads * lin_vdim_pad]
+  float eps, lin_scale;
+  void* out;                // the same rows as attention.out
+  int out_stride, lin_offset;
+};
+template <typename T>
+void launch_mixer_finish(const MixerFinishParams& p, cudaStream_t stream, bool pdl);
+
+// ---- gated recurrence (minGRU) ----
+struct MinGruParams {
+  const void* fused;        // [rows, stride]: gate | candidate | output gate pre-activations, width_pad each
+  int rows, stride, width_pad;
+  float *ring_gate, *ring_candidate;  // [kRingRows, width_pad]
+  float* state;             // [width_pad]: as of Control::state_base
+  const Control* control;
+  int capacity;
+  void* out;                // [rows, out_stride]; columns beyond width_pad are cleared
+  int out_stride;
+};
+template <typename T>
+void launch_min_gru_step(const MinGruParams& p, cudaStream_t stream, bool pdl);
+void launch_min_gru_prompt(const MinGruParams& p, cudaStream_t stream, bool pdl);
+
+// out[rows, ff] = gated unit of the pair [rows, 2 ff] (clamped).
+template <typename T>
+void launch_clamped_glu(const T* gate_up, int rows, int ff, float limit, T* out, int multiprocessors,
+                        cudaStream_t stream, bool pdl);
+// Rows `index[i]` of `source` (row stride in elements) to consecutive rows of `out`.
+template <typename T>
+void launch_gather_rows(const T* source, const int32_t* index, int count, int stride, T* out, cudaStream_t stream);
+// FP32 partial sums -> FP32 sums, and the argmax partials of FP32 logits (at most 16 rows).
+void launch_sum_partials(const float* partial, int ksplit, size_t count, float* out, int multiprocessors,
+                         cudaStream_t stream, bool pdl);
+// out[rows, out] (FP32) = x (FP32) * W^T (BF16) + bias with FP32 arithmetic, at most 16 rows.
+void launch_true32_linear(const float* x, int rows, const PreparedLinear& w, float* out, cudaStream_t stream, bool pdl);
+// (cos, sin) of position * base^(-2 i / dims), computed in double and rounded once.
+void launch_rotation_table(float2* table, size_t positions, int dims, double base, cudaStream_t stream);
+
+// ---- model and session ----
+struct LayeredModel {
+  struct Layer {
+    ei_layer_spec spec{};
+    DynamicTanh norm1, norm1b, norm2, norm2b;
+    PreparedLinear in, out, gate_up, down;  // fused mixer input, mixer output, feed-forward
+    // parallel mixer
+    int dim_pad = 0, vdim_pad = 0, lin_dim_pad = 0, lin_vdim_pad = 0, rotation = 0;
+    int attention_width = 0, linear_width = 0;  // columns of the mixer's activation row
+    const float* sink = nullptr;
+    const float* powers = nullptr;
+    const bf16* lin_norm = nullptr;
+    // gated recurrence
+    int width_pad = 0;
+    int ff_pad = 0;
+  };
+  struct Run {              // one pass through one layer: its own caches and state
+    int layer = 0;
+    int pass = -1;          // >= 0: the loop pass that starts here
+  };
+  struct Rotation {
+    int dims = 0;
+    double base = 0.0;
+  };
+  bool true32 = false;
+  int width = 0, residual_stride = 0, normed_stride = 0, vocab_stride = 0;
+  float eps = 0.0f;
+  std::vector<Layer> layers;
+  std::vector<Run> runs;
+  std::vector<Rotation> rotations;
+  const bf16* embedding = nullptr;   // [vocab, residual_stride]
+  const bf16* loop_step = nullptr;   // [times, residual_stride]
+  DynamicTanh final_norm;
+  PreparedLinear head;
+  int max_fused = 0, max_mixed = 0, max_gate_up = 0, max_ff = 0, max_linear = 0;  // widest rows
+  size_t max_chunk_state = 0;        // floats of one chunk's state
+  // prompt workspace (in ei_model::prompt's arena)
+  float *residual = nullptr, *linear_out = nullptr, *chunk_states = nullptr;
+};
+
+struct LayeredSession {
+  struct Run {
+    void *k_cache = nullptr, *v_cache = nullptr;
+    void *ring_k = nullptr, *ring_v = nullptr;          // activation type
+    float *ring_gate = nullptr, *ring_candidate = nullptr;
+    float* state = nullptr;
+  };
+  std::vector<Run> runs;
+  std::vector<float2*> rotations;
+  size_t token_rows = 0;             // cache rows allocated (the capacity, whole tiles)
+  float *residual = nullptr, *linear_out = nullptr, *logits = nullptr, *head_partial = nullptr;
+  void *normed = nullptr, *fused = nullptr, *mixed = nullptr, *gate_up = nullptr, *act = nullptr, *head_rows = nullptr;
+  float* tap = nullptr;              // caller's device buffer [runs][tap_rows][width], or null
+  size_t tap_rows = 0;
+};
+
+// Builds `model` (device and limits already set) from the description and the checkpoint's tensors.
+void create_layered_model(ei_model& model, const ei_layered_config& config, const ei_layer_spec* layers,
+                          const ei_named_tensor* tensors, size_t count);
+void create_layered_session(ei_session& s);
+void ensure_layered_workspace(ei_model& model);
+// One forward of at most 16 rows at the device-side context length / of a prompt segment. The segment leaves the
+// normed rows in the prompt workspace; the vocabulary head runs in enqueue_layered_head over gathered rows.
+void enqueue_layered_step(ei_session& s, int rows, StepKind kind);
+void enqueue_layered_segment(ei_session& s, int rows);
+// FP32 logits of `count` <= 16 rows of the segment (indices on the device) into the session's logits; with `greedy`
+// the greedy token of row 0 goes to s.targets[0].
+void enqueue_layered_head(ei_session& s, const int32_t* device_rows, int count, bool greedy);
+
+}  // namespace ei

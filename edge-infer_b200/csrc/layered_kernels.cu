@@ -1,0 +1,531 @@
+// Elementwise and per-row kernels of decoders described layer by layer: embedding, sublayer joins, the preparation of
+// a mixer's heads, the end of a mixer, the gated recurrence, the clamped gated unit, and FP32 linears.
+#include "layered.cuh"
+
+#include <algorithm>
+#include <cmath>
+#include <stdexcept>
+
+namespace ei {
+namespace {
+
+__device__ __forceinline__ float value_of(bf16 x) { return __bfloat162float(x); }
+__device__ __forceinline__ float value_of(float x) { return x; }
+__device__ __forceinline__ void store_value(bf16* p, float x) { *p = __float2bfloat16_rn(x); }
+__device__ __forceinline__ void store_value(float* p, float x) { *p = x; }
+__device__ __forceinline__ float2 load_pair(const bf16* p) {
+  const uint32_t v = *reinterpret_cast<const uint32_t*>(p);
+  return make_float2(bf16_lo(v), bf16_hi(v));
+}
+__device__ __forceinline__ float2 load_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ void store_pair(bf16* p, float a, float b) { *reinterpret_cast<uint32_t*>(p) = pack_bf16(a, b); }
+__device__ __forceinline__ void store_pair(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ float4 load_quad(const bf16* p) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y));
+}
+__device__ __forceinline__ float4 load_quad(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void store_quad(bf16* p, float4 v) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+}
+__device__ __forceinline__ void store_quad(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+
+__device__ __forceinline__ float sigmoid_value(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float4 add(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+
+__device__ __forceinline__ float4 dynamic_tanh(const DynamicTanh& n, int i, float4 x) {
+  const float4 w = load_quad(n.weight + i), b = load_quad(n.bias + i);
+  return make_float4(fmaf(tanhf(n.alpha * x.x), w.x, b.x), fmaf(tanhf(n.alpha * x.y), w.y, b.y),
+                     fmaf(tanhf(n.alpha * x.z), w.z, b.z), fmaf(tanhf(n.alpha * x.w), w.w, b.w));
+}
+
+constexpr int kEmbedThreads = 256;
+template <typename T>
+__global__ void __launch_bounds__(kEmbedThreads) layered_embed_kernel(const LayeredEmbedParams p) {
+  __shared__ uint32_t token_shared;
+  grid_dependency_wait();
+  const int row = blockIdx.x;
+  if (threadIdx.x == 0) token_shared = take_step_token(p.token, row);
+  __syncthreads();
+  grid_launch_dependents();
+  const uint32_t token = token_shared < uint32_t(p.token.vocab) ? token_shared : 0u;
+  T* normed = static_cast<T*>(p.normed) + size_t(row) * p.normed_stride;
+  for (int i = threadIdx.x * 4; i < p.normed_stride; i += kEmbedThreads * 4) {
+    float4 out = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (i < p.residual_stride) {
+      float4 x = load_quad(p.table + size_t(token) * p.residual_stride + i);
+      if (p.vector) x = add(x, load_quad(p.vector + i));
+      *reinterpret_cast<float4*>(p.residual + size_t(row) * p.residual_stride + i) = x;
+      out = dynamic_tanh(p.norm, i, x);
+    }
+    store_quad(normed + i, out);
+  }
+}
+
+// Four columns per thread, rows along y.
+constexpr int kJoinThreads = 128;
+template <typename T>
+__global__ void __launch_bounds__(kJoinThreads) sublayer_join_kernel(const SublayerJoinParams p) {
+  const int i = (blockIdx.x * kJoinThreads + threadIdx.x) * 4;
+  const bool live = i < p.residual_stride;
+  // Norm vectors do not come from the preceding kernel.
+  float4 wa = make_float4(0.0f, 0.0f, 0.0f, 0.0f), ba = wa, wb = wa, bb = wa;
+  if (live) {
+    wa = load_quad(p.after.weight + i);
+    ba = load_quad(p.after.bias + i);
+    wb = load_quad(p.before.weight + i);
+    bb = load_quad(p.before.bias + i);
+  }
+  grid_dependency_wait();
+  grid_launch_dependents();
+  if (i >= p.normed_stride) return;
+  for (int row = blockIdx.y; row < p.rows; row += gridDim.y) {
+    float4 out = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (live) {
+      const size_t at = size_t(row) * p.residual_stride + i;
+      const size_t slice = size_t(p.rows) * p.residual_stride;
+      float4 y = *reinterpret_cast<const float4*>(p.partial + at);
+      for (int s = 1; s < p.ksplit; ++s) y = add(y, *reinterpret_cast<const float4*>(p.partial + s * slice + at));
+      float4 x = *reinterpret_cast<const float4*>(p.residual + at);
+      x.x += fmaf(tanhf(p.after.alpha * y.x), wa.x, ba.x);
+      x.y += fmaf(tanhf(p.after.alpha * y.y), wa.y, ba.y);
+      x.z += fmaf(tanhf(p.after.alpha * y.z), wa.z, ba.z);
+      x.w += fmaf(tanhf(p.after.alpha * y.w), wa.w, ba.w);
+      if (p.tap) {
+        float* tap = p.tap + size_t(row) * p.tap_width;
+        const float values[4] = {x.x, x.y, x.z, x.w};
+        for (int j = 0; j < 4; ++j)
+          if (i + j < p.tap_width) tap[i + j] = values[j];
+      }
+      if (p.inject.table) {
+        const uint32_t token = p.inject.tokens[row];
+        x = add(x, load_quad(p.inject.table + size_t(token < uint32_t(p.inject.vocab) ? token : 0u) * p.residual_stride + i));
+      }
+      if (p.inject.vector) x = add(x, load_quad(p.inject.vector + i));
+      *reinterpret_cast<float4*>(p.residual + at) = x;
+      out = make_float4(fmaf(tanhf(p.before.alpha * x.x), wb.x, bb.x), fmaf(tanhf(p.before.alpha * x.y), wb.y, bb.y),
+                        fmaf(tanhf(p.before.alpha * x.z), wb.z, bb.z), fmaf(tanhf(p.before.alpha * x.w), wb.w, bb.w));
+    }
+    store_quad(static_cast<T*>(p.normed) + size_t(row) * p.normed_stride + i, out);
+  }
+}
+
+// One warp per (row, unit); units in the order of the fused projection: q heads, k heads, v heads, then the linear
+// attention's q, k and v heads.
+template <typename T>
+__global__ void __launch_bounds__(128) mixer_prepare_kernel(const MixerPrepareParams p) {
+  const int warp = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int units = p.heads + 2 * p.kv_heads + 3 * p.lin_heads;
+  const int context = p.control->context;  // written by the previous step
+  grid_dependency_wait();
+  grid_launch_dependents();
+  if (warp >= p.rows * units || context < 0 || context + p.rows > p.capacity) return;
+  const int row = warp / units;
+  int unit = warp - row * units;
+  const int position = context + row;
+  T* x = static_cast<T*>(p.fused) + size_t(row) * p.stride;
+
+  if (unit < p.heads + p.kv_heads) {  // rotation of a q or k head; k goes to the cache
+    const bool key = unit >= p.heads;
+    x += size_t(unit) * p.dim_pad;
+    T* to = key ? static_cast<T*>(p.k_cache) + (size_t(position) * p.kv_heads + (unit - p.heads)) * p.dim_pad : x;
+    const int half = p.rot_dims >> 1;
+    const float2* turn = p.rotation + size_t(position) * half;
+    if (half & 1) {
+      for (int i = lane; i < half; i += 32) {
+        const float u = value_of(x[i]), v = value_of(x[i + half]);
+        const float2 t = turn[i];
+        store_value(to + i, u * t.x - v * t.y);
+        store_value(to + i + half, v * t.x + u * t.y);
+      }
+    } else {
+      for (int i = lane * 2; i < half; i += 64) {
+        const float2 u = load_pair(x + i), v = load_pair(x + i + half);
+        const float2 t0 = turn[i], t1 = turn[i + 1];
+        store_pair(to + i, u.x * t0.x - v.x * t0.y, u.y * t1.x - v.y * t1.y);
+        store_pair(to + i + half, v.x * t0.x + u.x * t0.y, v.y * t1.x + u.y * t1.y);
+      }
+    }
+    if (key)
+      for (int i = p.rot_dims + lane * 2; i < p.dim_pad; i += 64) {
+        const float2 v = load_pair(x + i);
+        store_pair(to + i, v.x, v.y);
+      }
+    return;
+  }
+  unit -= p.heads + p.kv_heads;
+  x += size_t(p.heads + p.kv_heads) * p.dim_pad;
+  if (unit < p.kv_heads) {  // value norm, into the cache
+    x += size_t(unit) * p.vdim_pad;
+    T* to = static_cast<T*>(p.v_cache) + (size_t(position) * p.kv_heads + unit) * p.vdim_pad;
+    float sum = 0.0f;
+    for (int i = lane * 2; i < p.vdim_pad; i += 64) {
+      const float2 v = load_pair(x + i);
+      sum = fmaf(v.x, v.x, fmaf(v.y, v.y, sum));
+    }
+    const float root = sqrtf(warp_sum(sum) / float(p.vdim) + p.eps);
+    for (int i = lane * 2; i < p.vdim_pad; i += 64) {
+      const float2 v = load_pair(x + i);
+      store_pair(to + i, v.x / root, v.y / root);
+    }
+    return;
+  }
+  unit -= p.kv_heads;
+  x += size_t(p.kv_heads) * p.vdim_pad;
+  const int kind = unit / p.lin_heads, head = unit - kind * p.lin_heads;  // 0 q, 1 k, 2 v
+  const int pad = kind == 2 ? p.lin_vdim_pad : p.lin_dim_pad;
+  x += size_t(min(kind, 2)) * p.lin_heads * p.lin_dim_pad + size_t(head) * pad;
+  T* ring = nullptr;
+  if (p.ring_k && kind > 0)
+    ring = static_cast<T*>(kind == 1 ? p.ring_k : p.ring_v) + (size_t(position & (kRingRows - 1)) * p.lin_heads + head) * pad;
+  for (int i = lane * 2; i < pad; i += 64) {
+    float2 v = load_pair(x + i);
+    v.x = silu_exact(v.x);
+    v.y = silu_exact(v.y);
+    store_pair(x + i, v.x, v.y);
+    if (ring) store_pair(ring + i, v.x, v.y);
+  }
+}
+
+__device__ __forceinline__ float block_total(float v, float* shared) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) shared[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float total = 0.0f;
+  for (int w = 0; w < int(blockDim.x >> 5); ++w) total += shared[w];
+  return total;
+}
+
+// Blocks [0, rows * heads) merge one (row, head) of the split attention (when asked to); the last `rows` blocks finish
+// one row of the linear attention: RMS norm over all heads, weight, sigmoid gate, scale.
+constexpr int kFinishThreads = 128;
+template <typename T>
+__global__ void __launch_bounds__(kFinishThreads) mixer_finish_kernel(const MixerFinishParams p) {
+  __shared__ float weights[64];
+  __shared__ float shared[8];
+  const int merges = p.merge ? p.rows * p.attention.heads : 0;
+  if (int(blockIdx.x) < merges) {
+    const SizedAttentionParams& a = p.attention;
+    const int offset = *a.device_offset;
+    grid_dependency_wait();
+    grid_launch_dependents();
+    if (offset < 0 || offset + p.rows > a.capacity) return;
+    const int slot = blockIdx.x, row = slot / a.heads, head = slot - row * a.heads;
+    const int slots = p.rows * a.heads, pitch = a.vdim_pad + 4;
+    const int splits = min(64, (offset + p.rows + a.chunk - 1) / a.chunk);
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    float m = -INFINITY, l = 0.0f;
+    if (int(threadIdx.x) < splits) {
+      const float* src = a.scratch + (size_t(threadIdx.x) * slots + slot) * pitch + a.vdim_pad;
+      m = src[0];
+      l = src[1];
+    }
+    const float sink = a.sink ? a.sink[head] : -INFINITY;
+    float top = warp_max(m);
+    if (lane == 0) shared[warp] = top;
+    __syncthreads();
+    top = fmaxf(fmaxf(fmaxf(shared[0], shared[1]), fmaxf(shared[2], shared[3])), sink);
+    const float weight = m == -INFINITY ? 0.0f : expf(m - top);
+    if (threadIdx.x < 64) weights[threadIdx.x] = weight;
+    const float part = warp_sum(l * weight);
+    if (lane == 0) shared[4 + warp] = part;
+    __syncthreads();
+    const float denominator = ((shared[4] + shared[5]) + (shared[6] + shared[7])) + (a.sink ? expf(sink - top) : 0.0f);
+    const float factor = denominator > 0.0f ? a.out_scale / denominator : 0.0f;
+    T* out = static_cast<T*>(a.out) + size_t(row) * a.out_stride + size_t(head) * a.vdim_pad;
+    for (int i = threadIdx.x; i < a.vdim_pad; i += kFinishThreads) {
+      const float* src = a.scratch + size_t(slot) * pitch + i;
+      float sum = 0.0f;
+#pragma unroll 8
+      for (int s = 0; s < splits; ++s) sum = fmaf(src[size_t(s) * slots * pitch], weights[s], sum);
+      store_value(out + i, sum * factor);
+    }
+    return;
+  }
+  const int row = int(blockIdx.x) - merges;
+  grid_dependency_wait();
+  grid_launch_dependents();
+  const int width = p.lin_heads * p.lin_vdim_pad;
+  const float* x = p.lin_out + size_t(row) * width;
+  const T* gate = static_cast<const T*>(p.gate) + size_t(row) * p.gate_stride;
+  T* out = static_cast<T*>(p.out) + size_t(row) * p.out_stride + p.lin_offset;
+  float sum = 0.0f;
+  for (int i = threadIdx.x * 4; i < width; i += kFinishThreads * 4) {
+    const float4 v = *reinterpret_cast<const float4*>(x + i);
+    sum = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, sum))));
+  }
+  const float mean = block_total(sum, shared) / (float(p.lin_heads) * float(p.lin_vdim));
+  const float factor = p.lin_scale / sqrtf(mean + p.eps);
+  const int end = p.out_stride - p.lin_offset;  // the columns behind the heads pad the projection's input
+  for (int i = threadIdx.x * 4; i < end; i += kFinishThreads * 4) {
+    float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (i < width) {
+      const float4 v = *reinterpret_cast<const float4*>(x + i), w = load_quad(p.norm + i), z = load_quad(gate + i);
+      y = make_float4(v.x * factor * w.x * sigmoid_value(z.x), v.y * factor * w.y * sigmoid_value(z.y),
+                      v.z * factor * w.z * sigmoid_value(z.z), v.w * factor * w.w * sigmoid_value(z.w));
+    }
+    store_quad(out + i, y);
+  }
+}
+
+__device__ __forceinline__ float min_gru_candidate(float u) { return u >= 0.0f ? u + 0.5f : sigmoid_value(u); }
+
+// One thread per channel. Pending rows are folded into the state; the step's own rows stay pending in the ring.
+template <typename T>
+__global__ void __launch_bounds__(128) min_gru_step_kernel(const MinGruParams p) {
+  const int channel = blockIdx.x * 128 + threadIdx.x;
+  const int context = p.control->context, base = p.control->state_base;
+  const bool runs = context >= 0 && context + p.rows <= p.capacity;
+  const int pending = min(kPendingRows, max(0, context - base));
+  float s = 0.0f;
+  if (runs && channel < p.width_pad) {  // the ring and the state were written by earlier steps
+    if (base > 0) s = p.state[channel];
+    for (int i = 0; i < pending; ++i) {
+      const size_t at = size_t((base + i) & (kRingRows - 1)) * p.width_pad + channel;
+      const float z = p.ring_gate[at];
+      s = (1.0f - z) * s + z * p.ring_candidate[at];
+    }
+  }
+  grid_dependency_wait();
+  grid_launch_dependents();
+  if (!runs || channel >= p.out_stride) return;
+  T* out = static_cast<T*>(p.out) + channel;
+  if (channel >= p.width_pad) {
+    for (int r = 0; r < p.rows; ++r) store_value(out + size_t(r) * p.out_stride, 0.0f);
+    return;
+  }
+  if (pending) p.state[channel] = s;
+  for (int r = 0; r < p.rows; ++r) {
+    const T* x = static_cast<const T*>(p.fused) + size_t(r) * p.stride + channel;
+    const float z = sigmoid_value(value_of(x[0])), candidate = min_gru_candidate(value_of(x[p.width_pad]));
+    const size_t at = size_t((context + r) & (kRingRows - 1)) * p.width_pad + channel;
+    p.ring_gate[at] = z;
+    p.ring_candidate[at] = candidate;
+    s = (1.0f - z) * s + z * candidate;
+    store_value(out + size_t(r) * p.out_stride, s * silu_exact(value_of(x[2 * p.width_pad])));
+  }
+}
+
+// A prompt segment: a block owns 32 channels, its 1024 threads 64 time stretches of 16 channel pairs. Every stretch is
+// reduced to (product of 1 - z, value from zero), the stretches are chained, and a second pass emits the rows.
+constexpr int kStretches = 64;
+__global__ void __launch_bounds__(1024) min_gru_prompt_kernel(const MinGruParams p) {
+  __shared__ float keep[kStretches][32], value[kStretches][32];
+  const int context = p.control->context, base = p.control->state_base;
+  const bool runs = context >= 0 && context + p.rows <= p.capacity;
+  grid_dependency_wait();
+  grid_launch_dependents();
+  if (!runs) return;
+  const int pair = threadIdx.x & 15, stretch = threadIdx.x >> 4;
+  const int channel = blockIdx.x * 32 + pair * 2;
+  const int length = (p.rows + kStretches - 1) / kStretches;
+  const int begin = min(p.rows, stretch * length), end = min(p.rows, begin + length);
+  const bool live = channel < p.width_pad;
+  const bf16* x = static_cast<const bf16*>(p.fused) + channel;
+  float a0 = 1.0f, a1 = 1.0f, s0 = 0.0f, s1 = 0.0f;
+  if (live) {
+#pragma unroll 4
+    for (int t = begin; t < end; ++t) {
+      const float2 zr = load_pair(x + size_t(t) * p.stride), u = load_pair(x + size_t(t) * p.stride + p.width_pad);
+      const float z0 = sigmoid_value(zr.x), z1 = sigmoid_value(zr.y);
+      s0 = (1.0f - z0) * s0 + z0 * min_gru_candidate(u.x);
+      s1 = (1.0f - z1) * s1 + z1 * min_gru_candidate(u.y);
+      a0 *= 1.0f - z0;
+      a1 *= 1.0f - z1;
+    }
+  }
+  keep[stretch][pair * 2] = a0;
+  keep[stretch][pair * 2 + 1] = a1;
+  value[stretch][pair * 2] = s0;
+  value[stretch][pair * 2 + 1] = s1;
+  __syncthreads();
+  if (threadIdx.x < 32) {
+    const int own = blockIdx.x * 32 + threadIdx.x;
+    if (own < p.width_pad) {
+      float s = base > 0 ? p.state[own] : 0.0f;
+      const int pending = min(kPendingRows, max(0, context - base));
+      for (int i = 0; i < pending; ++i) {
+        const size_t at = size_t((base + i) & (kRingRows - 1)) * p.width_pad + own;
+        const float z = p.ring_gate[at];
+        s = (1.0f - z) * s + z * p.ring_candidate[at];
+      }
+      for (int i = 0; i < kStretches; ++i) {
+        const float next = keep[i][threadIdx.x] * s + value[i][threadIdx.x];
+        value[i][threadIdx.x] = s;  // the state ahead of the stretch
+        s = next;
+      }
+      p.state[own] = s;
+    }
+  }
+  __syncthreads();
+  if (channel >= p.out_stride) return;
+  bf16* out = static_cast<bf16*>(p.out) + channel;
+  s0 = value[stretch][pair * 2];
+  s1 = value[stretch][pair * 2 + 1];
+#pragma unroll 4
+  for (int t = begin; t < end; ++t) {
+    float y0 = 0.0f, y1 = 0.0f;
+    if (live) {
+      const bf16* row = x + size_t(t) * p.stride;
+      const float2 zr = load_pair(row), u = load_pair(row + p.width_pad), g = load_pair(row + 2 * p.width_pad);
+      const float z0 = sigmoid_value(zr.x), z1 = sigmoid_value(zr.y);
+      s0 = (1.0f - z0) * s0 + z0 * min_gru_candidate(u.x);
+      s1 = (1.0f - z1) * s1 + z1 * min_gru_candidate(u.y);
+      y0 = s0 * silu_exact(g.x);
+      y1 = s1 * silu_exact(g.y);
+    }
+    store_pair(out + size_t(t) * p.out_stride, y0, y1);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) clamped_glu_kernel(const T* gate_up, int rows, int ff, float limit, T* out) {
+  grid_dependency_wait();
+  grid_launch_dependents();
+  const int per_row = ff / 4;
+  const long long total = (long long)rows * per_row;
+  for (long long i = blockIdx.x * 256ll + threadIdx.x; i < total; i += gridDim.x * 256ll) {
+    const int row = int(i / per_row), n = int(i - (long long)row * per_row) * 4;
+    const float4 g = load_quad(gate_up + size_t(row) * 2 * ff + n), u = load_quad(gate_up + size_t(row) * 2 * ff + ff + n);
+    store_quad(out + size_t(row) * ff + n,
+               make_float4(clamped_glu_value(g.x, u.x, limit), clamped_glu_value(g.y, u.y, limit),
+                           clamped_glu_value(g.z, u.z, limit), clamped_glu_value(g.w, u.w, limit)));
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) gather_rows_kernel(const T* source, const int32_t* index, int stride, T* out) {
+  const T* from = source + size_t(index[blockIdx.x]) * stride;
+  for (int i = threadIdx.x; i < stride; i += 256) out[size_t(blockIdx.x) * stride + i] = from[i];
+}
+
+__global__ void __launch_bounds__(256) sum_partials_kernel(const float* partial, int ksplit, size_t count, float* out) {
+  grid_dependency_wait();
+  for (size_t i = size_t(blockIdx.x) * 256 + threadIdx.x; i < count; i += size_t(gridDim.x) * 256) {
+    float sum = partial[i];
+    for (int s = 1; s < ksplit; ++s) sum += partial[s * count + i];
+    out[i] = sum;
+  }
+}
+
+// A warp per output feature, the rows' products summed lane by lane and then across the warp.
+constexpr int kTrue32Tile = 256;
+__global__ void __launch_bounds__(256) true32_linear_kernel(const float* x, int rows, const bf16* w, const bf16* bias,
+                                                            int in, int out_features, float* out) {
+  __shared__ float tile[kMaxRows][kTrue32Tile];
+  grid_dependency_wait();
+  grid_launch_dependents();
+  const int n = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  float acc[kMaxRows];
+#pragma unroll
+  for (int r = 0; r < kMaxRows; ++r) acc[r] = 0.0f;
+  for (int first = 0; first < in; first += kTrue32Tile) {
+    const int width = min(kTrue32Tile, in - first);
+    __syncthreads();
+    for (int i = threadIdx.x; i < rows * kTrue32Tile; i += 256) {
+      const int r = i / kTrue32Tile, k = i - r * kTrue32Tile;
+      tile[r][k] = k < width ? x[size_t(r) * in + first + k] : 0.0f;
+    }
+    __syncthreads();
+    if (n < out_features) {
+      for (int k = lane; k < width; k += 32) {
+        const float weight = __bfloat162float(w[size_t(n) * in + first + k]);
+#pragma unroll
+        for (int r = 0; r < kMaxRows; ++r)
+          if (r < rows) acc[r] = fmaf(tile[r][k], weight, acc[r]);
+      }
+    }
+  }
+  if (n >= out_features) return;
+#pragma unroll
+  for (int r = 0; r < kMaxRows; ++r) {
+    if (r < rows) {
+      const float sum = warp_sum(acc[r]);
+      if (lane == 0) out[size_t(r) * out_features + n] = sum + (bias ? __bfloat162float(bias[n]) : 0.0f);
+    }
+  }
+}
+
+__global__ void rotation_table_kernel(float2* table, size_t positions, int half, int dims, double log_base) {
+  for (size_t i = size_t(blockIdx.x) * blockDim.x + threadIdx.x; i < positions * half; i += size_t(gridDim.x) * blockDim.x) {
+    const double angle = double(i / half) * exp(log_base * (-2.0 * double(i % half) / double(dims)));
+    double s, c;
+    sincos(angle, &s, &c);
+    table[i] = make_float2(float(c), float(s));
+  }
+}
+
+}  // namespace
+
+template <typename T>
+void launch_layered_embed(const LayeredEmbedParams& p, cudaStream_t stream, bool pdl) {
+  launch(layered_embed_kernel<T>, dim3(p.token.rows), dim3(kEmbedThreads), 0, stream, pdl, p);
+}
+template <typename T>
+void launch_sublayer_join(const SublayerJoinParams& p, cudaStream_t stream, bool pdl) {
+  const unsigned columns = unsigned((p.normed_stride / 4 + kJoinThreads - 1) / kJoinThreads);
+  launch(sublayer_join_kernel<T>, dim3(columns, unsigned(std::min(p.rows, 1024))), dim3(kJoinThreads), 0, stream, pdl, p);
+}
+template <typename T>
+void launch_mixer_prepare(const MixerPrepareParams& p, cudaStream_t stream, bool pdl) {
+  const int warps = p.rows * (p.heads + 2 * p.kv_heads + 3 * p.lin_heads);
+  launch(mixer_prepare_kernel<T>, dim3(unsigned((warps + 3) / 4)), dim3(128), 0, stream, pdl, p);
+}
+template <typename T>
+void launch_mixer_finish(const MixerFinishParams& p, cudaStream_t stream, bool pdl) {
+  const int blocks = p.rows + (p.merge ? p.rows * p.attention.heads : 0);
+  launch(mixer_finish_kernel<T>, dim3(unsigned(blocks)), dim3(kFinishThreads), 0, stream, pdl, p);
+}
+template <typename T>
+void launch_min_gru_step(const MinGruParams& p, cudaStream_t stream, bool pdl) {
+  launch(min_gru_step_kernel<T>, dim3(unsigned((p.out_stride + 127) / 128)), dim3(128), 0, stream, pdl, p);
+}
+void launch_min_gru_prompt(const MinGruParams& p, cudaStream_t stream, bool pdl) {
+  launch(min_gru_prompt_kernel, dim3(unsigned((p.out_stride + 31) / 32)), dim3(1024), 0, stream, pdl, p);
+}
+template <typename T>
+void launch_clamped_glu(const T* gate_up, int rows, int ff, float limit, T* out, int multiprocessors,
+                        cudaStream_t stream, bool pdl) {
+  const long long quads = (long long)rows * ff / 4;
+  const unsigned blocks = unsigned(std::max(1ll, std::min((quads + 255) / 256, (long long)multiprocessors * 8)));
+  launch(clamped_glu_kernel<T>, dim3(blocks), dim3(256), 0, stream, pdl, gate_up, rows, ff, limit, out);
+}
+template <typename T>
+void launch_gather_rows(const T* source, const int32_t* index, int count, int stride, T* out, cudaStream_t stream) {
+  launch(gather_rows_kernel<T>, dim3(count), dim3(256), 0, stream, false, source, index, stride, out);
+}
+void launch_sum_partials(const float* partial, int ksplit, size_t count, float* out, int multiprocessors,
+                         cudaStream_t stream, bool pdl) {
+  const unsigned blocks = unsigned(std::max<size_t>(1, std::min((count + 255) / 256, size_t(multiprocessors) * 8)));
+  launch(sum_partials_kernel, dim3(blocks), dim3(256), 0, stream, pdl, partial, ksplit, count, out);
+}
+void launch_true32_linear(const float* x, int rows, const PreparedLinear& w, float* out, cudaStream_t stream, bool pdl) {
+  if (rows < 1 || rows > kMaxRows) throw std::invalid_argument("32-bit linear takes 1..16 rows");
+  launch(true32_linear_kernel, dim3(unsigned((w.out + 7) / 8)), dim3(256), 0, stream, pdl, x, rows, w.dense, w.bias, w.in,
+         w.out, out);
+}
+void launch_rotation_table(float2* table, size_t positions, int dims, double base, cudaStream_t stream) {
+  const size_t count = positions * (dims / 2);
+  if (!count) return;
+  rotation_table_kernel<<<unsigned(std::min<size_t>((count + 255) / 256, 4096)), 256, 0, stream>>>(table, positions, dims / 2,
+                                                                                                   dims, std::log(base));
+  check_launch();
+}
+
+template void launch_layered_embed<bf16>(const LayeredEmbedParams&, cudaStream_t, bool);
+template void launch_layered_embed<float>(const LayeredEmbedParams&, cudaStream_t, bool);
+template void launch_sublayer_join<bf16>(const SublayerJoinParams&, cudaStream_t, bool);
+template void launch_sublayer_join<float>(const SublayerJoinParams&, cudaStream_t, bool);
+template void launch_mixer_prepare<bf16>(const MixerPrepareParams&, cudaStream_t, bool);
+template void launch_mixer_prepare<float>(const MixerPrepareParams&, cudaStream_t, bool);
+template void launch_mixer_finish<bf16>(const MixerFinishParams&, cudaStream_t, bool);
+template void launch_mixer_finish<float>(const MixerFinishParams&, cudaStream_t, bool);
+template void launch_min_gru_step<bf16>(const MinGruParams&, cudaStream_t, bool);
+template void launch_min_gru_step<float>(const MinGruParams&, cudaStream_t, bool);
+template void launch_clamped_glu<bf16>(const bf16*, int, int, float, bf16*, int, cudaStream_t, bool);
+template void launch_clamped_glu<float>(const float*, int, int, float, float*, int, cudaStream_t, bool);
+template void launch_gather_rows<bf16>(const bf16*, const int32_t*, int, int, bf16*, cudaStream_t);
+template void launch_gather_rows<float>(const float*, const int32_t*, int, int, float*, cudaStream_t);
+
+}  // namespace ei

@@ -7,44 +7,20 @@
 // What differs is the step itself: one fused kernel sequence per layer, the context length,
 // pending token, acceptance and KV commit kept on the device, the whole step replayed from a
 // CUDA graph per row count, and a single host synchronisation at its end.
-#include <algorithm>
 #include <cmath>
 #include <cstring>
 #include <limits>
-#include <map>
-#include <memory>
-#include <mutex>
-#include <string>
-#include <vector>
 
-#include "abi_util.cuh"
-#include "kernels.cuh"
-#include "smallm_gemm.cuh"
+#include "layered.cuh"
 
 namespace ei {
 namespace {
 
-constexpr size_t kAlign = 256;
-constexpr int kMaxRows = 16;
-
-size_t aligned(size_t bytes) { return (bytes + kAlign - 1) & ~(kAlign - 1); }
-
-struct PreparedLinear {
-  bool quantized = false;
-  int in = 0, out = 0;
-  const int32_t* qweight = nullptr;
-  const bf16* scales = nullptr;
-  const int32_t* zeros = nullptr;
-  int padded_groups = 0, zero_stride = 0, group_size = 0;
-  const bf16* dense = nullptr;  // [out, in]
-  const bf16* bias = nullptr;
-  size_t bytes = 0;  // weight bytes one call streams
-};
-
-__global__ void commit_rows_kernel(Control* control, int rows) {
+__global__ void commit_rows_kernel(Control* control, int rows, int folded) {
   grid_dependency_wait();
   if (threadIdx.x || blockIdx.x) return;
   if (control->status & 1) return;
+  control->state_base = control->context + (folded ? rows : 0);
   control->context += rows;
 }
 
@@ -113,39 +89,6 @@ __global__ void __launch_bounds__(512) residual_norm_bf16_kernel(const bf16* pro
 }  // namespace ei
 
 using namespace ei;
-
-struct ei_model {
-  ei_model_config config{};
-  int device = 0;
-  unsigned char* arena = nullptr;
-  size_t arena_bytes = 0;
-  const bf16* embedding = nullptr;
-  const bf16* output_norm = nullptr;
-  PreparedLinear lm_head;
-  struct Layer {
-    PreparedLinear qkv, o, gate_up, down;
-    const bf16 *attention_norm = nullptr, *ffn_norm = nullptr, *q_norm = nullptr, *k_norm = nullptr;
-  };
-  std::vector<Layer> layers;
-  float* rope_table = nullptr;
-  size_t weight_bytes = 0;
-  int multiprocessors = 1;  // queried at creation
-  size_t smem_limit = 227 * 1024;
-  // Activations of a prompt segment (up to kPromptSegment rows through every projection at once): one set per
-  // model, created by the first long prompt and lent, under the mutex, to one prefill at a time.
-  struct PromptWorkspace {
-    std::mutex mutex;
-    unsigned char* arena = nullptr;
-    size_t rows = 0;
-    bf16 *residual = nullptr, *normed = nullptr, *qkv = nullptr, *attention = nullptr, *gate_up = nullptr,
-         *act = nullptr, *projection = nullptr;
-    float* partial = nullptr;         // FP32 sums of the o / down projections: [K slices][rows][hidden]
-    size_t partial_bytes = 0;
-    uint32_t *tokens = nullptr, *step_tokens = nullptr;
-    uint32_t* host_tokens = nullptr;  // pinned
-  } prompt;
-  bool prompt_ready = false;  // every projection of every layer has a shape the prompt GEMM takes
-};
 
 namespace {
 
@@ -284,89 +227,7 @@ void validate_config(const ei_model_config& c) {
 
 }  // namespace
 
-struct ei_session {
-  ei_model* model = nullptr;
-  size_t capacity = 0;
-  bool use_graph = false;
-  cudaStream_t stream = nullptr;
-  unsigned char* arena = nullptr;
-  // workspace
-  bf16 *residual = nullptr, *normed = nullptr, *qkv = nullptr, *attention = nullptr, *act = nullptr,
-       *gate_up = nullptr, *projection = nullptr, *logits = nullptr;
-  float* partial = nullptr;
-  float* attention_scratch = nullptr;
-  float* best_value = nullptr;
-  int* best_index = nullptr;
-  uint32_t *tokens = nullptr, *step_tokens = nullptr, *targets = nullptr;
-  Control* control = nullptr;
-  DraftSource* draft_source = nullptr;
-  DraftSource draft_host{nullptr, 0, 0};
-  TokenSink* token_sink = nullptr;  // device; all zero unless a speculative decoder owns the session
-  bf16 *k_cache = nullptr, *v_cache = nullptr;
-  // pinned host staging
-  uint32_t* host_tokens = nullptr;
-  Control* host_control = nullptr;
-  // plans
-  int attention_chunk = 64, attention_splits = 1;
-  // state
-  size_t context = 0;
-  size_t bound = 0;  // upper bound of the context length after every step enqueued so far (full acceptance)
-  bool history_ready = false, poisoned = false;
-  int inject_launch = 0, inject_completion = 0;
-  uint32_t inject_attention_polls = 0;  // the same hook for the next attention launch (its K / V tile copies)
-  uint32_t inject_wait_polls = 0;  // test hook: the next weight-streaming GEMM gets this poll limit and a copy
-                                   // expectation it cannot meet, so that its bounded waits run out
-  size_t launches = 0, launches_per_step[kMaxRows + 1] = {};
-  size_t prefill_target_row = 0;  // where in `targets` the last prefill left the greedy token of its last row
-  // graphs: [kind][rows]; kind 0 verify (host tokens), 1 verify (device drafts), 2 decode (commit all)
-  cudaGraphExec_t graphs[3][kMaxRows + 1] = {};
-};
-
-// A fixed set of sessions of one model that are verified together: their rows are stacked into one
-// [sessions * rows, hidden] forward, so every weight is streamed once for all of them; attention, KV append
-// and acceptance stay per session. The first session lends its workspace and stream.
-struct ei_batch {
-  std::vector<ei_session*> sessions;
-  cudaGraphExec_t graphs[kMaxRows + 1] = {};  // by rows per session
-  // Wide form (more than 16 stacked rows): the sessions' slots on the device, and buffers sized on first use
-  // for sessions * rows stacked rows.
-  SessionSlot* slots = nullptr;
-  CUtensorMap* maps = nullptr;      // [sessions][2]: TMA descriptions of every session's K and V cache, all layers
-  unsigned char* wide_arena = nullptr;
-  size_t wide_rows = 0;
-  bf16* logits = nullptr;           // [stacked rows, vocab]
-  float* attention_scratch = nullptr;
-  size_t scratch_stride = 0;        // floats per session
-  float* best_value = nullptr;      // [stacked rows][kWideParts]
-  int* best_index = nullptr;
-  uint32_t* targets = nullptr;      // [stacked rows]
-  Control* controls = nullptr;      // [sessions] gathered after a step
-  Control* host_controls = nullptr; // pinned
-};
-constexpr int kWideParts = 8;       // argmax partials per row of the wide form
-constexpr size_t kMaxBatchSessions = 1024;
-
-// A target session and a draft session that generate together without host round trips: per round the draft
-// session decodes drafts_per_round + 1 tokens, each from the token the previous step left on the device, the
-// target session verifies [pending, d1..dk] in one forward, and the draft session adopts the target's context
-// length and pending token. One device array holds the token of every position for both: the draft session
-// writes its proposals into it, the target session reads them from it and overwrites them with what it emits.
-struct ei_speculative {
-  ei_session* target = nullptr;
-  ei_session* draft = nullptr;
-  size_t drafts = 0;             // k: drafts verified per round (rows = k + 1)
-  size_t capacity = 0;           // of both sessions
-  uint32_t* tokens = nullptr;    // device [capacity + kMaxRows + 1]: token of every absolute position
-  size_t token_count = 0;
-  cudaEvent_t drafted = nullptr, verified = nullptr;
-  size_t prompt_rows = 0;
-  size_t bound = 0;              // upper bound of the context length after everything enqueued so far
-  bool started = false;
-};
-
-namespace {
-
-enum StepKind { kVerifyHost = 0, kVerifyDevice = 1, kCommitAllWithHead = 2, kCommitAllNoHead = 3 };
+namespace ei {
 
 void tick(ei_session& s) {
   ++s.launches;
@@ -374,43 +235,8 @@ void tick(ei_session& s) {
     throw std::runtime_error("injected launch failure (test hook)");
 }
 
-void require_usable(const ei_session& s) {
-  if (s.poisoned) throw PoisonedError("Session is unusable after failed CUDA stream completion");
-}
-
-void synchronize(ei_session& s) {
-  cudaError_t status = cudaStreamSynchronize(s.stream);
-  if (status == cudaSuccess && s.inject_completion) {
-    s.inject_completion = 0;
-    status = cudaErrorUnknown;  // reported after a real wait; the context itself is intact
-  }
-  if (status != cudaSuccess) {
-    s.poisoned = true;
-    throw std::runtime_error(std::string("CUDA stream completion failed: ") + cudaGetErrorString(status));
-  }
-}
-
-// After a failed submission: drain this session's own stream; on success forget the history
-// (partially written KV is never restored), on failure poison. Mirrors runtime/src/qwen3.cpp:142-161.
-void drain_failed(ei_session& s) noexcept {
-  if (s.poisoned) return;
-  if (cudaStreamSynchronize(s.stream) != cudaSuccess) {
-    s.poisoned = true;
-    return;
-  }
-  Control zero{};
-  if (cudaMemcpyAsync(s.control, &zero, sizeof(Control), cudaMemcpyHostToDevice, s.stream) != cudaSuccess ||
-      cudaStreamSynchronize(s.stream) != cudaSuccess) {
-    s.poisoned = true;
-    return;
-  }
-  s.context = 0;
-  s.bound = 0;
-  s.history_ready = false;
-}
-
 void run_linear(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, int epilogue, bf16* out,
-                int out_stride, bool pdl, int* ksplit_out = nullptr) {
+                int out_stride, bool pdl, int* ksplit_out) {
   const ei_model& m = *s.model;
   const bool aligned_ok = (reinterpret_cast<uintptr_t>(x) & 15) == 0;
   GemmPlan plan;
@@ -433,6 +259,8 @@ void run_linear(ei_session& s, const PreparedLinear& w, const bf16* x, int rows,
   p.w = w.dense;
   p.ldw = w.in;
   p.bias = epilogue == kEpiPartial ? nullptr : w.bias;
+  p.glu = w.glu;
+  p.glu_limit = w.glu_limit;
   p.out = out;
   p.out_stride = out_stride;
   p.epilogue = epilogue;
@@ -458,48 +286,6 @@ bool has_plan(const ei_session& s, const PreparedLinear& w, int rows, int epilog
   return plan_gemm(w.quantized, rows, w.out, w.in, epilogue, m.multiprocessors, m.smem_limit, epilogue == kEpiPartial).fast;
 }
 
-void run_generic(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, bf16* out, bool pdl) {
-  (void)pdl;
-  const size_t count = size_t(rows) * w.out;
-  const unsigned blocks = unsigned(std::min<size_t>((count + 255) / 256, size_t(s.model->multiprocessors) * 32));
-  tick(s);
-  if (w.quantized)
-    awq_generic_kernel<<<blocks, 256, 0, s.stream>>>(x, w.in, w.qweight, w.scales, w.zeros, w.bias, out, w.out, rows,
-                                                    w.out, w.in, w.group_size, w.padded_groups);
-  else
-    dense_generic_kernel<<<blocks, 256, 0, s.stream>>>(x, w.in, w.dense, 1, w.in, w.bias, out, w.out, rows, w.out, w.in);
-  check_launch();
-}
-
-// projection -> residual add -> RMSNorm with `norm_weight`.
-void run_projection_residual_norm(ei_session& s, const PreparedLinear& w, const bf16* x, int rows,
-                                  const bf16* norm_weight, bool pdl) {
-  const auto& c = s.model->config;
-  if (has_plan(s, w, rows, kEpiPartial)) {
-    int ksplit = 1;
-    run_linear(s, w, x, rows, kEpiPartial, nullptr, 0, pdl, &ksplit);
-    ResidualNormParams p{};
-    p.partial = s.partial;
-    p.ksplit = ksplit;
-    p.rows = rows;
-    p.hidden = int(c.hidden_size);
-    p.bias = w.bias;
-    p.residual = s.residual;
-    p.norm_weight = norm_weight;
-    p.eps = c.rms_norm_eps;
-    p.normed = s.normed;
-    tick(s);
-    launch_residual_norm(p, s.stream, pdl);
-  } else {
-    run_generic(s, w, x, rows, s.projection, pdl);
-    tick(s);
-    launch(residual_norm_bf16_kernel, dim3(rows), dim3(512), 0, s.stream, pdl, (const bf16*)s.projection,
-           int(c.hidden_size), s.residual, norm_weight, c.rms_norm_eps, s.normed);
-  }
-}
-
-constexpr size_t kPromptSegment = 2048;  // rows of a long prompt that go through the layers together
-
 bool prompt_linear_ok(const PreparedLinear& w) {
   if (w.quantized && (w.in / 8) % 4) return false;
   const void* weights = w.quantized ? static_cast<const void*>(w.qweight) : static_cast<const void*>(w.dense);
@@ -507,49 +293,9 @@ bool prompt_linear_ok(const PreparedLinear& w) {
          prompt_gemm_eligible(w.quantized, w.group_size, w.out, w.in, nullptr, w.in, nullptr, w.out);
 }
 
-void ensure_prompt_workspace(ei_model& m) {
-  auto& ws = m.prompt;
-  if (ws.arena) return;
-  const auto& c = m.config;
-  const size_t rows = std::min<size_t>(kPromptSegment, c.max_position_embeddings);
-  const size_t H = c.hidden_size, F = c.intermediate_size, Q = c.n_heads * 128;
-  const size_t qkv_width = (c.n_heads + 2 * c.n_kv_heads) * 128;
-  size_t offset = 0;
-  auto take = [&](size_t bytes) {
-    const size_t at = offset;
-    offset += aligned(bytes);
-    return at;
-  };
-  const size_t o_residual = take(rows * H * 2), o_normed = take(rows * H * 2), o_qkv = take(rows * qkv_width * 2);
-  const size_t o_attention = take(rows * Q * 2), o_gate_up = take(rows * 2 * F * 2), o_act = take(rows * F * 2);
-  const size_t o_projection = take(rows * H * 2), o_tokens = take(rows * 4), o_step = take(rows * 4);
-  // Room for the FP32 sums of a full segment, or for 16 K slices of a short one.
-  const size_t partial_bytes = std::max(rows, size_t(16) * std::min<size_t>(rows, 256)) * H * sizeof(float);
-  const size_t o_partial = take(partial_bytes);
-  unsigned char* base = nullptr;
-  EI_CUDA(cudaMalloc(reinterpret_cast<void**>(&base), offset));
-  if (cudaMallocHost(reinterpret_cast<void**>(&ws.host_tokens), rows * 4) != cudaSuccess) {
-    cudaFree(base);
-    throw std::runtime_error("Prompt staging buffer could not be allocated");
-  }
-  ws.residual = reinterpret_cast<bf16*>(base + o_residual);
-  ws.normed = reinterpret_cast<bf16*>(base + o_normed);
-  ws.qkv = reinterpret_cast<bf16*>(base + o_qkv);
-  ws.attention = reinterpret_cast<bf16*>(base + o_attention);
-  ws.gate_up = reinterpret_cast<bf16*>(base + o_gate_up);
-  ws.act = reinterpret_cast<bf16*>(base + o_act);
-  ws.projection = reinterpret_cast<bf16*>(base + o_projection);
-  ws.tokens = reinterpret_cast<uint32_t*>(base + o_tokens);
-  ws.step_tokens = reinterpret_cast<uint32_t*>(base + o_step);
-  ws.partial = reinterpret_cast<float*>(base + o_partial);
-  ws.partial_bytes = partial_bytes;
-  ws.rows = rows;
-  ws.arena = base;
-}
-
 // ksplit == 0: BF16 output with bias; otherwise FP32 partial sums of `ksplit` K slices in the workspace.
 void run_prompt_linear(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, bf16* out, bool pdl,
-                       int ksplit = 0) {
+                       int ksplit) {
   GemmParams p{};
   p.epilogue = ksplit ? kEpiPartial : kEpiStore;
   p.ksplit = ksplit;
@@ -596,6 +342,172 @@ void run_prompt_linear_store(ei_session& s, const PreparedLinear& w, const bf16*
          pdl, (const float*)ws.partial, ksplit, rows, w.out, w.bias, out, w.out);
 }
 
+void enqueue_commit(ei_session& s, int rows, bool folded) {
+  tick(s);
+  launch(commit_rows_kernel, dim3(1), dim3(32), 0, s.stream, true, s.control, rows, folded ? 1 : 0);
+}
+
+}  // namespace ei
+
+// A fixed set of sessions of one model that are verified together: their rows are stacked into one
+// [sessions * rows, hidden] forward, so every weight is streamed once for all of them; attention, KV append
+// and acceptance stay per session. The first session lends its workspace and stream.
+struct ei_batch {
+  std::vector<ei_session*> sessions;
+  cudaGraphExec_t graphs[kMaxRows + 1] = {};  // by rows per session
+  // Wide form (more than 16 stacked rows): the sessions' slots on the device, and buffers sized on first use
+  // for sessions * rows stacked rows.
+  SessionSlot* slots = nullptr;
+  CUtensorMap* maps = nullptr;      // [sessions][2]: TMA descriptions of every session's K and V cache, all layers
+  unsigned char* wide_arena = nullptr;
+  size_t wide_rows = 0;
+  bf16* logits = nullptr;           // [stacked rows, vocab]
+  float* attention_scratch = nullptr;
+  size_t scratch_stride = 0;        // floats per session
+  float* best_value = nullptr;      // [stacked rows][kWideParts]
+  int* best_index = nullptr;
+  uint32_t* targets = nullptr;      // [stacked rows]
+  Control* controls = nullptr;      // [sessions] gathered after a step
+  Control* host_controls = nullptr; // pinned
+};
+constexpr int kWideParts = 8;       // argmax partials per row of the wide form
+constexpr size_t kMaxBatchSessions = 1024;
+
+// A target session and a draft session that generate together without host round trips: per round the draft
+// session decodes drafts_per_round + 1 tokens, each from the token the previous step left on the device, the
+// target session verifies [pending, d1..dk] in one forward, and the draft session adopts the target's context
+// length and pending token. One device array holds the token of every position for both: the draft session
+// writes its proposals into it, the target session reads them from it and overwrites them with what it emits.
+struct ei_speculative {
+  ei_session* target = nullptr;
+  ei_session* draft = nullptr;
+  size_t drafts = 0;             // k: drafts verified per round (rows = k + 1)
+  size_t capacity = 0;           // of both sessions
+  uint32_t* tokens = nullptr;    // device [capacity + kMaxRows + 1]: token of every absolute position
+  size_t token_count = 0;
+  cudaEvent_t drafted = nullptr, verified = nullptr;
+  size_t prompt_rows = 0;
+  size_t bound = 0;              // upper bound of the context length after everything enqueued so far
+  bool started = false;
+};
+
+namespace {
+
+void require_usable(const ei_session& s) {
+  if (s.poisoned) throw PoisonedError("Session is unusable after failed CUDA stream completion");
+}
+
+void synchronize(ei_session& s) {
+  cudaError_t status = cudaStreamSynchronize(s.stream);
+  if (status == cudaSuccess && s.inject_completion) {
+    s.inject_completion = 0;
+    status = cudaErrorUnknown;  // reported after a real wait; the context itself is intact
+  }
+  if (status != cudaSuccess) {
+    s.poisoned = true;
+    throw std::runtime_error(std::string("CUDA stream completion failed: ") + cudaGetErrorString(status));
+  }
+}
+
+// After a failed submission: drain this session's own stream; on success forget the history
+// (partially written KV is never restored), on failure poison. Mirrors runtime/src/qwen3.cpp:142-161.
+void drain_failed(ei_session& s) noexcept {
+  if (s.poisoned) return;
+  if (cudaStreamSynchronize(s.stream) != cudaSuccess) {
+    s.poisoned = true;
+    return;
+  }
+  Control zero{};
+  if (cudaMemcpyAsync(s.control, &zero, sizeof(Control), cudaMemcpyHostToDevice, s.stream) != cudaSuccess ||
+      cudaStreamSynchronize(s.stream) != cudaSuccess) {
+    s.poisoned = true;
+    return;
+  }
+  s.context = 0;
+  s.bound = 0;
+  s.history_ready = false;
+}
+
+void run_generic(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, bf16* out, bool pdl) {
+  (void)pdl;
+  const size_t count = size_t(rows) * w.out;
+  const unsigned blocks = unsigned(std::min<size_t>((count + 255) / 256, size_t(s.model->multiprocessors) * 32));
+  tick(s);
+  if (w.quantized)
+    awq_generic_kernel<<<blocks, 256, 0, s.stream>>>(x, w.in, w.qweight, w.scales, w.zeros, w.bias, out, w.out, rows,
+                                                    w.out, w.in, w.group_size, w.padded_groups);
+  else
+    dense_generic_kernel<<<blocks, 256, 0, s.stream>>>(x, w.in, w.dense, 1, w.in, w.bias, out, w.out, rows, w.out, w.in);
+  check_launch();
+}
+
+// projection -> residual add -> RMSNorm with `norm_weight`.
+void run_projection_residual_norm(ei_session& s, const PreparedLinear& w, const bf16* x, int rows,
+                                  const bf16* norm_weight, bool pdl) {
+  const auto& c = s.model->config;
+  if (has_plan(s, w, rows, kEpiPartial)) {
+    int ksplit = 1;
+    run_linear(s, w, x, rows, kEpiPartial, nullptr, 0, pdl, &ksplit);
+    ResidualNormParams p{};
+    p.partial = s.partial;
+    p.ksplit = ksplit;
+    p.rows = rows;
+    p.hidden = int(c.hidden_size);
+    p.bias = w.bias;
+    p.residual = s.residual;
+    p.norm_weight = norm_weight;
+    p.eps = c.rms_norm_eps;
+    p.normed = s.normed;
+    tick(s);
+    launch_residual_norm(p, s.stream, pdl);
+  } else {
+    run_generic(s, w, x, rows, s.projection, pdl);
+    tick(s);
+    launch(residual_norm_bf16_kernel, dim3(rows), dim3(512), 0, s.stream, pdl, (const bf16*)s.projection,
+           int(c.hidden_size), s.residual, norm_weight, c.rms_norm_eps, s.normed);
+  }
+}
+
+void ensure_prompt_workspace(ei_model& m) {
+  auto& ws = m.prompt;
+  if (ws.arena) return;
+  const auto& c = m.config;
+  const size_t rows = std::min<size_t>(kPromptSegment, c.max_position_embeddings);
+  const size_t H = c.hidden_size, F = c.intermediate_size, Q = c.n_heads * 128;
+  const size_t qkv_width = (c.n_heads + 2 * c.n_kv_heads) * 128;
+  size_t offset = 0;
+  auto take = [&](size_t bytes) {
+    const size_t at = offset;
+    offset += aligned(bytes);
+    return at;
+  };
+  const size_t o_residual = take(rows * H * 2), o_normed = take(rows * H * 2), o_qkv = take(rows * qkv_width * 2);
+  const size_t o_attention = take(rows * Q * 2), o_gate_up = take(rows * 2 * F * 2), o_act = take(rows * F * 2);
+  const size_t o_projection = take(rows * H * 2), o_tokens = take(rows * 4), o_step = take(rows * 4);
+  // Room for the FP32 sums of a full segment, or for 16 K slices of a short one.
+  const size_t partial_bytes = std::max(rows, size_t(16) * std::min<size_t>(rows, 256)) * H * sizeof(float);
+  const size_t o_partial = take(partial_bytes);
+  unsigned char* base = nullptr;
+  EI_CUDA(cudaMalloc(reinterpret_cast<void**>(&base), offset));
+  if (cudaMallocHost(reinterpret_cast<void**>(&ws.host_tokens), rows * 4) != cudaSuccess) {
+    cudaFree(base);
+    throw std::runtime_error("Prompt staging buffer could not be allocated");
+  }
+  ws.residual = reinterpret_cast<bf16*>(base + o_residual);
+  ws.normed = reinterpret_cast<bf16*>(base + o_normed);
+  ws.qkv = reinterpret_cast<bf16*>(base + o_qkv);
+  ws.attention = reinterpret_cast<bf16*>(base + o_attention);
+  ws.gate_up = reinterpret_cast<bf16*>(base + o_gate_up);
+  ws.act = reinterpret_cast<bf16*>(base + o_act);
+  ws.projection = reinterpret_cast<bf16*>(base + o_projection);
+  ws.tokens = reinterpret_cast<uint32_t*>(base + o_tokens);
+  ws.step_tokens = reinterpret_cast<uint32_t*>(base + o_step);
+  ws.partial = reinterpret_cast<float*>(base + o_partial);
+  ws.partial_bytes = partial_bytes;
+  ws.rows = rows;
+  ws.arena = base;
+}
+
 // projection -> residual add -> RMSNorm over all rows of a segment: the projection leaves FP32 sums (K split
 // over blocks when few token tiles would leave SMs idle) that the residual + norm kernel finishes, as in the
 // verify step.
@@ -625,6 +537,22 @@ void run_prompt_projection_residual_norm(ei_session& s, const PreparedLinear& w,
     launch(residual_norm_bf16_kernel, dim3(rows), dim3(512), 0, s.stream, pdl, (const bf16*)ws.projection,
            int(c.hidden_size), ws.residual, norm_weight, c.rms_norm_eps, ws.normed);
   }
+}
+
+// The vocabulary head of the uniform decoder over `rows` <= 16 normed rows: BF16 logits and argmax partials.
+int enqueue_uniform_head(ei_session& s, const bf16* normed, int rows) {
+  const ei_model& m = *s.model;
+  const auto& c = m.config;
+  int parts = 0;
+  if (has_plan(s, m.lm_head, rows, kEpiArgmax)) {
+    run_linear(s, m.lm_head, normed, rows, kEpiArgmax, s.logits, int(c.vocab_size), true, &parts);
+  } else {
+    run_generic(s, m.lm_head, normed, rows, s.logits, true);
+    parts = std::min(kSampleMaxParts, sample_partial_blocks(c.vocab_size, m.multiprocessors));
+    tick(s);
+    launch_argmax_partials(s.logits, rows, c.vocab_size, c.vocab_size, s.best_value, s.best_index, parts, s.stream, true);
+  }
+  return parts;
 }
 
 // One forward of `rows` prompt tokens (any number up to the workspace's) at the device-side context length:
@@ -709,26 +637,20 @@ void enqueue_prompt_segment(ei_session& s, int rows, bool head) {
   }
 
   if (head) {
-    const bf16* last = ws.normed + size_t(rows - 1) * hidden;
-    int parts = 0;
-    if (has_plan(s, m.lm_head, 1, kEpiArgmax)) {
-      run_linear(s, m.lm_head, last, 1, kEpiArgmax, s.logits, int(c.vocab_size), pdl, &parts);
-    } else {
-      run_generic(s, m.lm_head, last, 1, s.logits, pdl);
-      parts = std::min(kSampleMaxParts, sample_partial_blocks(c.vocab_size, m.multiprocessors));
-      tick(s);
-      launch_argmax_partials(s.logits, 1, c.vocab_size, c.vocab_size, s.best_value, s.best_index, parts, s.stream, pdl);
-    }
+    const int parts = enqueue_uniform_head(s, ws.normed + size_t(rows - 1) * hidden, 1);
     tick(s);
     launch_finalize(s.best_value, s.best_index, parts, 1, s.targets, nullptr, nullptr, nullptr, nullptr, nullptr,
                     s.stream, pdl);
   }
-  tick(s);
-  launch(commit_rows_kernel, dim3(1), dim3(32), 0, s.stream, pdl, s.control, rows);
+  enqueue_commit(s, rows, true);
 }
 
 // Enqueues one forward of `rows` tokens at the device-side context length.
 void enqueue_step(ei_session& s, int rows, StepKind kind, bf16* logits_out) {
+  if (s.model->layered) {
+    enqueue_layered_step(s, rows, kind);
+    return;
+  }
   const ei_model& m = *s.model;
   const auto& c = m.config;
   const int heads = int(c.n_heads), kv_heads = int(c.n_kv_heads), hidden = int(c.hidden_size), ffn = int(c.intermediate_size);
@@ -821,8 +743,7 @@ void enqueue_step(ei_session& s, int rows, StepKind kind, bf16* logits_out) {
   }
 
   if (kind == kCommitAllNoHead) {
-    tick(s);
-    launch(commit_rows_kernel, dim3(1), dim3(32), 0, s.stream, pdl, s.control, rows);
+    enqueue_commit(s, rows, false);
   } else {
     bf16* logits = logits_out ? logits_out : s.logits;
     int parts = 0;
@@ -838,8 +759,7 @@ void enqueue_step(ei_session& s, int rows, StepKind kind, bf16* logits_out) {
     if (kind == kCommitAllWithHead) {
       launch_finalize(s.best_value, s.best_index, parts, rows, s.targets, nullptr, nullptr, nullptr, nullptr, nullptr,
                       s.stream, pdl);
-      tick(s);
-      launch(commit_rows_kernel, dim3(1), dim3(32), 0, s.stream, pdl, s.control, rows);
+      enqueue_commit(s, rows, false);
     } else {
       launch_finalize(s.best_value, s.best_index, parts, rows, s.targets, s.step_tokens, s.control, nullptr, nullptr,
                       nullptr, s.stream, pdl, s.token_sink);
@@ -850,7 +770,8 @@ void enqueue_step(ei_session& s, int rows, StepKind kind, bf16* logits_out) {
 
 // Runs a step either eagerly or by replaying its graph (captured on first use after an eager warm run).
 void submit_step(ei_session& s, int rows, StepKind kind) {
-  if (!s.use_graph || kind == kCommitAllNoHead || s.inject_wait_polls || s.inject_attention_polls) {
+  if (!s.use_graph || kind == kCommitAllNoHead || s.inject_wait_polls || s.inject_attention_polls ||
+      (s.layered && s.layered->tap)) {
     enqueue_step(s, rows, kind, nullptr);
     return;
   }
@@ -1185,18 +1106,76 @@ void check_status(ei_session& s) {
 
 extern "C" {
 
+static void place_on_device(ei_model& model) {
+  EI_CUDA(cudaGetDevice(&model.device));
+  int value = 0;
+  EI_CUDA(cudaDeviceGetAttribute(&value, cudaDevAttrMultiProcessorCount, model.device));
+  model.multiprocessors = value;
+  EI_CUDA(cudaDeviceGetAttribute(&value, cudaDevAttrMaxSharedMemoryPerBlockOptin, model.device));
+  model.smem_limit = size_t(value);
+}
+
+// Workspace and caches of a session of the uniform decoder, in one arena.
+static void create_uniform_session(ei_session& session) {
+  ei_session* s = &session;
+  const auto& c = s->model->config;
+  const size_t capacity = s->capacity;
+  const size_t H = c.hidden_size, V = c.vocab_size, F = c.intermediate_size;
+  const size_t qkv_width = (c.n_heads + 2 * c.n_kv_heads) * 128, kv_width = c.n_kv_heads * 128;
+  s->attention_chunk = attention_chunk_for(capacity);
+  s->attention_splits = int((capacity + s->attention_chunk - 1) / s->attention_chunk);
+  size_t offset = 0;
+  auto take = [&](size_t bytes) {
+    const size_t at = offset;
+    offset += aligned(bytes);
+    return at;
+  };
+  const size_t o_residual = take(kMaxRows * H * 2), o_normed = take(kMaxRows * H * 2);
+  const size_t o_qkv = take(kMaxRows * qkv_width * 2), o_attention = take(kMaxRows * c.n_heads * 128 * 2);
+  const size_t o_act = take(kMaxRows * F * 2), o_gate_up = take(kMaxRows * 2 * F * 2);
+  const size_t o_projection = take(kMaxRows * H * 2), o_logits = take(kMaxRows * V * 2);
+  const size_t o_partial = take(size_t(16) * kMaxRows * H * sizeof(float));
+  const size_t o_scratch = take(attention_scratch_bytes(kMaxRows, c.n_heads, capacity));
+  const size_t o_best_value = take(size_t(kSampleMaxParts) * 16 * sizeof(float));
+  const size_t o_best_index = take(size_t(kSampleMaxParts) * 16 * sizeof(int));
+  const size_t o_tokens = take(kMaxRows * 4), o_step = take(kMaxRows * 4), o_targets = take(kMaxRows * 4);
+  const size_t o_gather = take(kMaxRows * sizeof(int32_t));
+  const size_t o_control = take(sizeof(Control)), o_source = take(sizeof(DraftSource));
+  const size_t o_sink = take(sizeof(TokenSink));
+  const size_t kv_bytes = c.n_layers * capacity * kv_width * 2;
+  const size_t o_k = take(kv_bytes), o_v = take(kv_bytes);
+  EI_CUDA(cudaMalloc(reinterpret_cast<void**>(&s->arena), offset));
+  unsigned char* base = s->arena;
+  s->residual = reinterpret_cast<bf16*>(base + o_residual);
+  s->normed = reinterpret_cast<bf16*>(base + o_normed);
+  s->qkv = reinterpret_cast<bf16*>(base + o_qkv);
+  s->attention = reinterpret_cast<bf16*>(base + o_attention);
+  s->act = reinterpret_cast<bf16*>(base + o_act);
+  s->gate_up = reinterpret_cast<bf16*>(base + o_gate_up);
+  s->projection = reinterpret_cast<bf16*>(base + o_projection);
+  s->logits = reinterpret_cast<bf16*>(base + o_logits);
+  s->partial = reinterpret_cast<float*>(base + o_partial);
+  s->attention_scratch = reinterpret_cast<float*>(base + o_scratch);
+  s->best_value = reinterpret_cast<float*>(base + o_best_value);
+  s->best_index = reinterpret_cast<int*>(base + o_best_index);
+  s->tokens = reinterpret_cast<uint32_t*>(base + o_tokens);
+  s->step_tokens = reinterpret_cast<uint32_t*>(base + o_step);
+  s->targets = reinterpret_cast<uint32_t*>(base + o_targets);
+  s->gather_index = reinterpret_cast<int32_t*>(base + o_gather);
+  s->control = reinterpret_cast<Control*>(base + o_control);
+  s->draft_source = reinterpret_cast<DraftSource*>(base + o_source);
+  s->token_sink = reinterpret_cast<TokenSink*>(base + o_sink);
+  s->k_cache = reinterpret_cast<bf16*>(base + o_k);
+  s->v_cache = reinterpret_cast<bf16*>(base + o_v);
+}
+
 ei_status ei_model_create(const ei_model_config* config, const ei_named_tensor* tensors, size_t count, ei_model** out) {
   return guarded([&] {
     if (!config || !tensors || !count || !out) throw std::invalid_argument("Model creation requires a config and tensors");
     validate_config(*config);
     auto model = std::make_unique<ei_model>();
     model->config = *config;
-    EI_CUDA(cudaGetDevice(&model->device));
-    int value = 0;
-    EI_CUDA(cudaDeviceGetAttribute(&value, cudaDevAttrMultiProcessorCount, model->device));
-    model->multiprocessors = value;
-    EI_CUDA(cudaDeviceGetAttribute(&value, cudaDevAttrMaxSharedMemoryPerBlockOptin, model->device));
-    model->smem_limit = size_t(value);
+    place_on_device(*model);
     Builder builder{*model};
     size_t bytes = 0;
     for (size_t i = 0; i < count; ++i) {
@@ -1291,6 +1270,18 @@ ei_status ei_model_config_of(const ei_model* model, ei_model_config* out) {
 
 size_t ei_model_weight_bytes(const ei_model* model) { return model ? model->weight_bytes : 0; }
 
+ei_status ei_model_create_layered(const ei_layered_config* config, const ei_layer_spec* layers,
+                                  const ei_named_tensor* tensors, size_t count, ei_model** out) {
+  return guarded([&] {
+    if (!config || !layers || !tensors || !count || !out)
+      throw std::invalid_argument("Model creation requires a config, its layers and tensors");
+    auto model = std::make_unique<ei_model>();
+    place_on_device(*model);
+    create_layered_model(*model, *config, layers, tensors, count);
+    *out = model.release();
+  });
+}
+
 ei_status ei_session_create(ei_model* model, size_t capacity, int graph, ei_session** out) {
   return guarded([&] {
     if (!model || !out || !capacity || capacity > model->config.max_position_embeddings)
@@ -1298,56 +1289,14 @@ ei_status ei_session_create(ei_model* model, size_t capacity, int graph, ei_sess
     int device = 0;
     EI_CUDA(cudaGetDevice(&device));
     if (device != model->device) throw std::invalid_argument("Session must be created on its model CUDA device");
-    const auto& c = model->config;
     auto s = std::make_unique<ei_session>();
     s->model = model;
     s->capacity = capacity;
     s->use_graph = graph != 0;
-    const size_t H = c.hidden_size, V = c.vocab_size, F = c.intermediate_size;
-    const size_t qkv_width = (c.n_heads + 2 * c.n_kv_heads) * 128, kv_width = c.n_kv_heads * 128;
-    s->attention_chunk = attention_chunk_for(capacity);
-    s->attention_splits = int((capacity + s->attention_chunk - 1) / s->attention_chunk);
-    size_t offset = 0;
-    auto take = [&](size_t bytes) {
-      const size_t at = offset;
-      offset += aligned(bytes);
-      return at;
-    };
-    const size_t o_residual = take(kMaxRows * H * 2), o_normed = take(kMaxRows * H * 2);
-    const size_t o_qkv = take(kMaxRows * qkv_width * 2), o_attention = take(kMaxRows * c.n_heads * 128 * 2);
-    const size_t o_act = take(kMaxRows * F * 2), o_gate_up = take(kMaxRows * 2 * F * 2);
-    const size_t o_projection = take(kMaxRows * H * 2), o_logits = take(kMaxRows * V * 2);
-    const size_t o_partial = take(size_t(16) * kMaxRows * H * sizeof(float));
-    const size_t o_scratch = take(attention_scratch_bytes(kMaxRows, c.n_heads, capacity));
-    const size_t o_best_value = take(size_t(kSampleMaxParts) * 16 * sizeof(float));
-    const size_t o_best_index = take(size_t(kSampleMaxParts) * 16 * sizeof(int));
-    const size_t o_tokens = take(kMaxRows * 4), o_step = take(kMaxRows * 4), o_targets = take(kMaxRows * 4);
-    const size_t o_control = take(sizeof(Control)), o_source = take(sizeof(DraftSource));
-    const size_t o_sink = take(sizeof(TokenSink));
-    const size_t kv_bytes = c.n_layers * capacity * kv_width * 2;
-    const size_t o_k = take(kv_bytes), o_v = take(kv_bytes);
-    EI_CUDA(cudaMalloc(reinterpret_cast<void**>(&s->arena), offset));
-    unsigned char* base = s->arena;
-    s->residual = reinterpret_cast<bf16*>(base + o_residual);
-    s->normed = reinterpret_cast<bf16*>(base + o_normed);
-    s->qkv = reinterpret_cast<bf16*>(base + o_qkv);
-    s->attention = reinterpret_cast<bf16*>(base + o_attention);
-    s->act = reinterpret_cast<bf16*>(base + o_act);
-    s->gate_up = reinterpret_cast<bf16*>(base + o_gate_up);
-    s->projection = reinterpret_cast<bf16*>(base + o_projection);
-    s->logits = reinterpret_cast<bf16*>(base + o_logits);
-    s->partial = reinterpret_cast<float*>(base + o_partial);
-    s->attention_scratch = reinterpret_cast<float*>(base + o_scratch);
-    s->best_value = reinterpret_cast<float*>(base + o_best_value);
-    s->best_index = reinterpret_cast<int*>(base + o_best_index);
-    s->tokens = reinterpret_cast<uint32_t*>(base + o_tokens);
-    s->step_tokens = reinterpret_cast<uint32_t*>(base + o_step);
-    s->targets = reinterpret_cast<uint32_t*>(base + o_targets);
-    s->control = reinterpret_cast<Control*>(base + o_control);
-    s->draft_source = reinterpret_cast<DraftSource*>(base + o_source);
-    s->token_sink = reinterpret_cast<TokenSink*>(base + o_sink);
-    s->k_cache = reinterpret_cast<bf16*>(base + o_k);
-    s->v_cache = reinterpret_cast<bf16*>(base + o_v);
+    if (model->layered)
+      create_layered_session(*s);
+    else
+      create_uniform_session(*s);
     try {
       EI_CUDA(cudaStreamCreateWithFlags(&s->stream, cudaStreamNonBlocking));
       EI_CUDA(cudaMallocHost(reinterpret_cast<void**>(&s->host_tokens), kMaxRows * 4));
@@ -1387,60 +1336,146 @@ static void require_device(const ei_session& s) {
   if (device != s.model->device) throw std::invalid_argument("Session CUDA device changed");
 }
 
+// Row `row` of the session's logits to host memory as FP32 (waits for the stream).
+static void copy_logits_row(ei_session& s, size_t row, float* host) {
+  const size_t vocab = s.model->config.vocab_size;
+  if (s.layered) {
+    EI_CUDA(cudaMemcpyAsync(host, s.layered->logits + row * s.model->layered->vocab_stride, vocab * sizeof(float),
+                            cudaMemcpyDeviceToHost, s.stream));
+    synchronize(s);
+    return;
+  }
+  std::vector<uint16_t> bits(vocab);
+  EI_CUDA(cudaMemcpyAsync(bits.data(), s.logits + row * vocab, vocab * 2, cudaMemcpyDeviceToHost, s.stream));
+  synchronize(s);
+  for (size_t i = 0; i < vocab; ++i) {
+    const uint32_t wide = uint32_t(bits[i]) << 16;
+    std::memcpy(host + i, &wide, 4);
+  }
+}
+
+// Runs `rows` tokens at the current context length and commits them. The FP32 logits of the rows named in `want`
+// (ascending) go to host_logits; with `last_logits` the last row's logits end up in row 0 of the session's logits and
+// its greedy token in `targets`. Long portions go through the layers in segments of up to kPromptSegment rows, on the
+// model's prompt workspace, which this call holds until its stream has drained; others in steps of up to 16 rows.
+static void append_tokens(ei_session& s, const uint32_t* host_tokens, size_t rows, const uint32_t* want, size_t want_count,
+                          float* host_logits, bool last_logits) {
+  ei_model& m = *s.model;
+  const size_t vocab = m.config.vocab_size;
+  const bool wide = rows > size_t(kPromptMinRows) && m.prompt_ready;
+  std::unique_lock<std::mutex> workspace(m.prompt.mutex, std::defer_lock);
+  if (wide) workspace.lock();
+  s.prefill_target_row = wide ? 0 : (rows - 1) % kMaxRows;
+  size_t next = 0;  // wanted rows handed out so far
+  const auto wanted_before = [&](size_t end) {
+    size_t stop = next;
+    while (stop < want_count && want[stop] < end) ++stop;
+    return stop;
+  };
+  if (wide) {
+    auto& ws = m.prompt;
+    m.layered ? ensure_layered_workspace(m) : ensure_prompt_workspace(m);
+    for (size_t first = 0; first < rows; first += ws.rows) {
+      const size_t count = std::min(ws.rows, rows - first);
+      const bool head = last_logits && first + count >= rows;
+      synchronize(s);  // the pinned staging buffer is reused by every segment
+      std::memcpy(ws.host_tokens, host_tokens + first, count * 4);
+      EI_CUDA(cudaMemcpyAsync(ws.tokens, ws.host_tokens, count * 4, cudaMemcpyHostToDevice, s.stream));
+      if (m.layered)
+        enqueue_layered_segment(s, int(count));
+      else
+        enqueue_prompt_segment(s, int(count), head);
+      // The segment's normed rows stay in the workspace: the head runs over the wanted ones, 16 at a time.
+      const auto head_over = [&](const int32_t* places, int places_count, bool greedy) {
+        EI_CUDA(cudaMemcpyAsync(s.gather_index, places, places_count * sizeof(int32_t), cudaMemcpyHostToDevice, s.stream));
+        if (m.layered) {
+          enqueue_layered_head(s, s.gather_index, places_count, greedy);
+        } else {
+          tick(s);
+          launch_gather_rows<bf16>(ws.normed, s.gather_index, places_count, int(m.config.hidden_size), s.normed, s.stream);
+          enqueue_uniform_head(s, s.normed, places_count);
+        }
+      };
+      for (const size_t stop = wanted_before(first + count); next < stop;) {
+        int32_t places[kMaxRows];
+        const int group = int(std::min<size_t>(kMaxRows, stop - next));
+        for (int i = 0; i < group; ++i) places[i] = int32_t(want[next + i] - first);
+        head_over(places, group, false);
+        for (int i = 0; i < group; ++i) copy_logits_row(s, size_t(i), host_logits + (next + i) * vocab);
+        next += size_t(group);
+      }
+      if (m.layered && head) {
+        const int32_t last = int32_t(count - 1);
+        head_over(&last, 1, true);
+      }
+    }
+    return;
+  }
+  for (size_t first = 0; first < rows; first += kMaxRows) {
+    const int chunk = int(std::min<size_t>(kMaxRows, rows - first));
+    const size_t stop = wanted_before(first + chunk);
+    const bool last = last_logits && first + chunk >= rows;
+    synchronize(s);  // the pinned staging buffer is reused by every chunk
+    std::memcpy(s.host_tokens, host_tokens + first, size_t(chunk) * 4);
+    EI_CUDA(cudaMemcpyAsync(s.tokens, s.host_tokens, size_t(chunk) * 4, cudaMemcpyHostToDevice, s.stream));
+    const StepKind kind = last || stop > next ? kCommitAllWithHead : kCommitAllNoHead;
+    if (rows == 1)
+      submit_step(s, 1, kind);
+    else
+      enqueue_step(s, chunk, kind, nullptr);
+    for (; next < stop; ++next) copy_logits_row(s, want[next] - first, host_logits + next * vocab);
+    if (last && chunk > 1) {
+      if (s.layered)
+        EI_CUDA(cudaMemcpyAsync(s.layered->logits, s.layered->logits + size_t(chunk - 1) * m.layered->vocab_stride,
+                                vocab * sizeof(float), cudaMemcpyDeviceToDevice, s.stream));
+      else
+        EI_CUDA(cudaMemcpyAsync(s.logits, s.logits + size_t(chunk - 1) * vocab, vocab * 2, cudaMemcpyDeviceToDevice, s.stream));
+    }
+  }
+}
+
+static const void* logits_of(const ei_session& s) {
+  return s.layered ? static_cast<const void*>(s.layered->logits) : static_cast<const void*>(s.logits);
+}
+
+static void require_tokens(const ei_session& s, const uint32_t* host_tokens, size_t rows, size_t room) {
+  if (!host_tokens || !rows) throw std::invalid_argument("Host input requires tokens; decode takes one token");
+  if (rows > room) throw LengthError("Host input exceeds session capacity");
+  if (s.layered && s.layered->tap && rows > s.layered->tap_rows)
+    throw std::invalid_argument("More rows than the residual tap holds");
+  for (size_t i = 0; i < rows; ++i)
+    if (host_tokens[i] >= s.model->config.vocab_size) throw std::invalid_argument("Token exceeds vocabulary");
+}
+
 ei_status ei_session_prefill(ei_session* session, const uint32_t* host_tokens, size_t rows, const void** last_logits,
                              void* all_logits) {
   return guarded([&] {
     if (!session) throw std::invalid_argument("session is null");
     ei_session& s = *session;
     require_usable(s);
-    if (!host_tokens || !rows) throw std::invalid_argument("Host input requires tokens; decode takes one token");
-    if (rows > s.capacity) throw LengthError("Host input exceeds session capacity");
+    require_tokens(s, host_tokens, rows, s.capacity);
     require_device(s);
+    if (all_logits && s.layered) throw std::invalid_argument("A layered model hands out rows through ei_session_extend");
     const size_t vocab = s.model->config.vocab_size;
-    for (size_t i = 0; i < rows; ++i)
-      if (host_tokens[i] >= vocab) throw std::invalid_argument("Token exceeds vocabulary");
-    // Long prompts go through the layers in segments of up to kPromptSegment rows, on the model's prompt
-    // workspace, which this call holds until its stream has drained.
-    const bool wide = rows > size_t(kPromptMinRows) && !all_logits && s.model->prompt_ready;
-    std::unique_lock<std::mutex> workspace(s.model->prompt.mutex, std::defer_lock);
-    if (wide) workspace.lock();
     try {
       // A prefill replaces the history (the reference resizes the managed cache to `rows`).
       EI_CUDA(cudaMemsetAsync(s.control, 0, sizeof(Control), s.stream));
       s.context = 0;
       s.bound = 0;
       s.history_ready = false;
-      s.prefill_target_row = wide ? 0 : (rows - 1) % kMaxRows;
-      if (wide) {
-        ensure_prompt_workspace(*s.model);
-        auto& ws = s.model->prompt;
-        for (size_t first = 0; first < rows; first += ws.rows) {
-          const size_t count = std::min(ws.rows, rows - first);
-          synchronize(s);  // the pinned staging buffer is reused by every segment
-          std::memcpy(ws.host_tokens, host_tokens + first, count * 4);
-          EI_CUDA(cudaMemcpyAsync(ws.tokens, ws.host_tokens, count * 4, cudaMemcpyHostToDevice, s.stream));
-          enqueue_prompt_segment(s, int(count), first + count >= rows);
-        }
-      }
-      for (size_t first = wide ? rows : 0; first < rows; first += kMaxRows) {
-        const int chunk = int(std::min<size_t>(kMaxRows, rows - first));
-        const bool last = first + chunk >= rows;
-        synchronize(s);  // the pinned staging buffer is reused by every chunk
-        std::memcpy(s.host_tokens, host_tokens + first, size_t(chunk) * 4);
-        EI_CUDA(cudaMemcpyAsync(s.tokens, s.host_tokens, size_t(chunk) * 4, cudaMemcpyHostToDevice, s.stream));
-        if (all_logits) {
+      if (!all_logits) {
+        append_tokens(s, host_tokens, rows, nullptr, 0, nullptr, true);
+      } else {
+        s.prefill_target_row = (rows - 1) % kMaxRows;
+        for (size_t first = 0; first < rows; first += kMaxRows) {
+          const int chunk = int(std::min<size_t>(kMaxRows, rows - first));
+          synchronize(s);  // the pinned staging buffer is reused by every chunk
+          std::memcpy(s.host_tokens, host_tokens + first, size_t(chunk) * 4);
+          EI_CUDA(cudaMemcpyAsync(s.tokens, s.host_tokens, size_t(chunk) * 4, cudaMemcpyHostToDevice, s.stream));
           enqueue_step(s, chunk, kCommitAllWithHead, static_cast<bf16*>(all_logits) + first * vocab);
-          if (last)
-            EI_CUDA(cudaMemcpyAsync(s.logits, static_cast<bf16*>(all_logits) + (rows - 1) * vocab, vocab * 2,
-                                    cudaMemcpyDeviceToDevice, s.stream));
-        } else if (last) {
-          enqueue_step(s, chunk, kCommitAllWithHead, nullptr);
-          if (chunk > 1)
-            EI_CUDA(cudaMemcpyAsync(s.logits, s.logits + size_t(chunk - 1) * vocab, vocab * 2, cudaMemcpyDeviceToDevice,
-                                    s.stream));
-        } else {
-          enqueue_step(s, chunk, kCommitAllNoHead, nullptr);
         }
+        EI_CUDA(cudaMemcpyAsync(s.logits, static_cast<bf16*>(all_logits) + (rows - 1) * vocab, vocab * 2,
+                                cudaMemcpyDeviceToDevice, s.stream));
       }
       read_control(s);
       check_status(s);
@@ -1451,7 +1486,33 @@ ei_status ei_session_prefill(ei_session* session, const uint32_t* host_tokens, s
       throw;
     }
     s.history_ready = true;
-    if (last_logits) *last_logits = s.logits;
+    if (last_logits) *last_logits = logits_of(s);
+  });
+}
+
+ei_status ei_session_extend(ei_session* session, const uint32_t* host_tokens, size_t rows, const uint32_t* want,
+                            size_t want_count, float* host_logits) {
+  return guarded([&] {
+    if (!session) throw std::invalid_argument("session is null");
+    ei_session& s = *session;
+    require_usable(s);
+    require_tokens(s, host_tokens, rows, s.capacity - std::min(s.capacity, s.context));
+    if (want_count && (!want || !host_logits)) throw std::invalid_argument("Wanted rows need an output");
+    for (size_t i = 0; i < want_count; ++i)
+      if (want[i] >= rows || (i && want[i] <= want[i - 1]))
+        throw std::invalid_argument("Wanted rows must be ascending places of this portion");
+    require_device(s);
+    try {
+      append_tokens(s, host_tokens, rows, want, want_count, host_logits, false);
+      read_control(s);
+      check_status(s);
+    } catch (const CapacityRefusal&) {
+      throw;  // refused on the device before any write: the history stays
+    } catch (...) {
+      drain_failed(s);
+      throw;
+    }
+    s.history_ready = true;
   });
 }
 
@@ -1476,7 +1537,7 @@ ei_status ei_session_decode(ei_session* session, uint32_t token, const void** lo
       drain_failed(s);
       throw;
     }
-    if (logits) *logits = s.logits;
+    if (logits) *logits = logits_of(s);
   });
 }
 
@@ -1490,6 +1551,8 @@ ei_status ei_session_verify(ei_session* session, const uint32_t* host_tokens, si
       throw std::invalid_argument("Verify takes 1..16 tokens [pending, drafts...] and a result");
     if (!s.history_ready) throw std::logic_error("Verify requires successful prefill");
     if (s.context + rows > s.capacity) throw LengthError("Verify rows exceed session capacity");
+    if (s.layered && s.layered->tap && rows > s.layered->tap_rows)
+      throw std::invalid_argument("More rows than the residual tap holds");
     require_device(s);
     const size_t vocab = s.model->config.vocab_size;
     for (size_t i = 0; i < rows; ++i)
@@ -1507,7 +1570,7 @@ ei_status ei_session_verify(ei_session* session, const uint32_t* host_tokens, si
       throw;
     }
     *result = s.host_control->last;
-    if (logits) *logits = s.logits;
+    if (logits) *logits = logits_of(s);
   });
 }
 
@@ -1519,6 +1582,7 @@ ei_status ei_batch_create(ei_session* const* sessions, size_t count, ei_batch** 
     for (size_t j = 0; j < count; ++j) {
       ei_session* s = sessions[j];
       if (!s) throw std::invalid_argument("session is null");
+      if (s->layered) throw std::invalid_argument("Sessions of a layered model run one at a time");
       if (s->model != sessions[0]->model) throw std::invalid_argument("Batched sessions must share one model");
       if (s->capacity != sessions[0]->capacity)
         throw std::invalid_argument("Batched sessions must have the same context capacity");
@@ -1690,7 +1754,14 @@ ei_status ei_session_truncate(ei_session* session, size_t length) {
     ei_session& s = *session;
     require_usable(s);
     if (length > s.capacity) throw std::runtime_error("KVCache: Attempted to resize beyond max_seq_len");
+    if (s.layered && length) {
+      // The recurrent state already holds the rows before state_base; those behind it can still be dropped.
+      read_control(s);
+      if (length < size_t(s.host_control->state_base) || length > s.context)
+        throw std::invalid_argument("A recurrent model can only drop rows of its last step");
+    }
     const int32_t value = int32_t(length);
+    if (s.layered && !length) EI_CUDA(cudaMemcpyAsync(&s.control->state_base, &value, sizeof(value), cudaMemcpyHostToDevice, s.stream));
     EI_CUDA(cudaMemcpyAsync(&s.control->context, &value, sizeof(value), cudaMemcpyHostToDevice, s.stream));
     synchronize(s);
     s.context = length;
@@ -1751,6 +1822,7 @@ void* ei_session_stream(const ei_session* session) { return session ? session->s
 ei_status ei_session_read_kv(ei_session* session, size_t layer, void* host_k, void* host_v) {
   return guarded([&] {
     if (!session || !host_k || !host_v) throw std::invalid_argument("session or output is null");
+    if (session->layered) throw std::invalid_argument("A layered model's caches and state have no K / V row form");
     ei_session& s = *session;
     require_usable(s);
     const auto& c = s.model->config;
@@ -1766,6 +1838,7 @@ ei_status ei_session_write_kv(ei_session* session, size_t layer, size_t first, s
                               const void* v) {
   return guarded([&] {
     if (!session || !k || !v) throw std::invalid_argument("session or source is null");
+    if (session->layered) throw std::invalid_argument("A layered model's caches and state have no K / V row form");
     ei_session& s = *session;
     require_usable(s);
     require_device(s);
@@ -1783,6 +1856,7 @@ ei_status ei_session_write_kv(ei_session* session, size_t layer, size_t first, s
 ei_status ei_session_adopt_history(ei_session* session, size_t length, uint32_t pending) {
   return guarded([&] {
     if (!session) throw std::invalid_argument("session is null");
+    if (session->layered) throw std::invalid_argument("A layered model's caches and state have no K / V row form");
     ei_session& s = *session;
     require_usable(s);
     require_device(s);
@@ -1806,7 +1880,35 @@ ei_status ei_session_read_logits(ei_session* session, size_t rows, void* host_lo
     ei_session& s = *session;
     require_usable(s);
     synchronize(s);
-    EI_CUDA(cudaMemcpy(host_logits, s.logits, rows * s.model->config.vocab_size * 2, cudaMemcpyDeviceToHost));
+    const size_t vocab = s.model->config.vocab_size;
+    if (!s.layered) {
+      EI_CUDA(cudaMemcpy(host_logits, s.logits, rows * vocab * 2, cudaMemcpyDeviceToHost));
+      return;
+    }
+    std::vector<float> row(vocab);
+    for (size_t r = 0; r < rows; ++r) {
+      copy_logits_row(s, r, row.data());
+      for (size_t i = 0; i < vocab; ++i) static_cast<bf16*>(host_logits)[r * vocab + i] = __float2bfloat16_rn(row[i]);
+    }
+  });
+}
+
+ei_status ei_session_read_logits_f32(ei_session* session, size_t rows, float* host_logits) {
+  return guarded([&] {
+    if (!session || !host_logits || !rows || rows > kMaxRows) throw std::invalid_argument("session, rows or output is invalid");
+    require_usable(*session);
+    for (size_t r = 0; r < rows; ++r) copy_logits_row(*session, r, host_logits + r * session->model->config.vocab_size);
+  });
+}
+
+ei_status ei_session_tap_residual(ei_session* session, float* device_buffer, size_t rows) {
+  return guarded([&] {
+    if (!session || (device_buffer && !rows)) throw std::invalid_argument("session is null or the buffer has no rows");
+    if (!session->layered) throw std::invalid_argument("Only layered models have a residual tap");
+    require_usable(*session);
+    synchronize(*session);
+    session->layered->tap = device_buffer;
+    session->layered->tap_rows = device_buffer ? rows : 0;
   });
 }
 
@@ -1822,6 +1924,8 @@ ei_status ei_speculative_create(ei_session* target, ei_session* draft, size_t dr
       throw std::invalid_argument("Invalid draft capacity");
     if (target->model->device != draft->model->device)
       throw std::invalid_argument("Target and draft sessions must live on one device");
+    if (draft->layered)
+      throw std::invalid_argument("A recurrent model cannot draft: its state cannot go back several steps");
     if (target->model->config.vocab_size != draft->model->config.vocab_size)
       throw std::invalid_argument("Target and draft models must share a vocabulary");
     require_usable(*target);

@@ -20,23 +20,26 @@ __device__ __forceinline__ void take_better(float& best, int& index, float value
   }
 }
 
+__device__ __forceinline__ float logit_value(bf16 x) { return __bfloat162float(x); }
+__device__ __forceinline__ float logit_value(float x) { return x; }
+
 // kWide: partials laid out [row][parts] for any number of rows; otherwise [part][16] for at most 16 rows.
-template <bool kWide>
-__global__ void __launch_bounds__(kArgmaxThreads) argmax_partial_kernel(const bf16* logits, int vocab,
+template <bool kWide, typename T = bf16>
+__global__ void __launch_bounds__(kArgmaxThreads) argmax_partial_kernel(const T* logits, int vocab,
                                                                         size_t row_stride, float* best_value,
                                                                         int* best_index) {
   __shared__ float values[kArgmaxThreads / 32];
   __shared__ int indices[kArgmaxThreads / 32];
   grid_dependency_wait();
   const int row = blockIdx.y;
-  const bf16* x = logits + size_t(row) * row_stride;
+  const T* x = logits + size_t(row) * row_stride;
   // Contiguous slice per block; the slice boundaries are multiples of 8 elements.
   const int per_block = ((vocab + gridDim.x - 1) / gridDim.x + 7) & ~7;
   const int begin = min(vocab, int(blockIdx.x) * per_block), end = min(vocab, begin + per_block);
   float best = -INFINITY;
   int index = 0x7fffffff;
-  const bool aligned = (reinterpret_cast<uintptr_t>(x) & 15) == 0;
-  if (aligned) {
+  const bool packed = sizeof(T) == 2 && (reinterpret_cast<uintptr_t>(x) & 15) == 0;  // eight BF16 logits per load
+  if (packed) {
     for (int i = begin + threadIdx.x * 8; i < end; i += kArgmaxThreads * 8) {
       if (i + 8 <= end) {
         const uint4 v = *reinterpret_cast<const uint4*>(x + i);
@@ -51,7 +54,7 @@ __global__ void __launch_bounds__(kArgmaxThreads) argmax_partial_kernel(const bf
         }
       } else {
         for (int j = i; j < end; ++j) {
-          float a = __bfloat162float(x[j]);
+          float a = logit_value(x[j]);
           if (isnan(a)) a = -INFINITY;
           take_better(best, index, a, j);
         }
@@ -59,7 +62,7 @@ __global__ void __launch_bounds__(kArgmaxThreads) argmax_partial_kernel(const bf
     }
   } else {
     for (int i = begin + threadIdx.x; i < end; i += kArgmaxThreads) {
-      float a = __bfloat162float(x[i]);
+      float a = logit_value(x[i]);
       if (isnan(a)) a = -INFINITY;
       take_better(best, index, a, i);
     }
@@ -105,6 +108,7 @@ __device__ void accept_commit(const uint32_t* chosen, int rows, const uint32_t* 
         if (at >= 0 && at < sink->count) sink->tokens[at] = chosen[i];
       }
     }
+    if (!skipped) control->state_base = control->context;  // this step's rows are pending until the next one
     control->context += emitted;
     if (emitted) control->pending = chosen[emitted - 1];
     control->steps += 1;
@@ -206,6 +210,12 @@ int sample_partial_blocks(size_t vocabulary, int multiprocessors) {
 void launch_argmax_partials(const bf16* logits, size_t rows, size_t vocab, size_t row_stride, float* best_value,
                             int* best_index, int blocks, cudaStream_t stream, bool pdl) {
   launch(argmax_partial_kernel<false>, dim3(blocks, unsigned(rows)), dim3(kArgmaxThreads), 0, stream, pdl, logits,
+         int(vocab), row_stride, best_value, best_index);
+}
+
+void launch_argmax_partials_f32(const float* logits, size_t rows, size_t vocab, size_t row_stride, float* best_value,
+                                int* best_index, int blocks, cudaStream_t stream, bool pdl) {
+  launch(argmax_partial_kernel<false, float>, dim3(blocks, unsigned(rows)), dim3(kArgmaxThreads), 0, stream, pdl, logits,
          int(vocab), row_stride, best_value, best_index);
 }
 

@@ -35,6 +35,11 @@ enum GemmEpilogue : int {
   kEpiArgmax = 3     // kEpiStore + per-block running argmax of every row
 };
 
+enum GluKind : int {
+  kGluSilu = 0,     // silu(gate) * up with the reference operator's BF16 staging
+  kGluClamped = 1   // g = min(gate, limit), u = clamp(up, -limit, limit): g * sigmoid(1.702 g) * (u + 1), rounded once
+};
+
 struct GemmParams {
   const bf16* x;          // [M, K], row stride x_stride
   int x_stride;
@@ -49,6 +54,8 @@ struct GemmParams {
   bf16* out;              // [M, out_stride]
   int out_stride;
   int epilogue;
+  int glu;                // kEpiSiluPair: a GluKind, and the clamp of kGluClamped
+  float glu_limit;
   int ksplit;             // blocks along K (>= 1); > 1 requires kEpiPartial
   float* partial;         // [ksplit, M, N]
   float* best_value;      // kEpiArgmax: [grid, 16]
@@ -84,6 +91,17 @@ __device__ __forceinline__ float silu_multiply_value(float gate, float up) {
   const float activated = round_bf16(silu_value(gate));
   const float zero = __uint_as_float((__float_as_uint(activated) ^ __float_as_uint(up)) & 0x80000000u);
   return round_bf16(__fmaf_ieee_rn(activated, up, zero));
+}
+
+__device__ __forceinline__ float clamped_glu_value(float gate, float up, float limit) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+
+// The gated unit of a gate|up pair from its two FP32 sums.
+__device__ __forceinline__ float gated_pair_value(int glu, float limit, float gate, float up) {
+  return glu == kGluClamped ? clamped_glu_value(gate, up, limit)
+                            : silu_multiply_value(round_bf16(gate), round_bf16(up));
 }
 
 // Two int4 weights (bits 0-3 of each 16-bit half of `shifted`) -> two BF16 values round_bf16((w - z) * scale):
@@ -301,7 +319,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1) smallm_gemm_kernel(const Gemm
               up += __bfloat162float(p.bias[n]);
             }
             p.out[size_t(row) * p.out_stride + out_n] =
-                __float2bfloat16_rn(silu_multiply_value(round_bf16(gate), round_bf16(up)));
+                __float2bfloat16_rn(gated_pair_value(p.glu, p.glu_limit, gate, up));
           }
         } else if (p.epilogue == kEpiPartial) {
           p.partial[(size_t(slice) * p.M + row) * p.N + n] = sum;

@@ -61,22 +61,24 @@ class Session:
                 callback(int(token))
             return
         self._session.prefill(prompt)
-        token = runtime.greedy_token(self._session.read_logits(1)[0])
+        token = self._session.greedy_next()
         for produced in range(budget):
             callback(int(token))
             if token == eos or produced + 1 == budget:
                 break
             self._session.decode(token)
-            token = runtime.greedy_token(self._session.read_logits(1)[0])
+            token = self._session.greedy_next()
 
 
 class Model:
     """Prepared immutable weights; sessions share them."""
 
-    def __init__(self, config: Mapping, weights: Mapping, model_type: str = "qwen3_bf16", device: Optional[str] = None):
+    def __init__(self, config: Mapping, weights: Mapping, model_type: Optional[str] = "qwen3_bf16",
+                 device: Optional[str] = None):
+        """model_type None: chosen by the config (checkpoint.model_type_of)."""
         if device not in (None, "cuda"):
             raise ValueError("this library runs on CUDA devices only")
-        shape, tensors = checkpoint.admit(config, weights, model_type)
+        shape, tensors = checkpoint.admit(config, weights, model_type or checkpoint.model_type_of(config))
         self._model = runtime.Model(shape, tensors)
 
     @property

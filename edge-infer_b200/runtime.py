@@ -7,7 +7,7 @@ from __future__ import annotations
 
 import ctypes as C
 from dataclasses import dataclass, field
-from typing import Dict, List, Optional, Sequence, Tuple
+from typing import Dict, List, Optional, Sequence, Tuple, Union
 
 import numpy as np
 
@@ -44,6 +44,96 @@ class Shape:
                                self.quant_type, self.group_size, 1 if self.qk_norm else 0)
 
 
+MIXER_MIN_GRU, MIXER_PARALLEL = 1, 2
+MLP_NONE, MLP_CLAMPED_GLU = 0, 1
+
+
+@dataclass
+class Attention:
+    """Grouped-query softmax attention: sizes, rotation, score scale."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    rot_dims: int
+    rot_base: float
+    scale: float
+
+
+@dataclass
+class LinearAttention:
+    """Decayed linear attention: sizes and one decay per head."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: Sequence[float]
+
+
+@dataclass
+class Layer:
+    """One layer of a LayeredShape. Either `rnn_width` (gated recurrence) or both attentions (parallel mixer) are set;
+    `ff` None: no feed-forward."""
+    rnn_width: Optional[int] = None
+    attention: Optional[Attention] = None
+    linear: Optional[LinearAttention] = None
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+    ff: Optional[int] = None
+    limit: float = 0.0
+
+    def to_c(self) -> abi.LayerSpec:
+        spec = abi.LayerSpec()
+        if self.rnn_width is not None:
+            spec.mixer, spec.rnn_width = MIXER_MIN_GRU, self.rnn_width
+        else:
+            a, l = self.attention, self.linear
+            spec.mixer = MIXER_PARALLEL
+            spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.rot_dims = a.heads, a.kv_heads, a.dim, a.vdim, a.rot_dims
+            spec.rot_base, spec.scale = a.rot_base, a.scale
+            if len(l.decay) != l.heads:
+                raise ValueError("Linear attention needs one decay per head")
+            spec.lin_heads, spec.lin_dim, spec.lin_vdim = l.heads, l.dim, l.vdim
+            spec.decay = (C.c_double * l.heads)(*[float(d) for d in l.decay])
+            spec.left_scale, spec.right_scale = self.left_scale, self.right_scale
+        if self.ff is not None:
+            spec.mlp, spec.ff, spec.limit = MLP_CLAMPED_GLU, self.ff, self.limit
+        return spec
+
+
+@dataclass
+class LayeredShape:
+    """A decoder described layer by layer (ei_model_create_layered). `loop` = (start, stop, times): layers
+    start .. stop - 1 run `times` times in a row. `true32`: FP32 activations, caches and products."""
+    vocab_size: int
+    hidden_size: int
+    layers: List[Layer]
+    norm_eps: float = 1e-6
+    loop: Optional[Tuple[int, int, int]] = None
+    true32: bool = False
+    max_position_embeddings: int = 1 << 20
+    bos_token_id: int = 0
+    eos_token_id: int = 0xFFFFFFFF
+
+    @property
+    def n_layers(self) -> int:
+        return len(self.layers)
+
+    def layer_runs(self) -> List[int]:
+        """The layers in the order they run, a looped layer once per pass."""
+        order = list(range(len(self.layers)))
+        if self.loop is None:
+            return order
+        start, stop, times = self.loop
+        return order[:start] + order[start:stop] * times + order[stop:]
+
+    def to_c(self):
+        start, stop, times = self.loop or (0, 0, 0)
+        config = abi.LayeredConfig(self.vocab_size, self.hidden_size, len(self.layers), self.max_position_embeddings,
+                                   start, stop, times, self.norm_eps, self.bos_token_id, self.eos_token_id,
+                                   1 if self.true32 else 0)
+        return config, (abi.LayerSpec * len(self.layers))(*[layer.to_c() for layer in self.layers])
+
+
 def _pointer(data) -> int:
     if isinstance(data, np.ndarray):
         return data.ctypes.data
@@ -51,13 +141,13 @@ def _pointer(data) -> int:
 
 
 def _shape(data) -> Tuple[int, ...]:
-    return tuple(int(x) for x in data.shape)
+    return tuple(int(x) for x in data.shape) or (1,)  # a scalar travels as one element
 
 
 class Model:
     """Prepared weights on the current device. `tensors`: name -> list of (kind, array)."""
 
-    def __init__(self, shape: Shape, tensors: Dict[str, List[Tuple[int, object]]]):
+    def __init__(self, shape: Union[Shape, LayeredShape], tensors: Dict[str, List[Tuple[int, object]]]):
         lib = abi.load_library()
         entries = []
         keep = []
@@ -70,8 +160,12 @@ class Model:
                 keep.append(data)
         array = (abi.NamedTensor * len(entries))(*entries)
         handle = C.c_void_p()
-        config = shape.to_c()
-        abi.check(lib.ei_model_create(C.byref(config), array, len(entries), C.byref(handle)))
+        if isinstance(shape, LayeredShape):
+            config, layers = shape.to_c()
+            abi.check(lib.ei_model_create_layered(C.byref(config), layers, array, len(entries), C.byref(handle)))
+        else:
+            config = shape.to_c()
+            abi.check(lib.ei_model_create(C.byref(config), array, len(entries), C.byref(handle)))
         self.shape = shape
         self._handle = handle
         self._lib = lib
@@ -124,6 +218,15 @@ class Session:
         abi.check(self._lib.ei_session_prefill(self._handle, ids.ctypes.data_as(C.c_void_p), len(ids), C.byref(out),
                                                C.c_void_p(all_logits.data_ptr()) if all_logits is not None else None))
         return out.value
+
+    def extend(self, tokens: Sequence[int], want: Sequence[int] = ()) -> np.ndarray:
+        """Appends a portion of a sequence; returns the FP32 logits of its rows `want` (ascending), [len(want), vocab]."""
+        ids = np.ascontiguousarray(tokens, dtype=np.uint32)
+        rows = np.ascontiguousarray(want, dtype=np.uint32)
+        out = np.empty((len(rows), self.model.shape.vocab_size), dtype=np.float32)
+        abi.check(self._lib.ei_session_extend(self._handle, ids.ctypes.data_as(C.c_void_p), len(ids),
+                                              rows.ctypes.data_as(C.c_void_p), len(rows), out.ctypes.data_as(C.c_void_p)))
+        return out
 
     def decode(self, token: int) -> int:
         out = C.c_void_p()
@@ -193,6 +296,24 @@ class Session:
         abi.check(self._lib.ei_session_read_logits(self._handle, rows, out.ctypes.data_as(C.c_void_p)))
         return out
 
+    def read_logits_f32(self, rows: int = 1) -> np.ndarray:
+        """FP32 logits of the first `rows` rows of the session's logits buffer."""
+        out = np.empty((rows, self.model.shape.vocab_size), dtype=np.float32)
+        abi.check(self._lib.ei_session_read_logits_f32(self._handle, rows, out.ctypes.data_as(C.c_void_p)))
+        return out
+
+    def greedy_next(self) -> int:
+        """Greedy token of the last prefill's or decode's logits."""
+        return greedy_of(self.read_logits_f32(1)[0])
+
+    def tap_residual(self, buffer) -> None:
+        """Layered models: copy the residual stream after every layer run into `buffer`, a float32 device tensor
+        [layer runs, rows, width]; None ends it. The caller keeps the tensor alive."""
+        if buffer is None:
+            abi.check(self._lib.ei_session_tap_residual(self._handle, None, 0))
+        else:
+            abi.check(self._lib.ei_session_tap_residual(self._handle, C.c_void_p(buffer.data_ptr()), buffer.shape[1]))
+
     def launches_per_step(self, rows: int) -> int:
         return self._lib.ei_session_launches_per_step(self._handle, rows)
 
@@ -234,7 +355,11 @@ def bf16_to_float(bits: np.ndarray) -> np.ndarray:
 
 def greedy_token(row_bits: np.ndarray) -> int:
     """Greedy token of one BF16 logit row with the reference's rules: NaN as -inf, lowest index on ties."""
-    values = bf16_to_float(row_bits)
+    return greedy_of(bf16_to_float(row_bits))
+
+
+def greedy_of(values: np.ndarray) -> int:
+    """The same for an FP32 logit row."""
     values = np.where(np.isnan(values), -np.inf, values)
     return int(np.argmax(values))  # numpy returns the first maximum
 
@@ -245,7 +370,7 @@ def speculative_generate(session: Session, prompt: Sequence[int], drafts_for, ma
     runtime/src/speculative_decoder.cpp:227-316) with the draft model replaced by `drafts_for(position, k)`,
     which proposes k tokens for positions position+1.. . Returns (emitted tokens, accept lengths)."""
     session.prefill(prompt)
-    pending = greedy_token(session.read_logits(1)[0])
+    pending = session.greedy_next()
     emitted = [pending]
     accepts: List[int] = []
     capacity = session.context_capacity()

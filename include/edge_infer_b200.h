@@ -219,6 +219,41 @@ typedef struct ei_session ei_session;
  * device arena on the current device, resolves prepared linears and builds the RoPE table. Allocates. */
 ei_status ei_model_create(const ei_model_config* config, const ei_named_tensor* tensors, size_t count,
                           ei_model** out);
+/* A decoder described layer by layer (no counterpart in the reference, whose models repeat one block): every layer
+ * names its token mixer with its sizes and constants and its feed-forward, each sublayer stands between two norms, and
+ * a stretch of layers may run several times in a row. The session verbs below serve such a model as they serve the
+ * others; differences are noted there.
+ * Mixers: EI_MIXER_MIN_GRU - gated recurrence of `rnn_width` channels whose gates read only the current token.
+ * EI_MIXER_PARALLEL - grouped-query softmax attention (partial rotation, value norm, per-head sink, own score scale)
+ * beside decayed linear attention (SiLU on q, k, v; one decay per head; normed and gated output), outputs weighted by
+ * left_scale and right_scale. Feed-forward: EI_MLP_CLAMPED_GLU - g = min(gate, limit), u = clamp(up, +-limit),
+ * g * sigmoid(1.702 g) * (u + 1). Norm: tanh(alpha x) * weight + bias. Residual stream, norms, angles, scores, softmax
+ * weights, gates and recurrent state are FP32; with `true32` so are all activations, caches and products. */
+enum { EI_MIXER_MIN_GRU = 1, EI_MIXER_PARALLEL = 2 };
+enum { EI_MLP_NONE = 0, EI_MLP_CLAMPED_GLU = 1 };
+typedef struct ei_layer_spec {
+  int32_t mixer, mlp;
+  uint32_t rnn_width;
+  uint32_t heads, kv_heads, dim, vdim, rot_dims;
+  uint32_t lin_heads, lin_dim, lin_vdim;
+  uint32_t ff;
+  double rot_base, scale, left_scale, right_scale, limit;
+  const double* decay; /* [lin_heads] */
+} ei_layer_spec;
+typedef struct ei_layered_config {
+  uint64_t vocab_size, width, n_layers, max_position_embeddings;
+  uint64_t loop_start, loop_stop, loop_times; /* loop_times 0: no loop */
+  double norm_eps;
+  uint32_t bos_token_id, eos_token_id;
+  int32_t true32; /* 1: FP32 activations and caches, FP32 products */
+} ei_layered_config;
+/* Tensors (kind 0, BF16; a scalar has rank 1 and one element): embed [V,W], head [V,W], final.norm [W], with a loop
+ * loop.step [times,W]; per layer i, prefix l<i>.: norm1, norm1b, and with a feed-forward norm2, norm2b, mlp.gate,
+ * mlp.up [ff,W], mlp.down [W,ff]; every norm also <name>.b [W] and <name>.alpha [1]. mix.z, mix.x (and their .b),
+ * mix.g [R,W], mix.o [W,R] for the gated recurrence; mix.left.{q,k,v,o,sink} and mix.right.{q,k,v,g,o,norm} for the
+ * parallel mixer, heads side by side. Linear weights are [out, in]. Allocates. */
+ei_status ei_model_create_layered(const ei_layered_config* config, const ei_layer_spec* layers,
+                                  const ei_named_tensor* tensors, size_t count, ei_model** out);
 void ei_model_destroy(ei_model* model);
 ei_status ei_model_config_of(const ei_model* model, ei_model_config* out);
 /* Bytes of prepared weights one verify step streams (layers + lm_head), the roofline numerator. */
@@ -231,11 +266,18 @@ ei_status ei_session_create(ei_model* model, size_t capacity, int graph, ei_sess
 void ei_session_destroy(ei_session* session);
 /* ref: Qwen3Session<T>::prefill(host tokens) (qwen3.cpp:399-447): replaces the history. Returns a
  * borrowed device pointer to BF16 logits of the LAST row ([1, vocab]) in *last_logits, valid until the
- * session's next operation; all_logits (optional, device, BF16 [rows, vocab]) receives every row. */
+ * session's next operation; all_logits (optional, device, BF16 [rows, vocab]) receives every row. A layered model's
+ * logits are FP32, and it refuses all_logits (ei_session_extend hands out any row). */
 ei_status ei_session_prefill(ei_session* session, const uint32_t* host_tokens, size_t rows,
                              const void** last_logits, void* all_logits);
 /* ref: Qwen3Session<T>::decode(token) (qwen3.cpp:449-467): appends one token; logits [1, vocab]. */
 ei_status ei_session_decode(ei_session* session, uint32_t token, const void** logits);
+/* Appends a portion of a sequence to the history (an empty one after create or reset): `rows` tokens run at the
+ * current context length from the caches and state that earlier calls left, however the sequence was cut. For the
+ * `want_count` rows named in `want` (ascending places in this portion) the FP32 logits [want_count, vocab] are copied
+ * to host_logits. No counterpart in the reference, whose prefill takes a whole prompt. */
+ei_status ei_session_extend(ei_session* session, const uint32_t* host_tokens, size_t rows, const uint32_t* want,
+                            size_t want_count, float* host_logits);
 /* The verify step. ref: SpeculativeDecoder<T>::verify_greedy (runtime/src/speculative_decoder.cpp:200-224)
  * + verify_logits (:190-198) + Qwen3Session::prefill_eager. tokens = [pending, d1..dk], 1 <= rows <= 16.
  * One forward of `rows` tokens at the current context, greedy token per row, acceptance and KV
@@ -272,7 +314,9 @@ ei_status ei_session_verify_enqueue(ei_session* session, const uint32_t* device_
  * previous drain. */
 ei_status ei_session_drain(ei_session* session, ei_verify_result* last, uint64_t* emitted_total);
 /* ref: KVCache<T>::resize (runtime/include/inference.hpp:41, runtime/src/inference.cpp:116-121) used for
- * EOS truncation (speculative_decoder.cpp:302-304): logical length only; must not exceed what is stored. */
+ * EOS truncation (speculative_decoder.cpp:302-304): logical length only; must not exceed what is stored. A recurrent
+ * model can only drop rows of its last step of at most 16 rows (its state is kept as of that step's start): an earlier
+ * length, other than 0, is refused with EI_INVALID_ARGUMENT. */
 ei_status ei_session_truncate(ei_session* session, size_t length);
 /* Overrides the device-resident pending token (row 0 of the next enqueued step). */
 ei_status ei_session_set_pending(ei_session* session, uint32_t token);
@@ -298,6 +342,12 @@ ei_status ei_session_adopt_history(ei_session* session, size_t length, uint32_t 
 /* Copies the first `rows` rows of the session's borrowed logits (BF16 [rows, vocab]) to the host: row 0 after
  * prefill / decode, rows 0..rows-1 after a verify step. */
 ei_status ei_session_read_logits(ei_session* session, size_t rows, void* host_logits);
+/* The same rows as FP32 (a layered model's own precision; BF16 logits widened otherwise). */
+ei_status ei_session_read_logits_f32(ei_session* session, size_t rows, float* host_logits);
+/* Layered models: from now on every forward copies the residual stream after each layer run, ahead of what is added
+ * before the next one, to `device_buffer` [layer runs][rows][width] FP32, row r of the forward in row r. Null ends it.
+ * Inspection aid; forwards run outside captured graphs while it is set and must not have more than `rows` rows. */
+ei_status ei_session_tap_residual(ei_session* session, float* device_buffer, size_t rows);
 /* Kernels launched by this session's last step (the launches inside one captured graph). */
 size_t ei_session_launches_per_step(const ei_session* session, size_t rows);
 
