@@ -29,6 +29,8 @@ Prints ONE JSON line:
                lengths in [256, 8192] split evenly over the GPUs, k = 4, p = 0.3, three sessions stacked per
                forward (ei_batch_verify)
 `--impl reference` times the CPU implementation alone (rank 0 only), whole 36-layer-deep steps.
+`--design zofesun` runs another workload instead: prefill and decode throughput of the layered Zofesun design at three
+sizes with real models' layers (random weights), each beside the uniform BF16 decoder of the same width and depth.
 """
 from __future__ import annotations
 
@@ -551,6 +553,115 @@ def run_sessions_leg(package, torch, dist, rank: int, world: int, rounds: int, p
     }
 
 
+DESIGN_SIZES = {
+    # name: (width, layers, heads, kv heads, linear attention heads, feed-forward width)
+    "w1024": (1024, 28, 16, 8, 8, 3072),
+    "w2048": (2048, 28, 16, 8, 16, 6144),
+    "w4096": (4096, 12, 32, 8, 32, 12288),
+}
+DESIGN_PROMPT, DESIGN_CAPACITY = 2048, 4096
+
+
+def design_costs(shape) -> dict:
+    """Weight bytes of one forward, projection and attention FLOPs of a whole prompt, and the cache and state bytes one
+    decoded token at the prompt's length moves."""
+    T, H = DESIGN_PROMPT, shape.hidden_size
+    params = flops = cache = 0
+    if hasattr(shape, "layers"):
+        for i in shape.layer_runs():
+            layer = shape.layers[i]
+            if layer.rnn_width is not None:
+                params += 4 * H * layer.rnn_width
+                cache += 2 * 4 * layer.rnn_width
+            else:
+                a, l = layer.attention, layer.linear
+                params += H * (a.heads * (a.dim + a.vdim) + a.kv_heads * (a.dim + a.vdim) + l.heads * (2 * l.dim + 3 * l.vdim))
+                flops += a.heads * (a.dim + a.vdim) * T * T                       # causal: half of 2 T^2 per dimension
+                flops += l.heads * T * (4 * l.dim * l.vdim + 128 * (l.dim + l.vdim))
+                cache += 2 * a.kv_heads * (a.dim + a.vdim) * T + 2 * 4 * l.heads * l.dim * l.vdim
+            params += 3 * H * (layer.ff or 0)
+    else:
+        qkv = (shape.n_heads + 2 * shape.n_kv_heads) * shape.head_dim
+        params = shape.n_layers * H * (qkv + shape.n_heads * shape.head_dim + 3 * shape.intermediate_size)
+        flops = shape.n_layers * 2 * shape.n_heads * shape.head_dim * T * T
+        cache = shape.n_layers * 4 * shape.n_kv_heads * shape.head_dim * T
+    return {"layer_params": params, "prompt_flops": 2 * params * T + flops,
+            "decode_bytes": 2 * (params + H * shape.vocab_size) + cache}
+
+
+def run_design(args):
+    """Prefill of a 2048-token prompt (host tokens in, median of five calls, host clock around the public call, which
+    ends synchronised) and one-token decode steps chained on the device behind it (CUDA events, weights larger than L2)."""
+    import torch
+
+    torch.cuda.set_device(0)
+    package = entry.load_package()
+    syn = package.synthetic
+    peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
+    hbm, tensor = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops_sustained", 1400.0))
+    line = {"design": "zofesun", "prompt": DESIGN_PROMPT, "data": "synthetic", "dtype": "bf16 weights and activations, "
+            "fp32 residual, norms, scores, softmax weights and recurrent state", "peaks": {"hbm_gbs": hbm, "tflops": tensor},
+            "sizes": {}}
+    sampler = ClockSampler(0)
+    sampler.start()
+    for name in (args.design_sizes or ",".join(DESIGN_SIZES)).split(","):
+        width, layers, heads, kv_heads, lin_heads, ff = DESIGN_SIZES[name]
+        shapes = {"zofesun": syn.layered_decoder(width, layers, heads, kv_heads, lin_heads, ff),
+                  "uniform": package.Shape(vocab_size=151936, n_layers=layers, n_heads=heads, n_kv_heads=kv_heads,
+                                           hidden_size=width, intermediate_size=ff, max_position_embeddings=DESIGN_CAPACITY)}
+        line["sizes"][name] = {"layers": layers, "width": width, "ff": ff}
+        for family, shape in shapes.items():
+            make = syn.make_device_layered_model if family == "zofesun" else syn.make_device_model
+            model = package.Model(shape, make(shape, seed=0))
+            torch.cuda.empty_cache()
+            session = model.new_session(DESIGN_CAPACITY, graph=True)
+            prompt = syn.make_prompt(SEED, DESIGN_PROMPT, shape.vocab_size)
+            drafts = torch.zeros(1, dtype=torch.int32, device="cuda")
+            stream = torch.cuda.ExternalStream(session.stream())
+
+            def decode(steps):
+                start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                start.record(stream)
+                for _ in range(steps):
+                    session.verify_enqueue(drafts, 0, 1)
+                end.record(stream)
+                session.drain()
+                return start.elapsed_time(end) / steps
+
+            for _ in range(3):
+                session.prefill(prompt)
+            session.set_pending(1)
+            decode(5)
+            if args.profile_design:
+                if family == args.profile_design:
+                    torch.cuda.profiler.start()
+                    session.prefill(prompt)
+                    session.set_pending(1)
+                    session.verify([1])
+                    torch.cuda.synchronize()
+                    torch.cuda.profiler.stop()
+                continue
+            times = []
+            for _ in range(5):
+                begin = time.perf_counter()
+                session.prefill(prompt)
+                times.append((time.perf_counter() - begin) * 1e3)
+            session.set_pending(1)
+            decode(5)
+            steps = [decode(50) for _ in range(5)]
+            prefill_ms, decode_ms, cost = statistics.median(times), statistics.median(steps), design_costs(shape)
+            line["sizes"][name][family] = {
+                "layer_params": cost["layer_params"], "launches_per_step": session.launches_per_step(1),
+                "prefill_ms": prefill_ms, "prefill_tokens_per_s": DESIGN_PROMPT / prefill_ms * 1e3,
+                "prefill_tensor_frac": cost["prompt_flops"] / (prefill_ms * 1e-3) / 1e12 / tensor,
+                "decode_ms": decode_ms, "decode_tokens_per_s": 1e3 / decode_ms,
+                "decode_hbm_frac": cost["decode_bytes"] / (decode_ms * 1e-3) / 1e9 / hbm}
+            del session, model
+            torch.cuda.empty_cache()
+    line["clocks"] = sampler.stop()
+    print(json.dumps(line))
+
+
 def run_native(args, rank: int, world: int, local_rank: int):
     import torch
 
@@ -730,7 +841,7 @@ def run_native(args, rank: int, world: int, local_rank: int):
                               "ms_per_step_max": times[order[-1]] / args.steps},
             "tokens_per_step_measured": totals[median] / (args.steps * world),
             "clocks": clocks,
-            "e2e": {"value": e2e_value, "unit": UNIT, "h2d_bytes_per_step": rows * 4, "d2h_bytes_per_step": 96,
+            "e2e": {"value": e2e_value, "unit": UNIT, "h2d_bytes_per_step": rows * 4, "d2h_bytes_per_step": 104,
                     "ms_per_step": times[regions] / args.steps},
             "gpu_launches": int(launches * args.steps),
             "prompt_leg": prompt_leg(shape, sorted(prompt_ms)[1]),
@@ -817,13 +928,20 @@ def main():
                         help="run only the 64-session leg and bracket one forward of all sessions the same way")
     parser.add_argument("--profile-prompt", action="store_true",
                         help="bracket one prefill of the prompt the same way and stop after it")
+    parser.add_argument("--design", choices=["zofesun"],
+                        help="time this layered design beside the uniform decoder instead of the headline workload")
+    parser.add_argument("--design-sizes", default="", help="sizes of --design, with commas between them")
+    parser.add_argument("--profile-design", choices=["zofesun", "uniform"],
+                        help="with --design: bracket one prefill and one decode step of this family and stop")
     args = parser.parse_args()
     if args.steps is None:
         args.steps = 5 if args.impl == "reference" else 60
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
-    if args.impl == "reference":
+    if args.design:
+        run_design(args)
+    elif args.impl == "reference":
         run_reference(args, rank)
     else:
         run_native(args, rank, world, local_rank)

@@ -163,7 +163,10 @@ def layered_tensor_shapes(shape: LayeredShape) -> Dict[str, Tuple[int, ...]]:
 
 def _admit_layered(shape: LayeredShape, weights: Mapping):
     expected = layered_tensor_shapes(shape)
-    missing, extra = sorted(set(expected) - set(weights)), sorted(set(weights) - set(expected))
+    # Norms around a feed-forward that a layer does not have, and the vectors of a loop that is not run, are passed over.
+    spare = {f"l{i}.{norm}{part}" for i, layer in enumerate(shape.layers) if layer.ff is None
+             for norm in ("norm2", "norm2b") for part in ("", ".b", ".alpha")} | {"loop.step"}
+    missing, extra = sorted(set(expected) - set(weights)), sorted(set(weights) - set(expected) - spare)
     if missing:
         raise ValueError("Decoder checkpoint lacks " + missing[0])
     if extra:

@@ -282,6 +282,8 @@ class Session:
 
     def read_kv(self, layer: int) -> Tuple[np.ndarray, np.ndarray]:
         shape = self.model.shape
+        if isinstance(shape, LayeredShape):
+            raise ValueError("A layered model's caches and state have no K / V row form")
         width = shape.n_kv_heads * shape.head_dim
         n = self.context_size()
         k = np.empty((n, width), dtype=np.uint16)

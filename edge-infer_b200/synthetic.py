@@ -15,7 +15,7 @@ from typing import Dict, List, Tuple
 
 import numpy as np
 
-from .runtime import DENSE, QWEIGHT, SCALES, ZEROS, Shape
+from .runtime import (DENSE, QWEIGHT, SCALES, ZEROS, Attention, Layer, LayeredShape, LinearAttention, Shape)
 
 Tensors = Dict[str, List[Tuple[int, np.ndarray]]]
 
@@ -167,6 +167,41 @@ def make_device_model(shape: Shape, seed: int = 0) -> Dict[str, List[Tuple[int, 
                 b.normal_(0.0, 0.02, generator=gen)
                 tensors[f"layers.{i}.self_attn.{proj}_proj.bias"] = [(DENSE, b)]
     return tensors
+
+
+def make_device_layered_model(shape: LayeredShape, seed: int = 0) -> Dict[str, List[Tuple[int, object]]]:
+    """Random weights of a layered decoder in device memory: linears N(0, 1 / sqrt(inputs)), norm weights 1, alphas 0.5,
+    biases and sinks 0."""
+    import torch
+
+    from .checkpoint import layered_tensor_shapes
+    gen = torch.Generator(device="cuda")
+    gen.manual_seed(seed)
+    tensors: Dict[str, List[Tuple[int, object]]] = {}
+    for name, dims in layered_tensor_shapes(shape).items():
+        t = torch.empty(dims, dtype=torch.bfloat16, device="cuda")
+        if len(dims) == 2:
+            t.normal_(0.0, 1.0 if name == "embed" else dims[1] ** -0.5, generator=gen)
+        elif name.endswith(".alpha"):
+            t.fill_(0.5)
+        elif name.endswith((".b", ".sink")):
+            t.zero_()
+        else:
+            t.fill_(1.0)
+        tensors[name] = [(DENSE, t)]
+    return tensors
+
+
+def layered_decoder(width: int, n_layers: int, heads: int, kv_heads: int, lin_heads: int, ff: int, vocab: int = 151936,
+                    head_dim: int = 128, **kw) -> LayeredShape:
+    """A layered decoder with a real model's sizes: the parallel mixer and the gated recurrence take turns."""
+    attention = Attention(heads=heads, kv_heads=kv_heads, dim=head_dim, vdim=head_dim, rot_dims=head_dim // 2, rot_base=1e6,
+                          scale=head_dim ** -0.5)
+    linear = LinearAttention(heads=lin_heads, dim=head_dim, vdim=head_dim,
+                             decay=[1.0 - 2.0 ** (-1.0 - 7.0 * h / max(1, lin_heads - 1)) for h in range(lin_heads)])
+    layers = [Layer(attention=attention, linear=linear, ff=ff, limit=7.0) if i % 2 == 0 else
+              Layer(rnn_width=width, ff=ff, limit=7.0) for i in range(n_layers)]
+    return LayeredShape(vocab_size=vocab, hidden_size=width, layers=layers, **kw)
 
 
 def make_prompt(seed: int, length: int, vocab: int) -> np.ndarray:
