@@ -477,6 +477,7 @@ MinGruParams min_gru_params(const ei_session& s, const LayeredModel::Layer& l, c
   g.ring_gate = r.ring_gate;
   g.ring_candidate = r.ring_candidate;
   g.state = r.state;
+  g.stretches = s.model->layered->stretches;
   g.control = s.control;
   g.capacity = int(s.capacity);
   g.out = b.mixed;
@@ -636,6 +637,7 @@ void create_layered_model(ei_model& model, const ei_layered_config& c, const ei_
     m.max_gate_up = std::max(m.max_gate_up, l.gate_up.out);
     m.max_ff = std::max(m.max_ff, l.ff_pad);
     m.max_linear = std::max(m.max_linear, l.linear_width);
+    m.max_rnn = std::max(m.max_rnn, l.width_pad);
     if (l.spec.mixer == EI_MIXER_PARALLEL) {
       m.max_chunk_state = std::max(m.max_chunk_state, size_t(l.linear_width) * l.lin_dim_pad);
       model.prompt_ready = model.prompt_ready && sized_attention_ok(l.dim_pad, l.vdim_pad) &&
@@ -735,6 +737,7 @@ void ensure_layered_workspace(ei_model& model) {
   take(m.residual, rows * m.residual_stride * sizeof(float));
   take(m.linear_out, rows * m.max_linear * sizeof(float));
   take(m.chunk_states, chunks * m.max_chunk_state * sizeof(float));
+  take(m.stretches, ((rows + kMinGruStretch - 1) / kMinGruStretch + 1) * 2 * m.max_rnn * sizeof(float));
   take(ws.normed, rows * m.normed_stride * 2);
   take(ws.qkv, rows * m.max_fused * 2);
   take(ws.attention, rows * m.max_mixed * 2);
@@ -792,6 +795,7 @@ void enqueue_layered_segment(ei_session& s, int rows) {
     const LayeredSession::Run& r = L.runs[run];
     run_prompt_linear_store(s, l.in, ws.normed, rows, ws.qkv, pdl);
     if (l.spec.mixer == EI_MIXER_MIN_GRU) {
+      tick(s);
       tick(s);
       launch_min_gru_prompt(min_gru_params<bf16>(s, l, r, b), s.stream, pdl);
     } else {

@@ -15,6 +15,7 @@ namespace ei {
 
 constexpr int kPendingRows = 16;     // rows a step may leave pending behind the recurrent state
 constexpr int kRingRows = 32;        // ring of a recurrence's inputs: pending rows and the rows of the step
+constexpr int kMinGruStretch = 32;   // rows of a prompt stretch of the gated recurrence
 constexpr int kLightningChunk = 128; // tokens of a prompt chunk of the decayed linear attention
 constexpr int kMaxHeadDim = 512;
 
@@ -154,12 +155,13 @@ struct MinGruParams {
   float* state;             // [width_pad]: as of Control::state_base
   const Control* control;
   int capacity;
+  float* stretches;         // prompt form: [stretches + 1][2 * width_pad]
   void* out;                // [rows, out_stride]; columns beyond width_pad are cleared
   int out_stride;
 };
 template <typename T>
 void launch_min_gru_step(const MinGruParams& p, cudaStream_t stream, bool pdl);
-void launch_min_gru_prompt(const MinGruParams& p, cudaStream_t stream, bool pdl);
+void launch_min_gru_prompt(const MinGruParams& p, cudaStream_t stream, bool pdl);  // two launches
 
 // out[rows, ff] = gated unit of the pair [rows, 2 ff] (clamped).
 template <typename T>
@@ -210,10 +212,10 @@ struct LayeredModel {
   const bf16* loop_step = nullptr;   // [times, residual_stride]
   DynamicTanh final_norm;
   PreparedLinear head;
-  int max_fused = 0, max_mixed = 0, max_gate_up = 0, max_ff = 0, max_linear = 0;  // widest rows
+  int max_fused = 0, max_mixed = 0, max_gate_up = 0, max_ff = 0, max_linear = 0, max_rnn = 0;  // widest rows
   size_t max_chunk_state = 0;        // floats of one chunk's state
   // prompt workspace (in ei_model::prompt's arena)
-  float *residual = nullptr, *linear_out = nullptr, *chunk_states = nullptr;
+  float *residual = nullptr, *linear_out = nullptr, *chunk_states = nullptr, *stretches = nullptr;
 };
 
 struct LayeredSession {

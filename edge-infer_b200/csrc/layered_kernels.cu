@@ -132,7 +132,16 @@ __global__ void __launch_bounds__(128) mixer_prepare_kernel(const MixerPreparePa
     T* to = key ? static_cast<T*>(p.k_cache) + (size_t(position) * p.kv_heads + (unit - p.heads)) * p.dim_pad : x;
     const int half = p.rot_dims >> 1;
     const float2* turn = p.rotation + size_t(position) * half;
-    if (half & 1) {
+    if (half % 4 == 0) {
+      for (int i = lane * 4; i < half; i += 128) {
+        const float4 u = load_quad(x + i), v = load_quad(x + i + half);
+        const float4 t01 = *reinterpret_cast<const float4*>(turn + i), t23 = *reinterpret_cast<const float4*>(turn + i + 2);
+        store_quad(to + i, make_float4(u.x * t01.x - v.x * t01.y, u.y * t01.z - v.y * t01.w, u.z * t23.x - v.z * t23.y,
+                                       u.w * t23.z - v.w * t23.w));
+        store_quad(to + i + half, make_float4(v.x * t01.x + u.x * t01.y, v.y * t01.z + u.y * t01.w, v.z * t23.x + u.z * t23.y,
+                                              v.w * t23.z + u.w * t23.w));
+      }
+    } else if (half & 1) {
       for (int i = lane; i < half; i += 32) {
         const float u = value_of(x[i]), v = value_of(x[i + half]);
         const float2 t = turn[i];
@@ -160,14 +169,14 @@ __global__ void __launch_bounds__(128) mixer_prepare_kernel(const MixerPreparePa
     x += size_t(unit) * p.vdim_pad;
     T* to = static_cast<T*>(p.v_cache) + (size_t(position) * p.kv_heads + unit) * p.vdim_pad;
     float sum = 0.0f;
-    for (int i = lane * 2; i < p.vdim_pad; i += 64) {
-      const float2 v = load_pair(x + i);
-      sum = fmaf(v.x, v.x, fmaf(v.y, v.y, sum));
+    for (int i = lane * 4; i < p.vdim_pad; i += 128) {
+      const float4 v = load_quad(x + i);
+      sum = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, sum))));
     }
     const float root = sqrtf(warp_sum(sum) / float(p.vdim) + p.eps);
-    for (int i = lane * 2; i < p.vdim_pad; i += 64) {
-      const float2 v = load_pair(x + i);
-      store_pair(to + i, v.x / root, v.y / root);
+    for (int i = lane * 4; i < p.vdim_pad; i += 128) {
+      const float4 v = load_quad(x + i);
+      store_quad(to + i, make_float4(v.x / root, v.y / root, v.z / root, v.w / root));
     }
     return;
   }
@@ -179,12 +188,11 @@ __global__ void __launch_bounds__(128) mixer_prepare_kernel(const MixerPreparePa
   T* ring = nullptr;
   if (p.ring_k && kind > 0)
     ring = static_cast<T*>(kind == 1 ? p.ring_k : p.ring_v) + (size_t(position & (kRingRows - 1)) * p.lin_heads + head) * pad;
-  for (int i = lane * 2; i < pad; i += 64) {
-    float2 v = load_pair(x + i);
-    v.x = silu_exact(v.x);
-    v.y = silu_exact(v.y);
-    store_pair(x + i, v.x, v.y);
-    if (ring) store_pair(ring + i, v.x, v.y);
+  for (int i = lane * 4; i < pad; i += 128) {
+    float4 v = load_quad(x + i);
+    v = make_float4(silu_exact(v.x), silu_exact(v.y), silu_exact(v.z), silu_exact(v.w));
+    store_quad(x + i, v);
+    if (ring) store_quad(ring + i, v);
   }
 }
 
@@ -198,13 +206,17 @@ __device__ __forceinline__ float block_total(float v, float* shared) {
 }
 
 // Blocks [0, rows * heads) merge one (row, head) of the split attention (when asked to); the last `rows` blocks finish
-// one row of the linear attention: RMS norm over all heads, weight, sigmoid gate, scale.
-constexpr int kFinishThreads = 128;
+// one row of the linear attention: RMS norm over all heads, weight, sigmoid gate, scale. At most 64 splits.
+constexpr int kFinishWarps = 8;
+constexpr int kFinishThreads = kFinishWarps * 32;
+constexpr int kFinishHeld = 4;  // quads of a row a thread keeps between the two passes over it
 template <typename T>
 __global__ void __launch_bounds__(kFinishThreads) mixer_finish_kernel(const MixerFinishParams p) {
   __shared__ float weights[64];
-  __shared__ float shared[8];
+  __shared__ float shared[2 * kFinishWarps];
+  __shared__ float4 parts[kFinishWarps][32];
   const int merges = p.merge ? p.rows * p.attention.heads : 0;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   if (int(blockIdx.x) < merges) {
     const SizedAttentionParams& a = p.attention;
     const int offset = *a.device_offset;
@@ -214,58 +226,107 @@ __global__ void __launch_bounds__(kFinishThreads) mixer_finish_kernel(const Mixe
     const int slot = blockIdx.x, row = slot / a.heads, head = slot - row * a.heads;
     const int slots = p.rows * a.heads, pitch = a.vdim_pad + 4;
     const int splits = min(64, (offset + p.rows + a.chunk - 1) / a.chunk);
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const float* base = a.scratch + size_t(slot) * pitch;
+    const size_t step = size_t(slots) * pitch;
+    // A warp's splits are w, w + 8, ...; lane l owns columns 4 l .. 4 l + 3 of each 128. The first 128 columns are
+    // requested together with the maxima and sums.
+    float4 values[64 / kFinishWarps];
+    auto request = [&](int column) {
+#pragma unroll
+      for (int i = 0; i < 64 / kFinishWarps; ++i) {
+        const int s = warp + kFinishWarps * i;
+        values[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (s < splits && column < a.vdim_pad) values[i] = *reinterpret_cast<const float4*>(base + s * step + column);
+      }
+    };
+    request(lane * 4);
     float m = -INFINITY, l = 0.0f;
     if (int(threadIdx.x) < splits) {
-      const float* src = a.scratch + (size_t(threadIdx.x) * slots + slot) * pitch + a.vdim_pad;
-      m = src[0];
-      l = src[1];
+      const float2 ml = *reinterpret_cast<const float2*>(base + threadIdx.x * step + a.vdim_pad);
+      m = ml.x;
+      l = ml.y;
     }
     const float sink = a.sink ? a.sink[head] : -INFINITY;
-    float top = warp_max(m);
-    if (lane == 0) shared[warp] = top;
+    if (warp < 2) {
+      const float top = warp_max(m);
+      if (lane == 0) shared[warp] = top;
+    }
     __syncthreads();
-    top = fmaxf(fmaxf(fmaxf(shared[0], shared[1]), fmaxf(shared[2], shared[3])), sink);
-    const float weight = m == -INFINITY ? 0.0f : expf(m - top);
-    if (threadIdx.x < 64) weights[threadIdx.x] = weight;
-    const float part = warp_sum(l * weight);
-    if (lane == 0) shared[4 + warp] = part;
+    const float top = fmaxf(fmaxf(shared[0], shared[1]), sink);
+    if (warp < 2) {
+      const float weight = m == -INFINITY ? 0.0f : expf(m - top);
+      weights[threadIdx.x] = weight;
+      const float part = warp_sum(l * weight);
+      if (lane == 0) shared[2 + warp] = part;
+    }
     __syncthreads();
-    const float denominator = ((shared[4] + shared[5]) + (shared[6] + shared[7])) + (a.sink ? expf(sink - top) : 0.0f);
+    const float denominator = shared[2] + shared[3] + (a.sink ? expf(sink - top) : 0.0f);
     const float factor = denominator > 0.0f ? a.out_scale / denominator : 0.0f;
     T* out = static_cast<T*>(a.out) + size_t(row) * a.out_stride + size_t(head) * a.vdim_pad;
-    for (int i = threadIdx.x; i < a.vdim_pad; i += kFinishThreads) {
-      const float* src = a.scratch + size_t(slot) * pitch + i;
-      float sum = 0.0f;
-#pragma unroll 8
-      for (int s = 0; s < splits; ++s) sum = fmaf(src[size_t(s) * slots * pitch], weights[s], sum);
-      store_value(out + i, sum * factor);
+    for (int first = 0; first < a.vdim_pad; first += 128) {
+      const int column = first + lane * 4;
+      if (first) request(column);
+      float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+      for (int i = 0; i < 64 / kFinishWarps; ++i) {
+        const int s = warp + kFinishWarps * i;
+        const float w = s < splits ? weights[s] : 0.0f;
+        sum = make_float4(fmaf(values[i].x, w, sum.x), fmaf(values[i].y, w, sum.y), fmaf(values[i].z, w, sum.z),
+                          fmaf(values[i].w, w, sum.w));
+      }
+      parts[warp][lane] = sum;
+      __syncthreads();
+      if (warp == 0 && column < a.vdim_pad) {
+        for (int w = 1; w < kFinishWarps; ++w) sum = add(sum, parts[w][lane]);
+        store_quad(out + column, make_float4(sum.x * factor, sum.y * factor, sum.z * factor, sum.w * factor));
+      }
+      __syncthreads();
     }
     return;
   }
   const int row = int(blockIdx.x) - merges;
+  const int width = p.lin_heads * p.lin_vdim_pad;
+  const T* gate = static_cast<const T*>(p.gate) + size_t(row) * p.gate_stride;
+  const float* x = p.lin_out + size_t(row) * width;
+  T* out = static_cast<T*>(p.out) + size_t(row) * p.out_stride + p.lin_offset;
   grid_dependency_wait();
   grid_launch_dependents();
-  const int width = p.lin_heads * p.lin_vdim_pad;
-  const float* x = p.lin_out + size_t(row) * width;
-  const T* gate = static_cast<const T*>(p.gate) + size_t(row) * p.gate_stride;
-  T* out = static_cast<T*>(p.out) + size_t(row) * p.out_stride + p.lin_offset;
+  float4 held[kFinishHeld], gates[kFinishHeld];
   float sum = 0.0f;
-  for (int i = threadIdx.x * 4; i < width; i += kFinishThreads * 4) {
+#pragma unroll
+  for (int j = 0; j < kFinishHeld; ++j) {
+    const int i = (threadIdx.x + j * kFinishThreads) * 4;
+    held[j] = gates[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (i < width) {
+      held[j] = *reinterpret_cast<const float4*>(x + i);
+      gates[j] = load_quad(gate + i);
+    }
+    sum = fmaf(held[j].x, held[j].x, fmaf(held[j].y, held[j].y, fmaf(held[j].z, held[j].z, fmaf(held[j].w, held[j].w, sum))));
+  }
+  for (int i = (threadIdx.x + kFinishHeld * kFinishThreads) * 4; i < width; i += kFinishThreads * 4) {
     const float4 v = *reinterpret_cast<const float4*>(x + i);
     sum = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, sum))));
   }
   const float mean = block_total(sum, shared) / (float(p.lin_heads) * float(p.lin_vdim));
   const float factor = p.lin_scale / sqrtf(mean + p.eps);
   const int end = p.out_stride - p.lin_offset;  // the columns behind the heads pad the projection's input
-  for (int i = threadIdx.x * 4; i < end; i += kFinishThreads * 4) {
+  auto finish = [&](int i, float4 v, float4 z) {
     float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     if (i < width) {
-      const float4 v = *reinterpret_cast<const float4*>(x + i), w = load_quad(p.norm + i), z = load_quad(gate + i);
+      const float4 w = load_quad(p.norm + i);
       y = make_float4(v.x * factor * w.x * sigmoid_value(z.x), v.y * factor * w.y * sigmoid_value(z.y),
                       v.z * factor * w.z * sigmoid_value(z.z), v.w * factor * w.w * sigmoid_value(z.w));
     }
     store_quad(out + i, y);
+  };
+#pragma unroll
+  for (int j = 0; j < kFinishHeld; ++j) {
+    const int i = (threadIdx.x + j * kFinishThreads) * 4;
+    if (i < end) finish(i, held[j], gates[j]);
+  }
+  for (int i = (threadIdx.x + kFinishHeld * kFinishThreads) * 4; i < end; i += kFinishThreads * 4) {
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    finish(i, i < width ? *reinterpret_cast<const float4*>(x + i) : zero, i < width ? load_quad(gate + i) : zero);
   }
 }
 
@@ -307,76 +368,88 @@ __global__ void __launch_bounds__(128) min_gru_step_kernel(const MinGruParams p)
   }
 }
 
-// A prompt segment: a block owns 32 channels, its 1024 threads 64 time stretches of 16 channel pairs. Every stretch is
-// reduced to (product of 1 - z, value from zero), the stretches are chained, and a second pass emits the rows.
-constexpr int kStretches = 64;
-__global__ void __launch_bounds__(1024) min_gru_prompt_kernel(const MinGruParams p) {
-  __shared__ float keep[kStretches][32], value[kStretches][32];
+// A prompt segment runs in stretches of 32 rows, two channels per thread. The first kernel reduces every stretch to
+// (product of 1 - z, value from zero) and leaves the state with its pending rows folded in behind the stretches; the
+// second chains the stretches before its own from that state and emits the rows, the last stretch writes the new state.
+// Exponential and quotient are the fast forms (a few units in the last place of FP32).
+constexpr int kStretch = kMinGruStretch;
+constexpr int kGruThreads = 64;
+__device__ __forceinline__ float quick_sigmoid(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+__device__ __forceinline__ float quick_candidate(float u) { return u >= 0.0f ? u + 0.5f : quick_sigmoid(u); }
+
+template <bool kEmit>
+__global__ void __launch_bounds__(kGruThreads) min_gru_prompt_kernel(const MinGruParams p) {
   const int context = p.control->context, base = p.control->state_base;
   const bool runs = context >= 0 && context + p.rows <= p.capacity;
   grid_dependency_wait();
   grid_launch_dependents();
-  if (!runs) return;
-  const int pair = threadIdx.x & 15, stretch = threadIdx.x >> 4;
-  const int channel = blockIdx.x * 32 + pair * 2;
-  const int length = (p.rows + kStretches - 1) / kStretches;
-  const int begin = min(p.rows, stretch * length), end = min(p.rows, begin + length);
-  const bool live = channel < p.width_pad;
-  const bf16* x = static_cast<const bf16*>(p.fused) + channel;
-  float a0 = 1.0f, a1 = 1.0f, s0 = 0.0f, s1 = 0.0f;
-  if (live) {
-#pragma unroll 4
-    for (int t = begin; t < end; ++t) {
-      const float2 zr = load_pair(x + size_t(t) * p.stride), u = load_pair(x + size_t(t) * p.stride + p.width_pad);
-      const float z0 = sigmoid_value(zr.x), z1 = sigmoid_value(zr.y);
-      s0 = (1.0f - z0) * s0 + z0 * min_gru_candidate(u.x);
-      s1 = (1.0f - z1) * s1 + z1 * min_gru_candidate(u.y);
-      a0 *= 1.0f - z0;
-      a1 *= 1.0f - z1;
-    }
-  }
-  keep[stretch][pair * 2] = a0;
-  keep[stretch][pair * 2 + 1] = a1;
-  value[stretch][pair * 2] = s0;
-  value[stretch][pair * 2 + 1] = s1;
-  __syncthreads();
-  if (threadIdx.x < 32) {
-    const int own = blockIdx.x * 32 + threadIdx.x;
-    if (own < p.width_pad) {
-      float s = base > 0 ? p.state[own] : 0.0f;
-      const int pending = min(kPendingRows, max(0, context - base));
-      for (int i = 0; i < pending; ++i) {
-        const size_t at = size_t((base + i) & (kRingRows - 1)) * p.width_pad + own;
-        const float z = p.ring_gate[at];
-        s = (1.0f - z) * s + z * p.ring_candidate[at];
-      }
-      for (int i = 0; i < kStretches; ++i) {
-        const float next = keep[i][threadIdx.x] * s + value[i][threadIdx.x];
-        value[i][threadIdx.x] = s;  // the state ahead of the stretch
-        s = next;
-      }
-      p.state[own] = s;
-    }
-  }
-  __syncthreads();
-  if (channel >= p.out_stride) return;
+  const int channel = (blockIdx.x * kGruThreads + threadIdx.x) * 2;
+  if (!runs || channel >= p.out_stride) return;
+  const int stretch = blockIdx.y, begin = stretch * kStretch, end = min(p.rows, begin + kStretch);
   bf16* out = static_cast<bf16*>(p.out) + channel;
-  s0 = value[stretch][pair * 2];
-  s1 = value[stretch][pair * 2 + 1];
-#pragma unroll 4
-  for (int t = begin; t < end; ++t) {
-    float y0 = 0.0f, y1 = 0.0f;
-    if (live) {
-      const bf16* row = x + size_t(t) * p.stride;
-      const float2 zr = load_pair(row), u = load_pair(row + p.width_pad), g = load_pair(row + 2 * p.width_pad);
-      const float z0 = sigmoid_value(zr.x), z1 = sigmoid_value(zr.y);
-      s0 = (1.0f - z0) * s0 + z0 * min_gru_candidate(u.x);
-      s1 = (1.0f - z1) * s1 + z1 * min_gru_candidate(u.y);
-      y0 = s0 * silu_exact(g.x);
-      y1 = s1 * silu_exact(g.y);
-    }
-    store_pair(out + size_t(t) * p.out_stride, y0, y1);
+  if (channel >= p.width_pad) {
+    if (kEmit)
+      for (int t = begin; t < end; ++t) store_pair(out + size_t(t) * p.out_stride, 0.0f, 0.0f);
+    return;
   }
+  float s0 = 0.0f, s1 = 0.0f, a0 = 1.0f, a1 = 1.0f;
+  float4* stretches = reinterpret_cast<float4*>(p.stretches) + channel / 2;
+  float4* folded = stretches + size_t(gridDim.y) * (p.width_pad / 2);
+  if (!kEmit && stretch == 0) {
+    float2 s = base > 0 ? load_pair(p.state + channel) : make_float2(0.0f, 0.0f);
+    const int pending = min(kPendingRows, max(0, context - base));
+    for (int i = 0; i < pending; ++i) {
+      const size_t at = size_t((base + i) & (kRingRows - 1)) * p.width_pad + channel;
+      const float2 z = load_pair(p.ring_gate + at), c = load_pair(p.ring_candidate + at);
+      s.x = (1.0f - z.x) * s.x + z.x * c.x;
+      s.y = (1.0f - z.y) * s.y + z.y * c.y;
+    }
+    *folded = make_float4(s.x, s.y, 0.0f, 0.0f);
+  }
+  if (kEmit) {
+    s0 = folded->x;
+    s1 = folded->y;
+#pragma unroll 8
+    for (int i = 0; i < stretch; ++i) {
+      const float4 r = stretches[size_t(i) * (p.width_pad / 2)];
+      s0 = fmaf(r.x, s0, r.z);
+      s1 = fmaf(r.y, s1, r.w);
+    }
+  }
+  // Eight rows are requested at once: stores to `out` would otherwise keep the next row's loads behind them.
+  constexpr int kBatch = 8;
+  const uint32_t* x = reinterpret_cast<const uint32_t*>(static_cast<const bf16*>(p.fused) + size_t(begin) * p.stride + channel);
+  const int pitch = p.stride / 2, section = p.width_pad / 2;
+  for (int t = begin; t < end; t += kBatch, x += size_t(kBatch) * pitch) {
+    uint32_t gates[kBatch], candidates[kBatch], outputs[kBatch];
+#pragma unroll
+    for (int j = 0; j < kBatch; ++j) {
+      if (t + j < end) {
+        gates[j] = __ldg(x + size_t(j) * pitch);
+        candidates[j] = __ldg(x + size_t(j) * pitch + section);
+        if (kEmit) outputs[j] = __ldg(x + size_t(j) * pitch + 2 * section);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < kBatch; ++j) {
+      if (t + j < end) {
+        const float z0 = quick_sigmoid(bf16_lo(gates[j])), z1 = quick_sigmoid(bf16_hi(gates[j]));
+        s0 = (1.0f - z0) * s0 + z0 * quick_candidate(bf16_lo(candidates[j]));
+        s1 = (1.0f - z1) * s1 + z1 * quick_candidate(bf16_hi(candidates[j]));
+        if (kEmit) {
+          const float g0 = bf16_lo(outputs[j]), g1 = bf16_hi(outputs[j]);
+          store_pair(out + size_t(t + j) * p.out_stride, s0 * g0 * quick_sigmoid(g0), s1 * g1 * quick_sigmoid(g1));
+        } else {
+          a0 *= 1.0f - z0;
+          a1 *= 1.0f - z1;
+        }
+      }
+    }
+  }
+  if (!kEmit)
+    stretches[size_t(stretch) * (p.width_pad / 2)] = make_float4(a0, a1, s0, s1);
+  else if (end == p.rows)
+    store_pair(p.state + channel, s0, s1);
 }
 
 template <typename T>
@@ -482,7 +555,9 @@ void launch_min_gru_step(const MinGruParams& p, cudaStream_t stream, bool pdl) {
   launch(min_gru_step_kernel<T>, dim3(unsigned((p.out_stride + 127) / 128)), dim3(128), 0, stream, pdl, p);
 }
 void launch_min_gru_prompt(const MinGruParams& p, cudaStream_t stream, bool pdl) {
-  launch(min_gru_prompt_kernel, dim3(unsigned((p.out_stride + 31) / 32)), dim3(1024), 0, stream, pdl, p);
+  const dim3 grid(unsigned((p.out_stride / 2 + kGruThreads - 1) / kGruThreads), unsigned((p.rows + kStretch - 1) / kStretch));
+  launch(min_gru_prompt_kernel<false>, grid, dim3(kGruThreads), 0, stream, pdl, p);
+  launch(min_gru_prompt_kernel<true>, grid, dim3(kGruThreads), 0, stream, pdl, p);
 }
 template <typename T>
 void launch_clamped_glu(const T* gate_up, int rows, int ff, float limit, T* out, int multiprocessors,
