@@ -32,6 +32,13 @@ __device__ __forceinline__ void store_quad(float* p, float4 v) { *reinterpret_ca
 
 __device__ __forceinline__ float sigmoid_value(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-x)); }
+// The fast exponential and quotient (a few units in the last place of FP32) for kernels on BF16 activations.
+__device__ __forceinline__ float quick_sigmoid(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+__device__ __forceinline__ float quick_candidate(float u) { return u >= 0.0f ? u + 0.5f : quick_sigmoid(u); }
+template <typename T>
+__device__ __forceinline__ float sigmoid_for(float x) { return sizeof(T) == 2 ? quick_sigmoid(x) : sigmoid_value(x); }
+template <typename T>
+__device__ __forceinline__ float silu_for(float x) { return sizeof(T) == 2 ? x * quick_sigmoid(x) : silu_exact(x); }
 __device__ __forceinline__ float4 add(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
 
 __device__ __forceinline__ float4 dynamic_tanh(const DynamicTanh& n, int i, float4 x) {
@@ -173,10 +180,10 @@ __global__ void __launch_bounds__(128) mixer_prepare_kernel(const MixerPreparePa
       const float4 v = load_quad(x + i);
       sum = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, sum))));
     }
-    const float root = sqrtf(warp_sum(sum) / float(p.vdim) + p.eps);
+    const float inverse = 1.0f / sqrtf(warp_sum(sum) / float(p.vdim) + p.eps);
     for (int i = lane * 4; i < p.vdim_pad; i += 128) {
       const float4 v = load_quad(x + i);
-      store_quad(to + i, make_float4(v.x / root, v.y / root, v.z / root, v.w / root));
+      store_quad(to + i, make_float4(v.x * inverse, v.y * inverse, v.z * inverse, v.w * inverse));
     }
     return;
   }
@@ -190,7 +197,7 @@ __global__ void __launch_bounds__(128) mixer_prepare_kernel(const MixerPreparePa
     ring = static_cast<T*>(kind == 1 ? p.ring_k : p.ring_v) + (size_t(position & (kRingRows - 1)) * p.lin_heads + head) * pad;
   for (int i = lane * 4; i < pad; i += 128) {
     float4 v = load_quad(x + i);
-    v = make_float4(silu_exact(v.x), silu_exact(v.y), silu_exact(v.z), silu_exact(v.w));
+    v = make_float4(silu_for<T>(v.x), silu_for<T>(v.y), silu_for<T>(v.z), silu_for<T>(v.w));
     store_quad(x + i, v);
     if (ring) store_quad(ring + i, v);
   }
@@ -314,8 +321,8 @@ __global__ void __launch_bounds__(kFinishThreads) mixer_finish_kernel(const Mixe
     float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     if (i < width) {
       const float4 w = load_quad(p.norm + i);
-      y = make_float4(v.x * factor * w.x * sigmoid_value(z.x), v.y * factor * w.y * sigmoid_value(z.y),
-                      v.z * factor * w.z * sigmoid_value(z.z), v.w * factor * w.w * sigmoid_value(z.w));
+      y = make_float4(v.x * factor * w.x * sigmoid_for<T>(z.x), v.y * factor * w.y * sigmoid_for<T>(z.y),
+                      v.z * factor * w.z * sigmoid_for<T>(z.z), v.w * factor * w.w * sigmoid_for<T>(z.w));
     }
     store_quad(out + i, y);
   };
@@ -371,12 +378,8 @@ __global__ void __launch_bounds__(128) min_gru_step_kernel(const MinGruParams p)
 // A prompt segment runs in stretches of 32 rows, two channels per thread. The first kernel reduces every stretch to
 // (product of 1 - z, value from zero) and leaves the state with its pending rows folded in behind the stretches; the
 // second chains the stretches before its own from that state and emits the rows, the last stretch writes the new state.
-// Exponential and quotient are the fast forms (a few units in the last place of FP32).
 constexpr int kStretch = kMinGruStretch;
 constexpr int kGruThreads = 64;
-__device__ __forceinline__ float quick_sigmoid(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
-__device__ __forceinline__ float quick_candidate(float u) { return u >= 0.0f ? u + 0.5f : quick_sigmoid(u); }
-
 template <bool kEmit>
 __global__ void __launch_bounds__(kGruThreads) min_gru_prompt_kernel(const MinGruParams p) {
   const int context = p.control->context, base = p.control->state_base;

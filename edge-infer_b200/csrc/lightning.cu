@@ -153,13 +153,17 @@ __device__ __forceinline__ void split_pair(float a, float b, uint32_t& leading, 
   rest = pack_bf16(a - bf16_lo(leading), b - bf16_hi(leading));
 }
 
-// Stages rows [0, live) of a [tokens][dim] BF16 operand, zeros behind them.
+// Requests a 16-byte piece into shared memory; a dead piece is filled with zeros and not read.
+__device__ __forceinline__ void request_piece(bf16* to, const bf16* from, bool live) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_address(to)), "l"(from), "r"(live ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void await_pieces() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+// Requests rows [0, live) of a [tokens][dim] BF16 operand, zeros behind them.
 __device__ __forceinline__ void stage_rows(bf16* to, const bf16* from, int stride, int live, int pieces, int pitch) {
-  for (int i = threadIdx.x; i < kChunk * pieces; i += blockDim.x) {
+#pragma unroll 8
+  for (int i = threadIdx.x; i < kChunk * pieces; i += kPromptThreads) {
     const int row = i / pieces, piece = i - row * pieces;
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (row < live) v = *reinterpret_cast<const uint4*>(from + size_t(row) * stride + piece * 8);
-    *reinterpret_cast<uint4*>(to + size_t(row) * pitch + piece * 8) = v;
+    request_piece(to + size_t(row) * pitch + piece * 8, from + (row < live ? size_t(row) * stride : 0) + piece * 8, row < live);
   }
 }
 
@@ -182,7 +186,8 @@ __global__ void __launch_bounds__(kPromptThreads) lightning_chunk_kernel(const L
   const float* powers = p.powers + size_t(head) * (kChunk + 1);
   stage_rows(keys, static_cast<const bf16*>(p.k) + size_t(first) * p.stride + size_t(head) * dim, p.stride, live, dim / 8,
              k_pitch);
-  for (int i = threadIdx.x; i < kChunk * (kSlice / 8); i += blockDim.x) {
+#pragma unroll
+  for (int i = threadIdx.x; i < kChunk * (kSlice / 8); i += kPromptThreads) {
     const int row = i >> 3, piece = i & 7;
     uint4 hi = make_uint4(0, 0, 0, 0), lo = hi;
     if (row < live && piece * 8 < values) {
@@ -197,6 +202,7 @@ __global__ void __launch_bounds__(kPromptThreads) lightning_chunk_kernel(const L
     *reinterpret_cast<uint4*>(leading + row * kPitch + piece * 8) = hi;
     *reinterpret_cast<uint4*>(rest + row * kPitch + piece * 8) = lo;
   }
+  await_pieces();
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
   const int matrix = lane >> 3, in_matrix = lane & 7;
@@ -300,16 +306,18 @@ __global__ void __launch_bounds__(kPromptThreads) lightning_output_kernel(const 
   for (int i = threadIdx.x; i <= kChunk; i += blockDim.x) powers[i] = p.powers[size_t(head) * (kChunk + 1) + i];
   stage_rows(keys, static_cast<const bf16*>(p.k) + size_t(first) * p.stride + size_t(head) * dim, p.stride, live, dim / 8,
              k_pitch);
-  for (int i = threadIdx.x; i < kChunk * (kSlice / 8); i += blockDim.x) {
-    const int row = i >> 3, piece = i & 7;
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (row < live && piece * 8 < values)
-      v = *reinterpret_cast<const uint4*>(static_cast<const bf16*>(p.v) + size_t(first + row) * p.stride +
-                                          size_t(head) * p.vdim_pad + first_value + piece * 8);
-    *reinterpret_cast<uint4*>(vals + row * kPitch + piece * 8) = v;
+  {
+    const bf16* v = static_cast<const bf16*>(p.v) + size_t(first) * p.stride + size_t(head) * p.vdim_pad + first_value;
+#pragma unroll
+    for (int i = threadIdx.x; i < kChunk * (kSlice / 8); i += kPromptThreads) {
+      const int row = i >> 3, piece = i & 7;
+      const bool on = row < live && piece * 8 < values;
+      request_piece(vals + row * kPitch + piece * 8, on ? v + size_t(row) * p.stride + piece * 8 : v, on);
+    }
   }
   const float* state = p.chunk_states + (size_t(chunk) * p.heads + head) * dim * p.vdim_pad;
-  for (int i = threadIdx.x; i < dim * (kSlice / 4); i += blockDim.x) {
+#pragma unroll 8
+  for (int i = threadIdx.x; i < dim * (kSlice / 4); i += kPromptThreads) {
     const int quad = i & 3, d = (i >> 2) % dim, slice = (i >> 2) / dim;  // consecutive threads: one slice's memory order
     const int value = slice * 16 + quad * 4;
     float4 s = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
@@ -321,6 +329,7 @@ __global__ void __launch_bounds__(kPromptThreads) lightning_output_kernel(const 
     *reinterpret_cast<uint2*>(leading + size_t(d) * kPitch + value) = hi;
     *reinterpret_cast<uint2*>(rest + size_t(d) * kPitch + value) = lo;
   }
+  await_pieces();
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
   const int matrix = lane >> 3, in_matrix = lane & 7;
