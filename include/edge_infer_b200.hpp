@@ -25,7 +25,12 @@ class Session {
   const void* prefill(const std::uint32_t* tokens, std::size_t rows, void* all_logits = nullptr) {
     const void* last = nullptr;
     check(ei_session_prefill(session_, tokens, rows, &last, all_logits));
-    return last;  // borrowed BF16 [1, vocab], valid until the next operation
+    return last;  // borrowed BF16 (layered models: FP32) [1, vocab], valid until the next operation
+  }
+  // Appends a portion of a sequence; FP32 logits [want_count, vocab] of its rows `want` go to `logits`.
+  void extend(const std::uint32_t* tokens, std::size_t rows, const std::uint32_t* want = nullptr,
+              std::size_t want_count = 0, float* logits = nullptr) {
+    check(ei_session_extend(session_, tokens, rows, want, want_count, logits));
   }
   const void* decode(std::uint32_t token) {
     const void* logits = nullptr;

@@ -47,6 +47,9 @@ CASES = {
     "loop_last": config(113, 88, [parallel((4, 2, 48, 32, 24, 1e3), (2, 32, 16)), mingru(88, ff=40, limit=2.0)],
                         loop=(1, 2, 2)),
     "loop_once": config(77, 66, [mingru(30), mingru(34)], loop=(0, 2, 1)),
+    # More inputs than one K slice of a step projection: FP32 slices summed by the joins, and BF16 results by a store.
+    "inputs_in_slices": config(60, 72, [mingru(4160, ff=4200, limit=1.2), mingru(1100)]),
+    "stream_in_slices": config(60, 4200, [mingru(40, ff=70), parallel((2, 1, 16, 16, 16, 1e3), (1, 16, 16))]),
     "mixed": config(203, 104, [mingru(56, ff=72), parallel((6, 3, 40, 24, 20, 1e4), (5, 24, 32), ff=60, limit=0.7),
                                parallel((6, 3, 40, 24, 20, 1e4), (5, 24, 32)), mingru(120)], loop=(1, 3, 2)),
 }
