@@ -1,4 +1,5 @@
-// Decayed linear attention: per head S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, the state in FP32.
+// Decayed linear attention. Per head a matrix M (key size x value size, FP32) becomes decay M + k v^T with every row,
+// and the row's output is q^T M.
 //
 // A step of at most 16 rows leaves its rows pending: their k and v stay in a ring indexed by position and the next
 // step folds those that were kept into the state it reads anyway, so a rejected draft costs nothing and no copy of a

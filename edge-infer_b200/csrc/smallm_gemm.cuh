@@ -37,7 +37,7 @@ enum GemmEpilogue : int {
 
 enum GluKind : int {
   kGluSilu = 0,     // silu(gate) * up with the reference operator's BF16 staging
-  kGluClamped = 1   // g = min(gate, limit), u = clamp(up, -limit, limit): g * sigmoid(1.702 g) * (u + 1), rounded once
+  kGluClamped = 1   // a = min(gate, limit), b = up held to +-limit: (1 + b) * a / (1 + exp(-1.702 a)), rounded once
 };
 
 struct GemmParams {

@@ -102,8 +102,8 @@ class Layer:
 
 @dataclass
 class LayeredShape:
-    """A decoder described layer by layer (ei_model_create_layered). `loop` = (start, stop, times): layers
-    start .. stop - 1 run `times` times in a row. `true32`: FP32 activations, caches and products."""
+    """A decoder described layer by layer (ei_model_create_layered). `loop` = (start, stop, times): the
+    stretch layers[start:stop] is repeated, `times` passes in all. `true32`: FP32 activations, caches and products."""
     vocab_size: int
     hidden_size: int
     layers: List[Layer]
@@ -309,7 +309,7 @@ class Session:
         return greedy_of(self.read_logits_f32(1)[0])
 
     def tap_residual(self, buffer) -> None:
-        """Layered models: copy the residual stream after every layer run into `buffer`, a float32 device tensor
+        """Layered models: every forward leaves each layer run's output stream in `buffer`, a float32 device tensor
         [layer runs, rows, width]; None ends it. The caller keeps the tensor alive."""
         if buffer is None:
             abi.check(self._lib.ei_session_tap_residual(self._handle, None, 0))

@@ -2,9 +2,9 @@
 
     bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N
 
-Standard input holds one JSON object a line,
+Every line of standard input is a step in JSON,
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "x", "tokens": [11, 4], "want": [1]}], "end": ["x"]}
 
 entries: the next tokens of each request and the places among them whose logits are wanted; end: requests that are over
 after the step. For a step that wants something DIR/<step>.f32 receives the logits, little-endian FP32 [wanted, vocab]
@@ -53,10 +53,10 @@ class Replay:
 
 def main(argv=None) -> int:
     parser = argparse.ArgumentParser(description="Replay a trace of token portions and write the wanted logits.")
-    parser.add_argument("--model", required=True, help="folder with config.json and model.safetensors")
+    parser.add_argument("--model", required=True, help="checkpoint folder (config.json, safetensors)")
     parser.add_argument("--dtype", required=True, choices=["bfloat16", "float32"])
     parser.add_argument("--out", required=True, help="folder for <step>.f32")
-    parser.add_argument("--max-tokens", type=int, required=True, help="most tokens live requests hold at any time")
+    parser.add_argument("--max-tokens", type=int, required=True, help="capacity of a request, in tokens")
     args = parser.parse_args(argv)
     config, weights = checkpoint.load_directory(args.model)
     try:

@@ -223,11 +223,12 @@ ei_status ei_model_create(const ei_model_config* config, const ei_named_tensor* 
  * names its token mixer with its sizes and constants and its feed-forward, each sublayer stands between two norms, and
  * a stretch of layers may run several times in a row. The session verbs below serve such a model as they serve the
  * others; differences are noted there.
- * Mixers: EI_MIXER_MIN_GRU - gated recurrence of `rnn_width` channels whose gates read only the current token.
+ * Mixers: EI_MIXER_MIN_GRU - `rnn_width` independent channels, each an exponential average whose gate depends on the
+ * row's own input alone.
  * EI_MIXER_PARALLEL - grouped-query softmax attention (partial rotation, value norm, per-head sink, own score scale)
  * beside decayed linear attention (SiLU on q, k, v; one decay per head; normed and gated output), outputs weighted by
- * left_scale and right_scale. Feed-forward: EI_MLP_CLAMPED_GLU - g = min(gate, limit), u = clamp(up, +-limit),
- * g * sigmoid(1.702 g) * (u + 1). Norm: tanh(alpha x) * weight + bias. Residual stream, norms, angles, scores, softmax
+ * left_scale and right_scale. Feed-forward: EI_MLP_CLAMPED_GLU - with a = min(gate, limit) and
+ * b = max(-limit, min(up, limit)): (1 + b) * a / (1 + exp(-1.702 a)). Norm: tanh(alpha x) * weight + bias. Residual stream, norms, angles, scores, softmax
  * weights, gates and recurrent state are FP32; with `true32` so are all activations, caches and products. */
 enum { EI_MIXER_MIN_GRU = 1, EI_MIXER_PARALLEL = 2 };
 enum { EI_MLP_NONE = 0, EI_MLP_CLAMPED_GLU = 1 };

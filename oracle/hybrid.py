@@ -21,7 +21,7 @@ def silu(x):
 
 
 def rms(x, eps):
-    """x divided by its root mean square over the last axis."""
+    """x scaled to unit mean square along the last axis."""
     return x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps)
 
 
@@ -80,8 +80,8 @@ def clamped_glu(gate, up, limit):
 
 
 class HybridOracle:
-    """One sequence: `forward(tokens)` appends tokens and returns their logits; `taps` then holds the residual
-    stream after every layer run, before what is added ahead of the next pass."""
+    """One sequence: `forward(tokens)` appends tokens and returns their logits; `taps` then holds the stream
+    as each layer run leaves it, without what the next pass adds."""
 
     def __init__(self, config, weights):
         self.c = config
