@@ -90,15 +90,21 @@ class LayerSpec(C.Structure):
     _fields_ = [("mixer", C.c_int32), ("mlp", C.c_int32), ("rnn_width", C.c_uint32), ("heads", C.c_uint32),
                 ("kv_heads", C.c_uint32), ("dim", C.c_uint32), ("vdim", C.c_uint32), ("rot_dims", C.c_uint32),
                 ("lin_heads", C.c_uint32), ("lin_dim", C.c_uint32), ("lin_vdim", C.c_uint32), ("ff", C.c_uint32),
+                ("rot_dim", C.c_uint32), ("kv_rank", C.c_uint32), ("state", C.c_uint32), ("groups", C.c_uint32),
+                ("norm_groups", C.c_uint32), ("taps", C.c_uint32), ("decay_rank", C.c_uint32), ("gate_rank", C.c_uint32),
                 ("rot_base", C.c_double), ("scale", C.c_double), ("left_scale", C.c_double),
-                ("right_scale", C.c_double), ("limit", C.c_double), ("decay", C.POINTER(C.c_double))]
+                ("right_scale", C.c_double), ("limit", C.c_double), ("rot_factor", C.c_double),
+                ("rot_original", C.c_double), ("rot_fast", C.c_double), ("rot_slow", C.c_double),
+                ("decay", C.POINTER(C.c_double))]
 
 
 class LayeredConfig(C.Structure):
     _fields_ = [("vocab_size", C.c_uint64), ("width", C.c_uint64), ("n_layers", C.c_uint64),
                 ("max_position_embeddings", C.c_uint64), ("loop_start", C.c_uint64), ("loop_stop", C.c_uint64),
                 ("loop_times", C.c_uint64), ("norm_eps", C.c_double), ("bos_token_id", C.c_uint32),
-                ("eos_token_id", C.c_uint32), ("true32", C.c_int32)]
+                ("eos_token_id", C.c_uint32), ("true32", C.c_int32), ("block", C.c_int32), ("tied_head", C.c_int32),
+                ("pair_buckets", C.c_uint64), ("pair_mul_prev", C.c_uint64), ("pair_mul_cur", C.c_uint64),
+                ("logit_softcap", C.c_double)]
 
 
 class NamedTensor(C.Structure):

@@ -24,11 +24,14 @@ from typing import Dict, List, Mapping, Optional, Tuple
 
 import numpy as np
 
-from .runtime import Attention, Layer, LayeredShape, LinearAttention, Shape
+from .runtime import (BLOCK_PARALLEL, MLP_RELU_SQUARED, Attention, ChannelDelta, LatentAttention, Layer, LayeredShape,
+                      LinearAttention, PairEmbedding, Shape, StateSpace, Yarn)
 
 DENSE, QWEIGHT, SCALES, ZEROS = 0, 1, 2, 3
 
-MODEL_TYPES = ("qwen_bf16", "qwen_awq", "qwen3_bf16", "qwen3_awq", "zofesun_bf16", "zofesun_f32")
+MODEL_TYPES = ("qwen_bf16", "qwen_awq", "qwen3_bf16", "qwen3_awq", "zofesun_bf16", "zofesun_f32",
+               "gikepel_bf16", "gikepel_f32")
+_DESIGNS = {"Zofesun": "zofesun", "Gikepel": "gikepel"}  # `architecture` of layered designs
 
 _PROJECTIONS = {
     "self_attn.q_proj": "wq", "self_attn.k_proj": "wk", "self_attn.v_proj": "wv", "self_attn.o_proj": "wo",
@@ -43,8 +46,9 @@ def model_type_of(config: Mapping, dtype: str = "bfloat16") -> str:
     `model_type` and quantization settings otherwise. dtype float32 is there for the layered designs only."""
     if dtype not in ("bfloat16", "float32"):
         raise ValueError("dtype must be bfloat16 or float32")
-    if config.get("architecture") == "Zofesun":
-        return "zofesun_f32" if dtype == "float32" else "zofesun_bf16"
+    design = _DESIGNS.get(config.get("architecture"))
+    if design is not None:
+        return design + ("_f32" if dtype == "float32" else "_bf16")
     family = {"qwen2": "qwen", "qwen3": "qwen3"}.get(config.get("model_type"))
     if family is None:
         raise ValueError("Unsupported model architecture: %r" % (config.get("architecture") or config.get("model_type")))
@@ -107,31 +111,98 @@ def _zofesun_layer(entry: Mapping, where: str) -> Layer:
     return layer
 
 
-def zofesun_shape(config: Mapping, true32: bool = False) -> LayeredShape:
-    """Decoder shape of a Zofesun config.json: every size and constant comes from it."""
+def _layer_entries(config: Mapping) -> List[Mapping]:
     entries = config.get("layers")
     if not isinstance(entries, list) or not entries or not all(isinstance(e, Mapping) for e in entries):
         raise ValueError("layers must be a nonempty list")
+    return entries
+
+
+def _layered_common(config: Mapping, true32: bool) -> Dict[str, object]:
+    return dict(vocab_size=_size(config, "vocab", "config"), hidden_size=_size(config, "width", "config"),
+                norm_eps=_number(_section(config, "norm", "config"), "eps", "norm"), true32=true32,
+                max_position_embeddings=int(config.get("max_position_embeddings", 1 << 20)),
+                bos_token_id=int(config.get("bos_token_id", 0) or 0),
+                eos_token_id=_first_int(config.get("eos_token_id", 0xFFFFFFFF)))
+
+
+def zofesun_shape(config: Mapping, true32: bool = False) -> LayeredShape:
+    """Decoder shape of a Zofesun config.json: every size and constant comes from it."""
+    entries = _layer_entries(config)
     loop = config.get("loop")
     if loop is not None:
         loop = (_size(loop, "start", "loop", 0), _size(loop, "stop", "loop"), _size(loop, "times", "loop"))
         if not loop[0] < loop[1] <= len(entries):
             raise ValueError("loop must span existing layers")
-    return LayeredShape(vocab_size=_size(config, "vocab", "config"), hidden_size=_size(config, "width", "config"),
-                        layers=[_zofesun_layer(e, f"layers[{i}]") for i, e in enumerate(entries)],
-                        norm_eps=_number(_section(config, "norm", "config"), "eps", "norm"), loop=loop, true32=true32,
-                        max_position_embeddings=int(config.get("max_position_embeddings", 1 << 20)),
-                        bos_token_id=int(config.get("bos_token_id", 0) or 0),
-                        eos_token_id=_first_int(config.get("eos_token_id", 0xFFFFFFFF)))
+    return LayeredShape(layers=[_zofesun_layer(e, f"layers[{i}]") for i, e in enumerate(entries)], loop=loop,
+                        **_layered_common(config, true32))
+
+
+def _gikepel_layer(entry: Mapping, where: str) -> Layer:
+    mixer, layer = _section(entry, "mixer", where), Layer(mlp=MLP_RELU_SQUARED)
+    kind, at = entry.get("type"), where + ".mixer"
+    if kind == "latent_attention":
+        rot = _section(mixer, "rot", at)
+        yarn = None
+        if rot.get("scaling") is not None:
+            scaling = _section(rot, "scaling", at + ".rot")
+            yarn = Yarn(*(_number(scaling, key, at + ".rot.scaling") for key in ("factor", "original", "fast", "slow")))
+        layer.latent = LatentAttention(*(_size(mixer, key, at) for key in ("heads", "dim", "rot_dim", "vdim", "kv_rank")),
+                                       rot_dims=_size(rot, "dims", at + ".rot", 0), rot_base=_number(rot, "base", at + ".rot"),
+                                       scale=_number(mixer, "scale", at), yarn=yarn)
+    elif kind == "mamba2":
+        layer.state_space = StateSpace(*(_size(mixer, key, at) for key in ("heads", "groups", "state", "vdim", "conv", "norm_groups")))
+    elif kind == "channel_delta":
+        layer.delta = ChannelDelta(*(_size(mixer, key, at) for key in ("heads", "kv_heads", "dim", "vdim", "conv")))
+    else:
+        raise ValueError(f"{where}: unsupported mixer type {kind!r}")
+    mlp = entry.get("mlp")
+    if mlp is not None:
+        if not isinstance(mlp, Mapping) or mlp.get("kind") != "dense":
+            raise ValueError(where + ": unsupported feed-forward")
+        layer.ff = _size(mlp, "ff", where + ".mlp")
+    return layer
+
+
+def gikepel_shape(config: Mapping, true32: bool = False) -> LayeredShape:
+    """Decoder shape of a Gikepel config.json. The ranks of the low-rank projections are not in it: they come from the
+    checkpoint's tensors (with_ranks)."""
+    pairs = config.get("embedding", {}).get("bigram")
+    if pairs is not None:
+        pairs = PairEmbedding(_size(pairs, "buckets", "embedding.bigram"), _size(pairs, "mul_prev", "embedding.bigram", 0),
+                              _size(pairs, "mul_cur", "embedding.bigram", 0))
+    softcap = 0.0 if config.get("logit_softcap") is None else _number(config, "logit_softcap", "config")
+    return LayeredShape(layers=[_gikepel_layer(e, f"layers[{i}]") for i, e in enumerate(_layer_entries(config))],
+                        block=BLOCK_PARALLEL, tied_embeddings=True, pairs=pairs, logit_softcap=softcap,
+                        **_layered_common(config, true32))
+
+
+def with_ranks(shape: LayeredShape, weights: Mapping) -> LayeredShape:
+    """Fills in the ranks that only the tensors tell."""
+    for i, layer in enumerate(shape.layers):
+        if layer.delta is None:
+            continue
+        for name, field in (("a1", "decay_rank"), ("g1", "gate_rank")):
+            tensor = weights.get(f"l{i}.mix.{name}")
+            if tensor is None:
+                raise ValueError(f"Decoder checkpoint lacks l{i}.mix.{name}")
+            setattr(layer.delta, field, int(tensor.shape[0]))
+    return shape
 
 
 def layered_tensor_shapes(shape: LayeredShape) -> Dict[str, Tuple[int, ...]]:
     """Every tensor a layered checkpoint must hold, with its shape ([out, in] for linears, () for scalars)."""
-    width = shape.hidden_size
-    shapes: Dict[str, Tuple[int, ...]] = {"embed": (shape.vocab_size, width), "head": (shape.vocab_size, width)}
+    width, parallel = shape.hidden_size, shape.block == BLOCK_PARALLEL
+    shapes: Dict[str, Tuple[int, ...]] = {"embed": (shape.vocab_size, width)}
+    if not shape.tied_embeddings:
+        shapes["head"] = (shape.vocab_size, width)
+    if shape.pairs is not None:
+        shapes["bigram"] = (shape.pairs.buckets + 1, width)
 
     def norm(name: str) -> None:
-        shapes.update({name: (width,), name + ".b": (width,), name + ".alpha": ()})
+        shapes[name] = (width,)
+        if not parallel:
+            shapes.update({name + ".b": (width,), name + ".alpha": ()})
 
     norm("final.norm")
     if shape.loop is not None:
@@ -139,33 +210,57 @@ def layered_tensor_shapes(shape: LayeredShape) -> Dict[str, Tuple[int, ...]]:
     for i, layer in enumerate(shape.layers):
         p = f"l{i}."
         norm(p + "norm1")
-        norm(p + "norm1b")
-        if layer.rnn_width is not None:
-            r = layer.rnn_width
-            shapes.update({p + "mix.z": (r, width), p + "mix.z.b": (r,), p + "mix.x": (r, width), p + "mix.x.b": (r,),
-                           p + "mix.g": (r, width), p + "mix.o": (width, r)})
+        if parallel:
+            shapes[p + "ls1"] = (width,)
         else:
-            a, l = layer.attention, layer.linear
-            left, right = p + "mix.left.", p + "mix.right."
-            shapes.update({left + "q": (a.heads * a.dim, width), left + "k": (a.kv_heads * a.dim, width),
-                           left + "v": (a.kv_heads * a.vdim, width), left + "sink": (a.heads,),
-                           left + "o": (width, a.heads * a.vdim), right + "q": (l.heads * l.dim, width),
-                           right + "k": (l.heads * l.dim, width), right + "v": (l.heads * l.vdim, width),
-                           right + "g": (l.heads * l.vdim, width), right + "o": (width, l.heads * l.vdim),
-                           right + "norm": (l.heads * l.vdim,)})
+            norm(p + "norm1b")
+        shapes.update({p + "mix." + name: dims for name, dims in _mixer_tensors(layer, width).items()})
         if layer.ff is not None:
             norm(p + "norm2")
-            norm(p + "norm2b")
-            shapes.update({p + "mlp.gate": (layer.ff, width), p + "mlp.up": (layer.ff, width),
-                           p + "mlp.down": (width, layer.ff)})
+            if parallel:
+                shapes[p + "ls2"] = (width,)
+            else:
+                norm(p + "norm2b")
+                shapes[p + "mlp.gate"] = (layer.ff, width)
+            shapes.update({p + "mlp.up": (layer.ff, width), p + "mlp.down": (width, layer.ff)})
     return shapes
 
 
+def _mixer_tensors(layer: Layer, width: int) -> Dict[str, Tuple[int, ...]]:
+    if layer.rnn_width is not None:
+        r = layer.rnn_width
+        return {"z": (r, width), "z.b": (r,), "x": (r, width), "x.b": (r,), "g": (r, width), "o": (width, r)}
+    if layer.latent is not None:
+        a = layer.latent
+        return {"q": (a.heads * (a.dim + a.rot_dim), width), "dkv": (a.kv_rank + a.rot_dim, width), "dkv.norm": (a.kv_rank,),
+                "uk": (a.heads * a.dim, a.kv_rank), "uv": (a.heads * a.vdim, a.kv_rank), "g": (a.heads * a.vdim, width),
+                "o": (width, a.heads * a.vdim)}
+    if layer.state_space is not None:
+        m = layer.state_space
+        inner, pairs = m.heads * m.vdim, m.groups * m.state
+        return {"in": (2 * inner + 2 * pairs + m.heads, width), "conv": (inner + 2 * pairs, m.taps),
+                "conv.b": (inner + 2 * pairs,), "dt_bias": (m.heads,), "A_log": (m.heads,), "D": (m.heads,),
+                "norm": (inner,), "o": (width, inner)}
+    if layer.delta is not None:
+        m = layer.delta
+        keys, values = m.kv_heads * m.dim, m.heads * m.vdim
+        return {"q": (keys, width), "q.conv": (keys, m.taps), "k": (keys, width), "k.conv": (keys, m.taps),
+                "v": (values, width), "v.conv": (values, m.taps), "b": (m.heads, width), "A_log": (m.heads,),
+                "norm": (m.vdim,), "a1": (m.decay_rank, width), "a2": (m.heads * m.dim, m.decay_rank),
+                "dt_bias": (m.heads * m.dim,), "g1": (m.gate_rank, width), "g2": (values, m.gate_rank), "o": (width, values)}
+    a, l = layer.attention, layer.linear
+    return {"left.q": (a.heads * a.dim, width), "left.k": (a.kv_heads * a.dim, width), "left.v": (a.kv_heads * a.vdim, width),
+            "left.sink": (a.heads,), "left.o": (width, a.heads * a.vdim), "right.q": (l.heads * l.dim, width),
+            "right.k": (l.heads * l.dim, width), "right.v": (l.heads * l.vdim, width), "right.g": (l.heads * l.vdim, width),
+            "right.o": (width, l.heads * l.vdim), "right.norm": (l.heads * l.vdim,)}
+
+
 def _admit_layered(shape: LayeredShape, weights: Mapping):
-    expected = layered_tensor_shapes(shape)
-    # Norms around a feed-forward that a layer does not have, and the vectors of a loop that is not run, are passed over.
+    expected = layered_tensor_shapes(with_ranks(shape, weights))
+    # Norms and scales of a feed-forward that a layer does not have, and the vectors of a loop that is not run, are
+    # passed over.
     spare = {f"l{i}.{norm}{part}" for i, layer in enumerate(shape.layers) if layer.ff is None
-             for norm in ("norm2", "norm2b") for part in ("", ".b", ".alpha")} | {"loop.step"}
+             for norm in ("norm2", "norm2b", "ls2") for part in ("", ".b", ".alpha")} | {"loop.step"}
     missing, extra = sorted(set(expected) - set(weights)), sorted(set(weights) - set(expected) - spare)
     if missing:
         raise ValueError("Decoder checkpoint lacks " + missing[0])
@@ -257,6 +352,8 @@ def shape_from_config(config: Mapping, model_type: str):
         raise ValueError(f"Unsupported model type: {model_type}")
     if model_type.startswith("zofesun"):
         return zofesun_shape(config, true32=model_type.endswith("_f32"))
+    if model_type.startswith("gikepel"):
+        return gikepel_shape(config, true32=model_type.endswith("_f32"))
     heads = int(config["num_attention_heads"])
     head_dim = int(config.get("head_dim", int(config["hidden_size"]) // heads))
     awq = model_type.endswith("_awq")

@@ -120,7 +120,7 @@ void run_prompt_operator(const ei_context* ctx, bool awq, GemmParams p, void* sc
   p.partial = static_cast<float*>(scratch);
   launch_prompt_gemm(awq, p, stream, false);
   splitk_store_kernel<<<std::min(ctx->multiprocessors * 8, (p.M * p.N + 255) / 256), 256, 0, stream>>>(
-      p.partial, ksplit, p.M, p.N, bias, out, p.out_stride);
+      p.partial, ksplit, p.M, p.N, bias, out, p.out_stride, int(kActNone));
   check_launch();
 }
 }  // namespace
@@ -256,7 +256,7 @@ ei_status ei_linear_bf16(const ei_context* ctx, ei_view2 input, const ei_dense_w
         launch_gemm(plan, false, p, stream, false);
         if (plan.ksplit > 1) {
           splitk_store_kernel<<<std::min(1024, (int(rows) * N + 255) / 256), 256, 0, stream>>>(
-              p.partial, plan.ksplit, int(rows), N, p.bias, out, N);
+              p.partial, plan.ksplit, int(rows), N, p.bias, out, N, int(kActNone));
           check_launch();
         }
       } else {
@@ -323,7 +323,7 @@ ei_status ei_awq_linear_bf16(const ei_context* ctx, ei_view2 input, const ei_awq
         launch_gemm(plan, true, p, stream, false);
         if (plan.ksplit > 1) {
           splitk_store_kernel<<<std::min(1024, (int(rows) * N + 255) / 256), 256, 0, stream>>>(
-              p.partial, plan.ksplit, int(rows), N, p.bias, out, N);
+              p.partial, plan.ksplit, int(rows), N, p.bias, out, N, int(kActNone));
           check_launch();
         }
       } else {

@@ -201,7 +201,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
         p.partial[(size_t(slice) * p.M + row) * p.N + n] = sum;
       } else {
         if (p.bias) sum += __bfloat162float(p.bias[n]);
-        const bf16 rounded = __float2bfloat16_rn(sum);
+        const bf16 rounded = __float2bfloat16_rn(activated_value(p.activation, sum));
         p.out[size_t(row) * p.out_stride + n] = rounded;
         if (p.epilogue == kEpiArgmax) {
           float value = __bfloat162float(rounded);

@@ -75,8 +75,16 @@ struct EmbedParams {
 void launch_embed_norm(const EmbedParams& p, cudaStream_t stream, bool pdl);
 
 #if defined(__CUDACC__)
-// The token of stacked row `row` of a step (given by the host, the pending token, or a draft), recorded in
-// step_tokens; raises the status bits for a bad id or a step that would pass the capacity. One thread per row.
+// The token of stacked row `row` of a step: given by the host, the pending token, or a draft.
+__device__ __forceinline__ uint32_t step_token_of(const EmbedParams& p, const Control* control, int row, int local) {
+  if (p.tokens) return p.tokens[row];
+  if (local == 0) return control->pending;
+  const DraftSource source = *p.source;
+  const long long index = (long long)control->context + local - source.base;
+  return (source.drafts && index >= 0 && index < source.count) ? source.drafts[index] : 0u;
+}
+// The same, recorded in step_tokens; raises the status bits for a bad id or a step that would pass the capacity. One
+// thread per row.
 __device__ __forceinline__ uint32_t take_step_token(const EmbedParams& p, int row) {
   Control* control = p.control;
   int local = row, step_rows = p.rows, capacity = p.capacity;
@@ -87,16 +95,7 @@ __device__ __forceinline__ uint32_t take_step_token(const EmbedParams& p, int ro
     control = p.slots[session].control;
     capacity = p.slots[session].capacity;
   }
-  uint32_t token;
-  if (p.tokens) {
-    token = p.tokens[row];
-  } else if (local == 0) {
-    token = control->pending;
-  } else {
-    const DraftSource source = *p.source;
-    const long long index = (long long)control->context + local - source.base;
-    token = (source.drafts && index >= 0 && index < source.count) ? source.drafts[index] : 0u;
-  }
+  const uint32_t token = step_token_of(p, control, row, local);
   p.step_tokens[row] = token;
   if (token >= uint32_t(p.vocab)) atomicOr(&control->status, 2);
   if (local == 0 && control->context + step_rows > capacity) atomicOr(&control->status, 1);

@@ -86,6 +86,37 @@ struct Placement {
     if (base) n.alpha = read(alpha)[0];
     return n;
   }
+  // A vector's values as FP32 on the host (zeros while only sizes are added up).
+  std::vector<float> values(const std::string& name, size_t width) {
+    const ei_named_tensor& t = find(name, width, 0);
+    return base ? read(t) : std::vector<float>(width);
+  }
+  // The same spread over `heads` heads `pad` entries apart, on the device.
+  const float* head_values(const std::string& name, int heads, int size, int pad) {
+    const std::vector<float> from = values(name, size_t(heads) * size);
+    std::vector<float> to(size_t(heads) * pad, 0.0f);
+    for (int h = 0; h < heads; ++h) std::copy_n(from.begin() + size_t(h) * size, size, to.begin() + size_t(h) * pad);
+    return host_values(to);
+  }
+  // Values `first`.. of a vector as `heads` heads `pad` entries apart from entry `at` on of `to`.
+  static void spread(std::vector<float>& to, size_t at, const std::vector<float>& from, size_t first, int heads, int size, int pad) {
+    for (int h = 0; h < heads; ++h)
+      std::copy_n(from.begin() + first + size_t(h) * size, size, to.begin() + at + size_t(h) * pad);
+  }
+  // Rows `first`.. of a [channels, taps] convolution to the same places of every tap of [taps][channels].
+  void conv_of(std::vector<float>& to, size_t channels, size_t at, const std::string& name, size_t rows, size_t first, int heads,
+               int size, int pad, int taps) {
+    const ei_named_tensor& t = find(name, rows, taps);
+    if (!base) return;
+    std::vector<uint16_t> bits(rows * taps);
+    EI_CUDA(cudaMemcpy(bits.data(), t.data, bits.size() * 2, cudaMemcpyDefault));
+    for (int h = 0; h < heads; ++h)
+      for (int i = 0; i < size; ++i)
+        for (int tap = 0; tap < taps; ++tap) {
+          const uint32_t wide = uint32_t(bits[(first + size_t(h) * size + i) * taps + tap]) << 16;
+          std::memcpy(&to[size_t(tap) * channels + at + size_t(h) * pad + i], &wide, 4);
+        }
+  }
   // A zeroed linear [out, in] to be filled section by section.
   PreparedLinear linear(int in, int out, bf16** weights) {
     PreparedLinear l;
@@ -96,13 +127,18 @@ struct Placement {
     l.bytes = size_t(out) * in * 2;
     return l;
   }
-  // Output rows of `heads` heads of `size` features, `pad` rows apart; returns the row behind them.
+  // Output rows of `heads` heads of `size` features, `pad` rows apart; returns the row behind them. A head's rows may be
+  // part of `spacing` rows in the source, from row `first` of a tensor of `total` rows on.
   int rows_of(bf16* weights, int pitch, int row, const std::string& name, int heads, int size, int pad, size_t inputs) {
-    const ei_named_tensor& t = find(name, size_t(heads) * size, inputs);
+    return some_rows_of(weights, pitch, row, name, size_t(heads) * size, 0, heads, size, size, pad, inputs);
+  }
+  int some_rows_of(bf16* weights, int pitch, int row, const std::string& name, size_t total, size_t first, int heads, int size,
+                   int spacing, int pad, size_t inputs) {
+    const ei_named_tensor& t = find(name, total, inputs);
     if (base)
       for (int h = 0; h < heads; ++h)
         copy(weights + (size_t(row) + size_t(h) * pad) * pitch, pitch,
-             static_cast<const bf16*>(t.data) + size_t(h) * size * inputs, inputs, size, inputs);
+             static_cast<const bf16*>(t.data) + (first + size_t(h) * spacing) * inputs, inputs, size, inputs);
     return row + heads * pad;
   }
   // Input columns of `heads` heads of `size` values, `pad` columns apart.
@@ -128,11 +164,230 @@ void validate_layer(const ei_layer_spec& l) {
       throw std::invalid_argument("Layered decoder: invalid linear attention sizes (head sizes are limited to 512)");
     if (!std::isfinite(l.left_scale) || !std::isfinite(l.right_scale))
       throw std::invalid_argument("Layered decoder: invalid mixer scale");
+  } else if (l.mixer == EI_MIXER_LATENT_ATTENTION) {
+    if (!in_range(l.heads, 4096) || !in_range(l.dim, kMaxHeadDim) || !in_range(l.rot_dim, kMaxHeadDim) ||
+        !in_range(l.vdim, kMaxHeadDim) || !in_range(l.kv_rank, kMaxLatent) || l.rot_dims > l.rot_dim || l.rot_dims % 2 ||
+        !(l.rot_base > 0.0) || !std::isfinite(l.scale))
+      throw std::invalid_argument("Layered decoder: invalid latent attention sizes (head sizes up to 512, latents up to 1024)");
+    if (l.rot_factor != 0.0 && (!(l.rot_factor > 0.0) || !(l.rot_original > 0.0) || !(l.rot_fast > 0.0) || !(l.rot_slow > 0.0) ||
+                                l.rot_base == 1.0 || !std::isfinite(l.rot_factor)))
+      throw std::invalid_argument("Layered decoder: invalid rotation scaling");
+  } else if (l.mixer == EI_MIXER_STATE_SPACE) {
+    if (!in_range(l.heads, 4096) || !in_range(l.groups, 4096) || l.heads % l.groups || !in_range(l.state, kMaxHeadDim) ||
+        !in_range(l.vdim, kMaxHeadDim) || !in_range(l.taps, 1024) || !in_range(l.norm_groups, kMany) ||
+        (l.heads * l.vdim) % l.norm_groups)
+      throw std::invalid_argument("Layered decoder: invalid state-space sizes (head sizes are limited to 512)");
+  } else if (l.mixer == EI_MIXER_CHANNEL_DELTA) {
+    if (!in_range(l.heads, 4096) || !in_range(l.kv_heads, 4096) || l.heads % l.kv_heads || !in_range(l.dim, kMaxHeadDim) ||
+        !in_range(l.vdim, kMaxHeadDim) || !in_range(l.taps, 1024) || !in_range(l.decay_rank, kMany) || !in_range(l.gate_rank, kMany))
+      throw std::invalid_argument("Layered decoder: invalid delta rule sizes (head sizes are limited to 512)");
   } else {
     throw std::invalid_argument("Layered decoder: unknown mixer");
   }
-  if (l.mlp != EI_MLP_NONE && (l.mlp != EI_MLP_CLAMPED_GLU || !in_range(l.ff, kMany) || std::isnan(l.limit)))
+  const bool known = l.mlp == EI_MLP_NONE || l.mlp == EI_MLP_RELU_SQUARED || (l.mlp == EI_MLP_CLAMPED_GLU && !std::isnan(l.limit));
+  if (!known || (l.mlp != EI_MLP_NONE && !in_range(l.ff, kMany)))
     throw std::invalid_argument("Layered decoder: invalid feed-forward");
+}
+
+// The rotation table's entry for these constants; equal ones share it.
+int rotation_of(LayeredModel& m, Placement& at, const ei_layer_spec& s) {
+  LayeredModel::Rotation r;
+  r.dims = int(s.rot_dims);
+  r.base = s.rot_base;
+  r.factor = s.rot_factor;
+  if (r.factor != 0.0) {
+    r.original = s.rot_original;
+    r.fast = s.rot_fast;
+    r.slow = s.rot_slow;
+  }
+  for (size_t i = 0; i < m.rotations.size(); ++i) {
+    const auto& o = m.rotations[i];
+    if (o.dims == r.dims && o.base == r.base && o.factor == r.factor && o.original == r.original && o.fast == r.fast && o.slow == r.slow)
+      return int(i);
+  }
+  // YaRN: frequencies that turn more than `fast` times over the original length stay, those below `slow` turns are
+  // divided by the factor, a ramp in between; lengths grow by 0.1 ln(factor) + 1.
+  double low = 0.0, high = 0.0;
+  if (r.factor != 0.0) {
+    const auto pair_of = [&](double turns) {
+      return r.dims * std::log(r.original / (2.0 * M_PI * turns)) / (2.0 * std::log(r.base));
+    };
+    low = std::max(std::floor(pair_of(r.fast)), 0.0);
+    high = std::min(std::ceil(pair_of(r.slow)), double(r.dims - 1));
+    r.length = 0.1 * std::log(r.factor) + 1.0;
+  }
+  std::vector<double> frequencies;
+  for (int i = 0; i < r.dims / 2; ++i) {
+    const double f = std::pow(r.base, -2.0 * i / r.dims);
+    const double ramp = r.factor != 0.0 ? std::min(std::max((i - low) / std::max(high - low, 0.001), 0.0), 1.0) : 0.0;
+    frequencies.push_back(ramp == 0.0 ? f : f / r.factor * ramp + f * (1.0 - ramp));
+  }
+  r.frequencies = at.host_values(frequencies);
+  m.rotations.push_back(r);
+  return int(m.rotations.size()) - 1;
+}
+
+void place_min_gru(LayeredModel::Layer& L, Placement& at, const std::string& mix, size_t W, int K, int R) {
+  bf16* weights = nullptr;
+  const int width = int(L.spec.rnn_width);
+  L.width_pad = round_up(width, 16);
+  L.in = at.linear(K, 3 * L.width_pad, &weights);
+  int row = at.rows_of(weights, K, 0, mix + "z", 1, width, L.width_pad, W);
+  row = at.rows_of(weights, K, row, mix + "x", 1, width, L.width_pad, W);
+  at.rows_of(weights, K, row, mix + "g", 1, width, L.width_pad, W);
+  bf16* bias = at.reserve<bf16>(L.in.out);
+  at.copy(bias, width, at.find(mix + "z.b", width, 0).data, width, 1, width);
+  at.copy(bias + L.width_pad, width, at.find(mix + "x.b", width, 0).data, width, 1, width);
+  L.in.bias = bias;
+  L.out = at.linear(round_up(width, 64), R, &weights);
+  at.columns_of(weights, L.out.in, 0, mix + "o", 1, width, L.width_pad, W);
+}
+
+void place_parallel(LayeredModel& m, LayeredModel::Layer& L, Placement& at, const std::string& mix, size_t W, int K, int R,
+                    const double* decay) {
+  bf16* weights = nullptr;
+  const ei_layer_spec& s = L.spec;
+  const std::string left = mix + "left.", right = mix + "right.";
+  L.dim_pad = round_up(s.dim, 16);
+  L.vdim_pad = round_up(s.vdim, 16);
+  L.lin_dim_pad = round_up(s.lin_dim, 16);
+  L.lin_vdim_pad = round_up(s.lin_vdim, 16);
+  L.attention_width = int(s.heads) * L.vdim_pad;
+  L.linear_width = int(s.lin_heads) * L.lin_vdim_pad;
+  const int H = int(s.heads), G = int(s.kv_heads), N = int(s.lin_heads);
+  L.in = at.linear(K, (H + G) * L.dim_pad + G * L.vdim_pad + 2 * N * (L.lin_dim_pad + L.lin_vdim_pad), &weights);
+  int row = at.rows_of(weights, K, 0, left + "q", H, int(s.dim), L.dim_pad, W);
+  row = at.rows_of(weights, K, row, left + "k", G, int(s.dim), L.dim_pad, W);
+  row = at.rows_of(weights, K, row, left + "v", G, int(s.vdim), L.vdim_pad, W);
+  row = at.rows_of(weights, K, row, right + "q", N, int(s.lin_dim), L.lin_dim_pad, W);
+  row = at.rows_of(weights, K, row, right + "k", N, int(s.lin_dim), L.lin_dim_pad, W);
+  row = at.rows_of(weights, K, row, right + "v", N, int(s.lin_vdim), L.lin_vdim_pad, W);
+  at.rows_of(weights, K, row, right + "g", N, int(s.lin_vdim), L.lin_vdim_pad, W);
+  L.out = at.linear(round_up(L.attention_width + L.linear_width, 64), R, &weights);
+  at.columns_of(weights, L.out.in, 0, left + "o", H, int(s.vdim), L.vdim_pad, W);
+  at.columns_of(weights, L.out.in, L.attention_width, right + "o", N, int(s.lin_vdim), L.lin_vdim_pad, W);
+  L.sink = at.host_values(at.values(left + "sink", H));
+  bf16* norm = at.reserve<bf16>(L.linear_width);
+  at.copy(norm, L.lin_vdim_pad, at.find(right + "norm", size_t(N) * s.lin_vdim, 0).data, s.lin_vdim, N, s.lin_vdim);
+  L.lin_norm = norm;
+  std::vector<float> powers;
+  for (int h = 0; h < N; ++h)
+    for (int n = 0; n <= kLightningChunk; ++n) powers.push_back(float(std::pow(decay[h], n)));
+  L.powers = at.host_values(powers);
+  L.rotation = rotation_of(m, at, s);
+}
+
+// Fused projection: q heads (unrotated | rotated) | latent | rotated key | gate.
+void place_latent(LayeredModel& m, LayeredModel::Layer& L, Placement& at, const std::string& mix, size_t W, int K, int R) {
+  bf16* weights = nullptr;
+  const ei_layer_spec& s = L.spec;
+  const int H = int(s.heads), dim = int(s.dim), rot = int(s.rot_dim), vdim = int(s.vdim), rank = int(s.kv_rank);
+  L.dim_pad = round_up(dim, 16);
+  L.rot_pad = round_up(rot, 16);
+  L.vdim_pad = round_up(vdim, 16);
+  L.rank_pad = round_up(rank, 64);
+  L.row_pad = round_up(L.rank_pad + L.rot_pad, 64);
+  const int query = L.dim_pad + L.rot_pad;
+  L.latent_at = H * query;
+  L.gate_at = L.latent_at + L.rank_pad + L.rot_pad;
+  L.in = at.linear(K, L.gate_at + H * L.vdim_pad, &weights);
+  const size_t q_rows = size_t(H) * (dim + rot);
+  at.some_rows_of(weights, K, 0, mix + "q", q_rows, 0, H, dim, dim + rot, query, W);
+  at.some_rows_of(weights, K, L.dim_pad, mix + "q", q_rows, dim, H, rot, dim + rot, query, W);
+  at.some_rows_of(weights, K, L.latent_at, mix + "dkv", size_t(rank) + rot, 0, 1, rank, rank, L.rank_pad, W);
+  at.some_rows_of(weights, K, L.latent_at + L.rank_pad, mix + "dkv", size_t(rank) + rot, rank, 1, rot, rot, L.rot_pad, W);
+  at.rows_of(weights, K, L.gate_at, mix + "g", H, vdim, L.vdim_pad, W);
+  L.latent_norm = at.vector(mix + "dkv.norm", rank, L.rank_pad);
+  L.expand = at.linear(L.rank_pad, H * (L.dim_pad + L.vdim_pad), &weights);
+  const int row = at.rows_of(weights, L.rank_pad, 0, mix + "uk", H, dim, L.dim_pad, rank);
+  at.rows_of(weights, L.rank_pad, row, mix + "uv", H, vdim, L.vdim_pad, rank);
+  L.out = at.linear(round_up(size_t(H) * L.vdim_pad, 64), R, &weights);
+  at.columns_of(weights, L.out.in, 0, mix + "o", H, vdim, L.vdim_pad, W);
+  L.rotation = rotation_of(m, at, s);
+}
+
+std::vector<float> exponentials(std::vector<float> v) {
+  for (float& x : v) x = float(std::exp(double(x)));
+  return v;
+}
+
+// Fused projection of both matrix recurrences: q heads | k heads | v heads | gate or first factors | step. A
+// state-space layer's C, B and x take the places of q, k and v.
+void place_state_space(LayeredModel::Layer& L, Placement& at, const std::string& mix, size_t W, int K, int R) {
+  bf16* weights = nullptr;
+  const ei_layer_spec& s = L.spec;
+  const int H = int(s.heads), G = L.key_heads = int(s.groups), state = int(s.state), vdim = int(s.vdim), taps = int(s.taps);
+  L.dim_pad = round_up(state, 16);
+  L.vdim_pad = round_up(vdim, 16);
+  const int keys = G * L.dim_pad, values = H * L.vdim_pad;
+  L.channels = 2 * keys + values;
+  L.gate_at = L.channels;
+  L.step_at = L.gate_at + values;
+  L.in = at.linear(K, L.step_at + round_up(H, 16), &weights);
+  // Rows of the checkpoint's projection: gate | x | B | C | step; its convolution covers x | B | C.
+  const size_t inner = size_t(H) * vdim, pairs = size_t(G) * state, rows = 2 * inner + 2 * pairs + H;
+  at.some_rows_of(weights, K, 0, mix + "in", rows, 2 * inner + pairs, G, state, state, L.dim_pad, W);
+  at.some_rows_of(weights, K, keys, mix + "in", rows, 2 * inner, G, state, state, L.dim_pad, W);
+  at.some_rows_of(weights, K, 2 * keys, mix + "in", rows, inner, H, vdim, vdim, L.vdim_pad, W);
+  at.some_rows_of(weights, K, L.gate_at, mix + "in", rows, 0, H, vdim, vdim, L.vdim_pad, W);
+  at.some_rows_of(weights, K, L.step_at, mix + "in", rows, 2 * inner + 2 * pairs, 1, H, H, H, W);
+  std::vector<float> conv(size_t(taps) * L.channels, 0.0f), bias(L.channels, 0.0f);
+  const size_t convolved = inner + 2 * pairs;
+  at.conv_of(conv, L.channels, 0, mix + "conv", convolved, inner + pairs, G, state, L.dim_pad, taps);
+  at.conv_of(conv, L.channels, keys, mix + "conv", convolved, inner, G, state, L.dim_pad, taps);
+  at.conv_of(conv, L.channels, 2 * keys, mix + "conv", convolved, 0, H, vdim, L.vdim_pad, taps);
+  L.conv = at.host_values(conv);
+  const std::vector<float> given = at.values(mix + "conv.b", convolved);
+  Placement::spread(bias, 0, given, inner + pairs, G, state, L.dim_pad);
+  Placement::spread(bias, keys, given, inner, G, state, L.dim_pad);
+  Placement::spread(bias, 2 * keys, given, 0, H, vdim, L.vdim_pad);
+  L.conv_bias = at.host_values(bias);
+  L.rate = at.host_values(exponentials(at.values(mix + "A_log", H)));
+  L.bias = at.host_values(at.values(mix + "dt_bias", H));
+  L.skip = at.host_values(at.values(mix + "D", H));
+  bf16* norm = at.reserve<bf16>(values);
+  at.copy(norm, L.vdim_pad, at.find(mix + "norm", inner, 0).data, vdim, H, vdim);
+  L.state_norm = norm;
+  L.out = at.linear(round_up(values, 64), R, &weights);
+  at.columns_of(weights, L.out.in, 0, mix + "o", H, vdim, L.vdim_pad, W);
+}
+
+void place_channel_delta(LayeredModel::Layer& L, Placement& at, const std::string& mix, size_t W, int K, int R) {
+  bf16* weights = nullptr;
+  const ei_layer_spec& s = L.spec;
+  const int H = int(s.heads), G = L.key_heads = int(s.kv_heads), dim = int(s.dim), vdim = int(s.vdim), taps = int(s.taps);
+  const int decay = int(s.decay_rank), gate = int(s.gate_rank);
+  L.dim_pad = round_up(dim, 16);
+  L.vdim_pad = round_up(vdim, 16);
+  const int keys = G * L.dim_pad, values = H * L.vdim_pad, decay_pad = round_up(decay, 64), gate_pad = round_up(gate, 64);
+  L.channels = 2 * keys + values;
+  L.first_at = L.channels;
+  L.step_at = L.first_at + decay_pad + gate_pad;
+  L.in = at.linear(K, L.step_at + round_up(H, 16), &weights);
+  at.rows_of(weights, K, 0, mix + "q", G, dim, L.dim_pad, W);
+  at.rows_of(weights, K, keys, mix + "k", G, dim, L.dim_pad, W);
+  at.rows_of(weights, K, 2 * keys, mix + "v", H, vdim, L.vdim_pad, W);
+  at.rows_of(weights, K, L.first_at, mix + "a1", 1, decay, decay_pad, W);
+  at.rows_of(weights, K, L.first_at + decay_pad, mix + "g1", 1, gate, gate_pad, W);
+  at.rows_of(weights, K, L.step_at, mix + "b", 1, H, H, W);
+  // Both second factors in one projection of both first factors' results: two blocks on the diagonal.
+  L.gate_at = H * L.dim_pad;
+  L.second = at.linear(decay_pad + gate_pad, H * L.dim_pad + values, &weights);
+  at.rows_of(weights, L.second.in, 0, mix + "a2", H, dim, L.dim_pad, decay);
+  at.rows_of(weights + decay_pad, L.second.in, L.gate_at, mix + "g2", H, vdim, L.vdim_pad, gate);
+  std::vector<float> conv(size_t(taps) * L.channels, 0.0f);
+  at.conv_of(conv, L.channels, 0, mix + "q.conv", size_t(G) * dim, 0, G, dim, L.dim_pad, taps);
+  at.conv_of(conv, L.channels, keys, mix + "k.conv", size_t(G) * dim, 0, G, dim, L.dim_pad, taps);
+  at.conv_of(conv, L.channels, 2 * keys, mix + "v.conv", size_t(H) * vdim, 0, H, vdim, L.vdim_pad, taps);
+  L.conv = at.host_values(conv);
+  L.rate = at.host_values(exponentials(at.values(mix + "A_log", H)));
+  L.bias = at.head_values(mix + "dt_bias", H, dim, L.dim_pad);
+  bf16* norm = at.reserve<bf16>(values);
+  const ei_named_tensor& shared = at.find(mix + "norm", vdim, 0);
+  for (int h = 0; h < H; ++h) at.copy(norm + size_t(h) * L.vdim_pad, vdim, shared.data, vdim, 1, vdim);
+  L.state_norm = norm;
+  L.out = at.linear(round_up(values, 64), R, &weights);
+  at.columns_of(weights, L.out.in, 0, mix + "o", H, vdim, L.vdim_pad, W);
 }
 
 void place(ei_model& model, const ei_layered_config& c, const ei_layer_spec* specs, Placement& at) {
@@ -142,77 +397,76 @@ void place(ei_model& model, const ei_layered_config& c, const ei_layer_spec* spe
   at.offset = 0;
   m.layers.assign(c.n_layers, {});
   m.rotations.clear();
-  m.embedding = at.matrix("embed", V, W, V, R);
-  if (c.loop_times) m.loop_step = at.matrix("loop.step", c.loop_times, W, c.loop_times, R);
-  m.final_norm = at.norm("final.norm", W, R);
   bf16* weights = nullptr;
   m.head = at.linear(K, m.vocab_stride, &weights);
-  at.rows_of(weights, K, 0, "head", 1, int(V), int(V), W);
+  if (c.tied_head) {
+    at.rows_of(weights, K, 0, "embed", 1, int(V), int(V), W);
+    m.embedding = weights;
+    m.embedding_stride = K;
+  } else {
+    at.rows_of(weights, K, 0, "head", 1, int(V), int(V), W);
+    m.embedding = at.matrix("embed", V, W, V, R);
+    m.embedding_stride = R;
+  }
+  if (c.pair_buckets) {
+    m.pairs.table = at.matrix("bigram", c.pair_buckets + 1, W, c.pair_buckets + 1, R);
+    m.pairs.stride = R;
+    m.pairs.buckets = c.pair_buckets;
+    m.pairs.mul_prev = c.pair_mul_prev % c.pair_buckets;
+    m.pairs.mul_cur = c.pair_mul_cur % c.pair_buckets;
+  }
+  if (c.loop_times) m.loop_step = at.matrix("loop.step", c.loop_times, W, c.loop_times, R);
+  if (m.parallel)
+    m.final_weight = at.vector("final.norm", W, R);
+  else
+    m.final_norm = at.norm("final.norm", W, R);
   for (size_t i = 0; i < c.n_layers; ++i) {
     const std::string p = "l" + std::to_string(i) + ".", mix = p + "mix.";
     LayeredModel::Layer& L = m.layers[i];
     const ei_layer_spec& s = L.spec = specs[i];
     L.spec.decay = nullptr;
-    L.norm1 = at.norm(p + "norm1", W, R);
-    L.norm1b = at.norm(p + "norm1b", W, R);
-    if (s.mixer == EI_MIXER_MIN_GRU) {
-      const int width = int(s.rnn_width);
-      L.width_pad = round_up(width, 16);
-      L.in = at.linear(K, 3 * L.width_pad, &weights);
-      int row = at.rows_of(weights, K, 0, mix + "z", 1, width, L.width_pad, W);
-      row = at.rows_of(weights, K, row, mix + "x", 1, width, L.width_pad, W);
-      at.rows_of(weights, K, row, mix + "g", 1, width, L.width_pad, W);
-      bf16* bias = at.reserve<bf16>(L.in.out);
-      at.copy(bias, width, at.find(mix + "z.b", width, 0).data, width, 1, width);
-      at.copy(bias + L.width_pad, width, at.find(mix + "x.b", width, 0).data, width, 1, width);
-      L.in.bias = bias;
-      L.out = at.linear(round_up(width, 64), R, &weights);
-      at.columns_of(weights, L.out.in, 0, mix + "o", 1, width, L.width_pad, W);
+    const bool feeds = s.mlp != EI_MLP_NONE;
+    if (m.parallel) {
+      L.norm1_weight = at.vector(p + "norm1", W, R);
+      L.scale1 = at.vector(p + "ls1", W, R);
+      if (feeds) {
+        L.norm2_weight = at.vector(p + "norm2", W, R);
+        L.scale2 = at.vector(p + "ls2", W, R);
+      }
     } else {
-      const std::string left = mix + "left.", right = mix + "right.";
-      L.dim_pad = round_up(s.dim, 16);
-      L.vdim_pad = round_up(s.vdim, 16);
-      L.lin_dim_pad = round_up(s.lin_dim, 16);
-      L.lin_vdim_pad = round_up(s.lin_vdim, 16);
-      L.attention_width = int(s.heads) * L.vdim_pad;
-      L.linear_width = int(s.lin_heads) * L.lin_vdim_pad;
-      const int H = int(s.heads), G = int(s.kv_heads), N = int(s.lin_heads);
-      L.in = at.linear(K, (H + G) * L.dim_pad + G * L.vdim_pad + 2 * N * (L.lin_dim_pad + L.lin_vdim_pad), &weights);
-      int row = at.rows_of(weights, K, 0, left + "q", H, int(s.dim), L.dim_pad, W);
-      row = at.rows_of(weights, K, row, left + "k", G, int(s.dim), L.dim_pad, W);
-      row = at.rows_of(weights, K, row, left + "v", G, int(s.vdim), L.vdim_pad, W);
-      row = at.rows_of(weights, K, row, right + "q", N, int(s.lin_dim), L.lin_dim_pad, W);
-      row = at.rows_of(weights, K, row, right + "k", N, int(s.lin_dim), L.lin_dim_pad, W);
-      row = at.rows_of(weights, K, row, right + "v", N, int(s.lin_vdim), L.lin_vdim_pad, W);
-      at.rows_of(weights, K, row, right + "g", N, int(s.lin_vdim), L.lin_vdim_pad, W);
-      L.out = at.linear(round_up(L.attention_width + L.linear_width, 64), R, &weights);
-      at.columns_of(weights, L.out.in, 0, left + "o", H, int(s.vdim), L.vdim_pad, W);
-      at.columns_of(weights, L.out.in, L.attention_width, right + "o", N, int(s.lin_vdim), L.lin_vdim_pad, W);
-      L.sink = at.host_values(at.base ? at.read(at.find(left + "sink", H, 0))
-                                      : (at.find(left + "sink", H, 0), std::vector<float>(H)));
-      bf16* norm = at.reserve<bf16>(L.linear_width);
-      at.copy(norm, L.lin_vdim_pad, at.find(right + "norm", size_t(N) * s.lin_vdim, 0).data, s.lin_vdim, N, s.lin_vdim);
-      L.lin_norm = norm;
-      std::vector<float> powers;
-      for (int h = 0; h < N; ++h)
-        for (int n = 0; n <= kLightningChunk; ++n) powers.push_back(float(std::pow(specs[i].decay[h], n)));
-      L.powers = at.host_values(powers);
-      for (L.rotation = 0; L.rotation < int(m.rotations.size()); ++L.rotation)
-        if (m.rotations[L.rotation].dims == int(s.rot_dims) && m.rotations[L.rotation].base == s.rot_base) break;
-      if (L.rotation == int(m.rotations.size())) m.rotations.push_back({int(s.rot_dims), s.rot_base});
+      L.norm1 = at.norm(p + "norm1", W, R);
+      L.norm1b = at.norm(p + "norm1b", W, R);
+      if (feeds) {
+        L.norm2 = at.norm(p + "norm2", W, R);
+        L.norm2b = at.norm(p + "norm2b", W, R);
+      }
     }
-    if (s.mlp != EI_MLP_NONE) {
-      L.norm2 = at.norm(p + "norm2", W, R);
-      L.norm2b = at.norm(p + "norm2b", W, R);
-      L.ff_pad = round_up(s.ff, 64);
+    switch (s.mixer) {
+      case EI_MIXER_MIN_GRU: place_min_gru(L, at, mix, W, K, R); break;
+      case EI_MIXER_PARALLEL: place_parallel(m, L, at, mix, W, K, R, specs[i].decay); break;
+      case EI_MIXER_LATENT_ATTENTION: place_latent(m, L, at, mix, W, K, R); break;
+      case EI_MIXER_STATE_SPACE: place_state_space(L, at, mix, W, K, R); break;
+      default: place_channel_delta(L, at, mix, W, K, R); break;
+    }
+    if (L.outer()) {
+      L.raw_rows = 1;  // a step reads the taps behind its first row while it records its own rows
+      while (L.raw_rows < kPendingRows + int(s.taps) - 1) L.raw_rows *= 2;
+    }
+    if (!feeds) continue;
+    L.ff_pad = round_up(s.ff, 64);
+    if (s.mlp == EI_MLP_RELU_SQUARED) {
+      L.up = at.linear(K, L.ff_pad, &weights);
+      L.up.activation = kActReluSquared;
+      at.rows_of(weights, K, 0, p + "mlp.up", 1, int(s.ff), L.ff_pad, W);
+    } else {
       L.gate_up = at.linear(K, 2 * L.ff_pad, &weights);
       L.gate_up.glu = kGluClamped;
       L.gate_up.glu_limit = float(s.limit);
       at.rows_of(weights, K, 0, p + "mlp.gate", 1, int(s.ff), L.ff_pad, W);
       at.rows_of(weights, K, L.ff_pad, p + "mlp.up", 1, int(s.ff), L.ff_pad, W);
-      L.down = at.linear(L.ff_pad, R, &weights);
-      at.columns_of(weights, L.ff_pad, 0, p + "mlp.down", 1, int(s.ff), L.ff_pad, W);
     }
+    L.down = at.linear(L.ff_pad, R, &weights);
+    at.columns_of(weights, L.ff_pad, 0, p + "mlp.down", 1, int(s.ff), L.ff_pad, W);
   }
 }
 
@@ -229,20 +483,20 @@ template <typename T>
 struct StepLinear;
 template <>
 struct StepLinear<bf16> {
-  static int sums(ei_session& s, const PreparedLinear& w, const bf16* x, int rows) {
+  static int sums(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, int x_stride = 0) {
     int ksplit = 1;
-    run_linear(s, w, x, rows, kEpiPartial, nullptr, 0, true, &ksplit);
+    run_linear(s, w, x, rows, kEpiPartial, nullptr, 0, true, &ksplit, x_stride);
     return ksplit;
   }
-  static void store(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, bf16* out) {
+  static void store(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, bf16* out, int x_stride = 0) {
     if (has_plan(s, w, rows, kEpiStore)) {
-      run_linear(s, w, x, rows, kEpiStore, out, w.out, true);
+      run_linear(s, w, x, rows, kEpiStore, out, w.out, true, nullptr, x_stride);
       return;
     }
-    const int ksplit = sums(s, w, x, rows);
+    const int ksplit = sums(s, w, x, rows, x_stride);
     tick(s);
     launch(splitk_store_kernel, dim3(std::min(s.model->multiprocessors * 8, (rows * w.out + 255) / 256)), dim3(256), 0,
-           s.stream, true, (const float*)s.partial, ksplit, rows, w.out, w.bias, out, w.out);
+           s.stream, true, (const float*)s.partial, ksplit, rows, w.out, w.bias, out, w.out, w.activation);
   }
   static void gated(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, bf16* pair, bf16* out) {
     if (has_plan(s, w, rows, kEpiSiluPair)) {
@@ -256,14 +510,13 @@ struct StepLinear<bf16> {
 };
 template <>
 struct StepLinear<float> {
-  static int sums(ei_session& s, const PreparedLinear& w, const float* x, int rows) {
-    tick(s);
-    launch_true32_linear(x, rows, w, s.partial, s.stream, true);
+  static int sums(ei_session& s, const PreparedLinear& w, const float* x, int rows, int x_stride = 0) {
+    store(s, w, x, rows, s.partial, x_stride);
     return 1;
   }
-  static void store(ei_session& s, const PreparedLinear& w, const float* x, int rows, float* out) {
+  static void store(ei_session& s, const PreparedLinear& w, const float* x, int rows, float* out, int x_stride = 0) {
     tick(s);
-    launch_true32_linear(x, rows, w, out, s.stream, true);
+    launch_true32_linear(x, x_stride ? x_stride : w.in, rows, w, out, s.stream, true);
   }
   static void gated(ei_session& s, const PreparedLinear& w, const float* x, int rows, float* pair, float* out) {
     store(s, w, x, rows, pair);
@@ -272,24 +525,28 @@ struct StepLinear<float> {
   }
 };
 
+// FP32 sums of a step projection in a buffer other than the session's.
+template <typename T>
+int sums_into(ei_session& s, const PreparedLinear& w, const T* x, int rows, float* buffer) {
+  struct Lend {
+    ei_session& s;
+    float* keep;
+    ~Lend() { s.partial = keep; }
+  } lend{s, s.partial};
+  s.partial = buffer;
+  return StepLinear<T>::sums(s, w, x, rows);
+}
+
 // The vocabulary head over at most 16 rows: FP32 logits in the session; with `parts` the argmax partials too.
 template <typename T>
 void run_head(ei_session& s, const T* rows_in, int rows, int* parts) {
   const LayeredModel& m = *s.model->layered;
   LayeredSession& L = *s.layered;
-  float* keep = s.partial;
-  s.partial = L.head_partial ? L.head_partial : L.logits;
-  int ksplit = 1;
-  try {
-    ksplit = StepLinear<T>::sums(s, m.head, rows_in, rows);
-  } catch (...) {
-    s.partial = keep;
-    throw;
-  }
-  s.partial = keep;
-  if (L.head_partial) {
+  const int ksplit = sums_into<T>(s, m.head, rows_in, rows, L.head_partial ? L.head_partial : L.logits);
+  if (L.head_partial || m.softcap > 0.0f) {
     tick(s);
-    launch_sum_partials(L.head_partial, ksplit, size_t(rows) * m.vocab_stride, L.logits, s.model->multiprocessors, s.stream, true);
+    launch_sum_partials(L.head_partial ? L.head_partial : L.logits, ksplit, size_t(rows) * m.vocab_stride, m.softcap, L.logits,
+                        s.model->multiprocessors, s.stream, true);
   }
   if (!parts) return;
   const size_t vocab = s.model->config.vocab_size;
@@ -304,6 +561,7 @@ struct Buffers {
   const uint32_t* tokens;  // of the rows, for the loop's embedding injection
   float *residual, *linear_out;
   void *normed, *fused, *mixed, *gate_up, *act;
+  void *second_normed, *second;  // a parallel block's other norm; second factors of a low-rank projection
 };
 
 DynamicTanh norm_ahead(const LayeredModel& m, size_t run) {
@@ -342,9 +600,40 @@ void end_of_run(const ei_session& s, const Buffers& b, size_t run, SublayerJoinP
   j.before = norm_ahead(m, run + 1);
 }
 
+// The norms that open layer run `run` of a parallel model, or the final one.
+RowNorms row_norms(const LayeredModel& m, const Buffers& b, size_t run) {
+  RowNorms n;
+  n.width = m.width;
+  n.stride = m.normed_stride;
+  n.eps = m.eps;
+  n.normed_first = b.normed;
+  n.first = m.final_weight;
+  if (run < m.runs.size()) {
+    const auto& l = m.layers[m.runs[run].layer];
+    n.first = l.norm1_weight;
+    n.second = l.norm2_weight;
+    n.normed_second = b.second_normed;
+  }
+  return n;
+}
+
 template <typename T>
 void enqueue_embed(ei_session& s, const Buffers& b, const EmbedParams& token) {
   const LayeredModel& m = *s.model->layered;
+  tick(s);
+  if (m.parallel) {
+    ParallelEmbedParams e{};
+    e.token = token;
+    e.table = m.embedding;
+    e.table_stride = m.embedding_stride;
+    e.pairs = m.pairs;
+    e.pairs.history = s.layered->history;
+    e.residual = b.residual;
+    e.residual_stride = m.residual_stride;
+    e.norms = row_norms(m, b, 0);
+    launch_parallel_embed<T>(e, s.stream, false);
+    return;
+  }
   LayeredEmbedParams e{};
   e.token = token;
   e.table = m.embedding;
@@ -354,8 +643,33 @@ void enqueue_embed(ei_session& s, const Buffers& b, const EmbedParams& token) {
   e.residual_stride = m.residual_stride;
   e.normed = b.normed;
   e.normed_stride = m.normed_stride;
-  tick(s);
   launch_layered_embed<T>(e, s.stream, false);
+}
+
+// The join that ends layer run `run` of a parallel model.
+template <typename T>
+void enqueue_parallel_join(ei_session& s, const Buffers& b, size_t run, const float* mixed, int mixed_ksplit, const float* fed,
+                           int fed_ksplit) {
+  const LayeredModel& m = *s.model->layered;
+  const LayeredSession& L = *s.layered;
+  const auto& l = m.layers[m.runs[run].layer];
+  ParallelJoinParams j{};
+  j.mixed = mixed;
+  j.mixed_ksplit = mixed_ksplit;
+  j.fed = fed;
+  j.fed_ksplit = fed_ksplit;
+  j.rows = b.rows;
+  j.mixed_scale = l.scale1;
+  j.fed_scale = l.scale2;
+  j.residual = b.residual;
+  j.residual_stride = m.residual_stride;
+  if (L.tap) {
+    j.tap = L.tap + run * L.tap_rows * m.width;
+    j.tap_width = m.width;
+  }
+  j.norms = row_norms(m, b, run + 1);
+  tick(s);
+  launch_parallel_join<T>(j, s.stream, true);
 }
 
 MixerPrepareParams prepare_params(const ei_session& s, const LayeredModel::Layer& l, const LayeredSession::Run& r,
@@ -394,6 +708,8 @@ SizedAttentionParams attention_params(ei_session& s, const LayeredModel::Layer& 
   a.q_stride = l.in.out;
   a.k = r.k_cache;
   a.v = r.v_cache;
+  a.k_stride = int(l.spec.kv_heads) * l.dim_pad;
+  a.v_stride = int(l.spec.kv_heads) * l.vdim_pad;
   a.rows = b.rows;
   a.heads = int(l.spec.heads);
   a.kv_heads = int(l.spec.kv_heads);
@@ -485,13 +801,185 @@ MinGruParams min_gru_params(const ei_session& s, const LayeredModel::Layer& l, c
   return g;
 }
 
+LatentParams latent_params(const ei_session& s, const LayeredModel::Layer& l, const LayeredSession::Run& r, const Buffers& b) {
+  LatentParams p{};
+  p.fused = b.fused;
+  p.rows = b.rows;
+  p.stride = l.in.out;
+  p.latent_at = l.latent_at;
+  p.gate_at = l.gate_at;
+  p.heads = int(l.spec.heads);
+  p.dim_pad = l.dim_pad;
+  p.vdim_pad = l.vdim_pad;
+  p.rank = int(l.spec.kv_rank);
+  p.rank_pad = l.rank_pad;
+  p.rot_pad = l.rot_pad;
+  p.rot_dims = int(l.spec.rot_dims);
+  p.row_pad = l.row_pad;
+  p.eps = s.model->layered->eps;
+  p.norm = l.latent_norm;
+  p.rotation = s.layered->rotations[l.rotation];
+  p.expand = l.expand.dense;
+  p.cache = r.latent;
+  p.control = s.control;
+  p.capacity = int(s.capacity);
+  p.query = s.layered->latent_query;
+  p.out = b.mixed;
+  p.out_stride = l.out.in;
+  return p;
+}
+
+// Attention of a step's queries over the latent cache; partials in the session's scratch, or (plain form) finished
+// latents in `out`.
+SizedAttentionParams latent_scores(ei_session& s, const LayeredModel::Layer& l, const LayeredSession::Run& r, const Buffers& b) {
+  SizedAttentionParams a{};
+  a.q = s.layered->latent_query;
+  a.q_stride = int(l.spec.heads) * l.row_pad;
+  a.k = a.v = r.latent;
+  a.k_stride = a.v_stride = l.row_pad;
+  a.rows = b.rows;
+  a.heads = int(l.spec.heads);
+  a.kv_heads = 1;
+  a.dim_pad = l.row_pad;
+  a.vdim_pad = l.rank_pad;
+  a.scale = float(l.spec.scale);
+  a.out_scale = 1.0f;
+  a.device_offset = &s.control->context;
+  a.capacity = int(s.capacity);
+  a.chunk = s.attention_chunk;
+  a.max_splits = s.attention_splits;
+  a.scratch = s.attention_scratch;
+  a.out = s.layered->latent_out;
+  a.out_stride = int(l.spec.heads) * l.rank_pad;
+  a.status = &s.control->status;
+  if (s.inject_attention_polls) {
+    a.wait_limit = s.inject_attention_polls;
+    a.fault_tx = 16;
+    s.inject_attention_polls = 0;  // one launch only
+  }
+  return a;
+}
+
+OuterStateParams outer_params(const ei_session& s, const LayeredModel::Layer& l, const LayeredSession::Run& r, const Buffers& b) {
+  OuterStateParams p{};
+  p.delta = l.delta();
+  p.fused = b.fused;
+  p.rows = b.rows;
+  p.stride = l.in.out;
+  p.step_at = l.step_at;
+  p.heads = int(l.spec.heads);
+  p.key_heads = l.key_heads;
+  p.dim = int(l.delta() ? l.spec.dim : l.spec.state);
+  p.dim_pad = l.dim_pad;
+  p.vdim = int(l.spec.vdim);
+  p.vdim_pad = l.vdim_pad;
+  p.taps = int(l.spec.taps);
+  p.conv = l.conv;
+  p.conv_bias = l.conv_bias;
+  p.raw = r.raw;
+  p.raw_rows = l.raw_rows;
+  p.decay = b.second;
+  p.decay_stride = l.second.out;
+  p.rate = l.rate;
+  p.bias = l.bias;
+  p.skip = l.skip;
+  p.ring_k = r.ring_key;
+  p.ring_g = r.ring_decay;
+  p.ring_u = r.ring_write;
+  p.q = s.layered->state_q;
+  p.v = s.layered->state_v;
+  p.beta = s.layered->state_beta;
+  p.state = r.state;
+  p.control = s.control;
+  p.capacity = int(s.capacity);
+  p.out = b.linear_out;
+  return p;
+}
+
+template <typename T>
+StateFinishParams state_finish_params(const ei_session& s, const LayeredModel::Layer& l, const Buffers& b) {
+  StateFinishParams f{};
+  f.in = b.linear_out;
+  f.rows = b.rows;
+  f.heads = int(l.spec.heads);
+  f.vdim = int(l.spec.vdim);
+  f.vdim_pad = l.vdim_pad;
+  f.gate_first = !l.delta();
+  f.groups = int(l.delta() ? l.spec.heads : l.spec.norm_groups);
+  f.gate = static_cast<const T*>(l.delta() ? b.second : b.fused) + l.gate_at;
+  f.gate_stride = l.delta() ? l.second.out : l.in.out;
+  f.norm = l.state_norm;
+  f.eps = s.model->layered->eps;
+  f.out = b.mixed;
+  f.out_stride = l.out.in;
+  return f;
+}
+
+// A layer's token mixer from the normed rows to the activations of its output projection, at most 16 rows.
+template <typename T>
+void enqueue_mixer_step(ei_session& s, const LayeredModel::Layer& l, const LayeredSession::Run& r, const Buffers& b) {
+  const ei_model& model = *s.model;
+  const bool pdl = true, true32 = model.layered->true32;
+  StepLinear<T>::store(s, l.in, static_cast<const T*>(b.normed), b.rows, static_cast<T*>(b.fused));
+  switch (l.spec.mixer) {
+    case EI_MIXER_MIN_GRU:
+      tick(s);
+      launch_min_gru_step<T>(min_gru_params<T>(s, l, r, b), s.stream, pdl);
+      return;
+    case EI_MIXER_PARALLEL: {
+      tick(s);
+      launch_mixer_prepare<T>(prepare_params(s, l, r, b, true), s.stream, pdl);
+      const SizedAttentionParams a = attention_params(s, l, r, b);
+      const bool tiled = !true32 && sized_attention_ok(l.dim_pad, l.vdim_pad);
+      tick(s);
+      if (tiled)
+        launch_sized_attention_step(a, s.stream, pdl);
+      else
+        launch_plain_attention<T>(a, s.stream, pdl);
+      tick(s);
+      launch_lightning_step<T>(lightning_params<T>(s, l, r, b), s.stream, pdl);
+      tick(s);
+      launch_mixer_finish<T>(finish_params<T>(s, l, b, a, tiled), s.stream, pdl);
+      return;
+    }
+    case EI_MIXER_LATENT_ATTENTION: {
+      const LatentParams p = latent_params(s, l, r, b);
+      const bool tiled = !true32 && latent_attention_ok(l.rank_pad, l.row_pad, model.smem_limit);
+      tick(s);
+      launch_latent_prepare<T>(p, true, s.stream, pdl);
+      const SizedAttentionParams a = latent_scores(s, l, r, b);
+      tick(s);
+      if (tiled)
+        launch_latent_attention(a, l.row_pad, model.smem_limit, s.stream, pdl);
+      else
+        launch_plain_attention<T>(a, s.stream, pdl);
+      tick(s);
+      launch_latent_expand<T>(p, a, tiled, s.stream, pdl);
+      return;
+    }
+    default: {
+      if (l.delta())
+        StepLinear<T>::store(s, l.second, static_cast<const T*>(b.fused) + l.first_at, b.rows, static_cast<T*>(b.second), l.in.out);
+      const OuterStateParams p = outer_params(s, l, r, b);
+      tick(s);
+      launch_outer_prepare<T>(p, s.stream, pdl);
+      tick(s);
+      launch_outer_step(p, s.stream, pdl);
+      tick(s);
+      launch_state_finish<T>(state_finish_params<T>(s, l, b), s.stream, pdl);
+      return;
+    }
+  }
+}
+
 template <typename T>
 void enqueue_step_as(ei_session& s, int rows, StepKind kind) {
   const LayeredModel& m = *s.model->layered;
   LayeredSession& L = *s.layered;
   const bool pdl = true;
   const size_t before = s.launches;
-  const Buffers b{rows, s.step_tokens, L.residual, L.linear_out, L.normed, L.fused, L.mixed, L.gate_up, L.act};
+  const Buffers b{rows,    s.step_tokens, L.residual, L.linear_out,    L.normed, L.fused,
+                  L.mixed, L.gate_up,     L.act,      L.second_normed, L.second};
   EmbedParams token{};
   token.tokens = kind == kVerifyDevice ? nullptr : s.tokens;
   token.source = kind == kVerifyDevice ? s.draft_source : nullptr;
@@ -504,38 +992,38 @@ void enqueue_step_as(ei_session& s, int rows, StepKind kind) {
 
   for (size_t run = 0; run < m.runs.size(); ++run) {
     const LayeredModel::Layer& l = m.layers[m.runs[run].layer];
-    const LayeredSession::Run& r = L.runs[run];
-    StepLinear<T>::store(s, l.in, static_cast<const T*>(b.normed), rows, static_cast<T*>(b.fused));
-    if (l.spec.mixer == EI_MIXER_MIN_GRU) {
-      tick(s);
-      launch_min_gru_step<T>(min_gru_params<T>(s, l, r, b), s.stream, pdl);
-    } else {
-      tick(s);
-      launch_mixer_prepare<T>(prepare_params(s, l, r, b, true), s.stream, pdl);
-      const SizedAttentionParams a = attention_params(s, l, r, b);
-      const bool tiled = !m.true32 && sized_attention_ok(l.dim_pad, l.vdim_pad);
-      tick(s);
-      if (tiled)
-        launch_sized_attention_step(a, s.stream, pdl);
+    enqueue_mixer_step<T>(s, l, L.runs[run], b);
+    const bool feeds = l.spec.mlp != EI_MLP_NONE;
+    const T *normed = static_cast<const T*>(m.parallel ? b.second_normed : b.normed), *mixed = static_cast<const T*>(b.mixed);
+    T* act = static_cast<T*>(b.act);
+    const auto activate = [&] {
+      if (l.spec.mlp == EI_MLP_RELU_SQUARED)
+        StepLinear<T>::store(s, l.up, normed, rows, act);
       else
-        launch_plain_attention<T>(a, s.stream, pdl);
-      tick(s);
-      launch_lightning_step<T>(lightning_params<T>(s, l, r, b), s.stream, pdl);
-      tick(s);
-      launch_mixer_finish<T>(finish_params<T>(s, l, b, a, tiled), s.stream, pdl);
+        StepLinear<T>::gated(s, l.gate_up, normed, rows, static_cast<T*>(b.gate_up), act);
+    };
+    if (m.parallel) {
+      const int mixed_ksplit = sums_into<T>(s, l.out, mixed, rows, L.mixed_partial);
+      int fed_ksplit = 0;
+      if (feeds) {
+        activate();
+        fed_ksplit = StepLinear<T>::sums(s, l.down, act, rows);
+      }
+      enqueue_parallel_join<T>(s, b, run, L.mixed_partial, mixed_ksplit, feeds ? s.partial : nullptr, fed_ksplit);
+      continue;
     }
-    int ksplit = StepLinear<T>::sums(s, l.out, static_cast<const T*>(b.mixed), rows);
+    int ksplit = StepLinear<T>::sums(s, l.out, mixed, rows);
     SublayerJoinParams j = join_params(s, b, s.partial, ksplit);
     j.after = l.norm1b;
-    if (l.spec.mlp == EI_MLP_NONE)
-      end_of_run(s, b, run, j);
-    else
+    if (feeds)
       j.before = l.norm2;
+    else
+      end_of_run(s, b, run, j);
     tick(s);
     launch_sublayer_join<T>(j, s.stream, pdl);
-    if (l.spec.mlp == EI_MLP_NONE) continue;
-    StepLinear<T>::gated(s, l.gate_up, static_cast<const T*>(b.normed), rows, static_cast<T*>(b.gate_up), static_cast<T*>(b.act));
-    ksplit = StepLinear<T>::sums(s, l.down, static_cast<const T*>(b.act), rows);
+    if (!feeds) continue;
+    activate();
+    ksplit = StepLinear<T>::sums(s, l.down, act, rows);
     j = join_params(s, b, s.partial, ksplit);
     j.after = l.norm2b;
     end_of_run(s, b, run, j);
@@ -572,11 +1060,18 @@ void create_layered_model(ei_model& model, const ei_layered_config& c, const ei_
     throw std::invalid_argument("Layered decoder: sizes must be positive and in range");
   if (c.loop_times && (c.loop_times > 65536 || c.loop_start >= c.loop_stop || c.loop_stop > c.n_layers))
     throw std::invalid_argument("Layered decoder: the loop must span existing layers");
+  if (c.pair_buckets && !positive(c.pair_buckets, kMany)) throw std::invalid_argument("Layered decoder: pair table out of range");
+  if (!std::isfinite(c.logit_softcap) || c.logit_softcap < 0.0) throw std::invalid_argument("Layered decoder: invalid logit cap");
+  if (c.block != EI_BLOCK_SANDWICH && c.block != EI_BLOCK_PARALLEL) throw std::invalid_argument("Layered decoder: unknown block form");
+  if (c.block == EI_BLOCK_PARALLEL ? c.loop_times != 0 : c.pair_buckets != 0)
+    throw std::invalid_argument("Layered decoder: loops go with sandwich blocks, the pair table with parallel ones");
   for (size_t i = 0; i < c.n_layers; ++i) validate_layer(specs[i]);
 
   model.layered = std::make_shared<LayeredModel>();
   LayeredModel& m = *model.layered;
   m.true32 = c.true32 != 0;
+  m.parallel = c.block == EI_BLOCK_PARALLEL;
+  m.softcap = float(c.logit_softcap);
   m.width = int(c.width);
   m.residual_stride = round_up(c.width, 16);
   m.normed_stride = round_up(c.width, 64);
@@ -628,7 +1123,7 @@ void create_layered_model(ei_model& model, const ei_layered_config& c, const ei_
   model.weight_bytes = m.head.bytes;
   for (const auto& run : m.runs) {
     const auto& l = m.layers[run.layer];
-    model.weight_bytes += l.in.bytes + l.out.bytes + l.gate_up.bytes + l.down.bytes;
+    model.weight_bytes += l.in.bytes + l.out.bytes + l.gate_up.bytes + l.up.bytes + l.down.bytes + l.expand.bytes + l.second.bytes;
   }
   model.prompt_ready = !m.true32;
   for (const auto& l : m.layers) {
@@ -636,15 +1131,23 @@ void create_layered_model(ei_model& model, const ei_layered_config& c, const ei_
     m.max_mixed = std::max(m.max_mixed, l.out.in);
     m.max_gate_up = std::max(m.max_gate_up, l.gate_up.out);
     m.max_ff = std::max(m.max_ff, l.ff_pad);
-    m.max_linear = std::max(m.max_linear, l.linear_width);
+    m.max_linear = std::max(m.max_linear, l.outer() ? int(l.spec.heads) * l.vdim_pad : l.linear_width);
     m.max_rnn = std::max(m.max_rnn, l.width_pad);
+    if (l.outer()) {
+      m.max_second = std::max(m.max_second, l.second.out);
+      m.max_state_keys = std::max(m.max_state_keys, l.key_heads * l.dim_pad);
+      m.max_state_heads = std::max(m.max_state_heads, int(l.spec.heads));
+      model.prompt_ready = false;
+    }
+    if (l.spec.mixer == EI_MIXER_LATENT_ATTENTION) model.prompt_ready = false;
     if (l.spec.mixer == EI_MIXER_PARALLEL) {
       m.max_chunk_state = std::max(m.max_chunk_state, size_t(l.linear_width) * l.lin_dim_pad);
       model.prompt_ready = model.prompt_ready && sized_attention_ok(l.dim_pad, l.vdim_pad) &&
                            lightning_prompt_ok(l.lin_dim_pad, l.lin_vdim_pad);
     }
+    const PreparedLinear& widen = l.spec.mlp == EI_MLP_RELU_SQUARED ? l.up : l.gate_up;
     model.prompt_ready = model.prompt_ready && prompt_linear_ok(l.in) && prompt_linear_ok(l.out) &&
-                         (l.spec.mlp == EI_MLP_NONE || (prompt_linear_ok(l.gate_up) && prompt_linear_ok(l.down)));
+                         (l.spec.mlp == EI_MLP_NONE || (prompt_linear_ok(widen) && prompt_linear_ok(l.down)));
   }
 }
 
@@ -657,9 +1160,15 @@ void create_layered_session(ei_session& s) {
   s.attention_chunk = attention_chunk_for(s.capacity);
   s.attention_splits = int((s.capacity + s.attention_chunk - 1) / s.attention_chunk);
   L.token_rows = (s.capacity + 63) / 64 * 64;
-  size_t partial = 0, scratch = 0;
+  size_t partial = 0, scratch = 0, mixed_partial = 0, latent_query = 0, latent_out = 0;
   for (const auto& l : m.layers) {
-    for (const PreparedLinear* w : {&l.in, &l.out, &l.gate_up, &l.down}) partial = std::max(partial, partial_floats(*w));
+    for (const PreparedLinear* w : {&l.in, &l.out, &l.gate_up, &l.up, &l.down, &l.second}) partial = std::max(partial, partial_floats(*w));
+    if (m.parallel) mixed_partial = std::max(mixed_partial, partial_floats(l.out));
+    if (l.spec.mixer == EI_MIXER_LATENT_ATTENTION) {
+      scratch = std::max(scratch, sized_attention_scratch_bytes(kMaxRows, l.spec.heads, l.rank_pad, s.capacity));
+      latent_query = std::max(latent_query, size_t(l.spec.heads) * l.row_pad);
+      latent_out = std::max(latent_out, size_t(l.spec.heads) * l.rank_pad);
+    }
     if (l.spec.mixer == EI_MIXER_PARALLEL)
       scratch = std::max(scratch, sized_attention_scratch_bytes(kMaxRows, l.spec.heads, l.vdim_pad, s.capacity));
   }
@@ -692,6 +1201,17 @@ void create_layered_session(ei_session& s) {
   take(L.act, kMaxRows * m.max_ff * T);
   take(L.head_rows, kMaxRows * m.normed_stride * T);
   take(s.gather_index, kMaxRows * sizeof(int32_t));
+  if (m.parallel) {
+    take(L.mixed_partial, mixed_partial * sizeof(float));
+    take(L.second_normed, kMaxRows * m.normed_stride * T);
+  }
+  if (m.pairs.table) take(L.history, s.capacity * sizeof(uint32_t));
+  take(L.second, size_t(kMaxRows) * m.max_second * T);
+  take(L.state_q, size_t(kMaxRows) * m.max_state_keys * sizeof(float));
+  take(L.state_v, size_t(kMaxRows) * m.max_linear * sizeof(float));
+  take(L.state_beta, size_t(kMaxRows) * m.max_state_heads * sizeof(float));
+  take(L.latent_query, kMaxRows * latent_query * T);
+  take(L.latent_out, kMaxRows * latent_out * T);
   L.rotations.resize(m.rotations.size());
   for (size_t i = 0; i < m.rotations.size(); ++i) take(L.rotations[i], s.capacity * (m.rotations[i].dims / 2) * sizeof(float2));
   L.runs.resize(m.runs.size());
@@ -702,6 +1222,15 @@ void create_layered_session(ei_session& s) {
       take(r.state, size_t(l.width_pad) * sizeof(float));
       take(r.ring_gate, size_t(kRingRows) * l.width_pad * sizeof(float));
       take(r.ring_candidate, size_t(kRingRows) * l.width_pad * sizeof(float));
+    } else if (l.spec.mixer == EI_MIXER_LATENT_ATTENTION) {
+      take(r.latent, L.token_rows * l.row_pad * T);
+    } else if (l.outer()) {
+      const size_t heads = l.spec.heads;
+      take(r.raw, size_t(l.raw_rows) * l.channels * T);
+      take(r.ring_key, size_t(kRingRows) * l.key_heads * l.dim_pad * sizeof(float));
+      take(r.ring_decay, size_t(kRingRows) * heads * (l.delta() ? l.dim_pad : 1) * sizeof(float));
+      take(r.ring_write, size_t(kRingRows) * heads * l.vdim_pad * sizeof(float));
+      take(r.state, heads * l.vdim_pad * l.dim_pad * sizeof(float));
     } else {
       take(r.k_cache, L.token_rows * l.spec.kv_heads * l.dim_pad * T);
       take(r.v_cache, L.token_rows * l.spec.kv_heads * l.vdim_pad * T);
@@ -717,7 +1246,7 @@ void create_layered_session(ei_session& s) {
   }
   EI_CUDA(cudaMemset(s.arena, 0, total));
   for (size_t i = 0; i < m.rotations.size(); ++i)
-    launch_rotation_table(L.rotations[i], s.capacity, m.rotations[i].dims, m.rotations[i].base, nullptr);
+    launch_rotation_table(L.rotations[i], s.capacity, m.rotations[i].frequencies, m.rotations[i].dims / 2, m.rotations[i].length, nullptr);
   EI_CUDA(cudaStreamSynchronize(nullptr));
 }
 
@@ -775,7 +1304,8 @@ void enqueue_layered_segment(ei_session& s, int rows) {
   LayeredSession& L = *s.layered;
   auto& ws = model.prompt;
   const bool pdl = true;
-  const Buffers b{rows, ws.step_tokens, m.residual, m.linear_out, ws.normed, ws.qkv, ws.attention, ws.gate_up, ws.act};
+  const Buffers b{rows,    ws.step_tokens, m.residual, m.linear_out,    ws.normed, ws.qkv,
+                  ws.attention, ws.gate_up, ws.act, nullptr, nullptr};
   EmbedParams token{};
   token.tokens = ws.tokens;
   token.control = s.control;

@@ -1,6 +1,6 @@
 // Elementwise and per-row kernels of decoders described layer by layer: embedding, sublayer joins, the preparation of
 // a mixer's heads, the end of a mixer, the gated recurrence, the clamped gated unit, and FP32 linears.
-#include "layered.cuh"
+#include "layered_device.cuh"
 
 #include <algorithm>
 #include <cmath>
@@ -8,38 +8,6 @@
 
 namespace ei {
 namespace {
-
-__device__ __forceinline__ float value_of(bf16 x) { return __bfloat162float(x); }
-__device__ __forceinline__ float value_of(float x) { return x; }
-__device__ __forceinline__ void store_value(bf16* p, float x) { *p = __float2bfloat16_rn(x); }
-__device__ __forceinline__ void store_value(float* p, float x) { *p = x; }
-__device__ __forceinline__ float2 load_pair(const bf16* p) {
-  const uint32_t v = *reinterpret_cast<const uint32_t*>(p);
-  return make_float2(bf16_lo(v), bf16_hi(v));
-}
-__device__ __forceinline__ float2 load_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
-__device__ __forceinline__ void store_pair(bf16* p, float a, float b) { *reinterpret_cast<uint32_t*>(p) = pack_bf16(a, b); }
-__device__ __forceinline__ void store_pair(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
-__device__ __forceinline__ float4 load_quad(const bf16* p) {
-  const uint2 v = *reinterpret_cast<const uint2*>(p);
-  return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y));
-}
-__device__ __forceinline__ float4 load_quad(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ void store_quad(bf16* p, float4 v) {
-  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
-}
-__device__ __forceinline__ void store_quad(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-
-__device__ __forceinline__ float sigmoid_value(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-x)); }
-// The fast exponential and quotient (a few units in the last place of FP32) for kernels on BF16 activations.
-__device__ __forceinline__ float quick_sigmoid(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
-__device__ __forceinline__ float quick_candidate(float u) { return u >= 0.0f ? u + 0.5f : quick_sigmoid(u); }
-template <typename T>
-__device__ __forceinline__ float sigmoid_for(float x) { return sizeof(T) == 2 ? quick_sigmoid(x) : sigmoid_value(x); }
-template <typename T>
-__device__ __forceinline__ float silu_for(float x) { return sizeof(T) == 2 ? x * quick_sigmoid(x) : silu_exact(x); }
-__device__ __forceinline__ float4 add(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
 
 __device__ __forceinline__ float4 dynamic_tanh(const DynamicTanh& n, int i, float4 x) {
   const float4 w = load_quad(n.weight + i), b = load_quad(n.bias + i);
@@ -201,15 +169,6 @@ __global__ void __launch_bounds__(128) mixer_prepare_kernel(const MixerPreparePa
     store_quad(x + i, v);
     if (ring) store_quad(ring + i, v);
   }
-}
-
-__device__ __forceinline__ float block_total(float v, float* shared) {
-  v = warp_sum(v);
-  if ((threadIdx.x & 31) == 0) shared[threadIdx.x >> 5] = v;
-  __syncthreads();
-  float total = 0.0f;
-  for (int w = 0; w < int(blockDim.x >> 5); ++w) total += shared[w];
-  return total;
 }
 
 // Blocks [0, rows * heads) merge one (row, head) of the split attention (when asked to); the last `rows` blocks finish
@@ -476,19 +435,20 @@ __global__ void __launch_bounds__(256) gather_rows_kernel(const T* source, const
   for (int i = threadIdx.x; i < stride; i += 256) out[size_t(blockIdx.x) * stride + i] = from[i];
 }
 
-__global__ void __launch_bounds__(256) sum_partials_kernel(const float* partial, int ksplit, size_t count, float* out) {
+__global__ void __launch_bounds__(256) sum_partials_kernel(const float* partial, int ksplit, size_t count, float cap, float* out) {
   grid_dependency_wait();
   for (size_t i = size_t(blockIdx.x) * 256 + threadIdx.x; i < count; i += size_t(gridDim.x) * 256) {
     float sum = partial[i];
     for (int s = 1; s < ksplit; ++s) sum += partial[s * count + i];
-    out[i] = sum;
+    out[i] = cap > 0.0f ? cap * tanhf(sum / cap) : sum;
   }
 }
 
 // A warp per output feature, the rows' products summed lane by lane and then across the warp.
 constexpr int kTrue32Tile = 256;
-__global__ void __launch_bounds__(256) true32_linear_kernel(const float* x, int rows, const bf16* w, const bf16* bias,
-                                                            int in, int out_features, float* out) {
+__global__ void __launch_bounds__(256) true32_linear_kernel(const float* x, int x_stride, int rows, const bf16* w,
+                                                            const bf16* bias, int activation, int in, int out_features,
+                                                            float* out) {
   __shared__ float tile[kMaxRows][kTrue32Tile];
   grid_dependency_wait();
   grid_launch_dependents();
@@ -501,7 +461,7 @@ __global__ void __launch_bounds__(256) true32_linear_kernel(const float* x, int 
     __syncthreads();
     for (int i = threadIdx.x; i < rows * kTrue32Tile; i += 256) {
       const int r = i / kTrue32Tile, k = i - r * kTrue32Tile;
-      tile[r][k] = k < width ? x[size_t(r) * in + first + k] : 0.0f;
+      tile[r][k] = k < width ? x[size_t(r) * x_stride + first + k] : 0.0f;
     }
     __syncthreads();
     if (n < out_features) {
@@ -518,17 +478,17 @@ __global__ void __launch_bounds__(256) true32_linear_kernel(const float* x, int 
   for (int r = 0; r < kMaxRows; ++r) {
     if (r < rows) {
       const float sum = warp_sum(acc[r]);
-      if (lane == 0) out[size_t(r) * out_features + n] = sum + (bias ? __bfloat162float(bias[n]) : 0.0f);
+      if (lane == 0)
+        out[size_t(r) * out_features + n] = activated_value(activation, sum + (bias ? __bfloat162float(bias[n]) : 0.0f));
     }
   }
 }
 
-__global__ void rotation_table_kernel(float2* table, size_t positions, int half, int dims, double log_base) {
+__global__ void rotation_table_kernel(float2* table, size_t positions, const double* frequencies, int half, double length) {
   for (size_t i = size_t(blockIdx.x) * blockDim.x + threadIdx.x; i < positions * half; i += size_t(gridDim.x) * blockDim.x) {
-    const double angle = double(i / half) * exp(log_base * (-2.0 * double(i % half) / double(dims)));
     double s, c;
-    sincos(angle, &s, &c);
-    table[i] = make_float2(float(c), float(s));
+    sincos(double(i / half) * frequencies[i % half], &s, &c);
+    table[i] = make_float2(float(c * length), float(s * length));
   }
 }
 
@@ -573,21 +533,23 @@ template <typename T>
 void launch_gather_rows(const T* source, const int32_t* index, int count, int stride, T* out, cudaStream_t stream) {
   launch(gather_rows_kernel<T>, dim3(count), dim3(256), 0, stream, false, source, index, stride, out);
 }
-void launch_sum_partials(const float* partial, int ksplit, size_t count, float* out, int multiprocessors,
+void launch_sum_partials(const float* partial, int ksplit, size_t count, float cap, float* out, int multiprocessors,
                          cudaStream_t stream, bool pdl) {
   const unsigned blocks = unsigned(std::max<size_t>(1, std::min((count + 255) / 256, size_t(multiprocessors) * 8)));
-  launch(sum_partials_kernel, dim3(blocks), dim3(256), 0, stream, pdl, partial, ksplit, count, out);
+  launch(sum_partials_kernel, dim3(blocks), dim3(256), 0, stream, pdl, partial, ksplit, count, cap, out);
 }
-void launch_true32_linear(const float* x, int rows, const PreparedLinear& w, float* out, cudaStream_t stream, bool pdl) {
+void launch_true32_linear(const float* x, int x_stride, int rows, const PreparedLinear& w, float* out, cudaStream_t stream,
+                          bool pdl) {
   if (rows < 1 || rows > kMaxRows) throw std::invalid_argument("32-bit linear takes 1..16 rows");
-  launch(true32_linear_kernel, dim3(unsigned((w.out + 7) / 8)), dim3(256), 0, stream, pdl, x, rows, w.dense, w.bias, w.in,
-         w.out, out);
+  launch(true32_linear_kernel, dim3(unsigned((w.out + 7) / 8)), dim3(256), 0, stream, pdl, x, x_stride, rows, w.dense, w.bias,
+         w.activation, w.in, w.out, out);
 }
-void launch_rotation_table(float2* table, size_t positions, int dims, double base, cudaStream_t stream) {
-  const size_t count = positions * (dims / 2);
+void launch_rotation_table(float2* table, size_t positions, const double* frequencies, int half, double length,
+                           cudaStream_t stream) {
+  const size_t count = positions * half;
   if (!count) return;
-  rotation_table_kernel<<<unsigned(std::min<size_t>((count + 255) / 256, 4096)), 256, 0, stream>>>(table, positions, dims / 2,
-                                                                                                   dims, std::log(base));
+  rotation_table_kernel<<<unsigned(std::min<size_t>((count + 255) / 256, 4096)), 256, 0, stream>>>(table, positions, frequencies,
+                                                                                                   half, length);
   check_launch();
 }
 

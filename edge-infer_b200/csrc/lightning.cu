@@ -12,15 +12,12 @@
 // values, the decayed scores) enters as two BF16 terms, i.e. with 16 significant bits.
 //
 // State layout: [head][slice of 16 values][key dimension][16], so that a block streams contiguous memory.
-#include "layered.cuh"
+#include "layered_device.cuh"
 
 #include <stdexcept>
 
 namespace ei {
 namespace {
-
-__device__ __forceinline__ float value_of(bf16 x) { return __bfloat162float(x); }
-__device__ __forceinline__ float value_of(float x) { return x; }
 
 constexpr int kStepThreads = 128;
 constexpr int kDimStep = kStepThreads / 4;       // key dimensions a block covers at once: 4 threads x float4 = 16 values
@@ -148,11 +145,6 @@ constexpr int kChunk = kLightningChunk;
 constexpr int kSlice = 64;               // values per block
 constexpr int kPitch = kSlice + 8;       // BF16 elements per staged value row: an odd number of 16-byte pieces
 constexpr int kPromptThreads = 256;
-
-__device__ __forceinline__ void split_pair(float a, float b, uint32_t& leading, uint32_t& rest) {
-  leading = pack_bf16(a, b);
-  rest = pack_bf16(a - bf16_lo(leading), b - bf16_hi(leading));
-}
 
 // Requests a 16-byte piece into shared memory; a dead piece is filled with zeros and not read.
 __device__ __forceinline__ void request_piece(bf16* to, const bf16* from, bool live) {

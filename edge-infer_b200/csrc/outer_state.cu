@@ -1,0 +1,266 @@
+// Recurrences over one FP32 matrix per head, S (key size x value size): S <- g S, S <- S + k u^T, out = S^T q.
+//
+// Two rules for the written vector u: the gated delta rule u = beta (v - S^T k) with one decay per key channel, and a
+// state-space layer's u = t v with one decay per head. q, k and v come out of a short causal convolution and SiLU.
+//
+// A step of at most 16 rows leaves its rows pending, as linear attention does (lightning.cu): the ring keeps every row's
+// k, g and u, so the next step rebuilds the state from those rows that were kept by plain rank-one updates, without
+// running the delta rule again. The convolution's inputs sit in a ring of their own, by position.
+#include "layered_device.cuh"
+
+#include <algorithm>
+#include <stdexcept>
+
+namespace ei {
+namespace {
+
+// One warp per (row, unit): q heads, k heads, v heads (convolution, SiLU, unit length), then the decays - per head for the
+// delta rule, 32 heads at a time otherwise.
+constexpr int kHeadColumns = kMaxHeadDim / 32;
+template <typename T>
+__global__ void __launch_bounds__(128) outer_prepare_kernel(const OuterStateParams p) {
+  const int warp = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int units = 2 * p.key_heads + p.heads + (p.delta ? p.heads : (p.heads + 31) / 32);
+  const int context = p.control->context;  // written by the previous step
+  grid_dependency_wait();
+  grid_launch_dependents();
+  if (warp >= p.rows * units || context < 0 || context + p.rows > p.capacity) return;
+  const int row = warp / units, position = context + row;
+  int unit = warp - row * units;
+  const int slot = position & (kRingRows - 1);
+  const T* fused = static_cast<const T*>(p.fused);
+
+  if (unit < 2 * p.key_heads + p.heads) {
+    const int kind = unit < p.key_heads ? 0 : unit < 2 * p.key_heads ? 1 : 2;  // q, k, v
+    const int head = unit - kind * p.key_heads, pad = kind == 2 ? p.vdim_pad : p.dim_pad;
+    const int first = kind * p.key_heads * p.dim_pad + head * pad;
+    const int channels = 2 * p.key_heads * p.dim_pad + p.heads * p.vdim_pad;
+    T* raw = static_cast<T*>(p.raw);
+    float values[kHeadColumns], squares = 0.0f;
+#pragma unroll
+    for (int j = 0; j < kHeadColumns; ++j) {
+      const int c = lane + 32 * j;
+      values[j] = 0.0f;
+      if (c >= pad) continue;
+      const int channel = first + c;
+      float sum = p.conv_bias ? p.conv_bias[channel] : 0.0f;
+      for (int tap = 0; tap < p.taps; ++tap) {
+        const int r = row - (p.taps - 1) + tap, at = context + r;
+        if (at < 0) continue;
+        const T x = r >= 0 ? fused[size_t(r) * p.stride + channel] : raw[size_t(at & (p.raw_rows - 1)) * channels + channel];
+        sum = fmaf(value_of(x), p.conv[size_t(tap) * channels + channel], sum);
+      }
+      raw[size_t(position & (p.raw_rows - 1)) * channels + channel] = fused[size_t(row) * p.stride + channel];
+      values[j] = silu_for<T>(sum);
+      squares = fmaf(values[j], values[j], squares);
+    }
+    float scale = 1.0f;
+    if (p.delta && kind < 2) {
+      scale = 1.0f / sqrtf(warp_sum(squares) + 1e-6f);
+      if (kind == 0) scale /= sqrtf(float(p.dim));
+    }
+    float* to = kind == 0 ? p.q + size_t(row) * p.key_heads * p.dim_pad + head * pad
+                : kind == 1 ? p.ring_k + size_t(slot) * p.key_heads * p.dim_pad + head * pad
+                            : p.v + size_t(row) * p.heads * p.vdim_pad + head * pad;
+#pragma unroll
+    for (int j = 0; j < kHeadColumns; ++j)
+      if (lane + 32 * j < pad) to[lane + 32 * j] = values[j] * scale;
+    return;
+  }
+  unit -= 2 * p.key_heads + p.heads;
+  const T* step = fused + size_t(row) * p.stride + p.step_at;
+  if (p.delta) {
+    const int head = unit;
+    const T* decay = static_cast<const T*>(p.decay) + size_t(row) * p.decay_stride + head * p.dim_pad;
+    float* to = p.ring_g + (size_t(slot) * p.heads + head) * p.dim_pad;
+    for (int d = lane; d < p.dim_pad; d += 32)
+      to[d] = expf(-p.rate[head] * softplus_value(value_of(decay[d]) + p.bias[head * p.dim_pad + d]));
+    if (lane == 0) p.beta[size_t(row) * p.heads + head] = sigmoid_value(value_of(step[head]));
+    return;
+  }
+  const int head = unit * 32 + lane;
+  if (head >= p.heads) return;
+  const float t = softplus_value(value_of(step[head]) + p.bias[head]);
+  p.ring_g[size_t(slot) * p.heads + head] = expf(-p.rate[head] * t);
+  p.beta[size_t(row) * p.heads + head] = t;
+}
+
+// Block (head, slice of 16 values): a warp owns four values over all key channels, lane l the channels l, l + 32, ...
+template <bool kDelta, int kStrips>
+__global__ void __launch_bounds__(128) outer_step_kernel(const OuterStateParams p) {
+  const int head = blockIdx.x, slice = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int key_head = head / (p.heads / p.key_heads);
+  const int key_width = p.key_heads * p.dim_pad, value_width = p.heads * p.vdim_pad;
+  const int value = head * p.vdim_pad + slice * 16 + warp * 4;
+  // Written by the previous step, several kernels ago: read, and the pending rows folded, before waiting.
+  const int context = p.control->context, base = p.control->state_base;
+  const bool runs = context >= 0 && context + p.rows <= p.capacity;
+  const int pending = min(kPendingRows, max(0, context - base));
+  float* state = p.state + ((size_t(head) * (p.vdim_pad / 16) + slice) * p.dim_pad) * 16 + warp * 4;
+  float4 s[kStrips];
+#pragma unroll
+  for (int i = 0; i < kStrips; ++i) {
+    const int d = lane + 32 * i;
+    s[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (runs && base > 0 && d < p.dim_pad) s[i] = *reinterpret_cast<const float4*>(state + size_t(d) * 16);
+  }
+  const float* keys = p.ring_k + key_head * p.dim_pad;
+  const float* decays = p.ring_g + (kDelta ? head * p.dim_pad : head);
+  const int decay_width = kDelta ? p.heads * p.dim_pad : p.heads;
+  if (runs && pending) {
+    for (int j = 0; j < pending; ++j) {
+      const int slot = (base + j) & (kRingRows - 1);
+      const float4 u = *reinterpret_cast<const float4*>(p.ring_u + size_t(slot) * value_width + value);
+      const float whole = kDelta ? 0.0f : decays[size_t(slot) * decay_width];
+#pragma unroll
+      for (int i = 0; i < kStrips; ++i) {
+        const int d = lane + 32 * i;
+        if (d >= p.dim_pad) continue;
+        const float k = keys[size_t(slot) * key_width + d], g = kDelta ? decays[size_t(slot) * decay_width + d] : whole;
+        s[i] = make_float4(fmaf(k, u.x, g * s[i].x), fmaf(k, u.y, g * s[i].y), fmaf(k, u.z, g * s[i].z), fmaf(k, u.w, g * s[i].w));
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < kStrips; ++i)
+      if (lane + 32 * i < p.dim_pad) *reinterpret_cast<float4*>(state + size_t(lane + 32 * i) * 16) = s[i];
+  }
+  grid_dependency_wait();
+  grid_launch_dependents();
+  if (!runs) return;
+  for (int row = 0; row < p.rows; ++row) {
+    const int slot = (context + row) & (kRingRows - 1);
+    const float4 v = *reinterpret_cast<const float4*>(p.v + size_t(row) * value_width + value);
+    const float rate = p.beta[size_t(row) * p.heads + head];
+    const float whole = kDelta ? 0.0f : decays[size_t(slot) * decay_width];
+    float k[kStrips];
+    float4 seen = make_float4(0.0f, 0.0f, 0.0f, 0.0f), read = seen;  // S^T k and S^T q after the decay
+    float match = 0.0f;                                              // q . k
+#pragma unroll
+    for (int i = 0; i < kStrips; ++i) {
+      const int d = lane + 32 * i;
+      k[i] = 0.0f;
+      if (d >= p.dim_pad) continue;
+      k[i] = keys[size_t(slot) * key_width + d];
+      const float q = p.q[size_t(row) * key_width + key_head * p.dim_pad + d];
+      const float g = kDelta ? decays[size_t(slot) * decay_width + d] : whole;
+      s[i] = make_float4(g * s[i].x, g * s[i].y, g * s[i].z, g * s[i].w);
+      if (kDelta) seen = make_float4(fmaf(k[i], s[i].x, seen.x), fmaf(k[i], s[i].y, seen.y), fmaf(k[i], s[i].z, seen.z), fmaf(k[i], s[i].w, seen.w));
+      read = make_float4(fmaf(q, s[i].x, read.x), fmaf(q, s[i].y, read.y), fmaf(q, s[i].z, read.z), fmaf(q, s[i].w, read.w));
+      match = fmaf(q, k[i], match);
+    }
+    if (kDelta) {
+      seen.x = warp_sum(seen.x); seen.y = warp_sum(seen.y); seen.z = warp_sum(seen.z); seen.w = warp_sum(seen.w);
+    }
+    read.x = warp_sum(read.x); read.y = warp_sum(read.y); read.z = warp_sum(read.z); read.w = warp_sum(read.w);
+    match = warp_sum(match);
+    const float4 u = make_float4(rate * (v.x - seen.x), rate * (v.y - seen.y), rate * (v.z - seen.z), rate * (v.w - seen.w));
+#pragma unroll
+    for (int i = 0; i < kStrips; ++i)
+      s[i] = make_float4(fmaf(k[i], u.x, s[i].x), fmaf(k[i], u.y, s[i].y), fmaf(k[i], u.z, s[i].z), fmaf(k[i], u.w, s[i].w));
+    if (lane == 0) {
+      const float skip = p.skip ? p.skip[head] : 0.0f;
+      *reinterpret_cast<float4*>(p.ring_u + size_t(slot) * value_width + value) = u;
+      *reinterpret_cast<float4*>(p.out + size_t(row) * value_width + value) =
+          make_float4(fmaf(match, u.x, fmaf(skip, v.x, read.x)), fmaf(match, u.y, fmaf(skip, v.y, read.y)),
+                      fmaf(match, u.z, fmaf(skip, v.z, read.z)), fmaf(match, u.w, fmaf(skip, v.w, read.w)));
+    }
+  }
+}
+
+// One warp (kWide: one block) per (row, norm group). Values of a group are those of its heads side by side, without the
+// heads' padding.
+constexpr int kFinishHeld = 8;
+template <typename T, bool kWide>
+__global__ void __launch_bounds__(256) state_finish_kernel(const StateFinishParams p) {
+  __shared__ float shared[8];
+  grid_dependency_wait();
+  grid_launch_dependents();
+  const int lanes = kWide ? blockDim.x : 32, lane = kWide ? threadIdx.x : threadIdx.x & 31;
+  const int item = kWide ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (item >= p.rows * p.groups) return;
+  const int row = item / p.groups, group = item - row * p.groups;
+  const int length = p.heads * p.vdim / p.groups, first = group * length;
+  const int width = p.heads * p.vdim_pad;
+  const bool packed = p.vdim == p.vdim_pad;
+  const float* in = p.in + size_t(row) * width;
+  const T* gate = static_cast<const T*>(p.gate) + size_t(row) * p.gate_stride;
+  T* out = static_cast<T*>(p.out) + size_t(row) * p.out_stride;
+  auto column = [&](int e) { return packed ? first + e : (first + e) / p.vdim * p.vdim_pad + (first + e) % p.vdim; };
+  auto value = [&](int at, float z) { return p.gate_first ? in[at] * silu_for<T>(z) : in[at]; };
+  float held[kFinishHeld], gates[kFinishHeld], sum = 0.0f;
+#pragma unroll
+  for (int j = 0; j < kFinishHeld; ++j) {
+    const int e = lane + j * lanes;
+    held[j] = gates[j] = 0.0f;
+    if (e < length) {
+      const int at = column(e);
+      gates[j] = value_of(gate[at]);
+      held[j] = value(at, gates[j]);
+    }
+    sum = fmaf(held[j], held[j], sum);
+  }
+  for (int e = lane + kFinishHeld * lanes; e < length; e += lanes) {
+    const int at = column(e);
+    const float x = value(at, value_of(gate[at]));
+    sum = fmaf(x, x, sum);
+  }
+  const float scale = 1.0f / sqrtf((kWide ? block_total(sum, shared) : warp_sum(sum)) / float(length) + p.eps);
+  auto finish = [&](int at, float x, float z) {
+    const float y = x * scale * __bfloat162float(p.norm[at]);
+    store_value(out + at, p.gate_first ? y : y * sigmoid_for<T>(z));
+  };
+#pragma unroll
+  for (int j = 0; j < kFinishHeld; ++j) {
+    const int e = lane + j * lanes;
+    if (e < length) finish(column(e), held[j], gates[j]);
+  }
+  for (int e = lane + kFinishHeld * lanes; e < length; e += lanes) {
+    const int at = column(e);
+    const float z = value_of(gate[at]);
+    finish(at, value(at, z), z);
+  }
+  if (group == 0) {
+    if (!packed)
+      for (int at = lane; at < width; at += lanes)
+        if (at % p.vdim_pad >= p.vdim) store_value(out + at, 0.0f);
+    for (int at = width + lane; at < p.out_stride; at += lanes) store_value(out + at, 0.0f);
+  }
+}
+
+template <bool kDelta>
+void launch_step_strips(const OuterStateParams& p, cudaStream_t stream, bool pdl) {
+  const dim3 grid(unsigned(p.heads), unsigned(p.vdim_pad / 16));
+  if (p.dim_pad <= 32) return launch(outer_step_kernel<kDelta, 1>, grid, dim3(128), 0, stream, pdl, p);
+  if (p.dim_pad <= 64) return launch(outer_step_kernel<kDelta, 2>, grid, dim3(128), 0, stream, pdl, p);
+  if (p.dim_pad <= 128) return launch(outer_step_kernel<kDelta, 4>, grid, dim3(128), 0, stream, pdl, p);
+  if (p.dim_pad <= 256) return launch(outer_step_kernel<kDelta, 8>, grid, dim3(128), 0, stream, pdl, p);
+  launch(outer_step_kernel<kDelta, 16>, grid, dim3(128), 0, stream, pdl, p);
+}
+
+}  // namespace
+
+template <typename T>
+void launch_outer_prepare(const OuterStateParams& p, cudaStream_t stream, bool pdl) {
+  if (p.rows < 1 || p.rows > kPendingRows) throw std::invalid_argument("a state step takes 1..16 rows");
+  const int warps = p.rows * (2 * p.key_heads + p.heads + (p.delta ? p.heads : (p.heads + 31) / 32));
+  launch(outer_prepare_kernel<T>, dim3(unsigned((warps + 3) / 4)), dim3(128), 0, stream, pdl, p);
+}
+void launch_outer_step(const OuterStateParams& p, cudaStream_t stream, bool pdl) {
+  if (p.rows < 1 || p.rows > kPendingRows || p.dim_pad > kMaxHeadDim)
+    throw std::invalid_argument("a state step takes 1..16 rows and key sizes up to 512");
+  p.delta ? launch_step_strips<true>(p, stream, pdl) : launch_step_strips<false>(p, stream, pdl);
+}
+template <typename T>
+void launch_state_finish(const StateFinishParams& p, cudaStream_t stream, bool pdl) {
+  const int items = p.rows * p.groups, length = p.heads * p.vdim / p.groups;
+  if (length > 256)
+    launch(state_finish_kernel<T, true>, dim3(unsigned(items)), dim3(256), 0, stream, pdl, p);
+  else
+    launch(state_finish_kernel<T, false>, dim3(unsigned((items + 3) / 4)), dim3(128), 0, stream, pdl, p);
+}
+template void launch_outer_prepare<bf16>(const OuterStateParams&, cudaStream_t, bool);
+template void launch_outer_prepare<float>(const OuterStateParams&, cudaStream_t, bool);
+template void launch_state_finish<bf16>(const StateFinishParams&, cudaStream_t, bool);
+template void launch_state_finish<float>(const StateFinishParams&, cudaStream_t, bool);
+
+}  // namespace ei

@@ -319,7 +319,7 @@ __global__ void __launch_bounds__(kPromptThreads, 1)
                 a += __bfloat162float(p.bias[column + 2 * i]);
                 b += __bfloat162float(p.bias[column + 2 * i + 1]);
               }
-              packed[i] = pack_bf16(a, b);
+              packed[i] = pack_bf16(activated_value(p.activation, a), activated_value(p.activation, b));
             }
             *reinterpret_cast<uint4*>(staged + lane * kPitch + cb * 32) = make_uint4(packed[0], packed[1], packed[2], packed[3]);
             *reinterpret_cast<uint4*>(staged + lane * kPitch + cb * 32 + 16) = make_uint4(packed[4], packed[5], packed[6], packed[7]);

@@ -236,7 +236,7 @@ void tick(ei_session& s) {
 }
 
 void run_linear(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, int epilogue, bf16* out,
-                int out_stride, bool pdl, int* ksplit_out) {
+                int out_stride, bool pdl, int* ksplit_out, int x_stride) {
   const ei_model& m = *s.model;
   const bool aligned_ok = (reinterpret_cast<uintptr_t>(x) & 15) == 0;
   GemmPlan plan;
@@ -247,7 +247,7 @@ void run_linear(ei_session& s, const PreparedLinear& w, const bf16* x, int rows,
   if (!plan.fast) throw std::invalid_argument("internal: linear shape has no streaming plan");
   GemmParams p{};
   p.x = x;
-  p.x_stride = w.in;
+  p.x_stride = x_stride ? x_stride : w.in;
   p.M = rows;
   p.K = w.in;
   p.N = w.out;
@@ -259,6 +259,7 @@ void run_linear(ei_session& s, const PreparedLinear& w, const bf16* x, int rows,
   p.w = w.dense;
   p.ldw = w.in;
   p.bias = epilogue == kEpiPartial ? nullptr : w.bias;
+  p.activation = w.activation;
   p.glu = w.glu;
   p.glu_limit = w.glu_limit;
   p.out = out;
@@ -295,13 +296,14 @@ bool prompt_linear_ok(const PreparedLinear& w) {
 
 // ksplit == 0: BF16 output with bias; otherwise FP32 partial sums of `ksplit` K slices in the workspace.
 void run_prompt_linear(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, bf16* out, bool pdl,
-                       int ksplit) {
+                       int ksplit, int x_stride, float* partial) {
   GemmParams p{};
   p.epilogue = ksplit ? kEpiPartial : kEpiStore;
   p.ksplit = ksplit;
-  p.partial = s.model->prompt.partial;
+  p.activation = w.activation;
+  p.partial = partial ? partial : s.model->prompt.partial;
   p.x = x;
-  p.x_stride = w.in;
+  p.x_stride = x_stride ? x_stride : w.in;
   p.M = rows;
   p.K = w.in;
   p.N = w.out;
@@ -328,18 +330,19 @@ void run_prompt_linear(ei_session& s, const PreparedLinear& w, const bf16* x, in
 // A projection with a BF16 output over all rows of a segment. Few output tiles (the q|k|v projection of a short
 // segment) would leave most SMs idle: K is then split over blocks that leave FP32 sums, and a second kernel adds
 // them, joins the bias and rounds once.
-void run_prompt_linear_store(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, bf16* out, bool pdl) {
+void run_prompt_linear_store(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, bf16* out, bool pdl,
+                             int x_stride) {
   ei_model& m = *s.model;
   auto& ws = m.prompt;
   const int ksplit = w.out % 4 == 0 ? prompt_gemm_ksplit(rows, w.out, w.in, m.multiprocessors, ws.partial_bytes) : 1;
   if (ksplit < 2) {
-    run_prompt_linear(s, w, x, rows, out, pdl);
+    run_prompt_linear(s, w, x, rows, out, pdl, 0, x_stride);
     return;
   }
-  run_prompt_linear(s, w, x, rows, nullptr, pdl, ksplit);
+  run_prompt_linear(s, w, x, rows, nullptr, pdl, ksplit, x_stride);
   tick(s);
   launch(splitk_store_kernel, dim3(std::min(m.multiprocessors * 8, (rows * w.out + 255) / 256)), dim3(256), 0, s.stream,
-         pdl, (const float*)ws.partial, ksplit, rows, w.out, w.bias, out, w.out);
+         pdl, (const float*)ws.partial, ksplit, rows, w.out, w.bias, out, w.out, w.activation);
 }
 
 void enqueue_commit(ei_session& s, int rows, bool folded) {

@@ -29,6 +29,7 @@ struct PreparedLinear {
   int padded_groups = 0, zero_stride = 0, group_size = 0;
   const bf16* dense = nullptr;  // [out, in]
   const bf16* bias = nullptr;
+  int activation = kActNone;    // of a stored result
   int glu = kGluSilu;           // a gate|up pair: which gated unit its epilogue applies
   float glu_limit = 0.0f;
   size_t bytes = 0;  // weight bytes one call streams
@@ -122,16 +123,17 @@ enum StepKind { kVerifyHost = 0, kVerifyDevice = 1, kCommitAllWithHead = 2, kCom
 // Counts a launch of the session (and fails it when the test hook is armed).
 void tick(ei_session& s);
 // One projection of at most 16 rows by the weight-streaming kernels (s.partial / s.best_* are its outputs where the
-// epilogue says so), and whether a plan exists for it.
+// epilogue says so), and whether a plan exists for it. x_stride 0: rows of w.in inputs side by side.
 void run_linear(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, int epilogue, bf16* out,
-                int out_stride, bool pdl, int* ksplit_out = nullptr);
+                int out_stride, bool pdl, int* ksplit_out = nullptr, int x_stride = 0);
 bool has_plan(const ei_session& s, const PreparedLinear& w, int rows, int epilogue);
 // One projection of a prompt segment on the tensor cores; ksplit == 0: BF16 output with bias, otherwise FP32 partial
-// sums of `ksplit` K slices in the model's prompt workspace.
+// sums of `ksplit` K slices in `partial` (null: the model's prompt workspace).
 bool prompt_linear_ok(const PreparedLinear& w);
 void run_prompt_linear(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, bf16* out, bool pdl,
-                       int ksplit = 0);
-void run_prompt_linear_store(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, bf16* out, bool pdl);
+                       int ksplit = 0, int x_stride = 0, float* partial = nullptr);
+void run_prompt_linear_store(ei_session& s, const PreparedLinear& w, const bf16* x, int rows, bf16* out, bool pdl,
+                             int x_stride = 0);
 // Commits all rows of a step. `folded`: the step's kernels already carried their recurrent state past these rows (a
 // prompt segment); otherwise the rows stay pending behind Control::state_base.
 void enqueue_commit(ei_session& s, int rows, bool folded);

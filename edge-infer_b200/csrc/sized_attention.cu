@@ -11,7 +11,7 @@
 //  * query rows of all heads of a KV group are stacked over the whole row range and dealt to blocks of up to four
 //    warps, 16 stacked rows per warp, so any group size and row count works;
 //  * kernels are compiled for sizes up to 64, 128 and 256, with the size known at compile time when it is exactly that.
-#include "layered.cuh"
+#include "layered_device.cuh"
 
 #include <algorithm>
 #include <stdexcept>
@@ -278,18 +278,13 @@ __global__ void __launch_bounds__(kMaxWarps * 32) sized_attention_kernel(const _
   }
 }
 
-__device__ __forceinline__ float value_of(bf16 x) { return __bfloat162float(x); }
-__device__ __forceinline__ float value_of(float x) { return x; }
-__device__ __forceinline__ void store_value(bf16* p, float x) { *p = __float2bfloat16_rn(x); }
-__device__ __forceinline__ void store_value(float* p, float x) { *p = x; }
-
 // Any head size, FP32 arithmetic: one block per (row, head), a lane scores one key of a warp's 32 and the warp's lanes
-// share the value columns; the four warps' running sums meet in shared memory.
-constexpr int kPlainColumns = kMaxHeadDim / 32;
-template <typename T>
+// share the value columns, kColumns each; the four warps' running sums meet in shared memory.
+template <typename T, int kColumns>
 __global__ void __launch_bounds__(128) plain_attention_kernel(const SizedAttentionParams p) {
-  __shared__ float query[kMaxHeadDim];
-  __shared__ float sums[4][kMaxHeadDim];
+  extern __shared__ float plain_smem[];
+  float* query = plain_smem;                       // [dim_pad]
+  float* sums = plain_smem + p.dim_pad;            // [4][vdim_pad]
   __shared__ float tops[4], denominators[4];
   grid_dependency_wait();
   grid_launch_dependents();
@@ -302,18 +297,17 @@ __global__ void __launch_bounds__(128) plain_attention_kernel(const SizedAttenti
   const T* q = static_cast<const T*>(p.q) + size_t(row) * p.q_stride + size_t(head) * p.dim_pad;
   for (int i = threadIdx.x; i < p.dim_pad; i += blockDim.x) query[i] = value_of(q[i]);
   __syncthreads();
-  const size_t k_pitch = size_t(p.kv_heads) * p.dim_pad, v_pitch = size_t(p.kv_heads) * p.vdim_pad;
   const T* keys = static_cast<const T*>(p.k) + size_t(kv_head) * p.dim_pad;
   const T* values = static_cast<const T*>(p.v) + size_t(kv_head) * p.vdim_pad;
-  float acc[kPlainColumns];
+  float acc[kColumns];
 #pragma unroll
-  for (int j = 0; j < kPlainColumns; ++j) acc[j] = 0.0f;
+  for (int j = 0; j < kColumns; ++j) acc[j] = 0.0f;
   float top = -INFINITY, denominator = 0.0f;
   for (int first = warp * 32; first < length; first += 128) {
     const int key = first + lane;
     float score = -INFINITY;
     if (key < length) {
-      const T* k = keys + size_t(key) * k_pitch;
+      const T* k = keys + size_t(key) * p.k_stride;
       float sum = 0.0f;
       for (int i = 0; i < p.dim_pad; ++i) sum = fmaf(query[i], value_of(k[i]), sum);
       score = sum * p.scale;
@@ -323,19 +317,19 @@ __global__ void __launch_bounds__(128) plain_attention_kernel(const SizedAttenti
     top = new_top;
     denominator = denominator * rescale + warp_sum(weight);
 #pragma unroll
-    for (int j = 0; j < kPlainColumns; ++j) acc[j] *= rescale;
+    for (int j = 0; j < kColumns; ++j) acc[j] *= rescale;
     const int live = min(32, length - first);
     for (int t = 0; t < live; ++t) {
       const float w = __shfl_sync(0xffffffffu, weight, t);
-      const T* v = values + size_t(first + t) * v_pitch;
+      const T* v = values + size_t(first + t) * p.v_stride;
 #pragma unroll
-      for (int j = 0; j < kPlainColumns; ++j)
+      for (int j = 0; j < kColumns; ++j)
         if (lane + 32 * j < p.vdim_pad) acc[j] = fmaf(w, value_of(v[lane + 32 * j]), acc[j]);
     }
   }
 #pragma unroll
-  for (int j = 0; j < kPlainColumns; ++j)
-    if (lane + 32 * j < p.vdim_pad) sums[warp][lane + 32 * j] = acc[j];
+  for (int j = 0; j < kColumns; ++j)
+    if (lane + 32 * j < p.vdim_pad) sums[warp * p.vdim_pad + lane + 32 * j] = acc[j];
   if (lane == 0) {
     tops[warp] = top;
     denominators[warp] = denominator;
@@ -353,7 +347,7 @@ __global__ void __launch_bounds__(128) plain_attention_kernel(const SizedAttenti
   for (int i = threadIdx.x; i < p.vdim_pad; i += blockDim.x) {
     float sum = 0.0f;
 #pragma unroll
-    for (int w = 0; w < 4; ++w) sum += sums[w][i] * weights[w];
+    for (int w = 0; w < 4; ++w) sum += sums[w * p.vdim_pad + i] * weights[w];
     store_value(out + i, sum / total * p.out_scale);
   }
 }
@@ -361,10 +355,10 @@ __global__ void __launch_bounds__(128) plain_attention_kernel(const SizedAttenti
 // 16-byte pieces per box row (as log2): the widest of 64, 32 and 16 values that divides the padded head.
 int box_shift(int pad) { return pad % 64 == 0 ? 3 : pad % 32 == 0 ? 2 : 1; }
 
-void encode_head_map(CUtensorMap* map, const void* base, int tokens, int kv_heads, int pad) {
+void encode_head_map(CUtensorMap* map, const void* base, int tokens, int token_stride, int kv_heads, int pad) {
   const int shift = box_shift(pad), values = 8 << shift;
   const cuuint64_t dims[4] = {cuuint64_t(values), cuuint64_t(tokens), cuuint64_t(pad / values), cuuint64_t(kv_heads)};
-  const cuuint64_t strides[3] = {cuuint64_t(kv_heads) * pad * 2, cuuint64_t(values) * 2, cuuint64_t(pad) * 2};
+  const cuuint64_t strides[3] = {cuuint64_t(token_stride) * 2, cuuint64_t(values) * 2, cuuint64_t(pad) * 2};
   const cuuint32_t box[4] = {cuuint32_t(values), cuuint32_t(kTile), cuuint32_t(pad / values), 1};
   encode_map(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, base, dims, strides, box,
              shift == 3 ? CU_TENSOR_MAP_SWIZZLE_128B : shift == 2 ? CU_TENSOR_MAP_SWIZZLE_64B : CU_TENSOR_MAP_SWIZZLE_32B,
@@ -401,8 +395,8 @@ void launch_sized(const SizedAttentionParams& given, bool direct, cudaStream_t s
   p.k_shift = box_shift(p.dim_pad);
   p.v_shift = box_shift(p.vdim_pad);
   const int tokens = (p.capacity + kTile - 1) / kTile * kTile;  // the caches are allocated in whole tiles
-  encode_head_map(&p.k_map, p.k, tokens, p.kv_heads, p.dim_pad);
-  encode_head_map(&p.v_map, p.v, tokens, p.kv_heads, p.vdim_pad);
+  encode_head_map(&p.k_map, p.k, tokens, p.k_stride, p.kv_heads, p.dim_pad);
+  encode_head_map(&p.v_map, p.v, tokens, p.v_stride, p.kv_heads, p.vdim_pad);
   const int widest = std::max(p.dim_pad, p.vdim_pad);
   const bool same = p.dim_pad == p.vdim_pad;
   if (widest <= 64) {
@@ -437,8 +431,13 @@ void launch_sized_attention_prompt(const SizedAttentionParams& p, cudaStream_t s
 
 template <typename T>
 void launch_plain_attention(const SizedAttentionParams& p, cudaStream_t stream, bool pdl) {
-  if (p.dim_pad > kMaxHeadDim || p.vdim_pad > kMaxHeadDim) throw std::invalid_argument("attention head size beyond 512");
-  launch(plain_attention_kernel<T>, dim3(unsigned(p.rows) * p.heads), dim3(128), 0, stream, pdl, p);
+  const size_t smem = (size_t(p.dim_pad) + 4 * size_t(p.vdim_pad)) * sizeof(float);
+  if (p.vdim_pad > kMaxLatent || smem > 47 * 1024) throw std::invalid_argument("attention head size beyond the supported range");
+  const dim3 grid(unsigned(p.rows) * p.heads);
+  if (p.vdim_pad <= 512)
+    launch(plain_attention_kernel<T, 16>, grid, dim3(128), smem, stream, pdl, p);
+  else
+    launch(plain_attention_kernel<T, 32>, grid, dim3(128), smem, stream, pdl, p);
 }
 template void launch_plain_attention<float>(const SizedAttentionParams&, cudaStream_t, bool);
 template void launch_plain_attention<bf16>(const SizedAttentionParams&, cudaStream_t, bool);

@@ -10,7 +10,7 @@
 namespace ei {
 
 __global__ void splitk_store_kernel(const float* partial, int ksplit, int M, int N, const bf16* bias,
-                                    bf16* out, int out_stride) {
+                                    bf16* out, int out_stride, int activation) {
   grid_dependency_wait();
   const int total = M * N;
   for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < total; i += gridDim.x * blockDim.x) {
@@ -18,7 +18,7 @@ __global__ void splitk_store_kernel(const float* partial, int ksplit, int M, int
     float sum = 0.0f;
     for (int s = 0; s < ksplit; ++s) sum += partial[(size_t(s) * M + row) * N + n];
     if (bias) sum += __bfloat162float(bias[n]);
-    out[size_t(row) * out_stride + n] = __float2bfloat16_rn(sum);
+    out[size_t(row) * out_stride + n] = __float2bfloat16_rn(activated_value(activation, sum));
   }
 }
 

@@ -40,6 +40,11 @@ enum GluKind : int {
   kGluClamped = 1   // a = min(gate, limit), b = up held to +-limit: (1 + b) * a / (1 + exp(-1.702 a)), rounded once
 };
 
+enum Activation : int {
+  kActNone = 0,
+  kActReluSquared = 1   // max(sum + bias, 0)^2, on the FP32 sum
+};
+
 struct GemmParams {
   const bf16* x;          // [M, K], row stride x_stride
   int x_stride;
@@ -56,6 +61,7 @@ struct GemmParams {
   int epilogue;
   int glu;                // kEpiSiluPair: a GluKind, and the clamp of kGluClamped
   float glu_limit;
+  int activation;         // kEpiStore: an Activation, applied ahead of the rounding
   int ksplit;             // blocks along K (>= 1); > 1 requires kEpiPartial
   float* partial;         // [ksplit, M, N]
   float* best_value;      // kEpiArgmax: [grid, 16]
@@ -96,6 +102,12 @@ __device__ __forceinline__ float silu_multiply_value(float gate, float up) {
 __device__ __forceinline__ float clamped_glu_value(float gate, float up, float limit) {
   const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
   return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+
+__device__ __forceinline__ float activated_value(int activation, float x) {
+  if (activation != kActReluSquared) return x;
+  const float r = fmaxf(x, 0.0f);
+  return r * r;
 }
 
 // The gated unit of a gate|up pair from its two FP32 sums.
@@ -325,7 +337,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1) smallm_gemm_kernel(const Gemm
           p.partial[(size_t(slice) * p.M + row) * p.N + n] = sum;
         } else {
           if (p.bias) sum += __bfloat162float(p.bias[n]);
-          const bf16 rounded = __float2bfloat16_rn(sum);
+          const bf16 rounded = __float2bfloat16_rn(activated_value(p.activation, sum));
           p.out[size_t(row) * p.out_stride + n] = rounded;
           if (p.epilogue == kEpiArgmax) {
             float value = __bfloat162float(rounded);
@@ -370,9 +382,9 @@ __global__ void __launch_bounds__(kGemmThreads, 1) smallm_gemm_kernel(const Gemm
   }
 }
 
-// Fixed-order reduction of split-K partials for a plain linear: out = round_bf16(sum_s partial + bias).
+// Fixed-order reduction of split-K partials for a plain linear: out = round_bf16(activation(sum_s partial + bias)).
 __global__ void splitk_store_kernel(const float* partial, int ksplit, int M, int N, const bf16* bias,
-                                    bf16* out, int out_stride);
+                                    bf16* out, int out_stride, int activation);
 
 // Any-shape fallbacks (one thread per output, sequential FP32 fma in input order like the
 // reference's scalar kernel, operators/src/cuda/kernels/awq_gemv_gemm.cu:579-604).

@@ -44,8 +44,9 @@ class Shape:
                                self.quant_type, self.group_size, 1 if self.qk_norm else 0)
 
 
-MIXER_MIN_GRU, MIXER_PARALLEL = 1, 2
-MLP_NONE, MLP_CLAMPED_GLU = 0, 1
+MIXER_MIN_GRU, MIXER_PARALLEL, MIXER_LATENT_ATTENTION, MIXER_STATE_SPACE, MIXER_CHANNEL_DELTA = 1, 2, 3, 4, 5
+MLP_NONE, MLP_CLAMPED_GLU, MLP_RELU_SQUARED = 0, 1, 2
+BLOCK_SANDWICH, BLOCK_PARALLEL = 0, 1
 
 
 @dataclass
@@ -70,9 +71,58 @@ class LinearAttention:
 
 
 @dataclass
+class Yarn:
+    """YaRN frequency scaling of a rotation."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass
+class LatentAttention:
+    """Softmax attention over latents: per head `dim` unrotated and `rot_dim` rotated query values (the first `rot_dims`
+    of them turned), values of `vdim`, latents of `kv_rank`."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    rot_dims: int
+    rot_base: float
+    scale: float
+    yarn: Optional[Yarn] = None
+
+
+@dataclass
+class StateSpace:
+    """State-space recurrence: per head a matrix `state` x `vdim`, inputs and outputs shared within `groups`, a
+    convolution of `taps` tokens, the result normed in `norm_groups` parts."""
+    heads: int
+    groups: int
+    state: int
+    vdim: int
+    taps: int
+    norm_groups: int
+
+
+@dataclass
+class ChannelDelta:
+    """Gated delta rule with one decay per key channel: sizes, convolution taps, ranks of the decay's and the gate's
+    projection (a checkpoint's tensors give them)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    taps: int
+    decay_rank: int = 0
+    gate_rank: int = 0
+
+
+@dataclass
 class Layer:
-    """One layer of a LayeredShape. Either `rnn_width` (gated recurrence) or both attentions (parallel mixer) are set;
-    `ff` None: no feed-forward."""
+    """One layer of a LayeredShape. One of `rnn_width` (gated recurrence), both attentions (parallel mixer), `latent`,
+    `state_space` and `delta` is set; `ff` None: no feed-forward."""
     rnn_width: Optional[int] = None
     attention: Optional[Attention] = None
     linear: Optional[LinearAttention] = None
@@ -80,11 +130,33 @@ class Layer:
     right_scale: float = 1.0
     ff: Optional[int] = None
     limit: float = 0.0
+    latent: Optional[LatentAttention] = None
+    state_space: Optional[StateSpace] = None
+    delta: Optional[ChannelDelta] = None
+    mlp: int = MLP_CLAMPED_GLU
 
     def to_c(self) -> abi.LayerSpec:
         spec = abi.LayerSpec()
         if self.rnn_width is not None:
             spec.mixer, spec.rnn_width = MIXER_MIN_GRU, self.rnn_width
+        elif self.latent is not None:
+            a = self.latent
+            spec.mixer = MIXER_LATENT_ATTENTION
+            spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank = a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank
+            spec.rot_dims, spec.rot_base, spec.scale = a.rot_dims, a.rot_base, a.scale
+            if a.yarn is not None:
+                spec.rot_factor, spec.rot_original = a.yarn.factor, a.yarn.original
+                spec.rot_fast, spec.rot_slow = a.yarn.fast, a.yarn.slow
+        elif self.state_space is not None:
+            m = self.state_space
+            spec.mixer = MIXER_STATE_SPACE
+            spec.heads, spec.groups, spec.state, spec.vdim = m.heads, m.groups, m.state, m.vdim
+            spec.taps, spec.norm_groups = m.taps, m.norm_groups
+        elif self.delta is not None:
+            m = self.delta
+            spec.mixer = MIXER_CHANNEL_DELTA
+            spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.taps = m.heads, m.kv_heads, m.dim, m.vdim, m.taps
+            spec.decay_rank, spec.gate_rank = m.decay_rank, m.gate_rank
         else:
             a, l = self.attention, self.linear
             spec.mixer = MIXER_PARALLEL
@@ -96,14 +168,24 @@ class Layer:
             spec.decay = (C.c_double * l.heads)(*[float(d) for d in l.decay])
             spec.left_scale, spec.right_scale = self.left_scale, self.right_scale
         if self.ff is not None:
-            spec.mlp, spec.ff, spec.limit = MLP_CLAMPED_GLU, self.ff, self.limit
+            spec.mlp, spec.ff, spec.limit = self.mlp, self.ff, self.limit
         return spec
+
+
+@dataclass
+class PairEmbedding:
+    """A second embedding picked by a token and the one before it: row (previous * mul_prev + token * mul_cur) mod
+    buckets, row `buckets` for a sequence's first token."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
 
 
 @dataclass
 class LayeredShape:
     """A decoder described layer by layer (ei_model_create_layered). `loop` = (start, stop, times): the
-    stretch layers[start:stop] is repeated, `times` passes in all. `true32`: FP32 activations, caches and products."""
+    stretch layers[start:stop] is repeated, `times` passes in all. `true32`: FP32 activations, caches and products.
+    `block`: how norms and sums join a layer's mixer and feed-forward."""
     vocab_size: int
     hidden_size: int
     layers: List[Layer]
@@ -113,6 +195,10 @@ class LayeredShape:
     max_position_embeddings: int = 1 << 20
     bos_token_id: int = 0
     eos_token_id: int = 0xFFFFFFFF
+    block: int = BLOCK_SANDWICH
+    tied_embeddings: bool = False
+    pairs: Optional[PairEmbedding] = None
+    logit_softcap: float = 0.0
 
     @property
     def n_layers(self) -> int:
@@ -130,7 +216,11 @@ class LayeredShape:
         start, stop, times = self.loop or (0, 0, 0)
         config = abi.LayeredConfig(self.vocab_size, self.hidden_size, len(self.layers), self.max_position_embeddings,
                                    start, stop, times, self.norm_eps, self.bos_token_id, self.eos_token_id,
-                                   1 if self.true32 else 0)
+                                   1 if self.true32 else 0, self.block, 1 if self.tied_embeddings else 0)
+        if self.pairs is not None:
+            config.pair_buckets = self.pairs.buckets
+            config.pair_mul_prev, config.pair_mul_cur = self.pairs.mul_prev, self.pairs.mul_cur
+        config.logit_softcap = self.logit_softcap
         return config, (abi.LayerSpec * len(self.layers))(*[layer.to_c() for layer in self.layers])
 
 

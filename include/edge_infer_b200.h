@@ -220,25 +220,50 @@ typedef struct ei_session ei_session;
 ei_status ei_model_create(const ei_model_config* config, const ei_named_tensor* tensors, size_t count,
                           ei_model** out);
 /* A decoder described layer by layer (no counterpart in the reference, whose models repeat one block): every layer
- * names its token mixer with its sizes and constants and its feed-forward, each sublayer stands between two norms, and
- * a stretch of layers may run several times in a row. The session verbs below serve such a model as they serve the
+ * names its token mixer with its sizes and constants and its feed-forward, the block form says how norms and sums join
+ * them, and a stretch of layers may run several times in a row. The session verbs below serve such a model as they serve the
  * others; differences are noted there.
  * Mixers: EI_MIXER_MIN_GRU - `rnn_width` independent channels, each an exponential average whose gate depends on the
  * row's own input alone.
  * EI_MIXER_PARALLEL - grouped-query softmax attention (partial rotation, value norm, per-head sink, own score scale)
  * beside decayed linear attention (SiLU on q, k, v; one decay per head; normed and gated output), outputs weighted by
- * left_scale and right_scale. Feed-forward: EI_MLP_CLAMPED_GLU - with a = min(gate, limit) and
- * b = max(-limit, min(up, limit)): (1 + b) * a / (1 + exp(-1.702 a)). Norm: tanh(alpha x) * weight + bias. Residual stream, norms, angles, scores, softmax
- * weights, gates and recurrent state are FP32; with `true32` so are all activations, caches and products. */
-enum { EI_MIXER_MIN_GRU = 1, EI_MIXER_PARALLEL = 2 };
-enum { EI_MLP_NONE = 0, EI_MLP_CLAMPED_GLU = 1 };
+ * left_scale and right_scale.
+ * EI_MIXER_LATENT_ATTENTION - softmax attention whose keys and values are made from one RMS-normed latent of `kv_rank`
+ * values per token; per head `dim` unrotated and `rot_dim` rotated query values (pairs of neighbours, rot_dims of them
+ * turned), the rotated key shared by all heads; sigmoid output gate. Only latent and rotated key are cached.
+ * EI_MIXER_STATE_SPACE - per head a matrix of `state` x `vdim` decayed by one factor per token and head, input and
+ * output vectors shared by the heads of a group, after a causal convolution of `taps` tokens and SiLU; the result is
+ * gated, then RMS-normed in `norm_groups` parts.
+ * EI_MIXER_CHANNEL_DELTA - per head a matrix of `dim` x `vdim` updated by the gated delta rule with one decay per key
+ * channel (a projection of rank `decay_rank`); convolved, unit-length q and k; per-head norm and a sigmoid gate of rank
+ * `gate_rank`.
+ * Feed-forward: EI_MLP_CLAMPED_GLU - with a = min(gate, limit) and b = max(-limit, min(up, limit)):
+ * (1 + b) * a / (1 + exp(-1.702 a)). EI_MLP_RELU_SQUARED - max(up, 0)^2.
+ * Blocks: EI_BLOCK_SANDWICH - mixer, then feed-forward, each between two norms tanh(alpha x) * weight + bias.
+ * EI_BLOCK_PARALLEL - mixer and feed-forward of the same stream, each behind its own layer norm (weight, no bias), their
+ * results multiplied by one vector each and added together.
+ * Residual stream, norms, angles, scores, softmax weights, gates, decays and recurrent state are FP32; with `true32` so
+ * are all activations, caches and products. */
+enum {
+  EI_MIXER_MIN_GRU = 1,
+  EI_MIXER_PARALLEL = 2,
+  EI_MIXER_LATENT_ATTENTION = 3,
+  EI_MIXER_STATE_SPACE = 4,
+  EI_MIXER_CHANNEL_DELTA = 5
+};
+enum { EI_MLP_NONE = 0, EI_MLP_CLAMPED_GLU = 1, EI_MLP_RELU_SQUARED = 2 };
+enum { EI_BLOCK_SANDWICH = 0, EI_BLOCK_PARALLEL = 1 };
 typedef struct ei_layer_spec {
   int32_t mixer, mlp;
   uint32_t rnn_width;
   uint32_t heads, kv_heads, dim, vdim, rot_dims;
   uint32_t lin_heads, lin_dim, lin_vdim;
   uint32_t ff;
+  uint32_t rot_dim, kv_rank;
+  uint32_t state, groups, norm_groups;
+  uint32_t taps, decay_rank, gate_rank;
   double rot_base, scale, left_scale, right_scale, limit;
+  double rot_factor, rot_original, rot_fast, rot_slow; /* YaRN frequency scaling; rot_factor 0: none */
   const double* decay; /* [lin_heads] */
 } ei_layer_spec;
 typedef struct ei_layered_config {
@@ -247,12 +272,23 @@ typedef struct ei_layered_config {
   double norm_eps;
   uint32_t bos_token_id, eos_token_id;
   int32_t true32; /* 1: FP32 activations and caches, FP32 products */
+  int32_t block;
+  int32_t tied_head; /* 1: the vocabulary head is the embedding table */
+  /* pair embedding: row (previous token * pair_mul_prev + token * pair_mul_cur) mod pair_buckets of `bigram` is added to
+   * a token's embedding, row pair_buckets to a sequence's first; pair_buckets 0: none */
+  uint64_t pair_buckets, pair_mul_prev, pair_mul_cur;
+  double logit_softcap; /* logits <- cap * tanh(logits / cap); 0: none */
 } ei_layered_config;
-/* Tensors (kind 0, BF16; a scalar has rank 1 and one element): embed [V,W], head [V,W], final.norm [W], with a loop
- * loop.step [times,W]; per layer i, prefix l<i>.: norm1, norm1b, and with a feed-forward norm2, norm2b, mlp.gate,
- * mlp.up [ff,W], mlp.down [W,ff]; every norm also <name>.b [W] and <name>.alpha [1]. mix.z, mix.x (and their .b),
- * mix.g [R,W], mix.o [W,R] for the gated recurrence; mix.left.{q,k,v,o,sink} and mix.right.{q,k,v,g,o,norm} for the
- * parallel mixer, heads side by side. Linear weights are [out, in]. Allocates. */
+/* Tensors (kind 0, BF16; a scalar has rank 1 and one element): embed [V,W], head [V,W] unless tied, bigram
+ * [pair_buckets + 1,W] with a pair embedding, final.norm [W], with a loop loop.step [times,W]; per layer i, prefix l<i>.:
+ * Sandwich blocks: norm1, norm1b, and with a feed-forward norm2, norm2b; every norm also <name>.b [W], <name>.alpha [1].
+ * Parallel blocks: norm1, ls1 [W], and with a feed-forward norm2, ls2 [W].
+ * Feed-forward: mlp.up [ff,W], mlp.down [W,ff], and mlp.gate [ff,W] for the gated unit.
+ * Gated recurrence: mix.z, mix.x (and their .b), mix.g [R,W], mix.o [W,R]. Parallel mixer: mix.left.{q,k,v,o,sink} and
+ * mix.right.{q,k,v,g,o,norm}, heads side by side. Latent attention: mix.{q,dkv,dkv.norm,uk,uv,g,o}. State space:
+ * mix.{in,conv,conv.b,dt_bias,A_log,D,norm,o}, rows of mix.in in the order gate, x, B, C, step. Channel delta:
+ * mix.{q,k,v} with their .conv, mix.{b,A_log,norm,a1,a2,dt_bias,g1,g2,o}. Convolutions are [channels,taps], the last
+ * column for the current token. Linear weights are [out, in]. Allocates. */
 ei_status ei_model_create_layered(const ei_layered_config* config, const ei_layer_spec* layers,
                                   const ei_named_tensor* tensors, size_t count, ei_model** out);
 void ei_model_destroy(ei_model* model);
