@@ -19,7 +19,7 @@ OBJ = HERE / "build"
 LIB = HERE / "libedge_infer_b200.so"
 SOURCES = ["abi_ops.cu", "smallm_gemm.cu", "prompt_gemm.cu", "elementwise.cu", "attention.cu", "sampling.cu", "runtime.cu",
            "layered.cu", "layered_kernels.cu", "lightning.cu", "sized_attention.cu",
-           "parallel_block.cu", "outer_state.cu", "latent_attention.cu"]
+           "parallel_block.cu", "outer_state.cu", "latent_attention.cu", "delta_prompt.cu"]
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 FLAGS = [
     "-std=c++17", "-O3", "-lineinfo",

@@ -1137,9 +1137,19 @@ void create_layered_model(ei_model& model, const ei_layered_config& c, const ei_
       m.max_second = std::max(m.max_second, l.second.out);
       m.max_state_keys = std::max(m.max_state_keys, l.key_heads * l.dim_pad);
       m.max_state_heads = std::max(m.max_state_heads, int(l.spec.heads));
-      model.prompt_ready = false;
+      m.max_channels = std::max(m.max_channels, l.channels);
+      if (l.delta()) {
+        model.prompt_ready = model.prompt_ready && delta_prompt_ok(l.dim_pad, l.vdim_pad) && prompt_linear_ok(l.second);
+        m.max_delta_chunks = std::max(m.max_delta_chunks, delta_prompt_bytes(kPromptSegment, l.spec.heads, l.dim_pad, l.vdim_pad));
+      } else {
+        model.prompt_ready = model.prompt_ready && lightning_prompt_ok(l.dim_pad, l.vdim_pad);
+        m.max_chunk_state = std::max(m.max_chunk_state, size_t(l.spec.heads) * l.vdim_pad * l.dim_pad);
+      }
     }
-    if (l.spec.mixer == EI_MIXER_LATENT_ATTENTION) model.prompt_ready = false;
+    if (l.spec.mixer == EI_MIXER_LATENT_ATTENTION) {
+      m.max_expand = std::max(m.max_expand, size_t(l.expand.out));
+      model.prompt_ready = model.prompt_ready && sized_attention_ok(l.dim_pad + l.rot_pad, l.vdim_pad) && prompt_linear_ok(l.expand);
+    }
     if (l.spec.mixer == EI_MIXER_PARALLEL) {
       m.max_chunk_state = std::max(m.max_chunk_state, size_t(l.linear_width) * l.lin_dim_pad);
       model.prompt_ready = model.prompt_ready && sized_attention_ok(l.dim_pad, l.vdim_pad) &&
@@ -1250,6 +1260,18 @@ void create_layered_session(ei_session& s) {
   EI_CUDA(cudaStreamSynchronize(nullptr));
 }
 
+void ensure_expanded(ei_model& model, size_t tokens) {
+  LayeredModel& m = *model.layered;
+  const size_t bytes = tokens * m.max_expand * sizeof(bf16);
+  if (bytes <= m.expanded_bytes) return;
+  if (m.expanded) EI_CUDA(cudaFree(m.expanded));
+  m.expanded = nullptr;
+  m.expanded_bytes = 0;
+  const size_t room = bytes + bytes / 4;
+  EI_CUDA(cudaMalloc(reinterpret_cast<void**>(&m.expanded), room));
+  m.expanded_bytes = room;
+}
+
 void ensure_layered_workspace(ei_model& model) {
   auto& ws = model.prompt;
   if (ws.arena) return;
@@ -1275,6 +1297,17 @@ void ensure_layered_workspace(ei_model& model) {
   take(ws.tokens, rows * 4);
   take(ws.step_tokens, rows * 4);
   take(ws.partial, partial_bytes);
+  if (m.parallel) {
+    take(m.mixed_partial, partial_bytes);
+    take(m.second_normed, rows * m.normed_stride * 2);
+  }
+  if (m.max_channels) {
+    take(m.second, rows * m.max_second * 2);
+    take(m.conv_out, rows * m.max_channels * 2);
+    take(m.inverse, rows * 2 * m.max_state_heads * sizeof(float));
+    take(m.decay_totals, chunks * m.max_state_heads * sizeof(float));
+    take(m.delta_chunks, m.max_delta_chunks);
+  }
   unsigned char* base = nullptr;
   EI_CUDA(cudaMalloc(reinterpret_cast<void**>(&base), total));
   if (cudaMemset(base, 0, total) != cudaSuccess || cudaStreamSynchronize(nullptr) != cudaSuccess ||
@@ -1298,37 +1331,20 @@ void enqueue_layered_step(ei_session& s, int rows, StepKind kind) {
     enqueue_step_as<bf16>(s, rows, kind);
 }
 
-void enqueue_layered_segment(ei_session& s, int rows) {
+// A layer's token mixer over a prompt segment, from the normed rows to the activations of its output projection.
+static void enqueue_mixer_segment(ei_session& s, const LayeredModel::Layer& l, const LayeredSession::Run& r, const Buffers& b, size_t context) {
   ei_model& model = *s.model;
   const LayeredModel& m = *model.layered;
-  LayeredSession& L = *s.layered;
-  auto& ws = model.prompt;
   const bool pdl = true;
-  const Buffers b{rows,    ws.step_tokens, m.residual, m.linear_out,    ws.normed, ws.qkv,
-                  ws.attention, ws.gate_up, ws.act, nullptr, nullptr};
-  EmbedParams token{};
-  token.tokens = ws.tokens;
-  token.control = s.control;
-  token.step_tokens = ws.step_tokens;
-  token.vocab = int(model.config.vocab_size);
-  token.rows = rows;
-  token.capacity = int(s.capacity);
-  enqueue_embed<bf16>(s, b, token);
-
-  const auto sums = [&](const PreparedLinear& w, const bf16* x) {
-    const int ksplit = prompt_gemm_ksplit(rows, w.out, w.in, model.multiprocessors, ws.partial_bytes);
-    run_prompt_linear(s, w, x, rows, nullptr, pdl, ksplit);
-    return ksplit;
-  };
-  for (size_t run = 0; run < m.runs.size(); ++run) {
-    const LayeredModel::Layer& l = m.layers[m.runs[run].layer];
-    const LayeredSession::Run& r = L.runs[run];
-    run_prompt_linear_store(s, l.in, ws.normed, rows, ws.qkv, pdl);
-    if (l.spec.mixer == EI_MIXER_MIN_GRU) {
+  const int rows = b.rows;
+  run_prompt_linear_store(s, l.in, static_cast<const bf16*>(b.normed), rows, static_cast<bf16*>(b.fused), pdl);
+  switch (l.spec.mixer) {
+    case EI_MIXER_MIN_GRU:
       tick(s);
       tick(s);
       launch_min_gru_prompt(min_gru_params<bf16>(s, l, r, b), s.stream, pdl);
-    } else {
+      return;
+    case EI_MIXER_PARALLEL: {
       tick(s);
       launch_mixer_prepare<bf16>(prepare_params(s, l, r, b, false), s.stream, pdl);
       const SizedAttentionParams a = attention_params(s, l, r, b);
@@ -1340,21 +1356,168 @@ void enqueue_layered_segment(ei_session& s, int rows) {
       s.launches += size_t(more - 1);
       tick(s);
       launch_mixer_finish<bf16>(finish_params<bf16>(s, l, b, a, false), s.stream, pdl);
+      return;
     }
-    int ksplit = sums(l.out, ws.attention);
+    case EI_MIXER_LATENT_ATTENTION: {
+      const LatentParams p = latent_params(s, l, r, b);
+      tick(s);
+      launch_latent_prepare<bf16>(p, false, s.stream, pdl);
+      // Keys and values of every token so far, from the cached latents.
+      const int tokens = int(context) + rows, keys = p.heads * l.dim_pad;
+      run_prompt_linear(s, l.expand, static_cast<const bf16*>(r.latent), tokens, m.expanded, pdl, 0, l.row_pad);
+      SizedAttentionParams a{};
+      a.q = b.fused;
+      a.q_stride = l.in.out;
+      a.k = m.expanded;
+      a.v = m.expanded + keys;
+      a.k_stride = a.v_stride = l.expand.out;
+      a.rows = rows;
+      a.heads = a.kv_heads = p.heads;
+      a.dim_pad = l.dim_pad + l.rot_pad;
+      a.vdim_pad = l.vdim_pad;
+      a.shared = static_cast<const bf16*>(r.latent) + l.rank_pad;
+      a.shared_stride = l.row_pad;
+      a.shared_pad = l.rot_pad;
+      a.tokens = tokens;
+      a.fresh = true;
+      a.gate = static_cast<const bf16*>(b.fused) + l.gate_at;
+      a.gate_stride = l.in.out;
+      a.scale = float(l.spec.scale);
+      a.out_scale = 1.0f;
+      a.device_offset = &s.control->context;
+      a.capacity = int(s.capacity);
+      a.out = b.mixed;
+      a.out_stride = l.out.in;
+      a.status = &s.control->status;
+      if (s.inject_attention_polls) {
+        a.wait_limit = s.inject_attention_polls;
+        a.fault_tx = 16;
+        s.inject_attention_polls = 0;  // one launch only
+      }
+      tick(s);
+      launch_sized_attention_prompt(a, s.stream, pdl);
+      return;
+    }
+    default: {
+      const OuterStateParams p = outer_params(s, l, r, b);
+      if (l.delta())
+        run_prompt_linear(s, l.second, static_cast<const bf16*>(b.fused) + l.first_at, rows, static_cast<bf16*>(b.second), pdl, 0, l.in.out);
+      tick(s);
+      launch_outer_conv(p, m.conv_out, m.inverse, s.stream, pdl);
+      const int keys = p.key_heads * p.dim_pad;
+      if (l.delta()) {
+        DeltaPromptParams d{};
+        d.outer = p;
+        d.conv = m.conv_out;
+        d.inverse = m.inverse;
+        d.channels = l.channels;
+        d.chunks = m.delta_chunks;
+        tick(s);
+        tick(s);
+        launch_delta_prompt(d, s.stream, pdl);
+      } else {
+        LightningParams q{};
+        q.q = m.conv_out;
+        q.k = m.conv_out + keys;
+        q.v = m.conv_out + 2 * keys;
+        q.stride = l.channels;
+        q.rows = rows;
+        q.heads = p.heads;
+        q.dim_pad = p.dim_pad;
+        q.vdim_pad = p.vdim_pad;
+        q.state = p.state;
+        q.chunk_states = m.chunk_states;
+        q.control = s.control;
+        q.capacity = p.capacity;
+        q.out = b.linear_out;
+        q.token.step = static_cast<const bf16*>(b.fused) + l.step_at;
+        q.token.step_stride = l.in.out;
+        q.token.bias = p.bias;
+        q.token.rate = p.rate;
+        q.token.skip = p.skip;
+        q.token.key_heads = p.key_heads;
+        q.token.ring_k = p.ring_k;
+        q.token.ring_g = p.ring_g;
+        q.token.ring_u = p.ring_u;
+        q.token.totals = m.decay_totals;
+        tick(s);
+        int more = 0;
+        launch_lightning_prompt(q, s.stream, pdl, &more);
+        s.launches += size_t(more - 1);
+      }
+      StateFinishParams f = state_finish_params<bf16>(s, l, b);
+      f.tail_rows = std::min(rows, p.taps - 1);
+      f.tail = b.fused;
+      f.tail_stride = l.in.out;
+      f.channels = l.channels;
+      f.raw_rows = l.raw_rows;
+      f.raw = r.raw;
+      f.control = s.control;
+      f.capacity = p.capacity;
+      tick(s);
+      launch_state_finish<bf16>(f, s.stream, pdl);
+      return;
+    }
+  }
+}
+
+void enqueue_layered_segment(ei_session& s, int rows, size_t context) {
+  ei_model& model = *s.model;
+  const LayeredModel& m = *model.layered;
+  LayeredSession& L = *s.layered;
+  auto& ws = model.prompt;
+  const bool pdl = true;
+  const Buffers b{rows,         ws.step_tokens, m.residual, m.linear_out,    ws.normed, ws.qkv,
+                  ws.attention, ws.gate_up,     ws.act,     m.second_normed, m.second};
+  EmbedParams token{};
+  token.tokens = ws.tokens;
+  token.control = s.control;
+  token.step_tokens = ws.step_tokens;
+  token.vocab = int(model.config.vocab_size);
+  token.rows = rows;
+  token.capacity = int(s.capacity);
+  enqueue_embed<bf16>(s, b, token);
+
+  const auto sums = [&](const PreparedLinear& w, const bf16* x, float* partial) {
+    const int ksplit = prompt_gemm_ksplit(rows, w.out, w.in, model.multiprocessors, ws.partial_bytes);
+    run_prompt_linear(s, w, x, rows, nullptr, pdl, ksplit, 0, partial);
+    return ksplit;
+  };
+  for (size_t run = 0; run < m.runs.size(); ++run) {
+    const LayeredModel::Layer& l = m.layers[m.runs[run].layer];
+    enqueue_mixer_segment(s, l, L.runs[run], b, context);
+    const bool feeds = l.spec.mlp != EI_MLP_NONE;
+    const auto activate = [&] {
+      if (l.spec.mlp == EI_MLP_RELU_SQUARED) {
+        run_prompt_linear(s, l.up, m.parallel ? m.second_normed : ws.normed, rows, ws.act, pdl);
+        return;
+      }
+      run_prompt_linear(s, l.gate_up, m.parallel ? m.second_normed : ws.normed, rows, ws.gate_up, pdl);
+      tick(s);
+      launch_clamped_glu<bf16>(ws.gate_up, rows, l.ff_pad, l.gate_up.glu_limit, ws.act, model.multiprocessors, s.stream, pdl);
+    };
+    if (m.parallel) {
+      const int mixed_ksplit = sums(l.out, ws.attention, m.mixed_partial);
+      int fed_ksplit = 0;
+      if (feeds) {
+        activate();
+        fed_ksplit = sums(l.down, ws.act, ws.partial);
+      }
+      enqueue_parallel_join<bf16>(s, b, run, m.mixed_partial, mixed_ksplit, feeds ? ws.partial : nullptr, fed_ksplit);
+      continue;
+    }
+    int ksplit = sums(l.out, ws.attention, ws.partial);
     SublayerJoinParams j = join_params(s, b, ws.partial, ksplit);
     j.after = l.norm1b;
-    if (l.spec.mlp == EI_MLP_NONE)
-      end_of_run(s, b, run, j);
-    else
+    if (feeds)
       j.before = l.norm2;
+    else
+      end_of_run(s, b, run, j);
     tick(s);
     launch_sublayer_join<bf16>(j, s.stream, pdl);
-    if (l.spec.mlp == EI_MLP_NONE) continue;
-    run_prompt_linear(s, l.gate_up, ws.normed, rows, ws.gate_up, pdl);
-    tick(s);
-    launch_clamped_glu<bf16>(ws.gate_up, rows, l.ff_pad, l.gate_up.glu_limit, ws.act, model.multiprocessors, s.stream, pdl);
-    ksplit = sums(l.down, ws.act);
+    if (!feeds) continue;
+    activate();
+    ksplit = sums(l.down, ws.act, ws.partial);
     j = join_params(s, b, ws.partial, ksplit);
     j.after = l.norm2b;
     end_of_run(s, b, run, j);

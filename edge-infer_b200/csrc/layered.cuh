@@ -131,6 +131,12 @@ struct SizedAttentionParams {
   const void *k, *v;        // token t, KV head g at k + t * k_stride + g * dim_pad, v + t * v_stride + g * vdim_pad
   int k_stride, v_stride;
   int rows, heads, kv_heads, dim_pad, vdim_pad;
+  const void* shared;       // the last shared_pad values of every head's key, token t at shared + t * shared_stride
+  int shared_stride, shared_pad;
+  int tokens;               // rows of k and v (0: the capacity in whole tiles)
+  bool fresh;               // k and v come from the preceding kernels, earlier tokens too
+  const void* gate;         // finished output times sigmoid of row r, head h at gate + r * gate_stride + h * vdim_pad; or null
+  int gate_stride;
   float scale, out_scale;   // out_scale multiplies the finished output
   const float* sink;        // [heads]: exp(sink) joins the denominator; or null
   const int32_t* device_offset;
@@ -139,7 +145,7 @@ struct SizedAttentionParams {
   float* scratch;           // [max_splits][rows * heads][vdim_pad + 4]
   void* out;                // row r, head h at out + r * out_stride + h * vdim_pad
   int out_stride;
-  CUtensorMap k_map, v_map; // filled by the launch functions
+  CUtensorMap k_map, v_map, shared_map;  // filled by the launch functions
   int k_shift, v_shift;     // log2 of the 16-byte pieces in one row of a staged box
   int* status;
   uint32_t wait_limit, fault_tx;
@@ -156,6 +162,17 @@ template <typename T>
 void launch_plain_attention(const SizedAttentionParams& p, cudaStream_t stream, bool pdl);
 
 // ---- decayed linear attention (lightning.cu) ----
+// One decay per token and head instead of one per head, for prompts of state-space layers: the row's step
+// t = softplus(step + bias) scales what it writes, and the state decays by exp(-rate t).
+struct TokenDecay {
+  const bf16* step;         // row r, head h at step + r * step_stride + h; null: decays are LightningParams::powers
+  int step_stride;
+  const float *bias, *rate;
+  const float* skip;        // [heads]: skip * v is added to the output; or null
+  int key_heads;            // head h reads q and k of head h / (heads / key_heads)
+  const float *ring_k, *ring_g, *ring_u;  // pending rows (outer_state.cu)
+  float* totals;            // [chunks][heads]: logarithm of a chunk's decay
+};
 struct LightningParams {
   const void *q, *k, *v;    // row r at + r * stride, heads side by side
   int stride, rows, heads, dim_pad, vdim_pad;
@@ -166,6 +183,7 @@ struct LightningParams {
   const Control* control;
   int capacity;
   float* out;               // [rows, heads * vdim_pad]
+  TokenDecay token;
 };
 // At most 16 rows: folds the pending rows into the state, reads it for the step's rows, leaves those pending.
 template <typename T>
@@ -252,6 +270,22 @@ struct OuterStateParams {
 template <typename T>
 void launch_outer_prepare(const OuterStateParams& p, cudaStream_t stream, bool pdl);
 void launch_outer_step(const OuterStateParams& p, cudaStream_t stream, bool pdl);
+// A prompt segment's convolution and SiLU, BF16: out [rows, channels] and, for the delta rule, one over the length of
+// every q and k head, inverse [rows, 2 key_heads].
+void launch_outer_conv(const OuterStateParams& p, bf16* out, float* inverse, cudaStream_t stream, bool pdl);
+// A prompt segment of the delta rule in chunks of 64 tokens (delta_prompt.cu), two launches: pending rows and all rows
+// end up in the state.
+struct DeltaPromptParams {
+  OuterStateParams outer;   // fused (step pre-activations), decay, state, rings, out
+  const bf16* conv;         // [rows, channels]
+  const float* inverse;     // [rows, 2 key_heads]
+  int channels;
+  unsigned char* chunks;    // delta_prompt_bytes(rows, heads, dim_pad, vdim_pad)
+};
+constexpr int kDeltaChunk = 64;
+bool delta_prompt_ok(int dim_pad, int vdim_pad);
+size_t delta_prompt_bytes(size_t rows, size_t heads, size_t dim_pad, size_t vdim_pad);
+void launch_delta_prompt(const DeltaPromptParams& p, cudaStream_t stream, bool pdl);
 // RMS norm in `groups` equal parts of the heads' values side by side, weight, and the gate: SiLU ahead of the norm
 // (gate_first) or sigmoid behind it.
 struct StateFinishParams {
@@ -264,6 +298,12 @@ struct StateFinishParams {
   float eps;
   void* out;
   int out_stride;           // columns beyond the heads' values are cleared
+  // after a prompt segment: the convolution inputs of its last tail_rows rows go to the ring
+  int tail_rows, tail_stride, channels, raw_rows;
+  const void* tail;         // row r at tail + r * tail_stride
+  void* raw;
+  const Control* control;
+  int capacity;
 };
 template <typename T>
 void launch_state_finish(const StateFinishParams& p, cudaStream_t stream, bool pdl);
@@ -358,6 +398,20 @@ struct LayeredModel {
   size_t max_chunk_state = 0;        // floats of one chunk's state
   // prompt workspace (in ei_model::prompt's arena)
   float *residual = nullptr, *linear_out = nullptr, *chunk_states = nullptr, *stretches = nullptr;
+  float *mixed_partial = nullptr, *inverse = nullptr, *decay_totals = nullptr;
+  bf16 *second_normed = nullptr, *second = nullptr, *conv_out = nullptr;
+  unsigned char* delta_chunks = nullptr;
+  int max_channels = 0;
+  size_t max_delta_chunks = 0;       // bytes for a whole segment
+  // Latent attention over a prompt: keys and values of every cached token of one layer, grown when a longer history
+  // comes by.
+  bf16* expanded = nullptr;
+  size_t expanded_bytes = 0, max_expand = 0;  // max_expand: widest row
+  LayeredModel() = default;
+  LayeredModel(const LayeredModel&) = delete;
+  ~LayeredModel() {
+    if (expanded) cudaFree(expanded);
+  }
 };
 
 struct LayeredSession {
@@ -387,10 +441,13 @@ void create_layered_model(ei_model& model, const ei_layered_config& config, cons
                           const ei_named_tensor* tensors, size_t count);
 void create_layered_session(ei_session& s);
 void ensure_layered_workspace(ei_model& model);
+// Room for the expanded keys and values of `tokens` tokens; the caller holds the prompt workspace and its stream is idle.
+void ensure_expanded(ei_model& model, size_t tokens);
 // One forward of at most 16 rows at the device-side context length / of a prompt segment. The segment leaves the
 // normed rows in the prompt workspace; the vocabulary head runs in enqueue_layered_head over gathered rows.
 void enqueue_layered_step(ei_session& s, int rows, StepKind kind);
-void enqueue_layered_segment(ei_session& s, int rows);
+// `context`: the context length the segment starts at, as the device will find it.
+void enqueue_layered_segment(ei_session& s, int rows, size_t context);
 // FP32 logits of `count` <= 16 rows of the segment (indices on the device) into the session's logits; with `greedy`
 // the greedy token of row 0 goes to s.targets[0].
 void enqueue_layered_head(ei_session& s, const int32_t* device_rows, int count, bool greedy);

@@ -12,6 +12,10 @@
 // values, the decayed scores) enters as two BF16 terms, i.e. with 16 significant bits.
 //
 // State layout: [head][slice of 16 values][key dimension][16], so that a block streams contiguous memory.
+//
+// The prompt kernels also run a state-space layer, whose decay and write strength belong to the token (TokenDecay): the
+// powers of the head's decay become exponentials of differences of cumulative logarithms, never above zero. Its step form
+// is in outer_state.cu.
 #include "layered_device.cuh"
 
 #include <stdexcept>
@@ -160,9 +164,36 @@ __device__ __forceinline__ void stage_rows(bf16* to, const bf16* from, int strid
   }
 }
 
+// Logarithms of the decays from the chunk's start through each of its rows, and the rows' steps; `cumulative` [kChunk]
+// and `strengths` [kChunk] are complete after the next block-wide barrier. All threads of the block take part.
+__device__ __forceinline__ void token_decays(const TokenDecay& t, int head, int first, int live, float* cumulative,
+                                             float* strengths, float* warp_totals) {
+  static_assert(kChunk == 128, "four warps scan a chunk");
+  const int row = threadIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float sum = 0.0f;
+  if (row < kChunk) {
+    float step = 0.0f;
+    if (row < live) step = softplus_value(__bfloat162float(t.step[size_t(first + row) * t.step_stride + head]) + t.bias[head]);
+    strengths[row] = step;
+    sum = -t.rate[head] * step;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float below = __shfl_up_sync(0xffffffffu, sum, o);
+      if (lane >= o) sum += below;
+    }
+    if (lane == 31) warp_totals[warp] = sum;
+  }
+  __syncthreads();
+  if (row < kChunk) {
+    for (int w = 0; w < warp; ++w) sum += warp_totals[w];
+    cumulative[row] = sum;
+  }
+}
+
 size_t chunk_state_shared(int dim_pad) { return size_t(kChunk) * (dim_pad + 8) * 2 + size_t(2) * kChunk * kPitch * 2; }
 
 // Block (chunk, head, slice of 64 values): chunk_states[chunk][head] = sum_j decay^(n-1-j) k_j v_j^T.
+template <bool kToken>
 __global__ void __launch_bounds__(kPromptThreads) lightning_chunk_kernel(const LightningParams p) {
   extern __shared__ __align__(16) unsigned char chunk_smem[];
   const int dim = p.dim_pad, k_pitch = dim + 8;
@@ -176,9 +207,16 @@ __global__ void __launch_bounds__(kPromptThreads) lightning_chunk_kernel(const L
   const int chunk = blockIdx.x, head = blockIdx.y, first_value = blockIdx.z * kSlice;
   const int first = chunk * kChunk, live = min(kChunk, p.rows - first);
   const int values = min(kSlice, p.vdim_pad - first_value);
-  const float* powers = p.powers + size_t(head) * (kChunk + 1);
-  stage_rows(keys, static_cast<const bf16*>(p.k) + size_t(first) * p.stride + size_t(head) * dim, p.stride, live, dim / 8,
+  const float* powers = kToken ? nullptr : p.powers + size_t(head) * (kChunk + 1);
+  const int key_head = kToken ? head / (p.heads / p.token.key_heads) : head;
+  stage_rows(keys, static_cast<const bf16*>(p.k) + size_t(first) * p.stride + size_t(key_head) * dim, p.stride, live, dim / 8,
              k_pitch);
+  __shared__ float cumulative[kToken ? kChunk : 1], strengths[kToken ? kChunk : 1], warp_totals[4];
+  if (kToken) {
+    token_decays(p.token, head, first, live, cumulative, strengths, warp_totals);
+    __syncthreads();
+    if (threadIdx.x == 0 && blockIdx.z == 0) p.token.totals[size_t(chunk) * p.heads + head] = cumulative[kChunk - 1];
+  }
 #pragma unroll
   for (int i = threadIdx.x; i < kChunk * (kSlice / 8); i += kPromptThreads) {
     const int row = i >> 3, piece = i & 7;
@@ -186,7 +224,7 @@ __global__ void __launch_bounds__(kPromptThreads) lightning_chunk_kernel(const L
     if (row < live && piece * 8 < values) {
       const uint4 v = *reinterpret_cast<const uint4*>(static_cast<const bf16*>(p.v) + size_t(first + row) * p.stride +
                                                       size_t(head) * p.vdim_pad + first_value + piece * 8);
-      const float w = powers[live - 1 - row];
+      const float w = kToken ? __expf(cumulative[kChunk - 1] - cumulative[row]) * strengths[row] : powers[live - 1 - row];
       split_pair(bf16_lo(v.x) * w, bf16_hi(v.x) * w, hi.x, lo.x);
       split_pair(bf16_lo(v.y) * w, bf16_hi(v.y) * w, hi.y, lo.y);
       split_pair(bf16_lo(v.z) * w, bf16_hi(v.z) * w, hi.z, lo.z);
@@ -234,6 +272,7 @@ __global__ void __launch_bounds__(kPromptThreads) lightning_chunk_kernel(const L
 
 // A thread owns four values of one key dimension: folds the pending rows into the state, then walks the chunks,
 // replacing each contribution by the state ahead of it; the state after the last chunk goes back.
+template <bool kToken>
 __global__ void __launch_bounds__(256) lightning_scan_kernel(const LightningParams p) {
   grid_dependency_wait();
   grid_launch_dependents();
@@ -246,10 +285,18 @@ __global__ void __launch_bounds__(256) lightning_scan_kernel(const LightningPara
   if (i >= quads) return;
   const int column = int(i & 3) * 4;
   const int d = int((i >> 2) % dim), slice = int((i >> 2) / dim % slices), head = int((i >> 2) / dim / slices);
-  const float* powers = p.powers + size_t(head) * (kChunk + 1);
+  const float* powers = kToken ? nullptr : p.powers + size_t(head) * (kChunk + 1);
   float4* state = reinterpret_cast<float4*>(p.state) + i;
   float4 s = base > 0 ? *state : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-  if (pending) {
+  if (kToken) {
+    const int key_head = head / (p.heads / p.token.key_heads);
+    for (int j = 0; j < pending; ++j) {
+      const size_t slot = (base + j) & (kRingRows - 1);
+      const float k = p.token.ring_k[(slot * p.token.key_heads + key_head) * dim + d], g = p.token.ring_g[slot * p.heads + head];
+      const float4 u = *reinterpret_cast<const float4*>(p.token.ring_u + (slot * p.heads + head) * p.vdim_pad + slice * 16 + column);
+      s = make_float4(fmaf(k, u.x, g * s.x), fmaf(k, u.y, g * s.y), fmaf(k, u.z, g * s.z), fmaf(k, u.w, g * s.w));
+    }
+  } else if (pending) {
     const float whole = powers[pending];
     s.x *= whole; s.y *= whole; s.z *= whole; s.w *= whole;
     for (int j = 0; j < pending; ++j) {
@@ -268,7 +315,7 @@ __global__ void __launch_bounds__(256) lightning_scan_kernel(const LightningPara
     const float4 add = next;
     if (chunk + 1 < chunks) next = own[size_t(chunk + 1) * quads];
     own[size_t(chunk) * quads] = s;
-    const float whole = powers[min(kChunk, p.rows - chunk * kChunk)];
+    const float whole = kToken ? expf(p.token.totals[size_t(chunk) * p.heads + head]) : powers[min(kChunk, p.rows - chunk * kChunk)];
     s.x = fmaf(whole, s.x, add.x); s.y = fmaf(whole, s.y, add.y);
     s.z = fmaf(whole, s.z, add.z); s.w = fmaf(whole, s.w, add.w);
   }
@@ -281,6 +328,7 @@ size_t output_shared(int dim_pad) {
 }
 
 // Block (chunk, head, slice of 64 values), eight warps of 16 tokens each.
+template <bool kToken>
 __global__ void __launch_bounds__(kPromptThreads) lightning_output_kernel(const LightningParams p) {
   extern __shared__ __align__(16) unsigned char output_smem[];
   const int dim = p.dim_pad, k_pitch = dim + 8;
@@ -296,9 +344,13 @@ __global__ void __launch_bounds__(kPromptThreads) lightning_output_kernel(const 
   const int chunk = blockIdx.x, head = blockIdx.y, first_value = blockIdx.z * kSlice;
   const int first = chunk * kChunk, live = min(kChunk, p.rows - first);
   const int values = min(kSlice, p.vdim_pad - first_value);
-  for (int i = threadIdx.x; i <= kChunk; i += blockDim.x) powers[i] = p.powers[size_t(head) * (kChunk + 1) + i];
-  stage_rows(keys, static_cast<const bf16*>(p.k) + size_t(first) * p.stride + size_t(head) * dim, p.stride, live, dim / 8,
+  __shared__ float cumulative[kToken ? kChunk : 1], strengths[kToken ? kChunk : 1], warp_totals[4];
+  if (!kToken)
+    for (int i = threadIdx.x; i <= kChunk; i += blockDim.x) powers[i] = p.powers[size_t(head) * (kChunk + 1) + i];
+  const int key_head = kToken ? head / (p.heads / p.token.key_heads) : head;
+  stage_rows(keys, static_cast<const bf16*>(p.k) + size_t(first) * p.stride + size_t(key_head) * dim, p.stride, live, dim / 8,
              k_pitch);
+  if (kToken) token_decays(p.token, head, first, live, cumulative, strengths, warp_totals);
   {
     const bf16* v = static_cast<const bf16*>(p.v) + size_t(first) * p.stride + size_t(head) * p.vdim_pad + first_value;
 #pragma unroll
@@ -328,7 +380,7 @@ __global__ void __launch_bounds__(kPromptThreads) lightning_output_kernel(const 
   const int matrix = lane >> 3, in_matrix = lane & 7;
   const int lo_row = warp * 16 + g, hi_row = lo_row + 8;
   if (warp * 16 >= live) return;
-  const bf16* q = static_cast<const bf16*>(p.q) + size_t(first) * p.stride + size_t(head) * dim;
+  const bf16* q = static_cast<const bf16*>(p.q) + size_t(first) * p.stride + size_t(key_head) * dim;
   const int key_tiles = 2 * (warp + 1);  // tiles of eight keys this warp's rows can see
   float acc[8][4], s[16][4];
 #pragma unroll
@@ -366,7 +418,12 @@ __global__ void __launch_bounds__(kPromptThreads) lightning_output_kernel(const 
       }
     }
   }
-  const float lo_power = powers[lo_row + 1], hi_power = powers[hi_row + 1];
+  // What a row's query sees of the state ahead of the chunk, and of the write of row j of the chunk.
+  const float lo_power = kToken ? __expf(cumulative[lo_row]) : powers[lo_row + 1];
+  const float hi_power = kToken ? __expf(cumulative[hi_row]) : powers[hi_row + 1];
+  auto reach = [&](int row, int j) {
+    return kToken ? __expf(cumulative[row] - cumulative[j]) * strengths[j] : powers[row - j];
+  };
 #pragma unroll
   for (int n = 0; n < 8; ++n) {
     acc[n][0] *= lo_power;
@@ -381,10 +438,10 @@ __global__ void __launch_bounds__(kPromptThreads) lightning_output_kernel(const 
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int n = 2 * t + half, j0 = n * 8 + 2 * c, j1 = j0 + 1;
-        const float s0 = j0 <= lo_row ? s[n][0] * powers[lo_row - j0] : 0.0f;
-        const float s1 = j1 <= lo_row ? s[n][1] * powers[lo_row - j1] : 0.0f;
-        const float s2 = j0 <= hi_row ? s[n][2] * powers[hi_row - j0] : 0.0f;
-        const float s3 = j1 <= hi_row ? s[n][3] * powers[hi_row - j1] : 0.0f;
+        const float s0 = j0 <= lo_row ? s[n][0] * reach(lo_row, j0) : 0.0f;
+        const float s1 = j1 <= lo_row ? s[n][1] * reach(lo_row, j1) : 0.0f;
+        const float s2 = j0 <= hi_row ? s[n][2] * reach(hi_row, j0) : 0.0f;
+        const float s3 = j1 <= hi_row ? s[n][3] * reach(hi_row, j1) : 0.0f;
         split_pair(s0, s1, wl[2 * half], wr[2 * half]);
         split_pair(s2, s3, wl[2 * half + 1], wr[2 * half + 1]);
       }
@@ -397,6 +454,18 @@ __global__ void __launch_bounds__(kPromptThreads) lightning_output_kernel(const 
         mma_bf16_16816(acc[n], wr[0], wr[1], wr[2], wr[3], b0, b1);
         mma_bf16_16816(acc[n + 1], wr[0], wr[1], wr[2], wr[3], b2, b3);
       }
+    }
+  }
+  if (kToken && p.token.skip) {
+    const float skip = p.token.skip[head];
+#pragma unroll
+    for (int n = 0; n < 8; ++n) {
+      const uint32_t lo = *reinterpret_cast<const uint32_t*>(vals + lo_row * kPitch + n * 8 + 2 * c);
+      const uint32_t hi = *reinterpret_cast<const uint32_t*>(vals + hi_row * kPitch + n * 8 + 2 * c);
+      acc[n][0] = fmaf(skip, bf16_lo(lo), acc[n][0]);
+      acc[n][1] = fmaf(skip, bf16_hi(lo), acc[n][1]);
+      acc[n][2] = fmaf(skip, bf16_lo(hi), acc[n][2]);
+      acc[n][3] = fmaf(skip, bf16_hi(hi), acc[n][3]);
     }
   }
   const size_t pitch = size_t(p.heads) * p.vdim_pad;
@@ -439,21 +508,28 @@ template void launch_lightning_step<bf16>(const LightningParams&, cudaStream_t, 
 
 bool lightning_prompt_ok(int dim_pad, int vdim_pad) { return dim_pad <= 256 && dim_pad % 16 == 0 && vdim_pad % 16 == 0; }
 
-void launch_lightning_prompt(const LightningParams& p, cudaStream_t stream, bool pdl, int* launches) {
+namespace {
+template <bool kToken>
+void launch_prompt_kernels(const LightningParams& p, cudaStream_t stream, bool pdl) {
   static thread_local int configured_device = -1;
   int device = 0;
   EI_CUDA(cudaGetDevice(&device));
   if (configured_device != device) {
-    EI_CUDA(cudaFuncSetAttribute(lightning_chunk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(chunk_state_shared(256))));
-    EI_CUDA(cudaFuncSetAttribute(lightning_output_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(output_shared(256))));
+    EI_CUDA(cudaFuncSetAttribute(lightning_chunk_kernel<kToken>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(chunk_state_shared(256))));
+    EI_CUDA(cudaFuncSetAttribute(lightning_output_kernel<kToken>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(output_shared(256))));
     configured_device = device;
   }
-  if (!lightning_prompt_ok(p.dim_pad, p.vdim_pad)) throw std::invalid_argument("linear attention prompt takes key sizes up to 256");
   const unsigned chunks = unsigned((p.rows + kChunk - 1) / kChunk), slices = unsigned((p.vdim_pad + kSlice - 1) / kSlice);
   const size_t quads = size_t(p.heads) * p.vdim_pad / 4 * p.dim_pad;
-  launch(lightning_chunk_kernel, dim3(chunks, p.heads, slices), dim3(kPromptThreads), chunk_state_shared(p.dim_pad), stream, pdl, p);
-  launch(lightning_scan_kernel, dim3(unsigned((quads + 255) / 256)), dim3(256), 0, stream, pdl, p);
-  launch(lightning_output_kernel, dim3(chunks, p.heads, slices), dim3(kPromptThreads), output_shared(p.dim_pad), stream, pdl, p);
+  launch(lightning_chunk_kernel<kToken>, dim3(chunks, p.heads, slices), dim3(kPromptThreads), chunk_state_shared(p.dim_pad), stream, pdl, p);
+  launch(lightning_scan_kernel<kToken>, dim3(unsigned((quads + 255) / 256)), dim3(256), 0, stream, pdl, p);
+  launch(lightning_output_kernel<kToken>, dim3(chunks, p.heads, slices), dim3(kPromptThreads), output_shared(p.dim_pad), stream, pdl, p);
+}
+}  // namespace
+
+void launch_lightning_prompt(const LightningParams& p, cudaStream_t stream, bool pdl, int* launches) {
+  if (!lightning_prompt_ok(p.dim_pad, p.vdim_pad)) throw std::invalid_argument("linear attention prompt takes key sizes up to 256");
+  p.token.step ? launch_prompt_kernels<true>(p, stream, pdl) : launch_prompt_kernels<false>(p, stream, pdl);
   if (launches) *launches += 3;
 }
 

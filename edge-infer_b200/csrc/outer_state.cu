@@ -167,6 +167,110 @@ __global__ void __launch_bounds__(128) outer_step_kernel(const OuterStateParams 
   }
 }
 
+// A prompt segment's convolution: a warp takes eight rows of one head of q, k or v, kVector channels per lane at a time.
+// kTaps 0: any number of taps.
+constexpr int kConvRows = 8;
+template <int kVector>
+struct Channels {
+  float v[kVector];
+};
+__device__ __forceinline__ Channels<4> load_channels(const bf16* p, Channels<4>) {
+  const float4 x = load_quad(p);
+  return {{x.x, x.y, x.z, x.w}};
+}
+__device__ __forceinline__ Channels<2> load_channels(const bf16* p, Channels<2>) {
+  const float2 x = load_pair(p);
+  return {{x.x, x.y}};
+}
+__device__ __forceinline__ void store_channels(bf16* p, Channels<4> x) { store_quad(p, make_float4(x.v[0], x.v[1], x.v[2], x.v[3])); }
+__device__ __forceinline__ void store_channels(bf16* p, Channels<2> x) { store_pair(p, x.v[0], x.v[1]); }
+
+template <int kTaps, int kVector>
+__device__ __forceinline__ void conv_head(const OuterStateParams& p, bf16* out, float* inverse, int context, int begin, int unit, int lane) {
+  using Vector = Channels<kVector>;
+  const int kind = unit < p.key_heads ? 0 : unit < 2 * p.key_heads ? 1 : 2;  // q, k, v
+  const int head = unit - kind * p.key_heads, pad = kind == 2 ? p.vdim_pad : p.dim_pad;
+  const int first = kind * p.key_heads * p.dim_pad + head * pad;
+  const int channels = 2 * p.key_heads * p.dim_pad + p.heads * p.vdim_pad;
+  const bf16* fused = static_cast<const bf16*>(p.fused);
+  const bf16* raw = static_cast<const bf16*>(p.raw);
+  const int taps = kTaps ? kTaps : p.taps;
+  float squares[kConvRows];
+#pragma unroll
+  for (int r = 0; r < kConvRows; ++r) squares[r] = 0.0f;
+  for (int c = lane * kVector; c < pad; c += 32 * kVector) {
+    const int channel = first + c;
+    auto input = [&](int r) {
+      if (r >= p.rows) return Vector{};
+      if (r >= 0) return load_channels(fused + size_t(r) * p.stride + channel, Vector{});
+      return context + r >= 0 ? load_channels(raw + size_t((context + r) & (p.raw_rows - 1)) * channels + channel, Vector{}) : Vector{};
+    };
+    Vector sums[kConvRows];
+#pragma unroll
+    for (int r = 0; r < kConvRows; ++r)
+#pragma unroll
+      for (int j = 0; j < kVector; ++j) sums[r].v[j] = p.conv_bias ? p.conv_bias[channel + j] : 0.0f;
+    if (kTaps) {
+      Vector window[kConvRows + (kTaps ? kTaps - 1 : 0)];
+#pragma unroll
+      for (int i = 0; i < kConvRows + kTaps - 1; ++i) window[i] = input(begin + i - (kTaps - 1));
+#pragma unroll
+      for (int tap = 0; tap < kTaps; ++tap)
+#pragma unroll
+        for (int j = 0; j < kVector; ++j) {
+          const float w = p.conv[size_t(tap) * channels + channel + j];
+#pragma unroll
+          for (int r = 0; r < kConvRows; ++r) sums[r].v[j] = fmaf(window[r + tap].v[j], w, sums[r].v[j]);
+        }
+    } else {
+      for (int tap = 0; tap < taps; ++tap) {
+        Vector w;
+#pragma unroll
+        for (int j = 0; j < kVector; ++j) w.v[j] = p.conv[size_t(tap) * channels + channel + j];
+#pragma unroll
+        for (int r = 0; r < kConvRows; ++r) {
+          const Vector x = input(begin + r - (taps - 1) + tap);
+#pragma unroll
+          for (int j = 0; j < kVector; ++j) sums[r].v[j] = fmaf(x.v[j], w.v[j], sums[r].v[j]);
+        }
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < kConvRows; ++r) {
+      if (begin + r >= p.rows) break;
+#pragma unroll
+      for (int j = 0; j < kVector; ++j) {
+        sums[r].v[j] = round_bf16(sums[r].v[j] * quick_sigmoid(sums[r].v[j]));
+        squares[r] = fmaf(sums[r].v[j], sums[r].v[j], squares[r]);
+      }
+      store_channels(out + size_t(begin + r) * channels + channel, sums[r]);
+    }
+  }
+  if (!p.delta || kind == 2) return;
+#pragma unroll
+  for (int r = 0; r < kConvRows; ++r) {
+    float scale = 1.0f / sqrtf(warp_sum(squares[r]) + 1e-6f);
+    if (kind == 0) scale /= sqrtf(float(p.dim));
+    if (lane == 0 && begin + r < p.rows) inverse[size_t(begin + r) * 2 * p.key_heads + unit] = scale;
+  }
+}
+
+template <int kTaps>
+__global__ void __launch_bounds__(128) outer_conv_kernel(const OuterStateParams p, bf16* out, float* inverse) {
+  const int context = p.control->context;  // written by the previous step
+  grid_dependency_wait();
+  grid_launch_dependents();
+  if (context < 0 || context + p.rows > p.capacity) return;
+  const int units = 2 * p.key_heads + p.heads;
+  const int warp = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int unit = warp % units, begin = warp / units * kConvRows;
+  if (begin >= p.rows) return;
+  if ((unit < 2 * p.key_heads ? p.dim_pad : p.vdim_pad) > 64)
+    conv_head<kTaps, 4>(p, out, inverse, context, begin, unit, lane);
+  else
+    conv_head<kTaps, 2>(p, out, inverse, context, begin, unit, lane);
+}
+
 // One warp (kWide: one block) per (row, norm group). Values of a group are those of its heads side by side, without the
 // heads' padding.
 constexpr int kFinishHeld = 8;
@@ -177,7 +281,18 @@ __global__ void __launch_bounds__(256) state_finish_kernel(const StateFinishPara
   grid_launch_dependents();
   const int lanes = kWide ? blockDim.x : 32, lane = kWide ? threadIdx.x : threadIdx.x & 31;
   const int item = kWide ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (item >= p.rows * p.groups) return;
+  if (item >= p.rows * p.groups) {
+    // Behind them: convolution inputs into the ring.
+    const int back = item - p.rows * p.groups, r = p.rows - 1 - back, context = p.control ? p.control->context : -1;
+    if (back >= p.tail_rows || context < 0 || context + p.rows > p.capacity) return;
+    const T* from = static_cast<const T*>(p.tail) + size_t(r) * p.tail_stride;
+    T* to = static_cast<T*>(p.raw) + size_t((context + r) & (p.raw_rows - 1)) * p.channels;
+    for (int i = lane * 2; i < p.channels; i += lanes * 2) {
+      const float2 v = load_pair(from + i);
+      store_pair(to + i, v.x, v.y);
+    }
+    return;
+  }
   const int row = item / p.groups, group = item - row * p.groups;
   const int length = p.heads * p.vdim / p.groups, first = group * length;
   const int width = p.heads * p.vdim_pad;
@@ -245,6 +360,14 @@ void launch_outer_prepare(const OuterStateParams& p, cudaStream_t stream, bool p
   const int warps = p.rows * (2 * p.key_heads + p.heads + (p.delta ? p.heads : (p.heads + 31) / 32));
   launch(outer_prepare_kernel<T>, dim3(unsigned((warps + 3) / 4)), dim3(128), 0, stream, pdl, p);
 }
+void launch_outer_conv(const OuterStateParams& p, bf16* out, float* inverse, cudaStream_t stream, bool pdl) {
+  const int warps = (p.rows + kConvRows - 1) / kConvRows * (2 * p.key_heads + p.heads);
+  const dim3 grid(unsigned((warps + 3) / 4));
+  if (p.taps == 2) return launch(outer_conv_kernel<2>, grid, dim3(128), 0, stream, pdl, p, out, inverse);
+  if (p.taps == 3) return launch(outer_conv_kernel<3>, grid, dim3(128), 0, stream, pdl, p, out, inverse);
+  if (p.taps == 4) return launch(outer_conv_kernel<4>, grid, dim3(128), 0, stream, pdl, p, out, inverse);
+  launch(outer_conv_kernel<0>, grid, dim3(128), 0, stream, pdl, p, out, inverse);
+}
 void launch_outer_step(const OuterStateParams& p, cudaStream_t stream, bool pdl) {
   if (p.rows < 1 || p.rows > kPendingRows || p.dim_pad > kMaxHeadDim)
     throw std::invalid_argument("a state step takes 1..16 rows and key sizes up to 512");
@@ -252,7 +375,7 @@ void launch_outer_step(const OuterStateParams& p, cudaStream_t stream, bool pdl)
 }
 template <typename T>
 void launch_state_finish(const StateFinishParams& p, cudaStream_t stream, bool pdl) {
-  const int items = p.rows * p.groups, length = p.heads * p.vdim / p.groups;
+  const int items = p.rows * p.groups + p.tail_rows, length = p.heads * p.vdim / p.groups;
   if (length > 256)
     launch(state_finish_kernel<T, true>, dim3(unsigned(items)), dim3(256), 0, stream, pdl, p);
   else

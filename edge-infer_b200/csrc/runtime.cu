@@ -1378,6 +1378,12 @@ static void append_tokens(ei_session& s, const uint32_t* host_tokens, size_t row
   if (wide) {
     auto& ws = m.prompt;
     m.layered ? ensure_layered_workspace(m) : ensure_prompt_workspace(m);
+    size_t start = 0;  // the context length on the device
+    if (m.layered && m.layered->max_expand) {
+      read_control(s);
+      start = size_t(s.host_control->context);
+      ensure_expanded(m, start + rows);
+    }
     for (size_t first = 0; first < rows; first += ws.rows) {
       const size_t count = std::min(ws.rows, rows - first);
       const bool head = last_logits && first + count >= rows;
@@ -1385,7 +1391,7 @@ static void append_tokens(ei_session& s, const uint32_t* host_tokens, size_t row
       std::memcpy(ws.host_tokens, host_tokens + first, count * 4);
       EI_CUDA(cudaMemcpyAsync(ws.tokens, ws.host_tokens, count * 4, cudaMemcpyHostToDevice, s.stream));
       if (m.layered)
-        enqueue_layered_segment(s, int(count));
+        enqueue_layered_segment(s, int(count), start + first);
       else
         enqueue_prompt_segment(s, int(count), head);
       // The segment's normed rows stay in the workspace: the head runs over the wanted ones, 16 at a time.

@@ -10,7 +10,10 @@
 //    cache needs no padding beyond a multiple of 16;
 //  * query rows of all heads of a KV group are stacked over the whole row range and dealt to blocks of up to four
 //    warps, 16 stacked rows per warp, so any group size and row count works;
-//  * kernels are compiled for sizes up to 64, 128 and 256, with the size known at compile time when it is exactly that.
+//  * kernels are compiled for sizes up to 64, 128 and 256, and for keys up to 256 with values up to 128, with the sizes
+//    known at compile time when they are exactly 64, 128 or 192 and 128;
+//  * a key may end in a part that all heads share (latent attention's rotated key), fetched from a tensor of its own;
+//  * the finished output may pass a sigmoid gate.
 #include "layered_device.cuh"
 
 #include <algorithm>
@@ -42,13 +45,13 @@ size_t sized_shared_bytes(int dim_pad, int vdim_pad) {
 // kDirect = false: block (kv head, split of the sequence, part of the stacked rows) writes (o, m, l) partials.
 // kDirect = true: block (kv head, part) covers its rows' whole history and writes the finished output; parts with the
 // longest histories start first.
-template <int kBucket, bool kExact, bool kDirect>
+template <int kKeys, int kValues, bool kExact, bool kDirect>
 __global__ void __launch_bounds__(kMaxWarps * 32) sized_attention_kernel(const __grid_constant__ SizedAttentionParams p) {
   extern __shared__ unsigned char sized_smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(sized_smem_raw) + 1023) &
                                                          ~uintptr_t(1023));
-  constexpr int kSteps = kBucket / 16;
-  const int dim = kExact ? kBucket : p.dim_pad, vdim = kExact ? kBucket : p.vdim_pad;
+  constexpr int kSteps = kKeys / 16, kTiles = kValues / 8;
+  const int dim = kExact ? kKeys : p.dim_pad, vdim = kExact ? kValues : p.vdim_pad;
   const int k_steps = dim / 16, v_tiles = vdim / 8;
   const int k_shift = kExact ? 3 : p.k_shift, v_shift = kExact ? 3 : p.v_shift;
   const int k_bytes = kTile * dim * 2, v_bytes = kTile * vdim * 2, stage_bytes = k_bytes + v_bytes;
@@ -86,9 +89,11 @@ __global__ void __launch_bounds__(kMaxWarps * 32) sized_attention_kernel(const _
     unsigned char* base = smem + size_t(stage) * stage_bytes;
     mbarrier_expect_tx(&sh->full[stage], uint32_t(stage_bytes) + (tile == 0 ? p.fault_tx : 0u));
     tma_load_4d(base, &p.k_map, 0, start + tile * kTile, 0, kv_head, &sh->full[stage]);
+    if (p.shared_pad)
+      tma_load_4d(base + kTile * (dim - p.shared_pad) * 2, &p.shared_map, 0, start + tile * kTile, 0, 0, &sh->full[stage]);
     tma_load_4d(base + k_bytes, &p.v_map, 0, start + tile * kTile, 0, kv_head, &sh->full[stage]);
   };
-  const bool settled = end <= offset;  // nothing in this chunk is written by the preceding kernel
+  const bool settled = end <= offset && !p.fresh;  // nothing in this chunk is written by the preceding kernel
   if (!settled) grid_dependency_wait();
   if (threadIdx.x == 0)
     for (int tile = 0; tile < min(kStages, tiles); ++tile) request(tile);
@@ -119,9 +124,9 @@ __global__ void __launch_bounds__(kMaxWarps * 32) sized_attention_kernel(const _
   const int warp_first = first_stacked + warp * 16;
   const int warp_limit = warp_first < stacked ? offset + min(stacked - 1, warp_first + 15) / group : -1;
 
-  float o[2 * kSteps][4];
+  float o[kTiles][4];
 #pragma unroll
-  for (int d = 0; d < 2 * kSteps; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.0f;
+  for (int d = 0; d < kTiles; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.0f;
   float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.0f, l_hi = 0.0f;
 
   int tile = 0;
@@ -195,7 +200,7 @@ __global__ void __launch_bounds__(kMaxWarps * 32) sized_attention_kernel(const _
       l_lo = l_lo * rescale_lo + sum_lo;
       l_hi = l_hi * rescale_hi + sum_hi;
 #pragma unroll
-      for (int d = 0; d < 2 * kSteps; ++d) {
+      for (int d = 0; d < kTiles; ++d) {
         o[d][0] *= rescale_lo;
         o[d][1] *= rescale_lo;
         o[d][2] *= rescale_hi;
@@ -204,7 +209,7 @@ __global__ void __launch_bounds__(kMaxWarps * 32) sized_attention_kernel(const _
 #pragma unroll
       for (int t = 0; t < 4; ++t) {
 #pragma unroll
-        for (int d = 0; d < 2 * kSteps; d += 2) {
+        for (int d = 0; d < kTiles; d += 2) {
           if (kExact || d < v_tiles) {
             uint32_t b0, b1, b2, b3;
             ldmatrix_x4_trans(b0, b1, b2, b3,
@@ -246,11 +251,20 @@ __global__ void __launch_bounds__(kMaxWarps * 32) sized_attention_kernel(const _
     bf16* out = static_cast<bf16*>(p.out);
     bf16* d_lo = out + size_t(r_lo) * p.out_stride + size_t(h_lo) * vdim;
     bf16* d_hi = out + size_t(r_hi) * p.out_stride + size_t(h_hi) * vdim;
+    const bf16* gate = static_cast<const bf16*>(p.gate);
+    const bf16* g_lo = gate ? gate + size_t(r_lo) * p.gate_stride + size_t(h_lo) * vdim : nullptr;
+    const bf16* g_hi = gate ? gate + size_t(r_hi) * p.gate_stride + size_t(h_hi) * vdim : nullptr;
+    auto gated = [&](const bf16* g, int at, float a, float b) {
+      if (!gate) return pack_bf16(a, b);
+      const float2 z = load_pair(g + at);
+      return pack_bf16(a * quick_sigmoid(z.x), b * quick_sigmoid(z.y));
+    };
 #pragma unroll
-    for (int d = 0; d < 2 * kSteps; ++d) {
+    for (int d = 0; d < kTiles; ++d) {
       if (kExact || d < v_tiles) {
-        if (live_lo) *reinterpret_cast<uint32_t*>(d_lo + d * 8 + 2 * c) = pack_bf16(o[d][0] * f_lo, o[d][1] * f_lo);
-        if (live_hi) *reinterpret_cast<uint32_t*>(d_hi + d * 8 + 2 * c) = pack_bf16(o[d][2] * f_hi, o[d][3] * f_hi);
+        const int at = d * 8 + 2 * c;
+        if (live_lo) *reinterpret_cast<uint32_t*>(d_lo + at) = gated(g_lo, at, o[d][0] * f_lo, o[d][1] * f_lo);
+        if (live_hi) *reinterpret_cast<uint32_t*>(d_hi + at) = gated(g_hi, at, o[d][2] * f_hi, o[d][3] * f_hi);
       }
     }
     return;
@@ -260,7 +274,7 @@ __global__ void __launch_bounds__(kMaxWarps * 32) sized_attention_kernel(const _
   float* d_lo = p.scratch + (size_t(split) * slots + size_t(r_lo) * p.heads + h_lo) * pitch;
   float* d_hi = p.scratch + (size_t(split) * slots + size_t(r_hi) * p.heads + h_hi) * pitch;
 #pragma unroll
-  for (int d = 0; d < 2 * kSteps; ++d) {
+  for (int d = 0; d < kTiles; ++d) {
     if (kExact || d < v_tiles) {
       if (live_lo) *reinterpret_cast<float2*>(d_lo + d * 8 + 2 * c) = make_float2(o[d][0], o[d][1]);
       if (live_hi) *reinterpret_cast<float2*>(d_hi + d * 8 + 2 * c) = make_float2(o[d][2], o[d][3]);
@@ -355,8 +369,8 @@ __global__ void __launch_bounds__(128) plain_attention_kernel(const SizedAttenti
 // 16-byte pieces per box row (as log2): the widest of 64, 32 and 16 values that divides the padded head.
 int box_shift(int pad) { return pad % 64 == 0 ? 3 : pad % 32 == 0 ? 2 : 1; }
 
-void encode_head_map(CUtensorMap* map, const void* base, int tokens, int token_stride, int kv_heads, int pad) {
-  const int shift = box_shift(pad), values = 8 << shift;
+void encode_head_map(CUtensorMap* map, const void* base, int tokens, int token_stride, int kv_heads, int pad, int shift) {
+  const int values = 8 << shift;
   const cuuint64_t dims[4] = {cuuint64_t(values), cuuint64_t(tokens), cuuint64_t(pad / values), cuuint64_t(kv_heads)};
   const cuuint64_t strides[3] = {cuuint64_t(token_stride) * 2, cuuint64_t(values) * 2, cuuint64_t(pad) * 2};
   const cuuint32_t box[4] = {cuuint32_t(values), cuuint32_t(kTile), cuuint32_t(pad / values), 1};
@@ -365,16 +379,16 @@ void encode_head_map(CUtensorMap* map, const void* base, int tokens, int token_s
              "sized K / V cache");
 }
 
-template <int kBucket, bool kExact>
+template <int kKeys, int kValues, bool kExact>
 void launch_bucket(const SizedAttentionParams& p, bool direct, cudaStream_t stream, bool pdl) {
   static thread_local int configured_device = -1;
   int device = 0;
   EI_CUDA(cudaGetDevice(&device));
   if (configured_device != device) {
-    const int bytes = int(sized_shared_bytes(kBucket, kBucket));
-    EI_CUDA(cudaFuncSetAttribute(sized_attention_kernel<kBucket, kExact, false>,
+    const int bytes = int(sized_shared_bytes(kKeys, kValues));
+    EI_CUDA(cudaFuncSetAttribute(sized_attention_kernel<kKeys, kValues, kExact, false>,
                                  cudaFuncAttributeMaxDynamicSharedMemorySize, bytes));
-    EI_CUDA(cudaFuncSetAttribute(sized_attention_kernel<kBucket, kExact, true>,
+    EI_CUDA(cudaFuncSetAttribute(sized_attention_kernel<kKeys, kValues, kExact, true>,
                                  cudaFuncAttributeMaxDynamicSharedMemorySize, bytes));
     configured_device = device;
   }
@@ -383,31 +397,38 @@ void launch_bucket(const SizedAttentionParams& p, bool direct, cudaStream_t stre
   const unsigned parts = unsigned((stacked + warps * 16 - 1) / (warps * 16));
   const size_t smem = sized_shared_bytes(p.dim_pad, p.vdim_pad);
   if (direct)
-    launch(sized_attention_kernel<kBucket, kExact, true>, dim3(p.kv_heads, parts), dim3(warps * 32), smem, stream, pdl, p);
+    launch(sized_attention_kernel<kKeys, kValues, kExact, true>, dim3(p.kv_heads, parts), dim3(warps * 32), smem, stream, pdl, p);
   else
-    launch(sized_attention_kernel<kBucket, kExact, false>, dim3(p.kv_heads, p.max_splits, parts), dim3(warps * 32), smem,
+    launch(sized_attention_kernel<kKeys, kValues, kExact, false>, dim3(p.kv_heads, p.max_splits, parts), dim3(warps * 32), smem,
            stream, pdl, p);
 }
 
 void launch_sized(const SizedAttentionParams& given, bool direct, cudaStream_t stream, bool pdl) {
   SizedAttentionParams p = given;
   if (!sized_attention_ok(p.dim_pad, p.vdim_pad)) throw std::invalid_argument("tiled attention takes head sizes up to 256");
-  p.k_shift = box_shift(p.dim_pad);
+  const int own = p.dim_pad - p.shared_pad;  // key values of each head's own
+  p.k_shift = p.shared_pad ? std::min(box_shift(own), box_shift(p.shared_pad)) : box_shift(own);
   p.v_shift = box_shift(p.vdim_pad);
-  const int tokens = (p.capacity + kTile - 1) / kTile * kTile;  // the caches are allocated in whole tiles
-  encode_head_map(&p.k_map, p.k, tokens, p.k_stride, p.kv_heads, p.dim_pad);
-  encode_head_map(&p.v_map, p.v, tokens, p.v_stride, p.kv_heads, p.vdim_pad);
+  // The caches are allocated in whole tiles.
+  const int tokens = p.tokens ? p.tokens : (p.capacity + kTile - 1) / kTile * kTile;
+  encode_head_map(&p.k_map, p.k, tokens, p.k_stride, p.kv_heads, own, p.k_shift);
+  if (p.shared_pad) encode_head_map(&p.shared_map, p.shared, tokens, p.shared_stride, 1, p.shared_pad, p.k_shift);
+  encode_head_map(&p.v_map, p.v, tokens, p.v_stride, p.kv_heads, p.vdim_pad, p.v_shift);
   const int widest = std::max(p.dim_pad, p.vdim_pad);
-  const bool same = p.dim_pad == p.vdim_pad;
+  const bool same = p.dim_pad == p.vdim_pad && p.k_shift == 3;
   if (widest <= 64) {
-    if (same && widest == 64) return launch_bucket<64, true>(p, direct, stream, pdl);
-    return launch_bucket<64, false>(p, direct, stream, pdl);
+    if (same && widest == 64) return launch_bucket<64, 64, true>(p, direct, stream, pdl);
+    return launch_bucket<64, 64, false>(p, direct, stream, pdl);
   }
   if (widest <= 128) {
-    if (same && widest == 128) return launch_bucket<128, true>(p, direct, stream, pdl);
-    return launch_bucket<128, false>(p, direct, stream, pdl);
+    if (same && widest == 128) return launch_bucket<128, 128, true>(p, direct, stream, pdl);
+    return launch_bucket<128, 128, false>(p, direct, stream, pdl);
   }
-  return launch_bucket<256, false>(p, direct, stream, pdl);
+  if (p.vdim_pad <= 128) {
+    if (p.dim_pad == 192 && p.vdim_pad == 128 && p.k_shift == 3) return launch_bucket<192, 128, true>(p, direct, stream, pdl);
+    return launch_bucket<256, 128, false>(p, direct, stream, pdl);
+  }
+  return launch_bucket<256, 256, false>(p, direct, stream, pdl);
 }
 
 }  // namespace

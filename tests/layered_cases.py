@@ -98,3 +98,23 @@ def logit_error(got, want):
     d = d - d.mean(axis=-1, keepdims=True)
     scale = np.sqrt(np.mean((want - want.mean(axis=-1, keepdims=True)) ** 2))
     return np.sqrt(np.mean(d * d, axis=-1)) / scale
+
+
+def run_portions(session, ids, sizes):
+    """All positions' logits, the sequence cut into portions (the last size repeats)."""
+    out, at, sizes = [], 0, list(sizes)
+    while at < len(ids):
+        size = min(sizes.pop(0) if len(sizes) > 1 else sizes[0], len(ids) - at)
+        out.append(session.extend(ids[at:at + size], range(size)))
+        at += size
+    return np.concatenate(out)
+
+
+def greedy(oracle, prompt, count):
+    """The restatement's own greedy continuation."""
+    logits = oracle.forward(prompt)[-1]
+    out = []
+    for _ in range(count):
+        out.append(int(np.argmax(logits)))
+        logits = oracle.forward([out[-1]])[0]
+    return out

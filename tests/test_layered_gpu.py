@@ -27,16 +27,6 @@ def build(package, c, kind, seed=0, sharp=1.0):
     return package.Model(shape, tensors), hybrid.HybridOracle(c, weights)
 
 
-def run_portions(session, ids, sizes):
-    """All positions' logits, the sequence cut into portions (the last size repeats)."""
-    out, at, sizes = [], 0, list(sizes)
-    while at < len(ids):
-        size = min(sizes.pop(0) if len(sizes) > 1 else sizes[0], len(ids) - at)
-        out.append(session.extend(ids[at:at + size], range(size)))
-        at += size
-    return np.concatenate(out)
-
-
 def check(got, want, kind, what=""):
     error = cases.logit_error(got, want)
     assert error.max() <= LIMIT[kind], f"{what}: position {int(error.argmax())} is off by {error.max():.3g}"
@@ -53,7 +43,7 @@ def test_every_case_whole_stepwise_and_in_portions(cuda, package, name, kind):
     session = model.new_session(160, graph=True)
     for sizes in ([150], [1], [2, 37, 16, 3, 64, 1]):
         session.reset()
-        check(run_portions(session, ids, sizes), want, kind, f"portions {sizes}")
+        check(cases.run_portions(session, ids, sizes), want, kind, f"portions {sizes}")
 
 
 @pytest.mark.parametrize("kind", KINDS)
@@ -119,7 +109,7 @@ def test_one_key_that_stands_out(cuda, package, kind):
         assert shift.min() > 0.1                             # the key matters at every probe
         for sizes in ([330], [62, 2, 1, 63, 129, 33, 40]) if kind == "bf16" else ([62, 2, 1],):
             session = model.new_session(330, graph=True)
-            check(run_portions(session, ids, sizes), want, kind, f"key at {place}, portions {sizes}")
+            check(cases.run_portions(session, ids, sizes), want, kind, f"key at {place}, portions {sizes}")
 
 
 # ---- cuts, long sequences, reuse ----
@@ -130,7 +120,7 @@ def test_portions_of_any_size(cuda, package, size, kind):
     model, oracle = build(package, c, kind, seed=2, sharp=1.5)
     ids = cases.tokens(c, 300, 5)
     session = model.new_session(300, graph=True)
-    check(run_portions(session, ids, [size]), oracle.forward(ids), kind, f"portions of {size}")
+    check(cases.run_portions(session, ids, [size]), oracle.forward(ids), kind, f"portions of {size}")
 
 
 def test_prompt_beyond_a_segment_then_long_decoding(cuda, package):
@@ -144,7 +134,7 @@ def test_prompt_beyond_a_segment_then_long_decoding(cuda, package):
     places = [0, 1, 63, 64, 127, 128, 129, 2046, 2047, 2048, 2049, 2175, 2176, 4095, 4096, 4249]
     got = session.extend(ids[:4250], places)
     check(got, want[places], "bf16", "prompt")
-    check(run_portions(session, ids[4250:], [1]), want[4250:], "bf16", "decoding")
+    check(cases.run_portions(session, ids[4250:], [1]), want[4250:], "bf16", "decoding")
 
 
 def test_long_decoding_in_32_bit(cuda, package):
@@ -152,7 +142,7 @@ def test_long_decoding_in_32_bit(cuda, package):
     model, oracle = build(package, c, "f32", seed=7)
     ids = cases.tokens(c, 700, 8)
     session = model.new_session(700, graph=True)
-    check(run_portions(session, ids, [60, 1]), oracle.forward(ids), "f32")
+    check(cases.run_portions(session, ids, [60, 1]), oracle.forward(ids), "f32")
 
 
 @pytest.mark.parametrize("kind", KINDS)
@@ -161,20 +151,20 @@ def test_reset_and_neighbours_leave_no_trace(cuda, package, kind):
     model, oracle = build(package, c, kind)
     first, second = cases.tokens(c, 140, 11), cases.tokens(c, 120, 12)
     fresh = model.new_session(160, graph=True)
-    alone = run_portions(fresh, second, [70, 1, 9])
+    alone = cases.run_portions(fresh, second, [70, 1, 9])
     check(alone, oracle.forward(second), kind)
     used = model.new_session(160, graph=True)
-    run_portions(used, first, [140])
+    cases.run_portions(used, first, [140])
     used.reset()
-    assert np.array_equal(run_portions(used, second, [70, 1, 9]), alone)
+    assert np.array_equal(cases.run_portions(used, second, [70, 1, 9]), alone)
     # Two requests taking turns.
     a, b = model.new_session(160, graph=True), model.new_session(160, graph=True)
     rows = []
     for at in range(0, 120, 40):
-        rows.append(run_portions(b, second[at:at + 40], [40]))
-        run_portions(a, first[at:at + 40], [33, 7])
+        rows.append(cases.run_portions(b, second[at:at + 40], [40]))
+        cases.run_portions(a, first[at:at + 40], [33, 7])
     other = model.new_session(160)
-    assert np.array_equal(np.concatenate(rows), run_portions(other, second, [40]))
+    assert np.array_equal(np.concatenate(rows), cases.run_portions(other, second, [40]))
     # A prefill replaces what was there.
     used.prefill(first)
     used.prefill(second)
@@ -240,22 +230,13 @@ def test_truncation_reaches_back_over_the_last_step_only(cuda, package):
 
 
 # ---- generation ----
-def greedy(oracle, prompt, count):
-    logits = oracle.forward(prompt)[-1]
-    out = []
-    for _ in range(count):
-        out.append(int(np.argmax(logits)))
-        logits = oracle.forward([out[-1]])[0]
-    return out
-
-
 @pytest.mark.parametrize("name", ["mixed", "loop_last"])
 def test_greedy_generation_through_the_model_surface(cuda, package, name):
     c = dict(cases.CASES[name])
     weights = cases.random_weights(package, c)
     bridge = package.model_bridge.Model(c, weights, "zofesun_f32")
     prompt = cases.tokens(c, 50, 15)
-    want = greedy(hybrid.HybridOracle(c, weights), prompt, 40)
+    want = cases.greedy(hybrid.HybridOracle(c, weights), prompt, 40)
     session, got = bridge.new_session(128), []
     session.generate(prompt, got.append, max_length=90)
     assert got == want
@@ -342,6 +323,6 @@ def test_the_uniform_decoder_takes_portions_too(cuda, package):
     want = whole.read_logits_f32(1)
     for sizes in ([120], [50, 2, 1, 33, 34], [16]):
         session = model.new_session(128, graph=True)
-        got = run_portions(session, ids, sizes)
+        got = cases.run_portions(session, ids, sizes)
         assert got.shape == (120, 512)
         assert cases.logit_error(got[-1:], want).max() < 0.02
