@@ -29,8 +29,9 @@ Prints ONE JSON line:
                lengths in [256, 8192] split evenly over the GPUs, k = 4, p = 0.3, three sessions stacked per
                forward (ei_batch_verify)
 `--impl reference` times the CPU implementation alone (rank 0 only), whole 36-layer-deep steps.
-`--design zofesun` runs another workload instead: prefill and decode throughput of the layered Zofesun design at three
-sizes with real models' layers (random weights), each beside the uniform BF16 decoder of the same width and depth.
+`--design zofesun` and `--design gikepel` run another workload instead: prefill and decode throughput of that layered
+design at three sizes with real models' layers (random weights), each beside the uniform BF16 decoder of the same width,
+depth and feed-forward width.
 """
 from __future__ import annotations
 
@@ -570,16 +571,36 @@ def design_costs(shape) -> dict:
     if hasattr(shape, "layers"):
         for i in shape.layer_runs():
             layer = shape.layers[i]
+            gated = 3
             if layer.rnn_width is not None:
                 params += 4 * H * layer.rnn_width
                 cache += 2 * 4 * layer.rnn_width
+            elif layer.latent is not None:
+                a, gated = layer.latent, 2
+                expand = a.heads * (a.dim + a.vdim) * a.kv_rank
+                params += H * (a.heads * (a.dim + a.rot_dim + 2 * a.vdim) + a.kv_rank + a.rot_dim) + expand
+                flops += a.heads * (a.dim + a.rot_dim + a.vdim) * T * T
+                cache += 2 * (a.kv_rank + a.rot_dim) * T
+            elif layer.state_space is not None:
+                m, gated = layer.state_space, 2
+                inner, pairs = m.heads * m.vdim, m.groups * m.state
+                params += H * (3 * inner + 2 * pairs + m.heads)
+                flops += m.heads * T * (4 * m.state * m.vdim + 128 * (m.state + m.vdim))
+                cache += 2 * 4 * m.heads * m.state * m.vdim
+            elif layer.delta is not None:
+                m, gated = layer.delta, 2
+                keys, values = m.kv_heads * m.dim, m.heads * m.vdim
+                params += H * (2 * keys + 2 * values + m.decay_rank + m.gate_rank + m.heads)
+                params += m.heads * m.dim * m.decay_rank + values * m.gate_rank
+                flops += m.heads * T * (6 * m.dim * m.vdim + 64 * (2 * m.dim + 2 * m.vdim))  # chunks of 64
+                cache += 2 * 4 * m.heads * m.dim * m.vdim
             else:
                 a, l = layer.attention, layer.linear
                 params += H * (a.heads * (a.dim + a.vdim) + a.kv_heads * (a.dim + a.vdim) + l.heads * (2 * l.dim + 3 * l.vdim))
                 flops += a.heads * (a.dim + a.vdim) * T * T                       # causal: half of 2 T^2 per dimension
                 flops += l.heads * T * (4 * l.dim * l.vdim + 128 * (l.dim + l.vdim))
                 cache += 2 * a.kv_heads * (a.dim + a.vdim) * T + 2 * 4 * l.heads * l.dim * l.vdim
-            params += 3 * H * (layer.ff or 0)
+            params += gated * H * (layer.ff or 0)
     else:
         qkv = (shape.n_heads + 2 * shape.n_kv_heads) * shape.head_dim
         params = shape.n_layers * H * (qkv + shape.n_heads * shape.head_dim + 3 * shape.intermediate_size)
@@ -599,19 +620,20 @@ def run_design(args):
     syn = package.synthetic
     peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
     hbm, tensor = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops_sustained", 1400.0))
-    line = {"design": "zofesun", "prompt": DESIGN_PROMPT, "data": "synthetic", "dtype": "bf16 weights and activations, "
+    line = {"design": args.design, "prompt": DESIGN_PROMPT, "data": "synthetic", "dtype": "bf16 weights and activations, "
             "fp32 residual, norms, scores, softmax weights and recurrent state", "peaks": {"hbm_gbs": hbm, "tflops": tensor},
             "sizes": {}}
     sampler = ClockSampler(0)
     sampler.start()
     for name in (args.design_sizes or ",".join(DESIGN_SIZES)).split(","):
         width, layers, heads, kv_heads, lin_heads, ff = DESIGN_SIZES[name]
-        shapes = {"zofesun": syn.layered_decoder(width, layers, heads, kv_heads, lin_heads, ff),
+        shapes = {args.design: syn.layered_decoder(width, layers, heads, kv_heads, lin_heads, ff) if args.design == "zofesun" else
+                  syn.parallel_block_decoder(width, layers, heads, lin_heads, ff),
                   "uniform": package.Shape(vocab_size=151936, n_layers=layers, n_heads=heads, n_kv_heads=kv_heads,
                                            hidden_size=width, intermediate_size=ff, max_position_embeddings=DESIGN_CAPACITY)}
         line["sizes"][name] = {"layers": layers, "width": width, "ff": ff}
         for family, shape in shapes.items():
-            make = syn.make_device_layered_model if family == "zofesun" else syn.make_device_model
+            make = syn.make_device_layered_model if family == args.design else syn.make_device_model
             model = package.Model(shape, make(shape, seed=0))
             torch.cuda.empty_cache()
             session = model.new_session(DESIGN_CAPACITY, graph=True)
@@ -928,10 +950,10 @@ def main():
                         help="run only the 64-session leg and bracket one forward of all sessions the same way")
     parser.add_argument("--profile-prompt", action="store_true",
                         help="bracket one prefill of the prompt the same way and stop after it")
-    parser.add_argument("--design", choices=["zofesun"],
+    parser.add_argument("--design", choices=["zofesun", "gikepel"],
                         help="time this layered design beside the uniform decoder instead of the headline workload")
     parser.add_argument("--design-sizes", default="", help="sizes of --design, with commas between them")
-    parser.add_argument("--profile-design", choices=["zofesun", "uniform"],
+    parser.add_argument("--profile-design", choices=["zofesun", "gikepel", "uniform"],
                         help="with --design: bracket one prefill and one decode step of this family and stop")
     args = parser.parse_args()
     if args.steps is None:

@@ -15,7 +15,8 @@ from typing import Dict, List, Tuple
 
 import numpy as np
 
-from .runtime import (DENSE, QWEIGHT, SCALES, ZEROS, Attention, Layer, LayeredShape, LinearAttention, Shape)
+from .runtime import (BLOCK_PARALLEL, DENSE, MLP_RELU_SQUARED, QWEIGHT, SCALES, ZEROS, Attention, ChannelDelta,
+                      LatentAttention, Layer, LayeredShape, LinearAttention, PairEmbedding, Shape, StateSpace, Yarn)
 
 Tensors = Dict[str, List[Tuple[int, np.ndarray]]]
 
@@ -170,8 +171,8 @@ def make_device_model(shape: Shape, seed: int = 0) -> Dict[str, List[Tuple[int, 
 
 
 def make_device_layered_model(shape: LayeredShape, seed: int = 0) -> Dict[str, List[Tuple[int, object]]]:
-    """Random weights of a layered decoder in device memory: linears N(0, 1 / sqrt(inputs)), norm weights 1, alphas 0.5,
-    biases and sinks 0."""
+    """Random weights of a layered decoder in device memory: linears N(0, 1 / sqrt(inputs)), norm weights and scales 1,
+    alphas 0.5, biases, sinks and logarithms of decay rates 0, step biases -2."""
     import torch
 
     from .checkpoint import layered_tensor_shapes
@@ -181,10 +182,12 @@ def make_device_layered_model(shape: LayeredShape, seed: int = 0) -> Dict[str, L
     for name, dims in layered_tensor_shapes(shape).items():
         t = torch.empty(dims, dtype=torch.bfloat16, device="cuda")
         if len(dims) == 2:
-            t.normal_(0.0, 1.0 if name == "embed" else dims[1] ** -0.5, generator=gen)
+            t.normal_(0.0, 1.0 if name in ("embed", "bigram") else dims[1] ** -0.5, generator=gen)
         elif name.endswith(".alpha"):
             t.fill_(0.5)
-        elif name.endswith((".b", ".sink")):
+        elif name.endswith(".dt_bias"):
+            t.fill_(-2.0)
+        elif name.endswith((".b", ".sink", ".A_log")):
             t.zero_()
         else:
             t.fill_(1.0)
@@ -202,6 +205,18 @@ def layered_decoder(width: int, n_layers: int, heads: int, kv_heads: int, lin_he
     layers = [Layer(attention=attention, linear=linear, ff=ff, limit=7.0) if i % 2 == 0 else
               Layer(rnn_width=width, ff=ff, limit=7.0) for i in range(n_layers)]
     return LayeredShape(vocab_size=vocab, hidden_size=width, layers=layers, **kw)
+
+
+def parallel_block_decoder(width: int, n_layers: int, heads: int, lin_heads: int, ff: int, vocab: int = 151936, **kw) -> LayeredShape:
+    """A Gikepel decoder with a real model's sizes: delta rule, latent attention and state space take turns."""
+    delta = ChannelDelta(heads=lin_heads, kv_heads=lin_heads, dim=128, vdim=128, taps=4, decay_rank=128, gate_rank=128)
+    latent = LatentAttention(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, rot_dims=64, rot_base=1e4,
+                             scale=192 ** -0.5, yarn=Yarn(4.0, 4096, 32.0, 1.0))
+    space = StateSpace(heads=2 * width // 64, groups=8, state=128, vdim=64, taps=4, norm_groups=8)
+    turns = [dict(delta=delta), dict(latent=latent), dict(state_space=space)]
+    layers = [Layer(ff=ff, mlp=MLP_RELU_SQUARED, **turns[i % 3]) for i in range(n_layers)]
+    return LayeredShape(vocab_size=vocab, hidden_size=width, layers=layers, block=BLOCK_PARALLEL, tied_embeddings=True,
+                        pairs=PairEmbedding(200003, 31337, 7919), logit_softcap=30.0, **kw)
 
 
 def make_prompt(seed: int, length: int, vocab: int) -> np.ndarray:

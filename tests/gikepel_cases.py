@@ -62,7 +62,8 @@ CASES = {
     "inputs_in_slices": config(60, 72, [delta(33, 3, 16, 128, 2, ff=4200), mamba(3, 1, 16, 16, 2, 1, ff=4160)]),
     "stream_in_slices": config(60, 4200, [delta(2, 1, 16, 16, 2, ff=70), mamba(2, 1, 16, 16, 2, 1), latent(2, 16, 8, 16, 24)],
                                cap=90.0),
-    "mixed": config(203, 104, [delta(4, 2, 40, 24, 3, ff=72), latent(6, 24, 16, 40, 56, ff=60), latent(3, 32, 20, 16, 88),
+    "mixed": config(203, 104, [delta(4, 2, 40, 24, 3, ff=72), latent(6, 24, 24, 40, 56, scaling=(40.0, 64, 32.0, 1.0), ff=60, scale=0.1),
+                               latent(3, 16, 20, 16, 88, base=300.0),
                                mamba(6, 2, 24, 32, 4, 3, ff=44), delta(3, 3, 32, 48, 4)], buckets=211, muls=(91, 17)),
 }
 
@@ -86,9 +87,9 @@ def random_weights(package, c, seed=0, sharp=1.0, ranks=(13, 21)):
         elif part == "mix.dt_bias":
             value = rng.uniform(-4.0, 0.5, dims)
         elif part == "mix.D":
-            value = rng.uniform(0.4, 1.0, dims)
+            value = rng.uniform(0.8, 1.6, dims)
         elif part == "mix.conv.b":
-            value = 0.2 * rng.standard_normal(dims)
+            value = 0.4 * rng.standard_normal(dims)
         elif part.endswith("conv"):
             value = rng.standard_normal(dims) * 1.2 / dims[-1] ** 0.5
         elif name in ("embed", "bigram"):
