@@ -22,7 +22,6 @@ namespace {
 
 constexpr int kChunk = kDeltaChunk;
 constexpr int kBlock = 16;
-constexpr int kThreads = 256;
 constexpr int kPitchA = kChunk;       // floats per row of A transposed, read four at a time
 constexpr int kPitchB = kChunk + 1;   // of B, written down its columns
 
@@ -43,8 +42,13 @@ __host__ __device__ inline ChunkLayout chunk_layout(int dim, int vdim) {
   return l;
 }
 
+// Floats per staged row: sixteen more than a multiple of 32 keeps four-value accesses of two rows apart in the banks.
+__host__ __device__ inline int row_pitch(int dim) {
+  if (dim > 192) return dim < 256 ? dim + 4 : dim;  // what shared memory has room for
+  return dim % 32 == 16 ? dim : dim + 16;
+}
 size_t prepare_shared(int dim) {
-  return (size_t(3) * kChunk * (dim + 1) + size_t(kChunk) * (kPitchA + kPitchB) + kChunk) * sizeof(float);
+  return (size_t(3) * kChunk * row_pitch(dim) + size_t(kChunk) * (kPitchA + kPitchB) + kChunk) * sizeof(float);
 }
 
 // Writes the A fragment of a 16 x 16 tile for this lane: values (g, 2c), (g, 2c+1), (g+8, ..), (g, 2c+8), .. in `x`.
@@ -57,17 +61,41 @@ __device__ __forceinline__ void store_fragment(uint4* to, const float (&x)[8]) {
   to[0] = leading;
   to[32] = rest;
 }
+// The same from four consecutive values of row g and of row g + 8: columns 4 c .. 4 c + 3 of the tile stand where the
+// fragment has 2 c, 2 c + 1, 2 c + 8, 2 c + 9. Both operands of a product use this order, so the sum is the same.
+__device__ __forceinline__ void store_fragment(uint4* to, float4 lo, float4 hi) {
+  const float x[8] = {lo.x, lo.y, hi.x, hi.y, lo.z, lo.w, hi.z, hi.w};
+  store_fragment(to, x);
+}
+__device__ __forceinline__ float4 quad_at(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 times(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+__device__ __forceinline__ float4 exp_of(float4 a) { return make_float4(__expf(a.x), __expf(a.y), __expf(a.z), __expf(a.w)); }
+__device__ __forceinline__ float4 exp_between(float4 a, float4 b) { return exp_of(make_float4(a.x - b.x, a.y - b.y, a.z - b.z, a.w - b.w)); }
+__device__ __forceinline__ float dot(float4 a, float4 b, float sum) {
+  return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, sum))));
+}
+// A operand registers (leading, rest) of rows g and g + 8 in that order, and B operand registers of one row.
+__device__ __forceinline__ void split_rows(float4 lo, float4 hi, uint32_t (&leading)[4], uint32_t (&rest)[4]) {
+  split_pair(lo.x, lo.y, leading[0], rest[0]);
+  split_pair(hi.x, hi.y, leading[1], rest[1]);
+  split_pair(lo.z, lo.w, leading[2], rest[2]);
+  split_pair(hi.z, hi.w, leading[3], rest[3]);
+}
 
-__global__ void __launch_bounds__(kThreads) delta_chunk_kernel(const DeltaPromptParams p) {
+// Sixteen warps. Warp w: part w & 3 of the key channels, and, of A and B, the diagonal block w >> 2 and one of four groups
+// of tiles below it.
+constexpr int kPrepareThreads = 512;
+constexpr int kParts = 4;
+__global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const DeltaPromptParams p) {
   extern __shared__ __align__(16) float chunk_smem[];
   const OuterStateParams& o = p.outer;
-  const int dim = o.dim_pad, pitch = dim + 1;
+  const int dim = o.dim_pad, pitch = row_pitch(dim), steps = dim / 16;
   float* at = chunk_smem;                          // diag(b) A transposed: at[j][t], j < t
-  float* bm = at + kChunk * kPitchA;               // B: bm[t][j], j <= t
-  float* beta = bm + kChunk * kPitchB;             // [kChunk]
-  float* gs = beta + kChunk;                       // [kChunk][pitch]: cumulative logarithms of the decays
+  float* gs = at + kChunk * kPitchA;               // [kChunk][pitch]: cumulative logarithms of the decays
   float* ks = gs + kChunk * pitch;                 // [kChunk][pitch]: unit k, then columns of W
   float* qs = ks + kChunk * pitch;                 // [kChunk][pitch]: scaled unit q, then columns of V'
+  float* bm = qs + kChunk * pitch;                 // B: bm[t][j], j <= t
+  float* beta = bm + kChunk * kPitchB;             // [kChunk]
   grid_dependency_wait();
   grid_launch_dependents();
   const int context = o.control->context;
@@ -75,6 +103,7 @@ __global__ void __launch_bounds__(kThreads) delta_chunk_kernel(const DeltaPrompt
   const int chunk = blockIdx.x, head = blockIdx.y, key_head = head / (o.heads / o.key_heads);
   const int first = chunk * kChunk, live = min(kChunk, o.rows - first);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
+  constexpr int kWarps = kPrepareThreads / 32;
   const ChunkLayout layout = chunk_layout(dim, o.vdim_pad);
   unsigned char* own = p.chunks + (size_t(chunk) * o.heads + head) * layout.total;
   const bf16* conv = p.conv + size_t(first) * p.channels;
@@ -85,119 +114,179 @@ __global__ void __launch_bounds__(kThreads) delta_chunk_kernel(const DeltaPrompt
     const int t = threadIdx.x;
     beta[t] = t < live ? sigmoid_value(__bfloat162float(static_cast<const bf16*>(o.fused)[size_t(first + t) * o.stride + o.step_at + head])) : 0.0f;
   }
-  for (int i = threadIdx.x; i < kChunk * (dim / 2); i += kThreads) {
-    const int t = i / (dim / 2), d = (i - t * (dim / 2)) * 2;
-    float2 q = make_float2(0.0f, 0.0f), k = q, l = q;
+  const int quads = dim / 4;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < kChunk * quads; i += kPrepareThreads) {
+    const int t = i / quads, d = (i - t * quads) * 4;
+    float4 q = make_float4(0.0f, 0.0f, 0.0f, 0.0f), k = q, l = q;
     if (t < live) {
       const float q_scale = inverse[size_t(t) * 2 * o.key_heads + key_head], k_scale = inverse[size_t(t) * 2 * o.key_heads + o.key_heads + key_head];
-      q = load_pair(conv + size_t(t) * p.channels + key_head * dim + d);
-      k = load_pair(conv + size_t(t) * p.channels + (o.key_heads + key_head) * dim + d);
-      q = make_float2(q.x * q_scale, q.y * q_scale);
-      k = make_float2(k.x * k_scale, k.y * k_scale);
-      const float2 a = load_pair(static_cast<const bf16*>(o.decay) + size_t(first + t) * o.decay_stride + head * dim + d);
-      const float2 bias = load_pair(o.bias + head * dim + d);
-      l = make_float2(-rate * softplus_value(a.x + bias.x), -rate * softplus_value(a.y + bias.y));
+      q = load_quad(conv + size_t(t) * p.channels + key_head * dim + d);
+      k = load_quad(conv + size_t(t) * p.channels + (o.key_heads + key_head) * dim + d);
+      l = add(load_quad(static_cast<const bf16*>(o.decay) + size_t(first + t) * o.decay_stride + head * dim + d),
+              quad_at(o.bias + head * dim + d));
+      q = make_float4(q.x * q_scale, q.y * q_scale, q.z * q_scale, q.w * q_scale);
+      k = make_float4(k.x * k_scale, k.y * k_scale, k.z * k_scale, k.w * k_scale);
+      l = make_float4(-rate * quick_softplus(l.x), -rate * quick_softplus(l.y), -rate * quick_softplus(l.z), -rate * quick_softplus(l.w));
     }
-    gs[t * pitch + d] = l.x;
-    gs[t * pitch + d + 1] = l.y;
-    ks[t * pitch + d] = k.x;
-    ks[t * pitch + d + 1] = k.y;
-    qs[t * pitch + d] = q.x;
-    qs[t * pitch + d + 1] = q.y;
+    *reinterpret_cast<float4*>(gs + t * pitch + d) = l;
+    *reinterpret_cast<float4*>(ks + t * pitch + d) = k;
+    *reinterpret_cast<float4*>(qs + t * pitch + d) = q;
   }
   __syncthreads();
   // Cumulative sums: inside blocks of 16 rows, then the blocks' totals.
-  for (int i = threadIdx.x; i < dim * (kChunk / kBlock); i += kThreads) {
+  for (int i = threadIdx.x; i < dim * (kChunk / kBlock); i += kPrepareThreads) {
     float* column = gs + (i / dim) * kBlock * pitch + i % dim;
-    float sum = 0.0f;
+    float sum = 0.0f, x[kBlock];
 #pragma unroll
-    for (int t = 0; t < kBlock; ++t) column[t * pitch] = sum += column[t * pitch];
+    for (int t = 0; t < kBlock; ++t) x[t] = column[t * pitch];
+#pragma unroll
+    for (int t = 0; t < kBlock; ++t) column[t * pitch] = sum += x[t];
   }
   __syncthreads();
-  for (int d = threadIdx.x; d < dim; d += kThreads) {
-    for (int b = 1; b < kChunk / kBlock; ++b) {
-      const float before = gs[(b * kBlock - 1) * pitch + d];
+  for (int i = threadIdx.x; i < dim; i += kPrepareThreads) {
+    float before[kChunk / kBlock];
+    before[0] = 0.0f;
 #pragma unroll
-      for (int t = 0; t < kBlock; ++t) gs[(b * kBlock + t) * pitch + d] += before;
+    for (int b = 1; b < kChunk / kBlock; ++b) before[b] = before[b - 1] + gs[(b * kBlock - 1) * pitch + i];
+#pragma unroll
+    for (int b = 1; b < kChunk / kBlock; ++b) {
+      float x[kBlock];
+#pragma unroll
+      for (int t = 0; t < kBlock; ++t) x[t] = gs[(b * kBlock + t) * pitch + i];
+#pragma unroll
+      for (int t = 0; t < kBlock; ++t) gs[(b * kBlock + t) * pitch + i] = x[t] + before[b];
     }
   }
   __syncthreads();
 
-  // A and B outside the diagonal blocks: tasks of 16 rows x 8 columns, through the end of the block ahead of the rows.
-  for (int task = warp; task < 12; task += kThreads / 32) {
-    const int block = task < 2 ? 1 : task < 6 ? 2 : 3, column = (task - (block == 1 ? 0 : block == 2 ? 2 : 6)) * 8;
-    const int t0 = block * kBlock;
-    const float* turn = gs + (t0 - 1) * pitch;
-    float ka[4] = {0.0f, 0.0f, 0.0f, 0.0f}, qa[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-    for (int kk = 0; kk < dim / 16; ++kk) {
-      uint32_t kh[4], kl[4], qh[4], ql[4], bh[2], bl[2];
+  // A and B. Every warp adds up its part of the key channels for one diagonal block, directly, and for a group of tiles of
+  // 16 rows x 8 columns below the diagonal, through the end of the block ahead of the rows; the parts are then added in
+  // order.
+  {
+    const int part = warp & (kParts - 1), group = warp >> 2;
+    const int kk_begin = steps * part / kParts, kk_end = steps * (part + 1) / kParts;
+    // Diagonal block `group`: rows g and g + 8 of it, columns 0..15; row g needs the first eight only.
+    float low_k[8], low_q[8], high_k[16], high_q[16];
 #pragma unroll
-      for (int part = 0; part < 4; ++part) {
-        const int t = t0 + g + (part & 1) * 8, d = kk * 16 + 2 * c + (part >> 1) * 8;
-        const float e0 = __expf(gs[t * pitch + d] - turn[d]), e1 = __expf(gs[t * pitch + d + 1] - turn[d + 1]);
-        split_pair(ks[t * pitch + d] * e0, ks[t * pitch + d + 1] * e1, kh[part], kl[part]);
-        split_pair(qs[t * pitch + d] * e0, qs[t * pitch + d + 1] * e1, qh[part], ql[part]);
+    for (int j = 0; j < 8; ++j) low_k[j] = low_q[j] = 0.0f;
+#pragma unroll
+    for (int j = 0; j < 16; ++j) high_k[j] = high_q[j] = 0.0f;
+    // Below the diagonal: groups 0 and 1 hold the row block 3 (columns 0..23 and 24..47), group 2 block 2, group 3 block 1.
+    const int block = group < 2 ? 3 : group == 2 ? 2 : 1, first_column = group == 1 ? 24 : 0;
+    const int tiles = group < 2 ? 3 : group == 2 ? 4 : 2;
+    float ka[4][4], qa[4][4];
+#pragma unroll
+    for (int n = 0; n < 4; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ka[n][e] = qa[n][e] = 0.0f;
+    for (int kk = kk_begin; kk < kk_end; ++kk) {
+      const int d = kk * 16 + 4 * c;
+      {
+        const int t = group * kBlock + g;
+        const float4 gl = quad_at(gs + t * pitch + d), gh = quad_at(gs + (t + 8) * pitch + d);
+        const float4 kl = quad_at(ks + t * pitch + d), kh = quad_at(ks + (t + 8) * pitch + d);
+        const float4 ql = quad_at(qs + t * pitch + d), qh = quad_at(qs + (t + 8) * pitch + d);
+#pragma unroll
+        for (int j = 0; j < 16; ++j) {
+          const float4 gj = quad_at(gs + (group * kBlock + j) * pitch + d), kj = quad_at(ks + (group * kBlock + j) * pitch + d);
+          // A row ahead of its column is not used; its exponent is held at zero so that it stays finite.
+          if (j < 8) {
+            const float4 x = times(kj, exp_of(make_float4(fminf(gl.x - gj.x, 0.0f), fminf(gl.y - gj.y, 0.0f), fminf(gl.z - gj.z, 0.0f),
+                                                          fminf(gl.w - gj.w, 0.0f))));
+            low_k[j & 7] = dot(kl, x, low_k[j & 7]);
+            low_q[j & 7] = dot(ql, x, low_q[j & 7]);
+          }
+          const float4 y = times(kj, exp_of(make_float4(fminf(gh.x - gj.x, 0.0f), fminf(gh.y - gj.y, 0.0f), fminf(gh.z - gj.z, 0.0f),
+                                                        fminf(gh.w - gj.w, 0.0f))));
+          high_k[j] = dot(kh, y, high_k[j]);
+          high_q[j] = dot(qh, y, high_q[j]);
+        }
+      }
+      const int t0 = block * kBlock;
+      const float4 turn = quad_at(gs + (t0 - 1) * pitch + d);
+      uint32_t kh[4], kl[4], qh[4], ql[4];
+      {
+        const float4 e_lo = exp_between(quad_at(gs + (t0 + g) * pitch + d), turn), e_hi = exp_between(quad_at(gs + (t0 + g + 8) * pitch + d), turn);
+        split_rows(times(quad_at(ks + (t0 + g) * pitch + d), e_lo), times(quad_at(ks + (t0 + g + 8) * pitch + d), e_hi), kh, kl);
+        split_rows(times(quad_at(qs + (t0 + g) * pitch + d), e_lo), times(quad_at(qs + (t0 + g + 8) * pitch + d), e_hi), qh, ql);
       }
 #pragma unroll
-      for (int part = 0; part < 2; ++part) {
-        const int j = column + g, d = kk * 16 + 2 * c + part * 8;
-        split_pair(ks[j * pitch + d] * __expf(turn[d] - gs[j * pitch + d]), ks[j * pitch + d + 1] * __expf(turn[d + 1] - gs[j * pitch + d + 1]),
-                   bh[part], bl[part]);
+      for (int n = 0; n < 4; ++n) {
+        if (n < tiles) {
+          const int j = first_column + n * 8 + g;
+          const float4 x = times(quad_at(ks + j * pitch + d), exp_between(turn, quad_at(gs + j * pitch + d)));
+          uint32_t bh[2], bl[2];
+          split_pair(x.x, x.y, bh[0], bl[0]);
+          split_pair(x.z, x.w, bh[1], bl[1]);
+          mma_bf16_16816(ka[n], kh[0], kh[1], kh[2], kh[3], bh[0], bh[1]);
+          mma_bf16_16816(qa[n], qh[0], qh[1], qh[2], qh[3], bh[0], bh[1]);
+          mma_bf16_16816(ka[n], kh[0], kh[1], kh[2], kh[3], bl[0], bl[1]);
+          mma_bf16_16816(qa[n], qh[0], qh[1], qh[2], qh[3], bl[0], bl[1]);
+          mma_bf16_16816(ka[n], kl[0], kl[1], kl[2], kl[3], bh[0], bh[1]);
+          mma_bf16_16816(qa[n], ql[0], ql[1], ql[2], ql[3], bh[0], bh[1]);
+        }
       }
-      mma_bf16_16816(ka, kh[0], kh[1], kh[2], kh[3], bh[0], bh[1]);
-      mma_bf16_16816(qa, qh[0], qh[1], qh[2], qh[3], bh[0], bh[1]);
-      mma_bf16_16816(ka, kh[0], kh[1], kh[2], kh[3], bl[0], bl[1]);
-      mma_bf16_16816(qa, qh[0], qh[1], qh[2], qh[3], bl[0], bl[1]);
-      mma_bf16_16816(ka, kl[0], kl[1], kl[2], kl[3], bh[0], bh[1]);
-      mma_bf16_16816(qa, ql[0], ql[1], ql[2], ql[3], bh[0], bh[1]);
+    }
+    auto across = [](float x) {
+      x += __shfl_xor_sync(0xffffffffu, x, 1);
+      return x + __shfl_xor_sync(0xffffffffu, x, 2);
+    };
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      low_k[j] = across(low_k[j]);
+      low_q[j] = across(low_q[j]);
     }
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int t = t0 + g + (i >> 1) * 8, j = column + 2 * c + (i & 1);
-      at[j * kPitchA + t] = ka[i] * beta[t];
-      bm[t * kPitchB + j] = qa[i];
+    for (int j = 0; j < 16; ++j) {
+      high_k[j] = across(high_k[j]);
+      high_q[j] = across(high_q[j]);
+    }
+    for (int turn_of = 0; turn_of < kParts; ++turn_of) {
+      if (part == turn_of) {
+        auto put = [&](int t, int j, float k_value, float q_value) {
+          float &a = at[j * kPitchA + t], &b = bm[t * kPitchB + j];
+          a = part ? a + k_value * beta[t] : k_value * beta[t];
+          b = part ? b + q_value : q_value;
+        };
+#pragma unroll
+        for (int j = 0; j < 16; ++j) {
+          if ((j & 3) != c) continue;  // the four lanes of a row hold the same sums and share the columns
+          const int t = group * kBlock + g, column = group * kBlock + j;
+          const bool low = j < 8 && j <= g, high = j <= g + 8;
+          put(t, column, low && j < g ? low_k[j & 7] : 0.0f, low ? low_q[j & 7] : 0.0f);
+          put(t + 8, column, high && j < g + 8 ? high_k[j] : 0.0f, high ? high_q[j] : 0.0f);
+        }
+#pragma unroll
+        for (int n = 0; n < 4; ++n)
+          if (n < tiles)
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              put(block * kBlock + g + (e >> 1) * 8, first_column + n * 8 + 2 * c + (e & 1), ka[n][e], qa[n][e]);
+      }
+      __syncthreads();
     }
   }
-  // Inside the diagonal blocks: a thread per (row, column).
-  for (int i = threadIdx.x; i < kChunk * kBlock; i += kThreads) {
-    const int t = i & (kChunk - 1), j = (t & ~(kBlock - 1)) + (i >> 6);  // a warp's threads: rows one after the other
-    float kk = 0.0f, qk = 0.0f;
-    if (j <= t) {
-      const float *gt = gs + t * pitch, *gj = gs + j * pitch, *kt = ks + t * pitch, *kj = ks + j * pitch, *qt = qs + t * pitch;
-#pragma unroll 4
-      for (int d = 0; d < dim; ++d) {
-        const float x = kj[d] * __expf(gt[d] - gj[d]);
-        kk = fmaf(kt[d], x, kk);
-        qk = fmaf(qt[d], x, qk);
-      }
-    }
-    at[j * kPitchA + t] = j < t ? kk * beta[t] : 0.0f;
-    bm[t * kPitchB + j] = j <= t ? qk : 0.0f;
-  }
-  __syncthreads();
 
   // Operands that need no solving: q e^G, k e^(G_end - G) transposed, B, and the chunk's decay.
   const float* last = gs + (kChunk - 1) * pitch;
   uint4* q_out = reinterpret_cast<uint4*>(own + layout.q);
   uint4* k_out = reinterpret_cast<uint4*>(own + layout.k);
   uint4* b_out = reinterpret_cast<uint4*>(own + layout.b);
-  const int steps = dim / 16;
-  for (int tile = warp; tile < 4 * steps; tile += kThreads / 32) {
+  for (int tile = warp; tile < 4 * steps; tile += kWarps) {
     const int mt = tile / steps, kk = tile - mt * steps;
-    float x[8], y[8];
+    const int row = (mt * 16 + g) * pitch + kk * 16 + 4 * c;
+    store_fragment(q_out + size_t(mt * steps + kk) * 64 + lane, times(quad_at(qs + row), exp_of(quad_at(gs + row))),
+                   times(quad_at(qs + row + 8 * pitch), exp_of(quad_at(gs + row + 8 * pitch))));
+    float y[8];  // tile (kk, mt) of the transpose: rows are key channels, columns tokens
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
-      const int row = g + ((e >> 1) & 1) * 8, col = 2 * c + (e & 1) + (e >> 2) * 8;
-      const int t = mt * 16 + row, d = kk * 16 + col;
-      x[e] = qs[t * pitch + d] * __expf(gs[t * pitch + d]);
-      // Tile (kk, mt) of the transpose: rows are key channels, columns tokens.
-      const int token = mt * 16 + col, channel = kk * 16 + row;
+      const int token = mt * 16 + 2 * c + (e & 1) + (e >> 2) * 8, channel = kk * 16 + g + ((e >> 1) & 1) * 8;
       y[e] = ks[token * pitch + channel] * __expf(last[channel] - gs[token * pitch + channel]);
     }
-    store_fragment(q_out + size_t(mt * steps + kk) * 64 + lane, x);
     store_fragment(k_out + size_t(kk * 4 + mt) * 64 + lane, y);
   }
-  for (int tile = warp; tile < 16; tile += kThreads / 32) {
+  for (int tile = warp; tile < 16; tile += kWarps) {
     const int mt = tile >> 2, kk = tile & 3;
     if (kk > mt) continue;
     float x[8];
@@ -206,7 +295,7 @@ __global__ void __launch_bounds__(kThreads) delta_chunk_kernel(const DeltaPrompt
       x[e] = bm[(mt * 16 + g + ((e >> 1) & 1) * 8) * kPitchB + kk * 16 + 2 * c + (e & 1) + (e >> 2) * 8];
     store_fragment(b_out + size_t(tile) * 64 + lane, x);
   }
-  for (int d = threadIdx.x; d < dim; d += kThreads) reinterpret_cast<float*>(own + layout.decay)[d] = __expf(last[d]);
+  for (int d = threadIdx.x; d < dim; d += kPrepareThreads) reinterpret_cast<float*>(own + layout.decay)[d] = __expf(last[d]);
   __syncthreads();
 
   // Solves (I + diag(b) A) X = right-hand side for one column in place, 16 rows at a time.
@@ -216,13 +305,13 @@ __global__ void __launch_bounds__(kThreads) delta_chunk_kernel(const DeltaPrompt
       float x[kBlock];
 #pragma unroll
       for (int i = 0; i < kBlock; ++i) x[i] = column[(b * kBlock + i) * pitch];
-#pragma unroll 2
+#pragma unroll 4
       for (int j = 0; j < b * kBlock; ++j) {
         const float known = column[j * pitch];
         const float* a = at + j * kPitchA + b * kBlock;
 #pragma unroll
         for (int i = 0; i < kBlock; i += 4) {
-          const float4 v = *reinterpret_cast<const float4*>(a + i);
+          const float4 v = quad_at(a + i);
           x[i] = fmaf(-v.x, known, x[i]);
           x[i + 1] = fmaf(-v.y, known, x[i + 1]);
           x[i + 2] = fmaf(-v.z, known, x[i + 2]);
@@ -234,7 +323,7 @@ __global__ void __launch_bounds__(kThreads) delta_chunk_kernel(const DeltaPrompt
         const float* a = at + (b * kBlock + j) * kPitchA + b * kBlock;
 #pragma unroll
         for (int i = (j + 1) & ~3; i < kBlock; i += 4) {
-          const float4 v = *reinterpret_cast<const float4*>(a + i);  // zero up to the diagonal
+          const float4 v = quad_at(a + i);  // zero up to the diagonal
           x[i] = i > j ? fmaf(-v.x, x[j], x[i]) : x[i];
           x[i + 1] = i + 1 > j ? fmaf(-v.y, x[j], x[i + 1]) : x[i + 1];
           x[i + 2] = i + 2 > j ? fmaf(-v.z, x[j], x[i + 2]) : x[i + 2];
@@ -249,27 +338,29 @@ __global__ void __launch_bounds__(kThreads) delta_chunk_kernel(const DeltaPrompt
   float4* v_out = reinterpret_cast<float4*>(own + layout.v);
   const bf16* values = conv + 2 * o.key_heads * dim + head * o.vdim_pad;
   for (int v0 = 0; v0 < o.vdim_pad; v0 += dim) {
-    const int width = min(dim, o.vdim_pad - v0);
-    for (int i = threadIdx.x; i < kChunk * (width / 2); i += kThreads) {
-      const int t = i / (width / 2), d = (i - t * (width / 2)) * 2;
-      const float2 v = t < live ? load_pair(values + size_t(t) * p.channels + v0 + d) : make_float2(0.0f, 0.0f);
-      qs[t * pitch + d] = v.x * beta[t];
-      qs[t * pitch + d + 1] = v.y * beta[t];
+    const int width = min(dim, o.vdim_pad - v0), width_quads = width / 4;
+    for (int i = threadIdx.x; i < kChunk * width_quads; i += kPrepareThreads) {
+      const int t = i / width_quads, d = (i - t * width_quads) * 4;
+      const float4 v = t < live ? load_quad(values + size_t(t) * p.channels + v0 + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      const float b = beta[t];
+      *reinterpret_cast<float4*>(qs + t * pitch + d) = make_float4(v.x * b, v.y * b, v.z * b, v.w * b);
     }
-    __syncthreads();
-    const int unsolved = v0 == 0 ? dim : 0;  // columns of W still to come, ahead of the value columns
-    for (int column = threadIdx.x; column < unsolved + width; column += kThreads) {
-      if (column < unsolved) {
-#pragma unroll 4
-        for (int t = 0; t < kChunk; ++t) ks[t * pitch + column] *= beta[t] * __expf(gs[t * pitch + column]);
-        solve(ks + column);
-      } else {
-        solve(qs + column - unsolved);
+    if (v0 == 0) {
+      for (int i = threadIdx.x; i < kChunk * quads; i += kPrepareThreads) {
+        const int t = i / quads, d = (i - t * quads) * 4;
+        const float4 e = exp_of(quad_at(gs + t * pitch + d));
+        const float b = beta[t];
+        float4* k = reinterpret_cast<float4*>(ks + t * pitch + d);
+        *k = times(*k, make_float4(e.x * b, e.y * b, e.z * b, e.w * b));
       }
     }
     __syncthreads();
+    const int unsolved = v0 == 0 ? dim : 0;  // columns of W still to come, ahead of the value columns
+    for (int column = threadIdx.x; column < unsolved + width; column += kPrepareThreads)
+      solve(column < unsolved ? ks + column : qs + column - unsolved);
+    __syncthreads();
     // V' in the order of the accumulators: [row tile][column tile of 8][lane].
-    for (int tile = warp; tile < 4 * (width / 8); tile += kThreads / 32) {
+    for (int tile = warp; tile < 4 * (width / 8); tile += kWarps) {
       const int mt = tile / (width / 8), nt = tile - mt * (width / 8);
       const float* x = qs + (mt * 16 + g) * pitch + nt * 8 + 2 * c;
       v_out[(size_t(mt) * (o.vdim_pad / 8) + v0 / 8 + nt) * 32 + lane] = make_float4(x[0], x[1], x[8 * pitch], x[8 * pitch + 1]);
@@ -277,18 +368,17 @@ __global__ void __launch_bounds__(kThreads) delta_chunk_kernel(const DeltaPrompt
     __syncthreads();
   }
   uint4* w_out = reinterpret_cast<uint4*>(own + layout.w);
-  for (int tile = warp; tile < 4 * steps; tile += kThreads / 32) {
+  for (int tile = warp; tile < 4 * steps; tile += kWarps) {
     const int mt = tile / steps, kk = tile - mt * steps;
-    float x[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e)
-      x[e] = ks[(mt * 16 + g + ((e >> 1) & 1) * 8) * pitch + kk * 16 + 2 * c + (e & 1) + (e >> 2) * 8];
-    store_fragment(w_out + size_t(tile) * 64 + lane, x);
+    const float* x = ks + (mt * 16 + g) * pitch + kk * 16 + 4 * c;
+    store_fragment(w_out + size_t(tile) * 64 + lane, quad_at(x), quad_at(x + 8 * pitch));
   }
 }
 
 // Block (head, kColumns values), eight warps, the chunks one after the other. Warps 0-3 hold 16 rows each of U, warps 4-7
-// of the output; every warp holds kTiles tiles of 16 key channels of the state.
+// of the output; every warp holds kTiles tiles of 16 key channels of the state. Operands are requested a phase ahead of
+// their use.
+constexpr int kThreads = 256;
 template <int kColumns, int kTiles>
 __global__ void __launch_bounds__(kThreads) delta_scan_kernel(const DeltaPromptParams p) {
   constexpr int kN = kColumns / 8;              // accumulator tiles per row tile
@@ -341,14 +431,17 @@ __global__ void __launch_bounds__(kThreads) delta_scan_kernel(const DeltaPromptP
       }
     }
   }
-  auto publish = [&](const float (&x)[kN][4], int row, bf16* leading, bf16* rest) {
+  // Accumulator rows into the two terms of an operand; key channels of a tile in the order of store_fragment's quads.
+  const int token_rows[2] = {g, g + 8};
+  const int channel_rows[2] = {(g >> 2) * 2 + (g & 1) + ((g >> 1) & 1) * 8, ((g >> 2) + 2) * 2 + (g & 1) + ((g >> 1) & 1) * 8};
+  auto publish = [&](const float (&x)[kN][4], int row, const int (&places)[2], bf16* leading, bf16* rest) {
 #pragma unroll
     for (int n = 0; n < kN; ++n) {
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         uint32_t hi, lo;
         split_pair(x[n][2 * half], x[n][2 * half + 1], hi, lo);
-        const int at = (row + g + half * 8) * kPitch + n * 8 + 2 * c;
+        const int at = (row + places[half]) * kPitch + n * 8 + 2 * c;
         *reinterpret_cast<uint32_t*>(leading + at) = hi;
         *reinterpret_cast<uint32_t*>(rest + at) = lo;
       }
@@ -356,14 +449,14 @@ __global__ void __launch_bounds__(kThreads) delta_scan_kernel(const DeltaPromptP
   };
 #pragma unroll
   for (int m = 0; m < kTiles; ++m)
-    if (warp + 8 * m < steps) publish(s[m], (warp + 8 * m) * 16, state_leading, state_rest);
+    if (warp + 8 * m < steps) publish(s[m], (warp + 8 * m) * 16, channel_rows, state_leading, state_rest);
   __syncthreads();
 
-  // acc += (two-term A fragment) x (two-term rows of `leading` / `rest` from `row` on).
+  // acc += (two-term A fragment) x (two-term rows of `leading` / `rest` at `row` + this lane's row of the 16).
   auto multiply = [&](float (&acc)[kN][4], const uint4& ah, const uint4& al, const bf16* leading, const bf16* rest, int row) {
 #pragma unroll
     for (int n = 0; n < kN; n += 2) {
-      const int at = (row + (matrix & 1) * 8 + in_matrix) * kPitch + (n + (matrix >> 1)) * 8;
+      const int at = row * kPitch + (n + (matrix >> 1)) * 8;
       uint32_t b0, b1, b2, b3;
       ldmatrix_x4_trans(b0, b1, b2, b3, leading + at);
       mma_bf16_16816(acc[n], ah.x, ah.y, ah.z, ah.w, b0, b1);
@@ -375,67 +468,104 @@ __global__ void __launch_bounds__(kThreads) delta_scan_kernel(const DeltaPromptP
       mma_bf16_16816(acc[n + 1], ah.x, ah.y, ah.z, ah.w, b2, b3);
     }
   };
+  const int own_row = (matrix & 1) * 8 + in_matrix;
   constexpr int kAhead = 8;  // K steps of an operand requested at once
   const int row_tile = warp & 3;
-  for (int chunk = 0; chunk < chunks; ++chunk) {
-    const unsigned char* own = p.chunks + (size_t(chunk) * o.heads + head) * layout.total;
-    const uint4* operand = reinterpret_cast<const uint4*>(own + (warp < 4 ? layout.w : layout.q)) + size_t(row_tile) * steps * 64 + lane;
+  const unsigned char* own = p.chunks + size_t(head) * layout.total;
+  const size_t chunk_bytes = size_t(o.heads) * layout.total;
+  auto operand_of = [&](const unsigned char* at) {
+    return reinterpret_cast<const uint4*>(at + (warp < 4 ? layout.w : layout.q)) + size_t(row_tile) * steps * 64 + lane;
+  };
+  uint4 ah[kAhead], al[kAhead];
+  auto request = [&](const uint4* operand, int kk) {
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) {
+      if (kk + i < steps) {
+        ah[i] = operand[size_t(kk + i) * 64];
+        al[i] = operand[size_t(kk + i) * 64 + 32];
+      }
+    }
+  };
+  request(operand_of(own), 0);
+  for (int chunk = 0; chunk < chunks; ++chunk, own += chunk_bytes) {
+    // Requested for the second phase: the keys of this warp's first tile, the decay, B or V'.
+    const uint4* keys = reinterpret_cast<const uint4*>(own + layout.k) + lane;
+    const float* decay = reinterpret_cast<const float*>(own + layout.decay);
+    const uint4* inside = reinterpret_cast<const uint4*>(own + layout.b) + size_t(row_tile) * 4 * 64 + lane;
+    uint4 kh[4], kl[4], bh[4], bl[4];
+    float4 v[kN];
+    float decay_lo = 1.0f, decay_hi = 1.0f;
+    if (warp < steps) {
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) {
+        kh[kk] = keys[size_t(warp * 4 + kk) * 64];
+        kl[kk] = keys[size_t(warp * 4 + kk) * 64 + 32];
+      }
+      decay_lo = decay[warp * 16 + g];
+      decay_hi = decay[warp * 16 + g + 8];
+    }
+    if (warp < 4) {
+      const float4* from = reinterpret_cast<const float4*>(own + layout.v) + (size_t(row_tile) * (o.vdim_pad / 8) + first_value / 8) * 32 + lane;
+#pragma unroll
+      for (int n = 0; n < kN; ++n) v[n] = n * 8 < live_columns ? from[n * 32] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    } else {
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) {
+        if (kk <= row_tile) {
+          bh[kk] = inside[size_t(kk) * 64];
+          bl[kk] = inside[size_t(kk) * 64 + 32];
+        }
+      }
+    }
     float acc[kN][4];
 #pragma unroll
     for (int n = 0; n < kN; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.0f;
     for (int kk = 0; kk < steps; kk += kAhead) {
-      uint4 ah[kAhead], al[kAhead];
-#pragma unroll
-      for (int i = 0; i < kAhead; ++i) {
-        if (kk + i < steps) {
-          ah[i] = operand[size_t(kk + i) * 64];
-          al[i] = operand[size_t(kk + i) * 64 + 32];
-        }
-      }
+      if (kk) request(operand_of(own), kk);
 #pragma unroll
       for (int i = 0; i < kAhead; ++i)
-        if (kk + i < steps) multiply(acc, ah[i], al[i], state_leading, state_rest, (kk + i) * 16);
+        if (kk + i < steps) multiply(acc, ah[i], al[i], state_leading, state_rest, (kk + i) * 16 + own_row);
     }
+    if (chunk + 1 < chunks) request(operand_of(own + chunk_bytes), 0);
     if (warp < 4) {
-      const float4* v = reinterpret_cast<const float4*>(own + layout.v) + (size_t(row_tile) * (o.vdim_pad / 8) + first_value / 8) * 32 + lane;
 #pragma unroll
       for (int n = 0; n < kN; ++n) {
-        const float4 x = n * 8 < live_columns ? v[n * 32] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        acc[n][0] = x.x - acc[n][0];
-        acc[n][1] = x.y - acc[n][1];
-        acc[n][2] = x.z - acc[n][2];
-        acc[n][3] = x.w - acc[n][3];
+        acc[n][0] = v[n].x - acc[n][0];
+        acc[n][1] = v[n].y - acc[n][1];
+        acc[n][2] = v[n].z - acc[n][2];
+        acc[n][3] = v[n].w - acc[n][3];
       }
-      publish(acc, row_tile * 16, write_leading, write_rest);
+      publish(acc, row_tile * 16, token_rows, write_leading, write_rest);
     }
     __syncthreads();  // the writes are there, and every warp is done with the staged state
-    const uint4* keys = reinterpret_cast<const uint4*>(own + layout.k) + lane;
-    const float* decay = reinterpret_cast<const float*>(own + layout.decay);
 #pragma unroll
     for (int m = 0; m < kTiles; ++m) {
       const int tile = warp + 8 * m;
       if (tile >= steps) break;
-      uint4 ah[4], al[4];
+      if (m) {
 #pragma unroll
-      for (int kk = 0; kk < 4; ++kk) {
-        ah[kk] = keys[size_t(tile * 4 + kk) * 64];
-        al[kk] = keys[size_t(tile * 4 + kk) * 64 + 32];
+        for (int kk = 0; kk < 4; ++kk) {
+          kh[kk] = keys[size_t(tile * 4 + kk) * 64];
+          kl[kk] = keys[size_t(tile * 4 + kk) * 64 + 32];
+        }
+        decay_lo = decay[tile * 16 + g];
+        decay_hi = decay[tile * 16 + g + 8];
       }
-      const float lo = decay[tile * 16 + g], hi = decay[tile * 16 + g + 8];
 #pragma unroll
       for (int n = 0; n < kN; ++n) {
-        s[m][n][0] *= lo;
-        s[m][n][1] *= lo;
-        s[m][n][2] *= hi;
-        s[m][n][3] *= hi;
+        s[m][n][0] *= decay_lo;
+        s[m][n][1] *= decay_lo;
+        s[m][n][2] *= decay_hi;
+        s[m][n][3] *= decay_hi;
       }
 #pragma unroll
-      for (int kk = 0; kk < 4; ++kk) multiply(s[m], ah[kk], al[kk], write_leading, write_rest, kk * 16);
-      publish(s[m], tile * 16, state_leading, state_rest);
+      for (int kk = 0; kk < 4; ++kk) multiply(s[m], kh[kk], kl[kk], write_leading, write_rest, kk * 16 + own_row);
+      publish(s[m], tile * 16, channel_rows, state_leading, state_rest);
     }
     if (warp >= 4) {
-      const uint4* inside = reinterpret_cast<const uint4*>(own + layout.b) + size_t(row_tile) * 4 * 64 + lane;
-      for (int kk = 0; kk <= row_tile; ++kk) multiply(acc, inside[size_t(kk) * 64], inside[size_t(kk) * 64 + 32], write_leading, write_rest, kk * 16);
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk)
+        if (kk <= row_tile) multiply(acc, bh[kk], bl[kk], write_leading, write_rest, kk * 16 + own_row);
       const int row = chunk * kChunk + row_tile * 16 + g;
       const size_t out_pitch = size_t(o.heads) * o.vdim_pad;
       float* out = o.out + size_t(row) * out_pitch + head * o.vdim_pad + first_value + 2 * c;
@@ -497,7 +627,7 @@ void launch_delta_prompt(const DeltaPromptParams& p, cudaStream_t stream, bool p
     configured_device = device;
   }
   const unsigned chunks = unsigned((p.outer.rows + kChunk - 1) / kChunk);
-  launch(delta_chunk_kernel, dim3(chunks, unsigned(p.outer.heads)), dim3(kThreads), prepare_shared(p.outer.dim_pad), stream, pdl, p);
+  launch(delta_chunk_kernel, dim3(chunks, unsigned(p.outer.heads)), dim3(kPrepareThreads), prepare_shared(p.outer.dim_pad), stream, pdl, p);
   // Narrow blocks where wide ones would leave most of the chip idle.
   const bool narrow = p.outer.heads * ((p.outer.vdim_pad + 31) / 32) * 3 < multiprocessors * 2;
   if (p.outer.dim_pad <= 128)

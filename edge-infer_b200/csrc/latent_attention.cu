@@ -17,54 +17,74 @@
 namespace ei {
 namespace {
 
-// Turns the pairs (2 i, 2 i + 1) of `x` and writes them to `to`; values behind them, up to `pad`, are copied.
+// Turns the pairs (2 i, 2 i + 1) of `x` and writes them to `to`; values behind them, up to `pad`, are copied. Lanes take
+// four values at a time (rotation sizes are even, padded ones multiples of 16).
 template <typename T>
-__device__ __forceinline__ void turn_pairs(const T* x, T* to, const float2* rotation, int dims, int pad, int lane) {
-  for (int i = lane; i < pad / 2; i += 32) {
-    float2 v = load_pair(x + 2 * i);
-    if (2 * i < dims) {
-      const float2 t = rotation[i];
-      v = make_float2(v.x * t.x - v.y * t.y, v.y * t.x + v.x * t.y);
-    }
-    store_pair(to + 2 * i, v.x, v.y);
+__device__ __forceinline__ void turn_quad(const T* x, T* to, const float2* rotation, int dims, int at) {
+  float4 v = load_quad(x + at);
+  if (at < dims) {
+    const float2 t = rotation[at / 2];
+    const float a = v.x * t.x - v.y * t.y;
+    v.y = v.y * t.x + v.x * t.y;
+    v.x = a;
   }
+  if (at + 2 < dims) {
+    const float2 t = rotation[at / 2 + 1];
+    const float a = v.z * t.x - v.w * t.y;
+    v.w = v.w * t.x + v.z * t.y;
+    v.z = a;
+  }
+  store_quad(to + at, v);
 }
 
-// One warp: latent norm and rotated key of a row (unit == heads), or the rotated part of one head's query.
+// One warp: latent norm and rotated key of a row into the cache.
 template <typename T>
-__device__ __forceinline__ void latent_row(const LatentParams& p, bool step, int context, int row, int unit, int lane) {
-  T* x = static_cast<T*>(p.fused) + size_t(row) * p.stride;
+__device__ __forceinline__ void cache_row(const LatentParams& p, int context, int row, int lane) {
+  const T* x = static_cast<const T*>(p.fused) + size_t(row) * p.stride + p.latent_at;
   const int position = context + row;
-  const float2* rotation = p.rotation + size_t(position) * (p.rot_dims / 2);
-  if (unit < p.heads) {
-    T* q = x + size_t(unit) * (p.dim_pad + p.rot_pad) + p.dim_pad;
-    T* to = q;
-    if (step) {
-      to = static_cast<T*>(p.query) + (size_t(row) * p.heads + unit) * p.row_pad + p.rank_pad;
-      for (int i = p.rot_pad + 2 * lane; i < p.row_pad - p.rank_pad; i += 64) store_pair(to + i, 0.0f, 0.0f);
-    }
-    turn_pairs(q, to, rotation, p.rot_dims, p.rot_pad, lane);
-    return;
-  }
-  x += p.latent_at;
   T* to = static_cast<T*>(p.cache) + size_t(position) * p.row_pad;
+  constexpr int kQuads = 4;
+  float4 held[kQuads];
   float sum = 0.0f;
-  for (int i = lane * 4; i < p.rank_pad; i += 128) {
-    const float4 v = load_quad(x + i);
-    sum = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, sum))));
+  auto square = [&](float4 v) { sum = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, sum)))); };
+#pragma unroll
+  for (int j = 0; j < kQuads; ++j) {
+    const int i = (lane + 32 * j) * 4;
+    held[j] = i < p.rank_pad ? load_quad(x + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
   }
+#pragma unroll
+  for (int j = 0; j < kQuads; ++j) square(held[j]);
+  for (int i = (lane + 32 * kQuads) * 4; i < p.rank_pad; i += 128) square(load_quad(x + i));
   const float scale = 1.0f / sqrtf(warp_sum(sum) / float(p.rank) + p.eps);
-  for (int i = lane * 4; i < p.rank_pad; i += 128) {
-    const float4 v = load_quad(x + i), w = load_quad(p.norm + i);
+  auto emit = [&](int i, float4 v) {
+    const float4 w = load_quad(p.norm + i);
     store_quad(to + i, make_float4(v.x * scale * w.x, v.y * scale * w.y, v.z * scale * w.z, v.w * scale * w.w));
-  }
-  turn_pairs(x + p.rank_pad, to + p.rank_pad, rotation, p.rot_dims, p.rot_pad, lane);
-  for (int i = p.rank_pad + p.rot_pad + 2 * lane; i < p.row_pad; i += 64) store_pair(to + i, 0.0f, 0.0f);
+  };
+#pragma unroll
+  for (int j = 0; j < kQuads; ++j)
+    if ((lane + 32 * j) * 4 < p.rank_pad) emit((lane + 32 * j) * 4, held[j]);
+  for (int i = (lane + 32 * kQuads) * 4; i < p.rank_pad; i += 128) emit(i, load_quad(x + i));
+  const float2* rotation = p.rotation + size_t(position) * (p.rot_dims / 2);
+  for (int i = lane * 4; i < p.rot_pad; i += 128) turn_quad(x + p.rank_pad, to + p.rank_pad, rotation, p.rot_dims, i);
+  for (int i = p.rank_pad + p.rot_pad + 4 * lane; i < p.row_pad; i += 128) store_quad(to + i, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
 }
 
-// Blocks [0, heads * rank_pad / 64) of a step: 64 latent columns of one head's queries, sum over the head's dim values
-// of query times key expansion, the eight warps taking every eighth value. The other blocks: eight rows of the above.
+// Four values of the rotated part of one head's query, in place or (step form) behind the absorbed query.
+template <typename T>
+__device__ __forceinline__ void query_quad(const LatentParams& p, bool step, int context, int row, int head, int at) {
+  T* q = static_cast<T*>(p.fused) + size_t(row) * p.stride + size_t(head) * (p.dim_pad + p.rot_pad) + p.dim_pad;
+  T* to = step ? static_cast<T*>(p.query) + (size_t(row) * p.heads + head) * p.row_pad + p.rank_pad : q;
+  if (at < p.rot_pad)
+    turn_quad(q, to, p.rotation + size_t(context + row) * (p.rot_dims / 2), p.rot_dims, at);
+  else
+    store_quad(to + at, make_float4(0.0f, 0.0f, 0.0f, 0.0f));  // a cache row's padding
+}
+
+// Blocks [0, absorbing) of a step: 64 latent columns of one head's queries, the sum over the head's dim values of query
+// times key expansion, the eight warps taking every eighth value. Then the cache rows, one per warp, then the rotated
+// query parts, four values per thread.
 constexpr int kPrepareThreads = 256;
+constexpr int kAhead = 16;  // rows of the expansion a warp requests before waiting
 template <typename T>
 __global__ void __launch_bounds__(kPrepareThreads) latent_prepare_kernel(const LatentParams p, int absorbing) {
   extern __shared__ __align__(16) unsigned char prepare_smem[];
@@ -72,16 +92,33 @@ __global__ void __launch_bounds__(kPrepareThreads) latent_prepare_kernel(const L
   float* query = reinterpret_cast<float*>(parts + size_t(8) * p.rows * 32);  // [rows][dim_pad]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int context = p.control->context;  // written by the previous step
-  grid_dependency_wait();
-  grid_launch_dependents();
-  if (context < 0 || context + p.rows > p.capacity) return;
+  const bool runs = context >= 0 && context + p.rows <= p.capacity;
   if (int(blockIdx.x) >= absorbing) {
-    const int item = (blockIdx.x - absorbing) * 8 + warp;
-    if (item < p.rows * (p.heads + 1))
-      latent_row<T>(p, absorbing > 0, context, item / (p.heads + 1), item % (p.heads + 1), lane);
+    grid_dependency_wait();
+    grid_launch_dependents();
+    if (!runs) return;
+    const bool step = absorbing > 0;
+    const int cache_blocks = (p.rows + 7) / 8, block = blockIdx.x - absorbing;
+    if (block < cache_blocks) {
+      if (block * 8 + warp < p.rows) cache_row<T>(p, context, block * 8 + warp, lane);
+      return;
+    }
+    const int quads = (step ? p.row_pad - p.rank_pad : p.rot_pad) / 4;
+    const int item = (block - cache_blocks) * kPrepareThreads + threadIdx.x, pair = item / quads;
+    if (pair < p.rows * p.heads) query_quad<T>(p, step, context, pair / p.heads, pair % p.heads, (item - pair * quads) * 4);
     return;
   }
   const int pieces = p.rank_pad / 64, head = blockIdx.x / pieces, column = (blockIdx.x - head * pieces) * 64 + 2 * lane;
+  const bf16* weights = p.expand + size_t(head) * p.dim_pad * p.rank_pad + column;
+  float2 held[kAhead];
+#pragma unroll
+  for (int i = 0; i < kAhead; ++i) {
+    const int d = warp + 8 * i;
+    held[i] = d < p.dim_pad ? load_pair(weights + size_t(d) * p.rank_pad) : make_float2(0.0f, 0.0f);
+  }
+  grid_dependency_wait();
+  grid_launch_dependents();
+  if (!runs) return;
   const T* q = static_cast<const T*>(p.fused) + size_t(head) * (p.dim_pad + p.rot_pad);
   for (int i = threadIdx.x; i < p.rows * p.dim_pad; i += kPrepareThreads)
     query[i] = value_of(q[size_t(i / p.dim_pad) * p.stride + i % p.dim_pad]);
@@ -89,10 +126,7 @@ __global__ void __launch_bounds__(kPrepareThreads) latent_prepare_kernel(const L
   float2 acc[kMaxRows];
 #pragma unroll
   for (int r = 0; r < kMaxRows; ++r) acc[r] = make_float2(0.0f, 0.0f);
-  const bf16* weights = p.expand + size_t(head) * p.dim_pad * p.rank_pad + column;
-#pragma unroll 4
-  for (int d = warp; d < p.dim_pad; d += 8) {
-    const float2 w = load_pair(weights + size_t(d) * p.rank_pad);
+  auto absorb = [&](int d, float2 w) {
 #pragma unroll
     for (int r = 0; r < kMaxRows; ++r) {
       if (r < p.rows) {
@@ -100,7 +134,11 @@ __global__ void __launch_bounds__(kPrepareThreads) latent_prepare_kernel(const L
         acc[r].y = fmaf(query[r * p.dim_pad + d], w.y, acc[r].y);
       }
     }
-  }
+  };
+#pragma unroll
+  for (int i = 0; i < kAhead; ++i)
+    if (warp + 8 * i < p.dim_pad) absorb(warp + 8 * i, held[i]);
+  for (int d = warp + 8 * kAhead; d < p.dim_pad; d += 8) absorb(d, load_pair(weights + size_t(d) * p.rank_pad));
 #pragma unroll
   for (int r = 0; r < kMaxRows; ++r)
     if (r < p.rows) parts[(warp * p.rows + r) * 32 + lane] = acc[r];
@@ -115,6 +153,8 @@ __global__ void __launch_bounds__(kPrepareThreads) latent_prepare_kernel(const L
     store_pair(static_cast<T*>(p.query) + (size_t(r) * p.heads + head) * p.row_pad + column, sum.x, sum.y);
   }
 }
+
+__device__ __forceinline__ float4 quad_of(const float* p) { return *reinterpret_cast<const float4*>(p); }
 
 // ---- split attention over the cache rows --------------------------------------------------------------------------
 constexpr int kTile = 64;
@@ -360,24 +400,49 @@ __global__ void __launch_bounds__(kWarps * 32) latent_attention_kernel(const __g
   }
 }
 
-// Block ((row, head), 32 values): the splits are merged into one latent, every warp then expands four values of it, and
-// the output gate is applied.
+// Block ((row, head), 32 values): the splits are merged into one latent - a thread sums four columns of every second
+// split -, every warp then expands four values of it, and the output gate is applied. The expansion's rows are requested
+// before waiting for the attention.
 constexpr int kExpandThreads = 256;
+constexpr int kExpandQuads = 4;   // quads of a row a lane requests ahead: 512 latent values
+constexpr int kMergeAhead = 8;    // splits a thread requests at once
 template <typename T>
 __global__ void __launch_bounds__(kExpandThreads) latent_expand_kernel(const LatentParams p, const SizedAttentionParams a, int merge) {
   __shared__ __align__(16) float latent[kMaxLatent];
+  __shared__ __align__(16) float other[kMaxLatent];
   __shared__ float weights[64];
-  __shared__ float shared[2];
+  __shared__ float shared[1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int offset = *a.device_offset;  // written by the previous step
+  const int pair = blockIdx.x, row = pair / p.heads, head = pair - row * p.heads;
+  const int first_value = blockIdx.y * 32 + warp * 4;
+  const bf16* values = p.expand + (size_t(p.heads) * p.dim_pad + size_t(head) * p.vdim_pad + first_value) * p.rank_pad;
+  uint2 held[4][kExpandQuads];
+#pragma unroll
+  for (int j = 0; j < 4; ++j)
+#pragma unroll
+    for (int i = 0; i < kExpandQuads; ++i) {
+      const int at = (lane + 32 * i) * 4;
+      held[j][i] = make_uint2(0, 0);
+      if (first_value + j < p.vdim_pad && at < p.rank_pad) held[j][i] = *reinterpret_cast<const uint2*>(values + size_t(j) * p.rank_pad + at);
+    }
   grid_dependency_wait();
   grid_launch_dependents();
   if (offset < 0 || offset + p.rows > p.capacity) return;
-  const int pair = blockIdx.x, row = pair / p.heads, head = pair - row * p.heads;
   if (merge) {
     const int splits = min(64, (offset + p.rows + a.chunk - 1) / a.chunk), pitch = p.rank_pad + 4;
     const float* base = a.scratch + size_t(pair) * pitch;
     const size_t step = size_t(p.rows) * p.heads * pitch;
+    const int half = threadIdx.x >> 7, column = (threadIdx.x & 127) * 4;  // splits half, half + 2, ..
+    float4 x[kMergeAhead];
+    auto request = [&](int s, int at) {
+#pragma unroll
+      for (int i = 0; i < kMergeAhead; ++i) {
+        x[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (s + 2 * i < splits && at < p.rank_pad) x[i] = quad_of(base + (s + 2 * i) * step + at);
+      }
+    };
+    request(half, column);
     if (warp == 0) {
       float m[2], l[2];
 #pragma unroll
@@ -399,18 +464,21 @@ __global__ void __launch_bounds__(kExpandThreads) latent_expand_kernel(const Lat
       if (lane == 0) shared[0] = sum > 0.0f ? 1.0f / sum : 0.0f;
     }
     __syncthreads();
-    for (int i = threadIdx.x * 2; i < p.rank_pad; i += kExpandThreads * 2) {
-      float2 sum = make_float2(0.0f, 0.0f);
-#pragma unroll 8
-      for (int s = 0; s < splits; ++s) {
+    for (int at = column; at < p.rank_pad; at += 512) {
+      float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      for (int s = half; s < splits; s += 2 * kMergeAhead) {
+        if (s != half || at != column) request(s, at);
         // A split in which this pair saw nothing has weight zero and finite sums.
-        const float2 v = *reinterpret_cast<const float2*>(base + s * step + i);
-        sum.x = fmaf(weights[s], v.x, sum.x);
-        sum.y = fmaf(weights[s], v.y, sum.y);
+#pragma unroll
+        for (int i = 0; i < kMergeAhead; ++i) {
+          const float w = s + 2 * i < splits ? weights[s + 2 * i] : 0.0f;
+          sum = make_float4(fmaf(w, x[i].x, sum.x), fmaf(w, x[i].y, sum.y), fmaf(w, x[i].z, sum.z), fmaf(w, x[i].w, sum.w));
+        }
       }
-      latent[i] = sum.x * shared[0];
-      latent[i + 1] = sum.y * shared[0];
+      *reinterpret_cast<float4*>((half ? other : latent) + at) = sum;
     }
+    __syncthreads();
+    for (int i = threadIdx.x; i < p.rank_pad; i += kExpandThreads) latent[i] = (latent[i] + other[i]) * shared[0];
   } else {
     const T* from = static_cast<const T*>(a.out) + size_t(row) * a.out_stride + size_t(head) * p.rank_pad;
     for (int i = threadIdx.x; i < p.rank_pad; i += kExpandThreads) latent[i] = value_of(from[i]);
@@ -418,16 +486,22 @@ __global__ void __launch_bounds__(kExpandThreads) latent_expand_kernel(const Lat
   __syncthreads();
   const T* gate = static_cast<const T*>(p.fused) + size_t(row) * p.stride + p.gate_at + size_t(head) * p.vdim_pad;
   T* out = static_cast<T*>(p.out) + size_t(row) * p.out_stride + size_t(head) * p.vdim_pad;
-  const bf16* values = p.expand + (size_t(p.heads) * p.dim_pad + size_t(head) * p.vdim_pad) * p.rank_pad;
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
-    const int v = blockIdx.y * 32 + warp * 4 + j;
+    const int v = first_value + j;
     if (v >= p.vdim_pad) break;
     float sum = 0.0f;
-    for (int i = lane * 4; i < p.rank_pad; i += 128) {
-      const float4 w = load_quad(values + size_t(v) * p.rank_pad + i), x = *reinterpret_cast<const float4*>(latent + i);
-      sum = fmaf(w.x, x.x, fmaf(w.y, x.y, fmaf(w.z, x.z, fmaf(w.w, x.w, sum))));
+    auto add_quad = [&](int at, float4 w) {
+      const float4 y = quad_of(latent + at);
+      sum = fmaf(w.x, y.x, fmaf(w.y, y.y, fmaf(w.z, y.z, fmaf(w.w, y.w, sum))));
+    };
+#pragma unroll
+    for (int i = 0; i < kExpandQuads; ++i) {
+      const int at = (lane + 32 * i) * 4;
+      if (at < p.rank_pad)
+        add_quad(at, make_float4(bf16_lo(held[j][i].x), bf16_hi(held[j][i].x), bf16_lo(held[j][i].y), bf16_hi(held[j][i].y)));
     }
+    for (int at = (lane + 32 * kExpandQuads) * 4; at < p.rank_pad; at += 128) add_quad(at, load_quad(values + size_t(j) * p.rank_pad + at));
     sum = warp_sum(sum);
     if (lane == 0) store_value(out + v, sum * sigmoid_for<T>(value_of(gate[v])));
   }
@@ -467,7 +541,8 @@ void launch_latent_prepare(const LatentParams& p, bool step, cudaStream_t stream
   }
   const int absorbing = step ? p.heads * (p.rank_pad / 64) : 0;
   const size_t smem = step ? size_t(p.rows) * (p.dim_pad * 4 + 2048) : 0;
-  const int blocks = absorbing + (p.rows * (p.heads + 1) + 7) / 8;
+  const int quads = (step ? p.row_pad - p.rank_pad : p.rot_pad) / 4;
+  const int blocks = absorbing + (p.rows + 7) / 8 + (p.rows * p.heads * quads + kPrepareThreads - 1) / kPrepareThreads;
   launch(latent_prepare_kernel<T>, dim3(unsigned(blocks)), dim3(kPrepareThreads), smem, stream, pdl, p, absorbing);
 }
 

@@ -38,6 +38,7 @@ template <typename T>
 __device__ __forceinline__ float silu_for(float x) { return sizeof(T) == 2 ? x * quick_sigmoid(x) : silu_exact(x); }
 __device__ __forceinline__ float4 add(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
 __device__ __forceinline__ float softplus_value(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
+__device__ __forceinline__ float quick_softplus(float x) { return x > 20.0f ? x : log1pf(__expf(x)); }
 
 // Sum over the block; `shared` holds a value per warp and is free again after the next block-wide barrier.
 __device__ __forceinline__ float block_total(float v, float* shared) {

@@ -15,16 +15,16 @@ namespace ei {
 namespace {
 
 // One warp per (row, unit): q heads, k heads, v heads (convolution, SiLU, unit length), then the decays - per head for the
-// delta rule, 32 heads at a time otherwise.
-constexpr int kHeadColumns = kMaxHeadDim / 32;
-template <typename T>
+// delta rule, 32 heads at a time otherwise. What does not come from the preceding kernel - weights, and the inputs of
+// earlier steps - is requested before waiting for it. kTaps 0: any number of taps.
+constexpr int kStrips = 4;  // strips of 32 channels in flight
+template <typename T, int kTaps>
 __global__ void __launch_bounds__(128) outer_prepare_kernel(const OuterStateParams p) {
+  constexpr int kHeldTaps = kTaps ? kTaps : 1;
   const int warp = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   const int units = 2 * p.key_heads + p.heads + (p.delta ? p.heads : (p.heads + 31) / 32);
   const int context = p.control->context;  // written by the previous step
-  grid_dependency_wait();
-  grid_launch_dependents();
-  if (warp >= p.rows * units || context < 0 || context + p.rows > p.capacity) return;
+  const bool runs = warp < p.rows * units && context >= 0 && context + p.rows <= p.capacity;
   const int row = warp / units, position = context + row;
   int unit = warp - row * units;
   const int slot = position & (kRingRows - 1);
@@ -36,23 +36,59 @@ __global__ void __launch_bounds__(128) outer_prepare_kernel(const OuterStatePara
     const int first = kind * p.key_heads * p.dim_pad + head * pad;
     const int channels = 2 * p.key_heads * p.dim_pad + p.heads * p.vdim_pad;
     T* raw = static_cast<T*>(p.raw);
-    float values[kHeadColumns], squares = 0.0f;
+    float weights[kStrips][kHeldTaps], inputs[kStrips][kHeldTaps], bias[kStrips];
+    auto settled = [&](int chunk) {  // weights, and inputs of earlier steps
 #pragma unroll
-    for (int j = 0; j < kHeadColumns; ++j) {
-      const int c = lane + 32 * j;
-      values[j] = 0.0f;
-      if (c >= pad) continue;
-      const int channel = first + c;
-      float sum = p.conv_bias ? p.conv_bias[channel] : 0.0f;
-      for (int tap = 0; tap < p.taps; ++tap) {
-        const int r = row - (p.taps - 1) + tap, at = context + r;
-        if (at < 0) continue;
-        const T x = r >= 0 ? fused[size_t(r) * p.stride + channel] : raw[size_t(at & (p.raw_rows - 1)) * channels + channel];
-        sum = fmaf(value_of(x), p.conv[size_t(tap) * channels + channel], sum);
+      for (int j = 0; j < kStrips; ++j) {
+        const int c = chunk + lane + 32 * j;
+        bias[j] = runs && c < pad && p.conv_bias ? p.conv_bias[first + c] : 0.0f;
+#pragma unroll
+        for (int tap = 0; tap < kTaps; ++tap) {
+          const int r = row - (kTaps - 1) + tap;
+          weights[j][tap] = inputs[j][tap] = 0.0f;
+          if (!runs || c >= pad) continue;
+          weights[j][tap] = p.conv[size_t(tap) * channels + first + c];
+          if (r < 0 && context + r >= 0) inputs[j][tap] = value_of(raw[size_t((context + r) & (p.raw_rows - 1)) * channels + first + c]);
+        }
       }
-      raw[size_t(position & (p.raw_rows - 1)) * channels + channel] = fused[size_t(row) * p.stride + channel];
-      values[j] = silu_for<T>(sum);
-      squares = fmaf(values[j], values[j], squares);
+    };
+    settled(0);
+    grid_dependency_wait();
+    grid_launch_dependents();
+    if (!runs) return;
+    float values[kMaxHeadDim / 32], squares = 0.0f;
+#pragma unroll
+    for (int chunk = 0; chunk < kMaxHeadDim; chunk += 32 * kStrips) {
+      if (chunk >= pad) break;
+      if (chunk) settled(chunk);
+#pragma unroll
+      for (int j = 0; j < kStrips; ++j) {
+        const int c = chunk + lane + 32 * j;
+        float sum = bias[j];
+        if (c < pad) {
+          const int channel = first + c;
+          const T own = fused[size_t(row) * p.stride + channel];
+          if (kTaps) {
+#pragma unroll
+            for (int tap = 0; tap < kTaps; ++tap) {
+              const int r = row - (kTaps - 1) + tap;
+              const float x = tap == kTaps - 1 ? value_of(own) : r >= 0 ? value_of(fused[size_t(r) * p.stride + channel]) : inputs[j][tap];
+              sum = fmaf(x, weights[j][tap], sum);
+            }
+          } else {
+            for (int tap = 0; tap < p.taps; ++tap) {
+              const int r = row - (p.taps - 1) + tap, at = context + r;
+              if (at < 0) continue;
+              const T x = r >= 0 ? fused[size_t(r) * p.stride + channel] : raw[size_t(at & (p.raw_rows - 1)) * channels + channel];
+              sum = fmaf(value_of(x), p.conv[size_t(tap) * channels + channel], sum);
+            }
+          }
+          raw[size_t(position & (p.raw_rows - 1)) * channels + channel] = own;
+        }
+        const float y = c < pad ? silu_for<T>(sum) : 0.0f;
+        values[chunk / 32 + j] = y;
+        squares = fmaf(y, y, squares);
+      }
     }
     float scale = 1.0f;
     if (p.delta && kind < 2) {
@@ -63,30 +99,35 @@ __global__ void __launch_bounds__(128) outer_prepare_kernel(const OuterStatePara
                 : kind == 1 ? p.ring_k + size_t(slot) * p.key_heads * p.dim_pad + head * pad
                             : p.v + size_t(row) * p.heads * p.vdim_pad + head * pad;
 #pragma unroll
-    for (int j = 0; j < kHeadColumns; ++j)
+    for (int j = 0; j < kMaxHeadDim / 32; ++j)
       if (lane + 32 * j < pad) to[lane + 32 * j] = values[j] * scale;
     return;
   }
   unit -= 2 * p.key_heads + p.heads;
+  const int head = p.delta ? unit : unit * 32 + lane;
+  const float rate = head < p.heads ? p.rate[head] : 0.0f;
+  const float bias = !p.delta && head < p.heads ? p.bias[head] : 0.0f;
+  grid_dependency_wait();
+  grid_launch_dependents();
+  if (!runs) return;
   const T* step = fused + size_t(row) * p.stride + p.step_at;
   if (p.delta) {
-    const int head = unit;
     const T* decay = static_cast<const T*>(p.decay) + size_t(row) * p.decay_stride + head * p.dim_pad;
     float* to = p.ring_g + (size_t(slot) * p.heads + head) * p.dim_pad;
-    for (int d = lane; d < p.dim_pad; d += 32)
-      to[d] = expf(-p.rate[head] * softplus_value(value_of(decay[d]) + p.bias[head * p.dim_pad + d]));
     if (lane == 0) p.beta[size_t(row) * p.heads + head] = sigmoid_value(value_of(step[head]));
+#pragma unroll 4
+    for (int d = lane; d < p.dim_pad; d += 32)
+      to[d] = expf(-rate * softplus_value(value_of(decay[d]) + p.bias[head * p.dim_pad + d]));
     return;
   }
-  const int head = unit * 32 + lane;
   if (head >= p.heads) return;
-  const float t = softplus_value(value_of(step[head]) + p.bias[head]);
-  p.ring_g[size_t(slot) * p.heads + head] = expf(-p.rate[head] * t);
+  const float t = softplus_value(value_of(step[head]) + bias);
+  p.ring_g[size_t(slot) * p.heads + head] = expf(-rate * t);
   p.beta[size_t(row) * p.heads + head] = t;
 }
 
 // Block (head, slice of 16 values): a warp owns four values over all key channels, lane l the channels l, l + 32, ...
-template <bool kDelta, int kStrips>
+template <bool kDelta, int kParts>
 __global__ void __launch_bounds__(128) outer_step_kernel(const OuterStateParams p) {
   const int head = blockIdx.x, slice = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int key_head = head / (p.heads / p.key_heads);
@@ -97,9 +138,9 @@ __global__ void __launch_bounds__(128) outer_step_kernel(const OuterStateParams 
   const bool runs = context >= 0 && context + p.rows <= p.capacity;
   const int pending = min(kPendingRows, max(0, context - base));
   float* state = p.state + ((size_t(head) * (p.vdim_pad / 16) + slice) * p.dim_pad) * 16 + warp * 4;
-  float4 s[kStrips];
+  float4 s[kParts];
 #pragma unroll
-  for (int i = 0; i < kStrips; ++i) {
+  for (int i = 0; i < kParts; ++i) {
     const int d = lane + 32 * i;
     s[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     if (runs && base > 0 && d < p.dim_pad) s[i] = *reinterpret_cast<const float4*>(state + size_t(d) * 16);
@@ -113,7 +154,7 @@ __global__ void __launch_bounds__(128) outer_step_kernel(const OuterStateParams 
       const float4 u = *reinterpret_cast<const float4*>(p.ring_u + size_t(slot) * value_width + value);
       const float whole = kDelta ? 0.0f : decays[size_t(slot) * decay_width];
 #pragma unroll
-      for (int i = 0; i < kStrips; ++i) {
+      for (int i = 0; i < kParts; ++i) {
         const int d = lane + 32 * i;
         if (d >= p.dim_pad) continue;
         const float k = keys[size_t(slot) * key_width + d], g = kDelta ? decays[size_t(slot) * decay_width + d] : whole;
@@ -121,7 +162,7 @@ __global__ void __launch_bounds__(128) outer_step_kernel(const OuterStateParams 
       }
     }
 #pragma unroll
-    for (int i = 0; i < kStrips; ++i)
+    for (int i = 0; i < kParts; ++i)
       if (lane + 32 * i < p.dim_pad) *reinterpret_cast<float4*>(state + size_t(lane + 32 * i) * 16) = s[i];
   }
   grid_dependency_wait();
@@ -132,11 +173,11 @@ __global__ void __launch_bounds__(128) outer_step_kernel(const OuterStateParams 
     const float4 v = *reinterpret_cast<const float4*>(p.v + size_t(row) * value_width + value);
     const float rate = p.beta[size_t(row) * p.heads + head];
     const float whole = kDelta ? 0.0f : decays[size_t(slot) * decay_width];
-    float k[kStrips];
+    float k[kParts];
     float4 seen = make_float4(0.0f, 0.0f, 0.0f, 0.0f), read = seen;  // S^T k and S^T q after the decay
     float match = 0.0f;                                              // q . k
 #pragma unroll
-    for (int i = 0; i < kStrips; ++i) {
+    for (int i = 0; i < kParts; ++i) {
       const int d = lane + 32 * i;
       k[i] = 0.0f;
       if (d >= p.dim_pad) continue;
@@ -155,7 +196,7 @@ __global__ void __launch_bounds__(128) outer_step_kernel(const OuterStateParams 
     match = warp_sum(match);
     const float4 u = make_float4(rate * (v.x - seen.x), rate * (v.y - seen.y), rate * (v.z - seen.z), rate * (v.w - seen.w));
 #pragma unroll
-    for (int i = 0; i < kStrips; ++i)
+    for (int i = 0; i < kParts; ++i)
       s[i] = make_float4(fmaf(k[i], u.x, s[i].x), fmaf(k[i], u.y, s[i].y), fmaf(k[i], u.z, s[i].z), fmaf(k[i], u.w, s[i].w));
     if (lane == 0) {
       const float skip = p.skip ? p.skip[head] : 0.0f;
@@ -171,23 +212,20 @@ __global__ void __launch_bounds__(128) outer_step_kernel(const OuterStateParams 
 // kTaps 0: any number of taps.
 constexpr int kConvRows = 8;
 template <int kVector>
-struct Channels {
-  float v[kVector];
+struct Packed {
+  uint32_t pair[kVector / 2];
 };
-__device__ __forceinline__ Channels<4> load_channels(const bf16* p, Channels<4>) {
-  const float4 x = load_quad(p);
-  return {{x.x, x.y, x.z, x.w}};
-}
-__device__ __forceinline__ Channels<2> load_channels(const bf16* p, Channels<2>) {
-  const float2 x = load_pair(p);
+__device__ __forceinline__ Packed<4> packed_at(const bf16* p, Packed<4>) {
+  const uint2 x = *reinterpret_cast<const uint2*>(p);
   return {{x.x, x.y}};
 }
-__device__ __forceinline__ void store_channels(bf16* p, Channels<4> x) { store_quad(p, make_float4(x.v[0], x.v[1], x.v[2], x.v[3])); }
-__device__ __forceinline__ void store_channels(bf16* p, Channels<2> x) { store_pair(p, x.v[0], x.v[1]); }
+__device__ __forceinline__ Packed<2> packed_at(const bf16* p, Packed<2>) { return {{*reinterpret_cast<const uint32_t*>(p)}}; }
+__device__ __forceinline__ void put_packed(bf16* p, Packed<4> x) { *reinterpret_cast<uint2*>(p) = make_uint2(x.pair[0], x.pair[1]); }
+__device__ __forceinline__ void put_packed(bf16* p, Packed<2> x) { *reinterpret_cast<uint32_t*>(p) = x.pair[0]; }
 
 template <int kTaps, int kVector>
 __device__ __forceinline__ void conv_head(const OuterStateParams& p, bf16* out, float* inverse, int context, int begin, int unit, int lane) {
-  using Vector = Channels<kVector>;
+  using Vector = Packed<kVector>;
   const int kind = unit < p.key_heads ? 0 : unit < 2 * p.key_heads ? 1 : 2;  // q, k, v
   const int head = unit - kind * p.key_heads, pad = kind == 2 ? p.vdim_pad : p.dim_pad;
   const int first = kind * p.key_heads * p.dim_pad + head * pad;
@@ -202,48 +240,67 @@ __device__ __forceinline__ void conv_head(const OuterStateParams& p, bf16* out, 
     const int channel = first + c;
     auto input = [&](int r) {
       if (r >= p.rows) return Vector{};
-      if (r >= 0) return load_channels(fused + size_t(r) * p.stride + channel, Vector{});
-      return context + r >= 0 ? load_channels(raw + size_t((context + r) & (p.raw_rows - 1)) * channels + channel, Vector{}) : Vector{};
+      if (r >= 0) return packed_at(fused + size_t(r) * p.stride + channel, Vector{});
+      return context + r >= 0 ? packed_at(raw + size_t((context + r) & (p.raw_rows - 1)) * channels + channel, Vector{}) : Vector{};
     };
-    Vector sums[kConvRows];
+    auto weight = [&](int tap, float (&w)[kVector]) {
 #pragma unroll
-    for (int r = 0; r < kConvRows; ++r)
+      for (int j = 0; j < kVector; j += 2) {
+        const float2 x = load_pair(p.conv + size_t(tap) * channels + channel + j);
+        w[j] = x.x;
+        w[j + 1] = x.y;
+      }
+    };
+    auto accumulate = [](float (&sum)[kVector], const Vector& x, const float (&w)[kVector]) {
 #pragma unroll
-      for (int j = 0; j < kVector; ++j) sums[r].v[j] = p.conv_bias ? p.conv_bias[channel + j] : 0.0f;
+      for (int j = 0; j < kVector; j += 2) {
+        sum[j] = fmaf(bf16_lo(x.pair[j / 2]), w[j], sum[j]);
+        sum[j + 1] = fmaf(bf16_hi(x.pair[j / 2]), w[j + 1], sum[j + 1]);
+      }
+    };
+    auto finish = [&](int r, float (&sum)[kVector]) {
+      if (begin + r >= p.rows) return;
+      Vector y;
+#pragma unroll
+      for (int j = 0; j < kVector; j += 2) {
+        const float a = sum[j], b = sum[j + 1];
+        y.pair[j / 2] = pack_bf16(a * quick_sigmoid(a), b * quick_sigmoid(b));
+        squares[r] = fmaf(bf16_lo(y.pair[j / 2]), bf16_lo(y.pair[j / 2]), fmaf(bf16_hi(y.pair[j / 2]), bf16_hi(y.pair[j / 2]), squares[r]));
+      }
+      put_packed(out + size_t(begin + r) * channels + channel, y);
+    };
+    float bias[kVector];
+#pragma unroll
+    for (int j = 0; j < kVector; ++j) bias[j] = p.conv_bias ? p.conv_bias[channel + j] : 0.0f;
     if (kTaps) {
-      Vector window[kConvRows + (kTaps ? kTaps - 1 : 0)];
+      constexpr int kHeld = kTaps ? kTaps : 1;
+      Vector window[kConvRows + kHeld - 1];
+      float w[kHeld][kVector];
 #pragma unroll
-      for (int i = 0; i < kConvRows + kTaps - 1; ++i) window[i] = input(begin + i - (kTaps - 1));
+      for (int i = 0; i < kConvRows + kHeld - 1; ++i) window[i] = input(begin + i - (kHeld - 1));
 #pragma unroll
-      for (int tap = 0; tap < kTaps; ++tap)
+      for (int tap = 0; tap < kHeld; ++tap) weight(tap, w[tap]);
 #pragma unroll
-        for (int j = 0; j < kVector; ++j) {
-          const float w = p.conv[size_t(tap) * channels + channel + j];
+      for (int r = 0; r < kConvRows; ++r) {
+        float sum[kVector];
 #pragma unroll
-          for (int r = 0; r < kConvRows; ++r) sums[r].v[j] = fmaf(window[r + tap].v[j], w, sums[r].v[j]);
-        }
+        for (int j = 0; j < kVector; ++j) sum[j] = bias[j];
+#pragma unroll
+        for (int tap = 0; tap < kHeld; ++tap) accumulate(sum, window[r + tap], w[tap]);
+        finish(r, sum);
+      }
     } else {
-      for (int tap = 0; tap < taps; ++tap) {
-        Vector w;
 #pragma unroll
-        for (int j = 0; j < kVector; ++j) w.v[j] = p.conv[size_t(tap) * channels + channel + j];
+      for (int r = 0; r < kConvRows; ++r) {
+        float sum[kVector], w[kVector];
 #pragma unroll
-        for (int r = 0; r < kConvRows; ++r) {
-          const Vector x = input(begin + r - (taps - 1) + tap);
-#pragma unroll
-          for (int j = 0; j < kVector; ++j) sums[r].v[j] = fmaf(x.v[j], w.v[j], sums[r].v[j]);
+        for (int j = 0; j < kVector; ++j) sum[j] = bias[j];
+        for (int tap = 0; tap < taps; ++tap) {
+          weight(tap, w);
+          accumulate(sum, input(begin + r - (taps - 1) + tap), w);
         }
+        finish(r, sum);
       }
-    }
-#pragma unroll
-    for (int r = 0; r < kConvRows; ++r) {
-      if (begin + r >= p.rows) break;
-#pragma unroll
-      for (int j = 0; j < kVector; ++j) {
-        sums[r].v[j] = round_bf16(sums[r].v[j] * quick_sigmoid(sums[r].v[j]));
-        squares[r] = fmaf(sums[r].v[j], sums[r].v[j], squares[r]);
-      }
-      store_channels(out + size_t(begin + r) * channels + channel, sums[r]);
     }
   }
   if (!p.delta || kind == 2) return;
@@ -273,7 +330,8 @@ __global__ void __launch_bounds__(128) outer_conv_kernel(const OuterStateParams 
 
 // One warp (kWide: one block) per (row, norm group). Values of a group are those of its heads side by side, without the
 // heads' padding.
-constexpr int kFinishHeld = 8;
+constexpr int kFinishHeld = 8;   // values a thread keeps between the two passes over a group
+constexpr int kFinishQuads = 4;  // the same, four at a time
 template <typename T, bool kWide>
 __global__ void __launch_bounds__(256) state_finish_kernel(const StateFinishParams p) {
   __shared__ float shared[8];
@@ -301,6 +359,51 @@ __global__ void __launch_bounds__(256) state_finish_kernel(const StateFinishPara
   const T* gate = static_cast<const T*>(p.gate) + size_t(row) * p.gate_stride;
   T* out = static_cast<T*>(p.out) + size_t(row) * p.out_stride;
   auto column = [&](int e) { return packed ? first + e : (first + e) / p.vdim * p.vdim_pad + (first + e) % p.vdim; };
+  if (packed && length % 4 == 0) {  // four values at a time
+    auto gated = [&](float4 x, float4 z) {
+      return p.gate_first ? make_float4(x.x * silu_for<T>(z.x), x.y * silu_for<T>(z.y), x.z * silu_for<T>(z.z), x.w * silu_for<T>(z.w)) : x;
+    };
+    float4 x[kFinishQuads], z[kFinishQuads];
+    float squares = 0.0f;
+#pragma unroll
+    for (int j = 0; j < kFinishQuads; ++j) {
+      const int e = (lane + j * lanes) * 4;
+      x[j] = z[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      if (e < length) {
+        x[j] = *reinterpret_cast<const float4*>(in + first + e);
+        z[j] = load_quad(gate + first + e);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < kFinishQuads; ++j) {
+      x[j] = gated(x[j], z[j]);
+      squares = fmaf(x[j].x, x[j].x, fmaf(x[j].y, x[j].y, fmaf(x[j].z, x[j].z, fmaf(x[j].w, x[j].w, squares))));
+    }
+    for (int e = (lane + kFinishQuads * lanes) * 4; e < length; e += lanes * 4) {
+      const float4 y = gated(*reinterpret_cast<const float4*>(in + first + e), load_quad(gate + first + e));
+      squares = fmaf(y.x, y.x, fmaf(y.y, y.y, fmaf(y.z, y.z, fmaf(y.w, y.w, squares))));
+    }
+    const float scale = 1.0f / sqrtf((kWide ? block_total(squares, shared) : warp_sum(squares)) / float(length) + p.eps);
+    auto finish = [&](int e, float4 y, float4 gates) {
+      const float4 w = load_quad(p.norm + first + e);
+      y = make_float4(y.x * scale * w.x, y.y * scale * w.y, y.z * scale * w.z, y.w * scale * w.w);
+      if (!p.gate_first)
+        y = make_float4(y.x * sigmoid_for<T>(gates.x), y.y * sigmoid_for<T>(gates.y), y.z * sigmoid_for<T>(gates.z), y.w * sigmoid_for<T>(gates.w));
+      store_quad(out + first + e, y);
+    };
+#pragma unroll
+    for (int j = 0; j < kFinishQuads; ++j) {
+      const int e = (lane + j * lanes) * 4;
+      if (e < length) finish(e, x[j], z[j]);
+    }
+    for (int e = (lane + kFinishQuads * lanes) * 4; e < length; e += lanes * 4) {
+      const float4 gates = load_quad(gate + first + e);
+      finish(e, gated(*reinterpret_cast<const float4*>(in + first + e), gates), gates);
+    }
+    if (group == 0)
+      for (int at = width + lane; at < p.out_stride; at += lanes) store_value(out + at, 0.0f);
+    return;
+  }
   auto value = [&](int at, float z) { return p.gate_first ? in[at] * silu_for<T>(z) : in[at]; };
   float held[kFinishHeld], gates[kFinishHeld], sum = 0.0f;
 #pragma unroll
@@ -358,7 +461,11 @@ template <typename T>
 void launch_outer_prepare(const OuterStateParams& p, cudaStream_t stream, bool pdl) {
   if (p.rows < 1 || p.rows > kPendingRows) throw std::invalid_argument("a state step takes 1..16 rows");
   const int warps = p.rows * (2 * p.key_heads + p.heads + (p.delta ? p.heads : (p.heads + 31) / 32));
-  launch(outer_prepare_kernel<T>, dim3(unsigned((warps + 3) / 4)), dim3(128), 0, stream, pdl, p);
+  const dim3 grid(unsigned((warps + 3) / 4));
+  if (p.taps == 2) return launch(outer_prepare_kernel<T, 2>, grid, dim3(128), 0, stream, pdl, p);
+  if (p.taps == 3) return launch(outer_prepare_kernel<T, 3>, grid, dim3(128), 0, stream, pdl, p);
+  if (p.taps == 4) return launch(outer_prepare_kernel<T, 4>, grid, dim3(128), 0, stream, pdl, p);
+  launch(outer_prepare_kernel<T, 0>, grid, dim3(128), 0, stream, pdl, p);
 }
 void launch_outer_conv(const OuterStateParams& p, bf16* out, float* inverse, cudaStream_t stream, bool pdl) {
   const int warps = (p.rows + kConvRows - 1) / kConvRows * (2 * p.key_heads + p.heads);
@@ -376,7 +483,7 @@ void launch_outer_step(const OuterStateParams& p, cudaStream_t stream, bool pdl)
 template <typename T>
 void launch_state_finish(const StateFinishParams& p, cudaStream_t stream, bool pdl) {
   const int items = p.rows * p.groups + p.tail_rows, length = p.heads * p.vdim / p.groups;
-  if (length > 256)
+  if (length > 512)
     launch(state_finish_kernel<T, true>, dim3(unsigned(items)), dim3(256), 0, stream, pdl, p);
   else
     launch(state_finish_kernel<T, false>, dim3(unsigned((items + 3) / 4)), dim3(128), 0, stream, pdl, p);

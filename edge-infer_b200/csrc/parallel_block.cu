@@ -17,16 +17,23 @@ __device__ __forceinline__ float masked_squares(float4 x, float mean, int i, int
   const float a = x.x - mean, b = x.y - mean, c = x.z - mean, d = x.w - mean;
   return (i < width ? a * a : 0.0f) + (i + 1 < width ? b * b : 0.0f) + (i + 2 < width ? c * c : 0.0f) + (i + 3 < width ? d * d : 0.0f);
 }
-__device__ __forceinline__ float4 weighted(float4 x, float mean, float scale, const bf16* weight, int i) {
-  const float4 w = load_quad(weight + i);
+__device__ __forceinline__ float4 weighted(float4 x, float mean, float scale, float4 w) {
   return make_float4((x.x - mean) * scale * w.x, (x.y - mean) * scale * w.y, (x.z - mean) * scale * w.z, (x.w - mean) * scale * w.w);
 }
 
 // The normed rows of a row whose quads are in `held` (and in `residual`, written by the same threads). `columns`: its
-// stride in the residual; the weights are zero beyond the width.
+// stride in the residual; the weights are zero beyond the width. `ahead`: both weights of a thread's first quad.
+struct FirstWeights {
+  float4 first, second;
+};
+__device__ __forceinline__ FirstWeights first_weights(const RowNorms& n, int columns) {
+  const int i = threadIdx.x * 4;
+  const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  return {i < columns ? load_quad(n.first + i) : zero, i < columns && n.second ? load_quad(n.second + i) : zero};
+}
 template <typename T>
 __device__ __forceinline__ void norm_row(const RowNorms& n, const float4 (&held)[kHeld], const float* residual, int columns,
-                                         int row, float* shared) {
+                                         int row, float* shared, const FirstWeights& ahead) {
   const int step = blockDim.x * 4;
   float sum = 0.0f;
 #pragma unroll
@@ -42,11 +49,11 @@ __device__ __forceinline__ void norm_row(const RowNorms& n, const float4 (&held)
   const float scale = 1.0f / sqrtf(block_total(squares, shared + kMostThreads / 32) / float(n.width) + n.eps);
   T* first = static_cast<T*>(n.normed_first) + size_t(row) * n.stride;
   T* second = n.second ? static_cast<T*>(n.normed_second) + size_t(row) * n.stride : nullptr;
+  const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
   auto emit = [&](int i, float4 x) {
-    const bool live = i < columns;
-    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-    store_quad(first + i, live ? weighted(x, mean, scale, n.first, i) : zero);
-    if (second) store_quad(second + i, live ? weighted(x, mean, scale, n.second, i) : zero);
+    const bool live = i < columns, held_ahead = i == int(threadIdx.x) * 4;
+    store_quad(first + i, live ? weighted(x, mean, scale, held_ahead ? ahead.first : load_quad(n.first + i)) : zero);
+    if (second) store_quad(second + i, live ? weighted(x, mean, scale, held_ahead ? ahead.second : load_quad(n.second + i)) : zero);
   };
 #pragma unroll
   for (int j = 0; j < kHeld; ++j) {
@@ -54,7 +61,7 @@ __device__ __forceinline__ void norm_row(const RowNorms& n, const float4 (&held)
     if (i < n.stride) emit(i, held[j]);
   }
   for (int i = threadIdx.x * 4 + kHeld * step; i < n.stride; i += step)
-    emit(i, i < columns ? *reinterpret_cast<const float4*>(residual + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f));
+    emit(i, i < columns ? *reinterpret_cast<const float4*>(residual + i) : zero);
 }
 
 template <typename T>
@@ -62,6 +69,7 @@ __global__ void __launch_bounds__(kMostThreads) parallel_embed_kernel(const Para
   __shared__ uint32_t token_shared;
   __shared__ unsigned long long pair_shared;
   __shared__ float shared[2 * kMostThreads / 32];
+  const FirstWeights ahead = first_weights(p.norms, p.residual_stride);
   grid_dependency_wait();
   const int row = blockIdx.x;
   if (threadIdx.x == 0) {
@@ -97,12 +105,18 @@ __global__ void __launch_bounds__(kMostThreads) parallel_embed_kernel(const Para
     held[j] = i < p.residual_stride ? fetch(i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
   }
   for (int i = (threadIdx.x + kHeld * blockDim.x) * 4; i < p.residual_stride; i += blockDim.x * 4) fetch(i);
-  norm_row<T>(p.norms, held, residual, p.residual_stride, row, shared);
+  norm_row<T>(p.norms, held, residual, p.residual_stride, row, shared, ahead);
 }
 
 template <typename T>
 __global__ void __launch_bounds__(kMostThreads) parallel_join_kernel(const ParallelJoinParams p) {
   __shared__ float shared[2 * kMostThreads / 32];
+  // Weights do not come from the preceding kernel.
+  const FirstWeights ahead = first_weights(p.norms, p.residual_stride);
+  const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  const bool live = int(threadIdx.x) * 4 < p.residual_stride;
+  const float4 mixed_ahead = live ? load_quad(p.mixed_scale + threadIdx.x * 4) : zero;
+  const float4 fed_ahead = live && p.fed ? load_quad(p.fed_scale + threadIdx.x * 4) : zero;
   grid_dependency_wait();
   grid_launch_dependents();
   const int row = blockIdx.x;
@@ -115,11 +129,12 @@ __global__ void __launch_bounds__(kMostThreads) parallel_join_kernel(const Paral
   };
   auto join = [&](int i) {
     float4 x = *reinterpret_cast<const float4*>(residual + i);
-    float4 y = total(p.mixed, p.mixed_ksplit, i), s = load_quad(p.mixed_scale + i);
+    const bool held_ahead = i == int(threadIdx.x) * 4;
+    float4 y = total(p.mixed, p.mixed_ksplit, i), s = held_ahead ? mixed_ahead : load_quad(p.mixed_scale + i);
     y = make_float4(y.x * s.x, y.y * s.y, y.z * s.z, y.w * s.w);
     if (p.fed) {
       const float4 f = total(p.fed, p.fed_ksplit, i);
-      s = load_quad(p.fed_scale + i);
+      s = held_ahead ? fed_ahead : load_quad(p.fed_scale + i);
       y = make_float4(fmaf(f.x, s.x, y.x), fmaf(f.y, s.y, y.y), fmaf(f.z, s.z, y.z), fmaf(f.w, s.w, y.w));
     }
     x = add(x, y);
@@ -139,7 +154,7 @@ __global__ void __launch_bounds__(kMostThreads) parallel_join_kernel(const Paral
     held[j] = i < p.residual_stride ? join(i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
   }
   for (int i = (threadIdx.x + kHeld * blockDim.x) * 4; i < p.residual_stride; i += blockDim.x * 4) join(i);
-  norm_row<T>(p.norms, held, residual, p.residual_stride, row, shared);
+  norm_row<T>(p.norms, held, residual, p.residual_stride, row, shared, ahead);
 }
 
 // A few rows: one quad per thread as far as a block goes. Many: blocks of 256.

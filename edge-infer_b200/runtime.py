@@ -234,6 +234,27 @@ def _shape(data) -> Tuple[int, ...]:
     return tuple(int(x) for x in data.shape) or (1,)  # a scalar travels as one element
 
 
+class _Owned:
+    """A library object and those made on top of it, which are destroyed before it whatever order Python finalizes its
+    wrappers in (members of a reference cycle are finalized in no particular order)."""
+
+    def __init__(self, handle, destroy, *below: "_Owned"):
+        self._handle, self._destroy, self._below = handle, destroy, below
+        self._above = set()
+        for owned in below:
+            owned._above.add(self)
+
+    def close(self) -> None:
+        if not self._handle:
+            return
+        for owned in list(self._above):
+            owned.close()
+        handle, self._handle = self._handle, None
+        self._destroy(handle)
+        for owned in self._below:
+            owned._above.discard(self)
+
+
 class Model:
     """Prepared weights on the current device. `tensors`: name -> list of (kind, array)."""
 
@@ -258,6 +279,7 @@ class Model:
             abi.check(lib.ei_model_create(C.byref(config), array, len(entries), C.byref(handle)))
         self.shape = shape
         self._handle = handle
+        self._owned = _Owned(handle, lib.ei_model_destroy)
         self._lib = lib
 
     @property
@@ -271,9 +293,8 @@ class Model:
         return Session(self, capacity, graph)
 
     def close(self) -> None:
-        if self._handle:
-            self._lib.ei_model_destroy(self._handle)
-            self._handle = None
+        self._owned.close()
+        self._handle = None
 
     def __del__(self):
         try:
@@ -299,6 +320,7 @@ class Session:
         handle = C.c_void_p()
         abi.check(self._lib.ei_session_create(model.handle, capacity, 1 if graph else 0, C.byref(handle)))
         self._handle = handle
+        self._owned = _Owned(handle, self._lib.ei_session_destroy, model._owned)
 
     # -- contract verbs ---------------------------------------------------------------------------
     def prefill(self, tokens: Sequence[int], all_logits=None) -> int:
@@ -430,9 +452,8 @@ class Session:
         abi.check(self._lib.ei_session_inject_attention_wait_timeout(self._handle, polls))
 
     def close(self) -> None:
-        if self._handle:
-            self._lib.ei_session_destroy(self._handle)
-            self._handle = None
+        self._owned.close()
+        self._handle = None
 
     def __del__(self):
         try:
@@ -498,6 +519,7 @@ class SessionBatch:
         out = C.c_void_p()
         abi.check(self._lib.ei_batch_create(handles, len(self.sessions), C.byref(out)))
         self._handle = out
+        self._owned = _Owned(out, self._lib.ei_batch_destroy, *(s._owned for s in self.sessions))
 
     def verify(self, tokens: Sequence[Sequence[int]]) -> List[VerifyOutput]:
         """tokens[j] = [pending, d1..dk] of session j (all of one length)."""
@@ -513,9 +535,8 @@ class SessionBatch:
         return outputs
 
     def close(self) -> None:
-        if self._handle:
-            self._lib.ei_batch_destroy(self._handle)
-            self._handle = None
+        self._owned.close()
+        self._handle = None
 
     def __del__(self):
         try:
@@ -537,6 +558,7 @@ class SpeculativeDecoder:
         out = C.c_void_p()
         abi.check(self._lib.ei_speculative_create(target._handle, draft._handle, self.drafts_per_round, C.byref(out)))
         self._handle = out
+        self._owned = _Owned(out, self._lib.ei_speculative_destroy, target._owned, draft._owned)
 
     def prefill(self, tokens: Sequence[int]) -> int:
         """Both sessions take the prompt; returns the first generated token."""
@@ -578,9 +600,8 @@ class SpeculativeDecoder:
         return out
 
     def close(self) -> None:
-        if self._handle:
-            self._lib.ei_speculative_destroy(self._handle)
-            self._handle = None
+        self._owned.close()
+        self._handle = None
 
     def __del__(self):
         try:

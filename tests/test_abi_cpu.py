@@ -114,3 +114,19 @@ def test_cpp_shim_compiles_links_and_maps_errors(package, tmp_path):
     result = subprocess.run([str(binary)], capture_output=True, text=True)
     assert result.returncode == 0, result.stdout + result.stderr
     assert result.stdout.startswith("1 ")
+
+
+def test_library_objects_are_destroyed_from_the_top_down(package):
+    """In whatever order the wrappers are finalized, a decoder goes before its sessions and a session before its model."""
+    owned, gone = package.runtime._Owned, []
+    for first in range(4):
+        gone.clear()
+        model = owned("model", gone.append)
+        sessions = [owned(name, gone.append, model) for name in ("target", "draft")]
+        decoder = owned("decoder", gone.append, *sessions)
+        order = [model, *sessions, decoder]
+        for item in order[first:] + order[:first]:
+            item.close()
+            item.close()
+        assert sorted(gone) == ["decoder", "draft", "model", "target"]
+        assert gone[0] == "decoder" and gone[-1] == "model"

@@ -322,7 +322,7 @@ def test_greedy_generation_through_the_model_surface(cuda, package, name):
 
 def test_speculative_rounds_on_the_target(cuda, package):
     """A uniform draft model proposes, the target verifies on the device: the output is the target's own."""
-    c = cases.CASES["mixed"]
+    c = {**cases.CASES["mixed"], "logit_softcap": 300.0}     # top logits apart from one another
     model, _ = build(package, c, "bf16")
     draft_shape = package.Shape(vocab_size=c["vocab"], n_layers=1, n_heads=2, n_kv_heads=1, hidden_size=128,
                                 intermediate_size=128, max_position_embeddings=256)
