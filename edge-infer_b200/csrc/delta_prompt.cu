@@ -452,22 +452,30 @@ __global__ void __launch_bounds__(kThreads) delta_scan_kernel(const DeltaPromptP
     if (warp + 8 * m < steps) publish(s[m], (warp + 8 * m) * 16, channel_rows, state_leading, state_rest);
   __syncthreads();
 
-  // acc += (two-term A fragment) x (two-term rows of `leading` / `rest` at `row` + this lane's row of the 16).
-  auto multiply = [&](float (&acc)[kN][4], const uint4& ah, const uint4& al, const bf16* leading, const bf16* rest, int row) {
+  // acc[0] += A leading x B leading, acc[1] += A rest x B leading, acc[2] += A leading x B rest: three short chains instead
+  // of a long one. A: a two-term fragment, B: two-term rows of `leading` / `rest` at `row`, this lane's row of the 16.
+  auto multiply = [&](float (&acc)[3][kN][4], const uint4& ah, const uint4& al, const bf16* leading, const bf16* rest, int row) {
 #pragma unroll
     for (int n = 0; n < kN; n += 2) {
       const int at = row * kPitch + (n + (matrix >> 1)) * 8;
       uint32_t b0, b1, b2, b3;
       ldmatrix_x4_trans(b0, b1, b2, b3, leading + at);
-      mma_bf16_16816(acc[n], ah.x, ah.y, ah.z, ah.w, b0, b1);
-      mma_bf16_16816(acc[n + 1], ah.x, ah.y, ah.z, ah.w, b2, b3);
-      mma_bf16_16816(acc[n], al.x, al.y, al.z, al.w, b0, b1);
-      mma_bf16_16816(acc[n + 1], al.x, al.y, al.z, al.w, b2, b3);
+      mma_bf16_16816(acc[0][n], ah.x, ah.y, ah.z, ah.w, b0, b1);
+      mma_bf16_16816(acc[0][n + 1], ah.x, ah.y, ah.z, ah.w, b2, b3);
+      mma_bf16_16816(acc[1][n], al.x, al.y, al.z, al.w, b0, b1);
+      mma_bf16_16816(acc[1][n + 1], al.x, al.y, al.z, al.w, b2, b3);
       ldmatrix_x4_trans(b0, b1, b2, b3, rest + at);
-      mma_bf16_16816(acc[n], ah.x, ah.y, ah.z, ah.w, b0, b1);
-      mma_bf16_16816(acc[n + 1], ah.x, ah.y, ah.z, ah.w, b2, b3);
+      mma_bf16_16816(acc[2][n], ah.x, ah.y, ah.z, ah.w, b0, b1);
+      mma_bf16_16816(acc[2][n + 1], ah.x, ah.y, ah.z, ah.w, b2, b3);
     }
   };
+  auto clear = [](float (&acc)[3][kN][4]) {
+#pragma unroll
+    for (int term = 0; term < 3; ++term)
+#pragma unroll
+      for (int n = 0; n < kN; ++n) acc[term][n][0] = acc[term][n][1] = acc[term][n][2] = acc[term][n][3] = 0.0f;
+  };
+  auto total = [](const float (&acc)[3][kN][4], int n, int e) { return acc[0][n][e] + (acc[1][n][e] + acc[2][n][e]); };
   const int own_row = (matrix & 1) * 8 + in_matrix;
   constexpr int kAhead = 8;  // K steps of an operand requested at once
   const int row_tile = warp & 3;
@@ -517,9 +525,8 @@ __global__ void __launch_bounds__(kThreads) delta_scan_kernel(const DeltaPromptP
         }
       }
     }
-    float acc[kN][4];
-#pragma unroll
-    for (int n = 0; n < kN; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.0f;
+    float acc[3][kN][4];
+    clear(acc);
     for (int kk = 0; kk < steps; kk += kAhead) {
       if (kk) request(operand_of(own), kk);
 #pragma unroll
@@ -528,14 +535,15 @@ __global__ void __launch_bounds__(kThreads) delta_scan_kernel(const DeltaPromptP
     }
     if (chunk + 1 < chunks) request(operand_of(own + chunk_bytes), 0);
     if (warp < 4) {
+      float u[kN][4];
 #pragma unroll
       for (int n = 0; n < kN; ++n) {
-        acc[n][0] = v[n].x - acc[n][0];
-        acc[n][1] = v[n].y - acc[n][1];
-        acc[n][2] = v[n].z - acc[n][2];
-        acc[n][3] = v[n].w - acc[n][3];
+        u[n][0] = v[n].x - total(acc, n, 0);
+        u[n][1] = v[n].y - total(acc, n, 1);
+        u[n][2] = v[n].z - total(acc, n, 2);
+        u[n][3] = v[n].w - total(acc, n, 3);
       }
-      publish(acc, row_tile * 16, token_rows, write_leading, write_rest);
+      publish(u, row_tile * 16, token_rows, write_leading, write_rest);
     }
     __syncthreads();  // the writes are there, and every warp is done with the staged state
 #pragma unroll
@@ -551,15 +559,17 @@ __global__ void __launch_bounds__(kThreads) delta_scan_kernel(const DeltaPromptP
         decay_lo = decay[tile * 16 + g];
         decay_hi = decay[tile * 16 + g + 8];
       }
+      float added[3][kN][4];
+      clear(added);
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) multiply(added, kh[kk], kl[kk], write_leading, write_rest, kk * 16 + own_row);
 #pragma unroll
       for (int n = 0; n < kN; ++n) {
-        s[m][n][0] *= decay_lo;
-        s[m][n][1] *= decay_lo;
-        s[m][n][2] *= decay_hi;
-        s[m][n][3] *= decay_hi;
+        s[m][n][0] = fmaf(decay_lo, s[m][n][0], total(added, n, 0));
+        s[m][n][1] = fmaf(decay_lo, s[m][n][1], total(added, n, 1));
+        s[m][n][2] = fmaf(decay_hi, s[m][n][2], total(added, n, 2));
+        s[m][n][3] = fmaf(decay_hi, s[m][n][3], total(added, n, 3));
       }
-#pragma unroll
-      for (int kk = 0; kk < 4; ++kk) multiply(s[m], kh[kk], kl[kk], write_leading, write_rest, kk * 16 + own_row);
       publish(s[m], tile * 16, channel_rows, state_leading, state_rest);
     }
     if (warp >= 4) {
@@ -572,8 +582,8 @@ __global__ void __launch_bounds__(kThreads) delta_scan_kernel(const DeltaPromptP
 #pragma unroll
       for (int n = 0; n < kN; ++n) {
         if (n * 8 >= live_columns) continue;
-        if (row < o.rows) *reinterpret_cast<float2*>(out + n * 8) = make_float2(acc[n][0], acc[n][1]);
-        if (row + 8 < o.rows) *reinterpret_cast<float2*>(out + 8 * out_pitch + n * 8) = make_float2(acc[n][2], acc[n][3]);
+        if (row < o.rows) *reinterpret_cast<float2*>(out + n * 8) = make_float2(total(acc, n, 0), total(acc, n, 1));
+        if (row + 8 < o.rows) *reinterpret_cast<float2*>(out + 8 * out_pitch + n * 8) = make_float2(total(acc, n, 2), total(acc, n, 3));
       }
     }
     __syncthreads();  // the next state is there, and every warp is done with the writes

@@ -38,7 +38,13 @@ template <typename T>
 __device__ __forceinline__ float silu_for(float x) { return sizeof(T) == 2 ? x * quick_sigmoid(x) : silu_exact(x); }
 __device__ __forceinline__ float4 add(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
 __device__ __forceinline__ float softplus_value(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
-__device__ __forceinline__ float quick_softplus(float x) { return x > 20.0f ? x : log1pf(__expf(x)); }
+// ln(1 + e^x) with the fast exponential and logarithm: max(x, 0) + ln(1 + y), y = e^-|x|, and for small y the start of
+// the logarithm's series, so that no digits are lost to the 1 (relative error below 1e-5).
+__device__ __forceinline__ float quick_softplus(float x) {
+  const float y = __expf(-fabsf(x));
+  const float series = y * fmaf(y, fmaf(y, fmaf(y, fmaf(y, 0.2f, -0.25f), 1.0f / 3.0f), -0.5f), 1.0f);
+  return fmaxf(x, 0.0f) + (y < 0.0625f ? series : __logf(1.0f + y));
+}
 
 // Sum over the block; `shared` holds a value per warp and is free again after the next block-wide barrier.
 __device__ __forceinline__ float block_total(float v, float* shared) {

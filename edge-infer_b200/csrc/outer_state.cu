@@ -313,7 +313,7 @@ __device__ __forceinline__ void conv_head(const OuterStateParams& p, bf16* out, 
 }
 
 template <int kTaps>
-__global__ void __launch_bounds__(128) outer_conv_kernel(const OuterStateParams p, bf16* out, float* inverse) {
+__global__ void __launch_bounds__(128, 5) outer_conv_kernel(const OuterStateParams p, bf16* out, float* inverse) {
   const int context = p.control->context;  // written by the previous step
   grid_dependency_wait();
   grid_launch_dependents();
@@ -332,6 +332,7 @@ __global__ void __launch_bounds__(128) outer_conv_kernel(const OuterStateParams 
 // heads' padding.
 constexpr int kFinishHeld = 8;   // values a thread keeps between the two passes over a group
 constexpr int kFinishQuads = 4;  // the same, four at a time
+constexpr int kTailPiece = 128;
 template <typename T, bool kWide>
 __global__ void __launch_bounds__(256) state_finish_kernel(const StateFinishParams p) {
   __shared__ float shared[8];
@@ -340,12 +341,14 @@ __global__ void __launch_bounds__(256) state_finish_kernel(const StateFinishPara
   const int lanes = kWide ? blockDim.x : 32, lane = kWide ? threadIdx.x : threadIdx.x & 31;
   const int item = kWide ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (item >= p.rows * p.groups) {
-    // Behind them: convolution inputs into the ring.
-    const int back = item - p.rows * p.groups, r = p.rows - 1 - back, context = p.control ? p.control->context : -1;
+    // Behind them: convolution inputs into the ring, kTailPiece channels per item.
+    const int pieces = (p.channels + kTailPiece - 1) / kTailPiece, tail = item - p.rows * p.groups;
+    const int back = tail / pieces, r = p.rows - 1 - back, context = p.control ? p.control->context : -1;
     if (back >= p.tail_rows || context < 0 || context + p.rows > p.capacity) return;
     const T* from = static_cast<const T*>(p.tail) + size_t(r) * p.tail_stride;
     T* to = static_cast<T*>(p.raw) + size_t((context + r) & (p.raw_rows - 1)) * p.channels;
-    for (int i = lane * 2; i < p.channels; i += lanes * 2) {
+    const int begin = (tail - back * pieces) * kTailPiece, end = min(p.channels, begin + kTailPiece);
+    for (int i = begin + lane * 2; i < end; i += lanes * 2) {
       const float2 v = load_pair(from + i);
       store_pair(to + i, v.x, v.y);
     }
@@ -482,7 +485,7 @@ void launch_outer_step(const OuterStateParams& p, cudaStream_t stream, bool pdl)
 }
 template <typename T>
 void launch_state_finish(const StateFinishParams& p, cudaStream_t stream, bool pdl) {
-  const int items = p.rows * p.groups + p.tail_rows, length = p.heads * p.vdim / p.groups;
+  const int items = p.rows * p.groups + p.tail_rows * ((p.channels + kTailPiece - 1) / kTailPiece), length = p.heads * p.vdim / p.groups;
   if (length > 512)
     launch(state_finish_kernel<T, true>, dim3(unsigned(items)), dim3(256), 0, stream, pdl, p);
   else

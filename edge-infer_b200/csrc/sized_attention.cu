@@ -3,7 +3,7 @@
 // weights keep 16 significant bits in the product with the values (each weight is split into two BF16 terms).
 //
 // The tile loop is that of the 128-wide verify attention (attention.cu): K and V tiles of 64 tokens by TMA through a
-// ring of three stages on mbarriers with bounded block-uniform waits, scores and running sums in FP32, mma.sync on
+// ring of two or three stages on mbarriers with bounded block-uniform waits, scores and running sums in FP32, mma.sync on
 // ldmatrix fragments. What differs:
 //  * a staged tile is [piece of a head row][token][up to 128 B]; a head row of `pad` values is cut into pieces of 64,
 //    32 or 16 values, whichever divides it, each with the TMA swizzle of its width (128 / 64 / 32 bytes), so the
@@ -23,11 +23,13 @@ namespace ei {
 namespace {
 
 constexpr int kTile = 64;
-constexpr int kStages = 3;
+constexpr int kMostStages = 3;
+// Tiles in flight: two where three would keep a second block off the SM.
+constexpr int stages_for(int keys, int values) { return keys + values > 256 ? 2 : kMostStages; }
 constexpr int kMaxWarps = 4;
 
 struct SizedShared {
-  uint64_t full[kStages];
+  uint64_t full[kMostStages];
   int failed;
 };
 
@@ -38,8 +40,8 @@ __device__ __forceinline__ int staged_offset(int token, int piece, int shift) {
   return at ^ (((at >> 7) & ((1 << shift) - 1)) << 4);
 }
 
-size_t sized_shared_bytes(int dim_pad, int vdim_pad) {
-  return size_t(kStages) * kTile * (dim_pad + vdim_pad) * 2 + 1024 + 64;
+size_t sized_shared_bytes(int stages, int dim_pad, int vdim_pad) {
+  return size_t(stages) * kTile * (dim_pad + vdim_pad) * 2 + 1024 + 64;
 }
 
 // kDirect = false: block (kv head, split of the sequence, part of the stacked rows) writes (o, m, l) partials.
@@ -50,7 +52,7 @@ __global__ void __launch_bounds__(kMaxWarps * 32) sized_attention_kernel(const _
   extern __shared__ unsigned char sized_smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(sized_smem_raw) + 1023) &
                                                          ~uintptr_t(1023));
-  constexpr int kSteps = kKeys / 16, kTiles = kValues / 8;
+  constexpr int kSteps = kKeys / 16, kTiles = kValues / 8, kStages = stages_for(kKeys, kValues);
   const int dim = kExact ? kKeys : p.dim_pad, vdim = kExact ? kValues : p.vdim_pad;
   const int k_steps = dim / 16, v_tiles = vdim / 8;
   const int k_shift = kExact ? 3 : p.k_shift, v_shift = kExact ? 3 : p.v_shift;
@@ -385,7 +387,7 @@ void launch_bucket(const SizedAttentionParams& p, bool direct, cudaStream_t stre
   int device = 0;
   EI_CUDA(cudaGetDevice(&device));
   if (configured_device != device) {
-    const int bytes = int(sized_shared_bytes(kKeys, kValues));
+    const int bytes = int(sized_shared_bytes(stages_for(kKeys, kValues), kKeys, kValues));
     EI_CUDA(cudaFuncSetAttribute(sized_attention_kernel<kKeys, kValues, kExact, false>,
                                  cudaFuncAttributeMaxDynamicSharedMemorySize, bytes));
     EI_CUDA(cudaFuncSetAttribute(sized_attention_kernel<kKeys, kValues, kExact, true>,
@@ -395,7 +397,7 @@ void launch_bucket(const SizedAttentionParams& p, bool direct, cudaStream_t stre
   const int stacked = p.rows * (p.heads / p.kv_heads);
   const int warps = std::min(kMaxWarps, (stacked + 15) / 16);
   const unsigned parts = unsigned((stacked + warps * 16 - 1) / (warps * 16));
-  const size_t smem = sized_shared_bytes(p.dim_pad, p.vdim_pad);
+  const size_t smem = sized_shared_bytes(stages_for(kKeys, kValues), p.dim_pad, p.vdim_pad);
   if (direct)
     launch(sized_attention_kernel<kKeys, kValues, kExact, true>, dim3(p.kv_heads, parts), dim3(warps * 32), smem, stream, pdl, p);
   else
