@@ -67,10 +67,26 @@ __device__ __forceinline__ void store_fragment(uint4* to, float4 lo, float4 hi) 
   const float x[8] = {lo.x, lo.y, hi.x, hi.y, lo.z, lo.w, hi.z, hi.w};
   store_fragment(to, x);
 }
+// Where tokens are summed over, value e of lane c's fragment belongs to this token of the tile's 16 (of both operands).
+__device__ __forceinline__ int token_of(int c, int e) { return c + 4 * (e & 1) + 8 * (e >> 2); }
+// Its place among the operand's rows, from the token.
+__device__ __forceinline__ int token_place(int t) { return 2 * (t & 3) + ((t >> 2) & 1) + 8 * (t >> 3); }
 __device__ __forceinline__ float4 quad_at(const float* p) { return *reinterpret_cast<const float4*>(p); }
 __device__ __forceinline__ float4 times(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
-__device__ __forceinline__ float4 exp_of(float4 a) { return make_float4(__expf(a.x), __expf(a.y), __expf(a.z), __expf(a.w)); }
-__device__ __forceinline__ float4 exp_between(float4 a, float4 b) { return exp_of(make_float4(a.x - b.x, a.y - b.y, a.z - b.z, a.w - b.w)); }
+// The decays' logarithms are kept to base two.
+__device__ __forceinline__ float power_of_two(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float4 exp_of(float4 a) { return make_float4(power_of_two(a.x), power_of_two(a.y), power_of_two(a.z), power_of_two(a.w)); }
+__device__ __forceinline__ float4 minus(float4 a, float4 b) { return make_float4(a.x - b.x, a.y - b.y, a.z - b.z, a.w - b.w); }
+__device__ __forceinline__ float4 exp_between(float4 a, float4 b) { return exp_of(minus(a, b)); }
+// The same for a difference that may be above zero where the result is not used: held at zero so that it stays finite.
+__device__ __forceinline__ float4 exp_below(float4 a, float4 b) {
+  const float4 x = minus(a, b);
+  return exp_of(make_float4(fminf(x.x, 0.0f), fminf(x.y, 0.0f), fminf(x.z, 0.0f), fminf(x.w, 0.0f)));
+}
 __device__ __forceinline__ float dot(float4 a, float4 b, float sum) {
   return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, sum))));
 }
@@ -82,10 +98,9 @@ __device__ __forceinline__ void split_rows(float4 lo, float4 hi, uint32_t (&lead
   split_pair(hi.z, hi.w, leading[3], rest[3]);
 }
 
-// Sixteen warps. Warp w: part w & 3 of the key channels, and, of A and B, the diagonal block w >> 2 and one of four groups
-// of tiles below it.
+// Sixteen warps. Of A and B, warp w takes four columns of a diagonal block and, up to the twelfth, a tile below the
+// diagonal.
 constexpr int kPrepareThreads = 512;
-constexpr int kParts = 4;
 __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const DeltaPromptParams p) {
   extern __shared__ __align__(16) float chunk_smem[];
   const OuterStateParams& o = p.outer;
@@ -108,7 +123,7 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
   unsigned char* own = p.chunks + (size_t(chunk) * o.heads + head) * layout.total;
   const bf16* conv = p.conv + size_t(first) * p.channels;
   const float* inverse = p.inverse + size_t(first) * 2 * o.key_heads;
-  const float rate = o.rate[head];
+  const float rate = o.rate[head] * 1.44269504f;  // logarithms to base two
 
   if (threadIdx.x < kChunk) {
     const int t = threadIdx.x;
@@ -160,129 +175,122 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
   }
   __syncthreads();
 
-  // A and B. Every warp adds up its part of the key channels for one diagonal block, directly, and for a group of tiles of
-  // 16 rows x 8 columns below the diagonal, through the end of the block ahead of the rows; the parts are then added in
-  // order.
+  // The value columns are requested now and used after A and B.
+  float4* v_out = reinterpret_cast<float4*>(own + layout.v);
+  const bf16* values = conv + 2 * o.key_heads * dim + head * o.vdim_pad;
+  constexpr int kValueQuads = 4;  // per thread: 64 rows of 128 values
+  uint2 ahead[kValueQuads];
+  const int first_width = min(dim, o.vdim_pad), first_quads = first_width / 4;
+#pragma unroll
+  for (int n = 0; n < kValueQuads; ++n) {
+    const int i = threadIdx.x + n * kPrepareThreads, t = i / first_quads;
+    ahead[n] = make_uint2(0, 0);
+    if (t < live && t < kChunk) ahead[n] = *reinterpret_cast<const uint2*>(values + size_t(t) * p.channels + (i - t * first_quads) * 4);
+  }
+
+  // A and B inside the diagonal blocks, directly. Warp w: block w >> 2; rows g and g + 8 of it against columns
+  // 2 (w & 3), + 1, and row g + 8 against the columns eight further on.
   {
-    const int part = warp & (kParts - 1), group = warp >> 2;
-    const int kk_begin = steps * part / kParts, kk_end = steps * (part + 1) / kParts;
-    // Diagonal block `group`: rows g and g + 8 of it, columns 0..15; row g needs the first eight only.
-    float low_k[8], low_q[8], high_k[16], high_q[16];
+    const int base = (warp >> 2) * kBlock, column = base + (warp & 3) * 2;
+    const int t = base + g;
+    float ka[3][2], qa[3][2];  // [row g, early column | row g + 8, early column | row g + 8, late column]
 #pragma unroll
-    for (int j = 0; j < 8; ++j) low_k[j] = low_q[j] = 0.0f;
+    for (int n = 0; n < 3; ++n) ka[n][0] = ka[n][1] = qa[n][0] = qa[n][1] = 0.0f;
+#pragma unroll 2
+    for (int d = 4 * c; d < dim; d += 16) {
+      const float4 gl = quad_at(gs + t * pitch + d), gh = quad_at(gs + (t + 8) * pitch + d);
+      const float4 kl = quad_at(ks + t * pitch + d), kh = quad_at(ks + (t + 8) * pitch + d);
+      const float4 ql = quad_at(qs + t * pitch + d), qh = quad_at(qs + (t + 8) * pitch + d);
 #pragma unroll
-    for (int j = 0; j < 16; ++j) high_k[j] = high_q[j] = 0.0f;
-    // Below the diagonal: groups 0 and 1 hold the row block 3 (columns 0..23 and 24..47), group 2 block 2, group 3 block 1.
-    const int block = group < 2 ? 3 : group == 2 ? 2 : 1, first_column = group == 1 ? 24 : 0;
-    const int tiles = group < 2 ? 3 : group == 2 ? 4 : 2;
-    float ka[4][4], qa[4][4];
-#pragma unroll
-    for (int n = 0; n < 4; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) ka[n][e] = qa[n][e] = 0.0f;
-    for (int kk = kk_begin; kk < kk_end; ++kk) {
-      const int d = kk * 16 + 4 * c;
-      {
-        const int t = group * kBlock + g;
-        const float4 gl = quad_at(gs + t * pitch + d), gh = quad_at(gs + (t + 8) * pitch + d);
-        const float4 kl = quad_at(ks + t * pitch + d), kh = quad_at(ks + (t + 8) * pitch + d);
-        const float4 ql = quad_at(qs + t * pitch + d), qh = quad_at(qs + (t + 8) * pitch + d);
-#pragma unroll
-        for (int j = 0; j < 16; ++j) {
-          const float4 gj = quad_at(gs + (group * kBlock + j) * pitch + d), kj = quad_at(ks + (group * kBlock + j) * pitch + d);
-          // A row ahead of its column is not used; its exponent is held at zero so that it stays finite.
-          if (j < 8) {
-            const float4 x = times(kj, exp_of(make_float4(fminf(gl.x - gj.x, 0.0f), fminf(gl.y - gj.y, 0.0f), fminf(gl.z - gj.z, 0.0f),
-                                                          fminf(gl.w - gj.w, 0.0f))));
-            low_k[j & 7] = dot(kl, x, low_k[j & 7]);
-            low_q[j & 7] = dot(ql, x, low_q[j & 7]);
-          }
-          const float4 y = times(kj, exp_of(make_float4(fminf(gh.x - gj.x, 0.0f), fminf(gh.y - gj.y, 0.0f), fminf(gh.z - gj.z, 0.0f),
-                                                        fminf(gh.w - gj.w, 0.0f))));
-          high_k[j] = dot(kh, y, high_k[j]);
-          high_q[j] = dot(qh, y, high_q[j]);
-        }
-      }
-      const int t0 = block * kBlock;
-      const float4 turn = quad_at(gs + (t0 - 1) * pitch + d);
-      uint32_t kh[4], kl[4], qh[4], ql[4];
-      {
-        const float4 e_lo = exp_between(quad_at(gs + (t0 + g) * pitch + d), turn), e_hi = exp_between(quad_at(gs + (t0 + g + 8) * pitch + d), turn);
-        split_rows(times(quad_at(ks + (t0 + g) * pitch + d), e_lo), times(quad_at(ks + (t0 + g + 8) * pitch + d), e_hi), kh, kl);
-        split_rows(times(quad_at(qs + (t0 + g) * pitch + d), e_lo), times(quad_at(qs + (t0 + g + 8) * pitch + d), e_hi), qh, ql);
-      }
-#pragma unroll
-      for (int n = 0; n < 4; ++n) {
-        if (n < tiles) {
-          const int j = first_column + n * 8 + g;
-          const float4 x = times(quad_at(ks + j * pitch + d), exp_between(turn, quad_at(gs + j * pitch + d)));
-          uint32_t bh[2], bl[2];
-          split_pair(x.x, x.y, bh[0], bl[0]);
-          split_pair(x.z, x.w, bh[1], bl[1]);
-          mma_bf16_16816(ka[n], kh[0], kh[1], kh[2], kh[3], bh[0], bh[1]);
-          mma_bf16_16816(qa[n], qh[0], qh[1], qh[2], qh[3], bh[0], bh[1]);
-          mma_bf16_16816(ka[n], kh[0], kh[1], kh[2], kh[3], bl[0], bl[1]);
-          mma_bf16_16816(qa[n], qh[0], qh[1], qh[2], qh[3], bl[0], bl[1]);
-          mma_bf16_16816(ka[n], kl[0], kl[1], kl[2], kl[3], bh[0], bh[1]);
-          mma_bf16_16816(qa[n], ql[0], ql[1], ql[2], ql[3], bh[0], bh[1]);
-        }
+      for (int e = 0; e < 2; ++e) {
+        const float4 early_g = quad_at(gs + (column + e) * pitch + d), early_k = quad_at(ks + (column + e) * pitch + d);
+        const float4 late_g = quad_at(gs + (column + e + 8) * pitch + d), late_k = quad_at(ks + (column + e + 8) * pitch + d);
+        const float4 x = times(early_k, exp_below(gl, early_g)), y = times(early_k, exp_between(gh, early_g)), z = times(late_k, exp_below(gh, late_g));
+        ka[0][e] = dot(kl, x, ka[0][e]);
+        qa[0][e] = dot(ql, x, qa[0][e]);
+        ka[1][e] = dot(kh, y, ka[1][e]);
+        qa[1][e] = dot(qh, y, qa[1][e]);
+        ka[2][e] = dot(kh, z, ka[2][e]);
+        qa[2][e] = dot(qh, z, qa[2][e]);
       }
     }
-    auto across = [](float x) {
-      x += __shfl_xor_sync(0xffffffffu, x, 1);
-      return x + __shfl_xor_sync(0xffffffffu, x, 2);
-    };
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      low_k[j] = across(low_k[j]);
-      low_q[j] = across(low_q[j]);
-    }
+    for (int n = 0; n < 3; ++n)
 #pragma unroll
-    for (int j = 0; j < 16; ++j) {
-      high_k[j] = across(high_k[j]);
-      high_q[j] = across(high_q[j]);
-    }
-    for (int turn_of = 0; turn_of < kParts; ++turn_of) {
-      if (part == turn_of) {
-        auto put = [&](int t, int j, float k_value, float q_value) {
-          float &a = at[j * kPitchA + t], &b = bm[t * kPitchB + j];
-          a = part ? a + k_value * beta[t] : k_value * beta[t];
-          b = part ? b + q_value : q_value;
-        };
-#pragma unroll
-        for (int j = 0; j < 16; ++j) {
-          if ((j & 3) != c) continue;  // the four lanes of a row hold the same sums and share the columns
-          const int t = group * kBlock + g, column = group * kBlock + j;
-          const bool low = j < 8 && j <= g, high = j <= g + 8;
-          put(t, column, low && j < g ? low_k[j & 7] : 0.0f, low ? low_q[j & 7] : 0.0f);
-          put(t + 8, column, high && j < g + 8 ? high_k[j] : 0.0f, high ? high_q[j] : 0.0f);
-        }
-#pragma unroll
-        for (int n = 0; n < 4; ++n)
-          if (n < tiles)
-#pragma unroll
-            for (int e = 0; e < 4; ++e)
-              put(block * kBlock + g + (e >> 1) * 8, first_column + n * 8 + 2 * c + (e & 1), ka[n][e], qa[n][e]);
+      for (int e = 0; e < 2; ++e) {
+        ka[n][e] += __shfl_xor_sync(0xffffffffu, ka[n][e], 1);
+        ka[n][e] += __shfl_xor_sync(0xffffffffu, ka[n][e], 2);
+        qa[n][e] += __shfl_xor_sync(0xffffffffu, qa[n][e], 1);
+        qa[n][e] += __shfl_xor_sync(0xffffffffu, qa[n][e], 2);
       }
-      __syncthreads();
+    if (c < 2) {  // the four lanes of a row hold the same sums; lane c writes column + c
+      const int e = c, early = column + e, late = early + 8;
+      const float ka0 = e ? ka[0][1] : ka[0][0], ka1 = e ? ka[1][1] : ka[1][0], ka2 = e ? ka[2][1] : ka[2][0];
+      const float qa0 = e ? qa[0][1] : qa[0][0], qa1 = e ? qa[1][1] : qa[1][0], qa2 = e ? qa[2][1] : qa[2][0];
+      at[early * kPitchA + t] = early < t ? ka0 * beta[t] : 0.0f;
+      bm[t * kPitchB + early] = early <= t ? qa0 : 0.0f;
+      at[early * kPitchA + t + 8] = ka1 * beta[t + 8];
+      bm[(t + 8) * kPitchB + early] = qa1;
+      at[late * kPitchA + t + 8] = late < t + 8 ? ka2 * beta[t + 8] : 0.0f;
+      bm[(t + 8) * kPitchB + late] = late <= t + 8 ? qa2 : 0.0f;
+    } else if (c == 2) {
+      for (int e = 0; e < 2; ++e) {
+        at[(column + 8 + e) * kPitchA + t] = 0.0f;
+        bm[t * kPitchB + column + 8 + e] = 0.0f;
+      }
     }
   }
+  // Below the diagonal: tiles of 16 rows x 8 columns, through the end of the block ahead of the rows.
+  if (warp < 12) {
+    const int block = warp < 2 ? 1 : warp < 6 ? 2 : 3, column = (warp - (block == 1 ? 0 : block == 2 ? 2 : 6)) * 8;
+    const int t0 = block * kBlock;
+    float ka[3][4], qa[3][4];  // a chain per product of terms
+#pragma unroll
+    for (int n = 0; n < 3; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ka[n][e] = qa[n][e] = 0.0f;
+#pragma unroll 2
+    for (int d = 4 * c; d < dim; d += 16) {
+      const float4 turn = quad_at(gs + (t0 - 1) * pitch + d);
+      const float4 e_lo = exp_between(quad_at(gs + (t0 + g) * pitch + d), turn), e_hi = exp_between(quad_at(gs + (t0 + g + 8) * pitch + d), turn);
+      uint32_t kh[4], kl[4], qh[4], ql[4], bh[2], bl[2];
+      split_rows(times(quad_at(ks + (t0 + g) * pitch + d), e_lo), times(quad_at(ks + (t0 + g + 8) * pitch + d), e_hi), kh, kl);
+      split_rows(times(quad_at(qs + (t0 + g) * pitch + d), e_lo), times(quad_at(qs + (t0 + g + 8) * pitch + d), e_hi), qh, ql);
+      const float4 x = times(quad_at(ks + (column + g) * pitch + d), exp_between(turn, quad_at(gs + (column + g) * pitch + d)));
+      split_pair(x.x, x.y, bh[0], bl[0]);
+      split_pair(x.z, x.w, bh[1], bl[1]);
+      mma_bf16_16816(ka[0], kh[0], kh[1], kh[2], kh[3], bh[0], bh[1]);
+      mma_bf16_16816(qa[0], qh[0], qh[1], qh[2], qh[3], bh[0], bh[1]);
+      mma_bf16_16816(ka[1], kh[0], kh[1], kh[2], kh[3], bl[0], bl[1]);
+      mma_bf16_16816(qa[1], qh[0], qh[1], qh[2], qh[3], bl[0], bl[1]);
+      mma_bf16_16816(ka[2], kl[0], kl[1], kl[2], kl[3], bh[0], bh[1]);
+      mma_bf16_16816(qa[2], ql[0], ql[1], ql[2], ql[3], bh[0], bh[1]);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int t = t0 + g + (e >> 1) * 8, j = column + 2 * c + (e & 1);
+      at[j * kPitchA + t] = (ka[0][e] + (ka[1][e] + ka[2][e])) * beta[t];
+      bm[t * kPitchB + j] = qa[0][e] + (qa[1][e] + qa[2][e]);
+    }
+  }
+  __syncthreads();
 
   // Operands that need no solving: q e^G, k e^(G_end - G) transposed, B, and the chunk's decay.
   const float* last = gs + (kChunk - 1) * pitch;
   uint4* q_out = reinterpret_cast<uint4*>(own + layout.q);
   uint4* k_out = reinterpret_cast<uint4*>(own + layout.k);
   uint4* b_out = reinterpret_cast<uint4*>(own + layout.b);
+#pragma unroll 2
   for (int tile = warp; tile < 4 * steps; tile += kWarps) {
     const int mt = tile / steps, kk = tile - mt * steps;
     const int row = (mt * 16 + g) * pitch + kk * 16 + 4 * c;
     store_fragment(q_out + size_t(mt * steps + kk) * 64 + lane, times(quad_at(qs + row), exp_of(quad_at(gs + row))),
                    times(quad_at(qs + row + 8 * pitch), exp_of(quad_at(gs + row + 8 * pitch))));
-    float y[8];  // tile (kk, mt) of the transpose: rows are key channels, columns tokens
+    float y[8];  // tile (kk, mt) of the transpose: rows are key channels, columns tokens in the order of token_of
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
-      const int token = mt * 16 + 2 * c + (e & 1) + (e >> 2) * 8, channel = kk * 16 + g + ((e >> 1) & 1) * 8;
-      y[e] = ks[token * pitch + channel] * __expf(last[channel] - gs[token * pitch + channel]);
+      const int token = mt * 16 + token_of(c, e), channel = kk * 16 + g + ((e >> 1) & 1) * 8;
+      y[e] = ks[token * pitch + channel] * power_of_two(last[channel] - gs[token * pitch + channel]);
     }
     store_fragment(k_out + size_t(kk * 4 + mt) * 64 + lane, y);
   }
@@ -292,62 +300,99 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
     float x[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e)
-      x[e] = bm[(mt * 16 + g + ((e >> 1) & 1) * 8) * kPitchB + kk * 16 + 2 * c + (e & 1) + (e >> 2) * 8];
+      x[e] = bm[(mt * 16 + g + ((e >> 1) & 1) * 8) * kPitchB + kk * 16 + token_of(c, e)];
     store_fragment(b_out + size_t(tile) * 64 + lane, x);
   }
-  for (int d = threadIdx.x; d < dim; d += kPrepareThreads) reinterpret_cast<float*>(own + layout.decay)[d] = __expf(last[d]);
+  for (int d = threadIdx.x; d < dim; d += kPrepareThreads) reinterpret_cast<float*>(own + layout.decay)[d] = power_of_two(last[d]);
   __syncthreads();
 
-  // Solves (I + diag(b) A) X = right-hand side for one column in place, 16 rows at a time.
-  auto solve = [&](float* column) {
+  // The inverses of the four unit lower triangular diagonal blocks, one column per thread, into the blocks' places in bm
+  // (B has been written out): inverse[i][j] at bm[(16 b + i) pitch + 16 b + j].
+  if (threadIdx.x < kChunk) {
+    const int base = threadIdx.x & ~(kBlock - 1), j = threadIdx.x & (kBlock - 1);
+    float x[kBlock];
+#pragma unroll
+    for (int i = 0; i < kBlock; ++i) x[i] = i == j ? 1.0f : 0.0f;
+#pragma unroll
+    for (int m = 0; m < kBlock - 1; ++m)
+#pragma unroll
+      for (int i = m + 1; i < kBlock; ++i) x[i] = fmaf(-at[(base + m) * kPitchA + base + i], x[m], x[i]);
+#pragma unroll
+    for (int i = 0; i < kBlock; ++i) bm[(base + i) * kPitchB + base + j] = x[i];
+  }
+  // Solves (I + diag(b) A) X = right-hand side in place, 16 rows at a time. Lanes l and l + 16 share a column: lane
+  // l + 16 h works on the rows 8 h .. 8 h + 7 of a block for the part below the diagonal blocks, and on every second row
+  // for the product with the block's inverse.
+  const int half = lane >> 4;
+  auto solve = [&](float* column, bool live_column) {
 #pragma unroll 1
     for (int b = 0; b < kChunk / kBlock; ++b) {
-      float x[kBlock];
+      float x[8];
+      float* own_rows = column + (b * kBlock + half * 8) * pitch;
+      if (live_column && b) {
 #pragma unroll
-      for (int i = 0; i < kBlock; ++i) x[i] = column[(b * kBlock + i) * pitch];
+        for (int i = 0; i < 8; ++i) x[i] = own_rows[i * pitch];
 #pragma unroll 4
-      for (int j = 0; j < b * kBlock; ++j) {
-        const float known = column[j * pitch];
-        const float* a = at + j * kPitchA + b * kBlock;
+        for (int j = 0; j < b * kBlock; ++j) {
+          const float known = column[j * pitch];
+          const float* a = at + j * kPitchA + b * kBlock + half * 8;
+          const float4 v = quad_at(a), w = quad_at(a + 4);
+          x[0] = fmaf(-v.x, known, x[0]);
+          x[1] = fmaf(-v.y, known, x[1]);
+          x[2] = fmaf(-v.z, known, x[2]);
+          x[3] = fmaf(-v.w, known, x[3]);
+          x[4] = fmaf(-w.x, known, x[4]);
+          x[5] = fmaf(-w.y, known, x[5]);
+          x[6] = fmaf(-w.z, known, x[6]);
+          x[7] = fmaf(-w.w, known, x[7]);
+        }
 #pragma unroll
-        for (int i = 0; i < kBlock; i += 4) {
-          const float4 v = quad_at(a + i);
-          x[i] = fmaf(-v.x, known, x[i]);
-          x[i + 1] = fmaf(-v.y, known, x[i + 1]);
-          x[i + 2] = fmaf(-v.z, known, x[i + 2]);
-          x[i + 3] = fmaf(-v.w, known, x[i + 3]);
+        for (int i = 0; i < 8; ++i) own_rows[i * pitch] = x[i];
+      }
+      __syncwarp();
+      float r[kBlock];
+      if (live_column) {
+#pragma unroll
+        for (int i = 0; i < kBlock; ++i) r[i] = column[(b * kBlock + i) * pitch];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const float* t = bm + (b * kBlock + 2 * i + half) * kPitchB + b * kBlock;
+          float sum = 0.0f;
+#pragma unroll
+          for (int j = 0; j < 2 * i + 2; ++j) sum = fmaf(t[j], r[j], sum);  // row 2 i has a zero at its end
+          x[i] = sum;
         }
       }
+      __syncwarp();
+      if (live_column)
 #pragma unroll
-      for (int j = 0; j < kBlock - 1; ++j) {
-        const float* a = at + (b * kBlock + j) * kPitchA + b * kBlock;
-#pragma unroll
-        for (int i = (j + 1) & ~3; i < kBlock; i += 4) {
-          const float4 v = quad_at(a + i);  // zero up to the diagonal
-          x[i] = i > j ? fmaf(-v.x, x[j], x[i]) : x[i];
-          x[i + 1] = i + 1 > j ? fmaf(-v.y, x[j], x[i + 1]) : x[i + 1];
-          x[i + 2] = i + 2 > j ? fmaf(-v.z, x[j], x[i + 2]) : x[i + 2];
-          x[i + 3] = i + 3 > j ? fmaf(-v.w, x[j], x[i + 3]) : x[i + 3];
-        }
-      }
-#pragma unroll
-      for (int i = 0; i < kBlock; ++i) column[(b * kBlock + i) * pitch] = x[i];
+        for (int i = 0; i < 8; ++i) column[(b * kBlock + 2 * i + half) * pitch] = x[i];
+      __syncwarp();
     }
   };
   // The columns of W in place of k, those of V' in place of q, `dim` value columns at a time.
-  float4* v_out = reinterpret_cast<float4*>(own + layout.v);
-  const bf16* values = conv + 2 * o.key_heads * dim + head * o.vdim_pad;
   for (int v0 = 0; v0 < o.vdim_pad; v0 += dim) {
     const int width = min(dim, o.vdim_pad - v0), width_quads = width / 4;
-    for (int i = threadIdx.x; i < kChunk * width_quads; i += kPrepareThreads) {
+    auto put_value = [&](int i, uint2 raw) {
       const int t = i / width_quads, d = (i - t * width_quads) * 4;
-      const float4 v = t < live ? load_quad(values + size_t(t) * p.channels + v0 + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
       const float b = beta[t];
-      *reinterpret_cast<float4*>(qs + t * pitch + d) = make_float4(v.x * b, v.y * b, v.z * b, v.w * b);
-    }
+      *reinterpret_cast<float4*>(qs + t * pitch + d) = make_float4(bf16_lo(raw.x) * b, bf16_hi(raw.x) * b, bf16_lo(raw.y) * b, bf16_hi(raw.y) * b);
+    };
+    auto fetch_value = [&](int i) {
+      const int t = i / width_quads, d = (i - t * width_quads) * 4;
+      return t < live ? *reinterpret_cast<const uint2*>(values + size_t(t) * p.channels + v0 + d) : make_uint2(0, 0);
+    };
+    int i = threadIdx.x;
     if (v0 == 0) {
-      for (int i = threadIdx.x; i < kChunk * quads; i += kPrepareThreads) {
-        const int t = i / quads, d = (i - t * quads) * 4;
+#pragma unroll
+      for (int n = 0; n < kValueQuads; ++n, i += kPrepareThreads)
+        if (i < kChunk * width_quads) put_value(i, ahead[n]);
+    }
+    for (; i < kChunk * width_quads; i += kPrepareThreads) put_value(i, fetch_value(i));
+    if (v0 == 0) {
+#pragma unroll 4
+      for (int n = threadIdx.x; n < kChunk * quads; n += kPrepareThreads) {
+        const int t = n / quads, d = (n - t * quads) * 4;
         const float4 e = exp_of(quad_at(gs + t * pitch + d));
         const float b = beta[t];
         float4* k = reinterpret_cast<float4*>(ks + t * pitch + d);
@@ -356,8 +401,10 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
     }
     __syncthreads();
     const int unsolved = v0 == 0 ? dim : 0;  // columns of W still to come, ahead of the value columns
-    for (int column = threadIdx.x; column < unsolved + width; column += kPrepareThreads)
-      solve(column < unsolved ? ks + column : qs + column - unsolved);
+    for (int begin = warp * 16; begin < unsolved + width; begin += kWarps * 16) {
+      const int column = begin + (lane & 15);
+      solve(column < unsolved ? ks + column : qs + column - unsolved, column < unsolved + width);
+    }
     __syncthreads();
     // V' in the order of the accumulators: [row tile][column tile of 8][lane].
     for (int tile = warp; tile < 4 * (width / 8); tile += kWarps) {
@@ -365,7 +412,7 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
       const float* x = qs + (mt * 16 + g) * pitch + nt * 8 + 2 * c;
       v_out[(size_t(mt) * (o.vdim_pad / 8) + v0 / 8 + nt) * 32 + lane] = make_float4(x[0], x[1], x[8 * pitch], x[8 * pitch + 1]);
     }
-    __syncthreads();
+    if (v0 + dim < o.vdim_pad) __syncthreads();
   }
   uint4* w_out = reinterpret_cast<uint4*>(own + layout.w);
   for (int tile = warp; tile < 4 * steps; tile += kWarps) {
@@ -431,8 +478,9 @@ __global__ void __launch_bounds__(kThreads) delta_scan_kernel(const DeltaPromptP
       }
     }
   }
-  // Accumulator rows into the two terms of an operand; key channels of a tile in the order of store_fragment's quads.
-  const int token_rows[2] = {g, g + 8};
+  // Accumulator rows into the two terms of an operand; tokens in the order of token_of, key channels of a tile in the order
+  // of store_fragment's quads.
+  const int token_rows[2] = {token_place(g), token_place(g + 8)};
   const int channel_rows[2] = {(g >> 2) * 2 + (g & 1) + ((g >> 1) & 1) * 8, ((g >> 2) + 2) * 2 + (g & 1) + ((g >> 1) & 1) * 8};
   auto publish = [&](const float (&x)[kN][4], int row, const int (&places)[2], bf16* leading, bf16* rest) {
 #pragma unroll
