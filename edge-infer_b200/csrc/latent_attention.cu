@@ -85,7 +85,7 @@ __device__ __forceinline__ void query_quad(const LatentParams& p, bool step, int
 // query parts, four values per thread.
 constexpr int kPrepareThreads = 256;
 constexpr int kAhead = 16;  // rows of the expansion a warp requests before waiting
-template <typename T>
+template <typename T, int kRows>
 __global__ void __launch_bounds__(kPrepareThreads) latent_prepare_kernel(const LatentParams p, int absorbing) {
   extern __shared__ __align__(16) unsigned char prepare_smem[];
   float2* parts = reinterpret_cast<float2*>(prepare_smem);                  // [8][rows][32]
@@ -123,12 +123,12 @@ __global__ void __launch_bounds__(kPrepareThreads) latent_prepare_kernel(const L
   for (int i = threadIdx.x; i < p.rows * p.dim_pad; i += kPrepareThreads)
     query[i] = value_of(q[size_t(i / p.dim_pad) * p.stride + i % p.dim_pad]);
   __syncthreads();
-  float2 acc[kMaxRows];
+  float2 acc[kRows];
 #pragma unroll
-  for (int r = 0; r < kMaxRows; ++r) acc[r] = make_float2(0.0f, 0.0f);
+  for (int r = 0; r < kRows; ++r) acc[r] = make_float2(0.0f, 0.0f);
   auto absorb = [&](int d, float2 w) {
 #pragma unroll
-    for (int r = 0; r < kMaxRows; ++r) {
+    for (int r = 0; r < kRows; ++r) {
       if (r < p.rows) {
         acc[r].x = fmaf(query[r * p.dim_pad + d], w.x, acc[r].x);
         acc[r].y = fmaf(query[r * p.dim_pad + d], w.y, acc[r].y);
@@ -140,7 +140,7 @@ __global__ void __launch_bounds__(kPrepareThreads) latent_prepare_kernel(const L
     if (warp + 8 * i < p.dim_pad) absorb(warp + 8 * i, held[i]);
   for (int d = warp + 8 * kAhead; d < p.dim_pad; d += 8) absorb(d, load_pair(weights + size_t(d) * p.rank_pad));
 #pragma unroll
-  for (int r = 0; r < kMaxRows; ++r)
+  for (int r = 0; r < kRows; ++r)
     if (r < p.rows) parts[(warp * p.rows + r) * 32 + lane] = acc[r];
   __syncthreads();
   for (int i = threadIdx.x; i < p.rows * 32; i += kPrepareThreads) {
@@ -178,13 +178,12 @@ size_t latent_shared_bytes(int row_pad, int stages) {
          sizeof(LatentShared) + 1024;
 }
 
-// Block (split of the sequence, 16 (row, head) pairs). kWarps warps share the tile: each scores kTile / kWarps tokens
-// for all 16 pairs, then sums every kWarps-th 16-value column of the latents.
-template <int kWarps>
+// Block (split of the sequence, 16 (row, head) pairs). Eight warps share the tile: each scores eight tokens for all 16
+// pairs, then sums every eighth 16-value column of the latents, kColumns at most.
+constexpr int kWarps = 8;
+template <int kColumns>
 __global__ void __launch_bounds__(kWarps * 32) latent_attention_kernel(const __grid_constant__ SizedAttentionParams p, int row_pad,
                                                                        int stages) {
-  constexpr int kOwn = kTile / kWarps / 8;  // tiles of eight tokens per warp: 2 or 1
-  constexpr int kColumns = 8;               // 16-value columns per warp
   extern __shared__ unsigned char latent_smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(latent_smem_raw) + 1023) & ~uintptr_t(1023));
   const int stage_bytes = kTile * row_pad * 2, query_pitch = row_pad + 8;
@@ -259,30 +258,25 @@ __global__ void __launch_bounds__(kWarps * 32) latent_attention_kernel(const __g
         *reinterpret_cast<uint4*>(rows + staged_offset(live + i / pieces, i % pieces)) = make_uint4(0, 0, 0, 0);
       __syncthreads();
     }
-    float s[kOwn][4];
-#pragma unroll
-    for (int j = 0; j < kOwn; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
+    float s[4], other[4];  // even and odd k-steps: two chains
+    s[0] = s[1] = s[2] = s[3] = other[0] = other[1] = other[2] = other[3] = 0.0f;
 #pragma unroll 4
-    for (int kk = 0; kk < steps; ++kk) {
+    for (int kk = 0; kk < steps; kk += 2) {  // a row has an even number of k-steps
       uint32_t a0, a1, a2, a3, b0, b1, b2, b3;
+      ldmatrix_x4(b0, b1, b2, b3, rows + staged_offset(warp * 8 + in_matrix, 2 * kk + matrix));
       ldmatrix_x4(a0, a1, a2, a3, query + ((matrix & 1) * 8 + in_matrix) * query_pitch + kk * 16 + (matrix >> 1) * 8);
-      // Fragments of this k-step for up to two tiles of eight tokens; with one, the second pair repeats it.
-      const int token = (warp * kOwn + (kOwn == 2 ? matrix >> 1 : 0)) * 8 + in_matrix;
-      ldmatrix_x4(b0, b1, b2, b3, rows + staged_offset(token, 2 * kk + (matrix & 1)));
-      mma_bf16_16816(s[0], a0, a1, a2, a3, b0, b1);
-      if (kOwn == 2) mma_bf16_16816(s[kOwn - 1], a0, a1, a2, a3, b2, b3);
+      mma_bf16_16816(s, a0, a1, a2, a3, b0, b1);
+      ldmatrix_x4(a0, a1, a2, a3, query + ((matrix & 1) * 8 + in_matrix) * query_pitch + (kk + 1) * 16 + (matrix >> 1) * 8);
+      mma_bf16_16816(other, a0, a1, a2, a3, b2, b3);
     }
-    float top_lo = -INFINITY, top_hi = -INFINITY;
-#pragma unroll
-    for (int j = 0; j < kOwn; ++j) {
-      const int t0 = first + (warp * kOwn + j) * 8 + 2 * c, t1 = t0 + 1;
-      s[j][0] = t0 <= limit_lo ? s[j][0] * p.scale : -INFINITY;
-      s[j][1] = t1 <= limit_lo ? s[j][1] * p.scale : -INFINITY;
-      s[j][2] = t0 <= limit_hi ? s[j][2] * p.scale : -INFINITY;
-      s[j][3] = t1 <= limit_hi ? s[j][3] * p.scale : -INFINITY;
-      top_lo = fmaxf(top_lo, fmaxf(s[j][0], s[j][1]));
-      top_hi = fmaxf(top_hi, fmaxf(s[j][2], s[j][3]));
-    }
+    float top_lo, top_hi;
+    const int t0 = first + warp * 8 + 2 * c, t1 = t0 + 1;
+    s[0] = t0 <= limit_lo ? (s[0] + other[0]) * p.scale : -INFINITY;
+    s[1] = t1 <= limit_lo ? (s[1] + other[1]) * p.scale : -INFINITY;
+    s[2] = t0 <= limit_hi ? (s[2] + other[2]) * p.scale : -INFINITY;
+    s[3] = t1 <= limit_hi ? (s[3] + other[3]) * p.scale : -INFINITY;
+    top_lo = fmaxf(s[0], s[1]);
+    top_hi = fmaxf(s[2], s[3]);
 #pragma unroll
     for (int d = 1; d <= 2; d <<= 1) {
       top_lo = fmaxf(top_lo, __shfl_xor_sync(0xffffffffu, top_lo, d));
@@ -303,14 +297,10 @@ __global__ void __launch_bounds__(kWarps * 32) latent_attention_kernel(const __g
     const float rescale_lo = __expf(m_lo - base_lo), rescale_hi = __expf(m_hi - base_hi);
     m_lo = new_lo;
     m_hi = new_hi;
-    float sum_lo = 0.0f, sum_hi = 0.0f;
-#pragma unroll
-    for (int j = 0; j < kOwn; ++j) {
-      const float p0 = __expf(s[j][0] - base_lo), p1 = __expf(s[j][1] - base_lo);
-      const float p2 = __expf(s[j][2] - base_hi), p3 = __expf(s[j][3] - base_hi);
-      sum_lo += p0 + p1;
-      sum_hi += p2 + p3;
-      const int at = (warp * kOwn + j) * 8 + 2 * c;
+    const float p0 = __expf(s[0] - base_lo), p1 = __expf(s[1] - base_lo);
+    const float p2 = __expf(s[2] - base_hi), p3 = __expf(s[3] - base_hi);
+    {
+      const int at = warp * 8 + 2 * c;
       uint32_t hi, lo;
       split_pair(p0, p1, hi, lo);
       *reinterpret_cast<uint32_t*>(leading + g * kWeightPitch + at) = hi;
@@ -319,8 +309,8 @@ __global__ void __launch_bounds__(kWarps * 32) latent_attention_kernel(const __g
       *reinterpret_cast<uint32_t*>(leading + (g + 8) * kWeightPitch + at) = hi;
       *reinterpret_cast<uint32_t*>(rest + (g + 8) * kWeightPitch + at) = lo;
     }
-    l_lo = l_lo * rescale_lo + sum_lo;
-    l_hi = l_hi * rescale_hi + sum_hi;
+    l_lo = l_lo * rescale_lo + (p0 + p1);
+    l_hi = l_hi * rescale_hi + (p2 + p3);
 #pragma unroll
     for (int j = 0; j < kColumns; ++j)
 #pragma unroll
@@ -513,37 +503,46 @@ __global__ void __launch_bounds__(kExpandThreads) latent_expand_kernel(const Lat
 
 int latent_stages(int row_pad, size_t smem_limit) { return latent_shared_bytes(row_pad, 2) <= smem_limit ? 2 : 1; }
 
-template <int kWarps>
-void launch_latent_warps(const SizedAttentionParams& p, int row_pad, size_t smem_limit, cudaStream_t stream, bool pdl) {
+template <int kColumns>
+void launch_latent_columns(const SizedAttentionParams& p, int row_pad, size_t smem_limit, cudaStream_t stream, bool pdl) {
   static thread_local int configured_device = -1;
   int device = 0;
   EI_CUDA(cudaGetDevice(&device));
   if (configured_device != device) {
-    EI_CUDA(cudaFuncSetAttribute(latent_attention_kernel<kWarps>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem_limit) - 1024));
+    EI_CUDA(cudaFuncSetAttribute(latent_attention_kernel<kColumns>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem_limit) - 1024));
     configured_device = device;
   }
   const int stages = latent_stages(row_pad, smem_limit - 1024);
-  launch(latent_attention_kernel<kWarps>, dim3(unsigned(p.max_splits), unsigned((p.rows * p.heads + 15) / 16)), dim3(kWarps * 32),
+  launch(latent_attention_kernel<kColumns>, dim3(unsigned(p.max_splits), unsigned((p.rows * p.heads + 15) / 16)), dim3(kWarps * 32),
          latent_shared_bytes(row_pad, stages), stream, pdl, p, row_pad, stages);
 }
 
 }  // namespace
 
-template <typename T>
-void launch_latent_prepare(const LatentParams& p, bool step, cudaStream_t stream, bool pdl) {
-  if (step && (p.rows > kMaxRows || p.dim_pad > kMaxHeadDim)) throw std::invalid_argument("a latent attention step takes 1..16 rows");
+namespace {
+template <typename T, int kRows>
+void launch_prepare_rows(const LatentParams& p, bool step, cudaStream_t stream, bool pdl) {
   static thread_local int configured_device = -1;
   int device = 0;
   EI_CUDA(cudaGetDevice(&device));
   if (configured_device != device) {
-    EI_CUDA(cudaFuncSetAttribute(latent_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxRows * (kMaxHeadDim * 4 + 2048)));
+    EI_CUDA(cudaFuncSetAttribute(latent_prepare_kernel<T, kRows>, cudaFuncAttributeMaxDynamicSharedMemorySize, kRows * (kMaxHeadDim * 4 + 2048)));
     configured_device = device;
   }
   const int absorbing = step ? p.heads * (p.rank_pad / 64) : 0;
   const size_t smem = step ? size_t(p.rows) * (p.dim_pad * 4 + 2048) : 0;
   const int quads = (step ? p.row_pad - p.rank_pad : p.rot_pad) / 4;
   const int blocks = absorbing + (p.rows + 7) / 8 + (p.rows * p.heads * quads + kPrepareThreads - 1) / kPrepareThreads;
-  launch(latent_prepare_kernel<T>, dim3(unsigned(blocks)), dim3(kPrepareThreads), smem, stream, pdl, p, absorbing);
+  launch(latent_prepare_kernel<T, kRows>, dim3(unsigned(blocks)), dim3(kPrepareThreads), smem, stream, pdl, p, absorbing);
+}
+}  // namespace
+
+template <typename T>
+void launch_latent_prepare(const LatentParams& p, bool step, cudaStream_t stream, bool pdl) {
+  if (step && (p.rows > kMaxRows || p.dim_pad > kMaxHeadDim)) throw std::invalid_argument("a latent attention step takes 1..16 rows");
+  if (!step || p.rows == 1) return launch_prepare_rows<T, 1>(p, step, stream, pdl);
+  if (p.rows <= 4) return launch_prepare_rows<T, 4>(p, step, stream, pdl);
+  launch_prepare_rows<T, kMaxRows>(p, step, stream, pdl);
 }
 
 bool latent_attention_ok(int rank_pad, int row_pad, size_t smem_limit) {
@@ -558,9 +557,9 @@ void launch_latent_attention(const SizedAttentionParams& given, int row_pad, siz
   const cuuint32_t box[3] = {64, kTile, cuuint32_t(row_pad / 64)};
   encode_map(&p.k_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, p.k, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B, "latent cache");
   if (p.vdim_pad <= 512)
-    launch_latent_warps<4>(p, row_pad, smem_limit, stream, pdl);
+    launch_latent_columns<4>(p, row_pad, smem_limit, stream, pdl);
   else
-    launch_latent_warps<8>(p, row_pad, smem_limit, stream, pdl);
+    launch_latent_columns<8>(p, row_pad, smem_limit, stream, pdl);
 }
 
 template <typename T>

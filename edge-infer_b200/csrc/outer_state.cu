@@ -56,11 +56,11 @@ __global__ void __launch_bounds__(128) outer_prepare_kernel(const OuterStatePara
     grid_dependency_wait();
     grid_launch_dependents();
     if (!runs) return;
-    float values[kMaxHeadDim / 32], squares = 0.0f;
-#pragma unroll
-    for (int chunk = 0; chunk < kMaxHeadDim; chunk += 32 * kStrips) {
-      if (chunk >= pad) break;
-      if (chunk) settled(chunk);
+    float* to = kind == 0 ? p.q + size_t(row) * p.key_heads * p.dim_pad + head * pad
+                : kind == 1 ? p.ring_k + size_t(slot) * p.key_heads * p.dim_pad + head * pad
+                            : p.v + size_t(row) * p.heads * p.vdim_pad + head * pad;
+    float values[kStrips], squares = 0.0f;
+    auto convolve = [&](int chunk) {
 #pragma unroll
       for (int j = 0; j < kStrips; ++j) {
         const int c = chunk + lane + 32 * j;
@@ -85,21 +85,29 @@ __global__ void __launch_bounds__(128) outer_prepare_kernel(const OuterStatePara
           }
           raw[size_t(position & (p.raw_rows - 1)) * channels + channel] = own;
         }
-        const float y = c < pad ? silu_for<T>(sum) : 0.0f;
-        values[chunk / 32 + j] = y;
-        squares = fmaf(y, y, squares);
+        values[j] = c < pad ? silu_for<T>(sum) : 0.0f;
+        squares = fmaf(values[j], values[j], squares);
       }
+    };
+    // Heads wider than the strips in flight: the rest is stored as it is and scaled once the length is known.
+#pragma unroll 1
+    for (int chunk = 32 * kStrips; chunk < pad; chunk += 32 * kStrips) {
+      settled(chunk);
+      convolve(chunk);
+#pragma unroll
+      for (int j = 0; j < kStrips; ++j)
+        if (chunk + lane + 32 * j < pad) to[chunk + lane + 32 * j] = values[j];
     }
+    if (pad > 32 * kStrips) settled(0);
+    convolve(0);
     float scale = 1.0f;
     if (p.delta && kind < 2) {
       scale = 1.0f / sqrtf(warp_sum(squares) + 1e-6f);
       if (kind == 0) scale /= sqrtf(float(p.dim));
+      for (int c = 32 * kStrips + lane; c < pad; c += 32) to[c] *= scale;  // written by this lane
     }
-    float* to = kind == 0 ? p.q + size_t(row) * p.key_heads * p.dim_pad + head * pad
-                : kind == 1 ? p.ring_k + size_t(slot) * p.key_heads * p.dim_pad + head * pad
-                            : p.v + size_t(row) * p.heads * p.vdim_pad + head * pad;
 #pragma unroll
-    for (int j = 0; j < kMaxHeadDim / 32; ++j)
+    for (int j = 0; j < kStrips; ++j)
       if (lane + 32 * j < pad) to[lane + 32 * j] = values[j] * scale;
     return;
   }
