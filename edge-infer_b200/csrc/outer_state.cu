@@ -41,14 +41,13 @@ __global__ void __launch_bounds__(128) outer_prepare_kernel(const OuterStatePara
 #pragma unroll
       for (int j = 0; j < kStrips; ++j) {
         const int c = chunk + lane + 32 * j;
-        bias[j] = runs && c < pad && p.conv_bias ? p.conv_bias[first + c] : 0.0f;
+        bias[j] = c < pad && p.conv_bias ? p.conv_bias[first + c] : 0.0f;
 #pragma unroll
         for (int tap = 0; tap < kTaps; ++tap) {
           const int r = row - (kTaps - 1) + tap;
-          weights[j][tap] = inputs[j][tap] = 0.0f;
-          if (!runs || c >= pad) continue;
-          weights[j][tap] = p.conv[size_t(tap) * channels + first + c];
-          if (r < 0 && context + r >= 0) inputs[j][tap] = value_of(raw[size_t((context + r) & (p.raw_rows - 1)) * channels + first + c]);
+          weights[j][tap] = c < pad ? p.conv[size_t(tap) * channels + first + c] : 0.0f;
+          inputs[j][tap] = 0.0f;
+          if (runs && c < pad && r < 0 && context + r >= 0) inputs[j][tap] = value_of(raw[size_t((context + r) & (p.raw_rows - 1)) * channels + first + c]);
         }
       }
     };
@@ -115,6 +114,10 @@ __global__ void __launch_bounds__(128) outer_prepare_kernel(const OuterStatePara
   const int head = p.delta ? unit : unit * 32 + lane;
   const float rate = head < p.heads ? p.rate[head] : 0.0f;
   const float bias = !p.delta && head < p.heads ? p.bias[head] : 0.0f;
+  float biases[kStrips];  // delta rule: of this lane's first key channels
+#pragma unroll
+  for (int j = 0; j < kStrips; ++j)
+    biases[j] = p.delta && head < p.heads && lane + 32 * j < p.dim_pad ? p.bias[head * p.dim_pad + lane + 32 * j] : 0.0f;
   grid_dependency_wait();
   grid_launch_dependents();
   if (!runs) return;
@@ -123,9 +126,11 @@ __global__ void __launch_bounds__(128) outer_prepare_kernel(const OuterStatePara
     const T* decay = static_cast<const T*>(p.decay) + size_t(row) * p.decay_stride + head * p.dim_pad;
     float* to = p.ring_g + (size_t(slot) * p.heads + head) * p.dim_pad;
     if (lane == 0) p.beta[size_t(row) * p.heads + head] = sigmoid_value(value_of(step[head]));
-#pragma unroll 4
-    for (int d = lane; d < p.dim_pad; d += 32)
-      to[d] = expf(-rate * softplus_value(value_of(decay[d]) + p.bias[head * p.dim_pad + d]));
+    auto decay_of = [&](int d, float b) { to[d] = expf(-rate * softplus_value(value_of(decay[d]) + b)); };
+#pragma unroll
+    for (int j = 0; j < kStrips; ++j)
+      if (lane + 32 * j < p.dim_pad) decay_of(lane + 32 * j, biases[j]);
+    for (int d = lane + 32 * kStrips; d < p.dim_pad; d += 32) decay_of(d, p.bias[head * p.dim_pad + d]);
     return;
   }
   if (head >= p.heads) return;
