@@ -45,6 +45,7 @@ __host__ __device__ inline ChunkLayout chunk_layout(int dim, int vdim) {
 // Floats per staged row: sixteen more than a multiple of 32 keeps four-value accesses of two rows apart in the banks.
 __host__ __device__ inline int row_pitch(int dim) {
   if (dim > 192) return dim < 256 ? dim + 4 : dim;  // what shared memory has room for
+  if (dim < 48) return 48;  // the decays' place holds ten 16 x 16 matrices later
   return dim % 32 == 16 ? dim : dim + 16;
 }
 size_t prepare_shared(int dim) {
@@ -98,8 +99,7 @@ __device__ __forceinline__ void split_rows(float4 lo, float4 hi, uint32_t (&lead
   split_pair(hi.z, hi.w, leading[3], rest[3]);
 }
 
-// Sixteen warps. Of A and B, warp w takes four columns of a diagonal block and, up to the twelfth, a tile below the
-// diagonal.
+// Sixteen warps. Of A and B, warp w takes columns of a diagonal block and one tile below the diagonal.
 constexpr int kPrepareThreads = 512;
 __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const DeltaPromptParams p) {
   extern __shared__ __align__(16) float chunk_smem[];
@@ -107,8 +107,8 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
   const int dim = o.dim_pad, pitch = row_pitch(dim), steps = dim / 16;
   float* at = chunk_smem;                          // diag(b) A transposed: at[j][t], j < t
   float* gs = at + kChunk * kPitchA;               // [kChunk][pitch]: cumulative logarithms of the decays
-  float* ks = gs + kChunk * pitch;                 // [kChunk][pitch]: unit k, then columns of W
-  float* qs = ks + kChunk * pitch;                 // [kChunk][pitch]: scaled unit q, then columns of V'
+  float* ks = gs + kChunk * pitch;                 // [kChunk][pitch]: unit k, then columns of V'
+  float* qs = ks + kChunk * pitch;                 // [kChunk][pitch]: scaled unit q, then columns of W
   float* bm = qs + kChunk * pitch;                 // B: bm[t][j], j <= t
   float* beta = bm + kChunk * kPitchB;             // [kChunk]
   grid_dependency_wait();
@@ -188,34 +188,29 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
     if (t < live && t < kChunk) ahead[n] = *reinterpret_cast<const uint2*>(values + size_t(t) * p.channels + (i - t * first_quads) * 4);
   }
 
-  // A and B inside the diagonal blocks, directly. Warp w: block w >> 2; rows g and g + 8 of it against columns
-  // 2 (w & 3), + 1, and row g + 8 against the columns eight further on.
+  // A and B inside the 8 x 8 blocks on the diagonal, directly. Warp w: row g of both blocks of the 16 x 16 block w >> 2
+  // against columns 2 (w & 3), + 1 of its own block.
   {
-    const int base = (warp >> 2) * kBlock, column = base + (warp & 3) * 2;
-    const int t = base + g;
-    float ka[3][2], qa[3][2];  // [row g, early column | row g + 8, early column | row g + 8, late column]
+    const int base = (warp >> 2) * kBlock, column = base + (warp & 3) * 2, t = base + g;
+    float ka[2][2], qa[2][2];  // [early block, late block][column]
 #pragma unroll
-    for (int n = 0; n < 3; ++n) ka[n][0] = ka[n][1] = qa[n][0] = qa[n][1] = 0.0f;
+    for (int n = 0; n < 2; ++n) ka[n][0] = ka[n][1] = qa[n][0] = qa[n][1] = 0.0f;
 #pragma unroll 2
     for (int d = 4 * c; d < dim; d += 16) {
-      const float4 gl = quad_at(gs + t * pitch + d), gh = quad_at(gs + (t + 8) * pitch + d);
-      const float4 kl = quad_at(ks + t * pitch + d), kh = quad_at(ks + (t + 8) * pitch + d);
-      const float4 ql = quad_at(qs + t * pitch + d), qh = quad_at(qs + (t + 8) * pitch + d);
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const float4 early_g = quad_at(gs + (column + e) * pitch + d), early_k = quad_at(ks + (column + e) * pitch + d);
-        const float4 late_g = quad_at(gs + (column + e + 8) * pitch + d), late_k = quad_at(ks + (column + e + 8) * pitch + d);
-        const float4 x = times(early_k, exp_below(gl, early_g)), y = times(early_k, exp_between(gh, early_g)), z = times(late_k, exp_below(gh, late_g));
-        ka[0][e] = dot(kl, x, ka[0][e]);
-        qa[0][e] = dot(ql, x, qa[0][e]);
-        ka[1][e] = dot(kh, y, ka[1][e]);
-        qa[1][e] = dot(qh, y, qa[1][e]);
-        ka[2][e] = dot(kh, z, ka[2][e]);
-        qa[2][e] = dot(qh, z, qa[2][e]);
+      for (int n = 0; n < 2; ++n) {
+        const float4 gt = quad_at(gs + (t + 8 * n) * pitch + d), kt = quad_at(ks + (t + 8 * n) * pitch + d), qt = quad_at(qs + (t + 8 * n) * pitch + d);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int j = (column + e + 8 * n) * pitch + d;
+          const float4 x = times(quad_at(ks + j), exp_below(gt, quad_at(gs + j)));
+          ka[n][e] = dot(kt, x, ka[n][e]);
+          qa[n][e] = dot(qt, x, qa[n][e]);
+        }
       }
     }
 #pragma unroll
-    for (int n = 0; n < 3; ++n)
+    for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         ka[n][e] += __shfl_xor_sync(0xffffffffu, ka[n][e], 1);
@@ -223,27 +218,22 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
         qa[n][e] += __shfl_xor_sync(0xffffffffu, qa[n][e], 1);
         qa[n][e] += __shfl_xor_sync(0xffffffffu, qa[n][e], 2);
       }
-    if (c < 2) {  // the four lanes of a row hold the same sums; lane c writes column + c
-      const int e = c, early = column + e, late = early + 8;
-      const float ka0 = e ? ka[0][1] : ka[0][0], ka1 = e ? ka[1][1] : ka[1][0], ka2 = e ? ka[2][1] : ka[2][0];
-      const float qa0 = e ? qa[0][1] : qa[0][0], qa1 = e ? qa[1][1] : qa[1][0], qa2 = e ? qa[2][1] : qa[2][0];
-      at[early * kPitchA + t] = early < t ? ka0 * beta[t] : 0.0f;
-      bm[t * kPitchB + early] = early <= t ? qa0 : 0.0f;
-      at[early * kPitchA + t + 8] = ka1 * beta[t + 8];
-      bm[(t + 8) * kPitchB + early] = qa1;
-      at[late * kPitchA + t + 8] = late < t + 8 ? ka2 * beta[t + 8] : 0.0f;
-      bm[(t + 8) * kPitchB + late] = late <= t + 8 ? qa2 : 0.0f;
-    } else if (c == 2) {
-      for (int e = 0; e < 2; ++e) {
-        at[(column + 8 + e) * kPitchA + t] = 0.0f;
-        bm[t * kPitchB + column + 8 + e] = 0.0f;
-      }
-    }
+    // The four lanes of a row hold the same sums: lane c writes column c & 1 of block c >> 1, and B's zeros beside it.
+    const float k_sum = c & 2 ? (c & 1 ? ka[1][1] : ka[1][0]) : (c & 1 ? ka[0][1] : ka[0][0]);
+    const float q_sum = c & 2 ? (c & 1 ? qa[1][1] : qa[1][0]) : (c & 1 ? qa[0][1] : qa[0][0]);
+    const int row = t + (c & 2) * 4, j = column + (c & 1) + (c & 2) * 4;
+    at[j * kPitchA + row] = j < row ? k_sum * beta[row] : 0.0f;
+    bm[row * kPitchB + j] = j <= row ? q_sum : 0.0f;
+    if (c < 2) bm[t * kPitchB + column + c + 8] = 0.0f;
   }
-  // Below the diagonal: tiles of 16 rows x 8 columns, through the end of the block ahead of the rows.
-  if (warp < 12) {
-    const int block = warp < 2 ? 1 : warp < 6 ? 2 : 3, column = (warp - (block == 1 ? 0 : block == 2 ? 2 : 6)) * 8;
-    const int t0 = block * kBlock;
+  // Everything else below the diagonal, through the end of the block ahead of the rows: twelve tiles of 16 rows x 8 columns
+  // below the 16 x 16 blocks, four of 8 x 8 inside them (rows g + 8 of those are not there).
+  {
+    const bool inside = warp >= 12;
+    const int block = inside ? warp - 12 : warp < 2 ? 1 : warp < 6 ? 2 : 3;
+    const int t0 = block * kBlock + (inside ? 8 : 0);
+    const int column = inside ? block * kBlock : (warp - (block == 1 ? 0 : block == 2 ? 2 : 6)) * 8;
+    const int high = inside ? 0 : 8;
     float ka[3][4], qa[3][4];  // a chain per product of terms
 #pragma unroll
     for (int n = 0; n < 3; ++n)
@@ -252,10 +242,11 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
 #pragma unroll 2
     for (int d = 4 * c; d < dim; d += 16) {
       const float4 turn = quad_at(gs + (t0 - 1) * pitch + d);
-      const float4 e_lo = exp_between(quad_at(gs + (t0 + g) * pitch + d), turn), e_hi = exp_between(quad_at(gs + (t0 + g + 8) * pitch + d), turn);
+      const int lo = (t0 + g) * pitch + d, hi = lo + high * pitch;
+      const float4 e_lo = exp_between(quad_at(gs + lo), turn), e_hi = exp_between(quad_at(gs + hi), turn);
       uint32_t kh[4], kl[4], qh[4], ql[4], bh[2], bl[2];
-      split_rows(times(quad_at(ks + (t0 + g) * pitch + d), e_lo), times(quad_at(ks + (t0 + g + 8) * pitch + d), e_hi), kh, kl);
-      split_rows(times(quad_at(qs + (t0 + g) * pitch + d), e_lo), times(quad_at(qs + (t0 + g + 8) * pitch + d), e_hi), qh, ql);
+      split_rows(times(quad_at(ks + lo), e_lo), times(quad_at(ks + hi), e_hi), kh, kl);
+      split_rows(times(quad_at(qs + lo), e_lo), times(quad_at(qs + hi), e_hi), qh, ql);
       const float4 x = times(quad_at(ks + (column + g) * pitch + d), exp_between(turn, quad_at(gs + (column + g) * pitch + d)));
       split_pair(x.x, x.y, bh[0], bl[0]);
       split_pair(x.z, x.w, bh[1], bl[1]);
@@ -268,6 +259,7 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
     }
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
+      if (e >= 2 && inside) break;
       const int t = t0 + g + (e >> 1) * 8, j = column + 2 * c + (e & 1);
       at[j * kPitchA + t] = (ka[0][e] + (ka[1][e] + ka[2][e])) * beta[t];
       bm[t * kPitchB + j] = qa[0][e] + (qa[1][e] + qa[2][e]);
@@ -275,7 +267,8 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
   }
   __syncthreads();
 
-  // Operands that need no solving: q e^G, k e^(G_end - G) transposed, B, and the chunk's decay.
+  // Operands that need no solving: q e^G, k e^(G_end - G) transposed, B, and the chunk's decay. A place of q that has been
+  // read takes the right-hand side of W, b k e^G.
   const float* last = gs + (kChunk - 1) * pitch;
   uint4* q_out = reinterpret_cast<uint4*>(own + layout.q);
   uint4* k_out = reinterpret_cast<uint4*>(own + layout.k);
@@ -283,9 +276,12 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
 #pragma unroll 2
   for (int tile = warp; tile < 4 * steps; tile += kWarps) {
     const int mt = tile / steps, kk = tile - mt * steps;
-    const int row = (mt * 16 + g) * pitch + kk * 16 + 4 * c;
-    store_fragment(q_out + size_t(mt * steps + kk) * 64 + lane, times(quad_at(qs + row), exp_of(quad_at(gs + row))),
-                   times(quad_at(qs + row + 8 * pitch), exp_of(quad_at(gs + row + 8 * pitch))));
+    const int t = mt * 16 + g, lo = t * pitch + kk * 16 + 4 * c, hi = lo + 8 * pitch;
+    const float4 e_lo = exp_of(quad_at(gs + lo)), e_hi = exp_of(quad_at(gs + hi));
+    store_fragment(q_out + size_t(mt * steps + kk) * 64 + lane, times(quad_at(qs + lo), e_lo), times(quad_at(qs + hi), e_hi));
+    const float b_lo = beta[t], b_hi = beta[t + 8];
+    *reinterpret_cast<float4*>(qs + lo) = times(quad_at(ks + lo), make_float4(e_lo.x * b_lo, e_lo.y * b_lo, e_lo.z * b_lo, e_lo.w * b_lo));
+    *reinterpret_cast<float4*>(qs + hi) = times(quad_at(ks + hi), make_float4(e_hi.x * b_hi, e_hi.y * b_hi, e_hi.z * b_hi, e_hi.w * b_hi));
     float y[8];  // tile (kk, mt) of the transpose: rows are key channels, columns tokens in the order of token_of
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
@@ -304,10 +300,8 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
     store_fragment(b_out + size_t(tile) * 64 + lane, x);
   }
   for (int d = threadIdx.x; d < dim; d += kPrepareThreads) reinterpret_cast<float*>(own + layout.decay)[d] = power_of_two(last[d]);
-  __syncthreads();
-
-  // The inverses of the four unit lower triangular diagonal blocks, one column per thread, into the blocks' places in bm
-  // (B has been written out): inverse[i][j] at bm[(16 b + i) pitch + 16 b + j].
+  // The inverses of the four unit lower triangular diagonal blocks, one column per thread, into the unused half of the
+  // blocks' places: inverse[i][j], j < i, at at[16 b + i][16 b + j].
   if (threadIdx.x < kChunk) {
     const int base = threadIdx.x & ~(kBlock - 1), j = threadIdx.x & (kBlock - 1);
     float x[kBlock];
@@ -318,65 +312,95 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
 #pragma unroll
       for (int i = m + 1; i < kBlock; ++i) x[i] = fmaf(-at[(base + m) * kPitchA + base + i], x[m], x[i]);
 #pragma unroll
-    for (int i = 0; i < kBlock; ++i) bm[(base + i) * kPitchB + base + j] = x[i];
+    for (int i = 1; i < kBlock; ++i)
+      if (i > j) at[(base + i) * kPitchA + base + j] = x[i];
   }
-  // Solves (I + diag(b) A) X = right-hand side in place, 16 rows at a time. Lanes l and l + 16 share a column: lane
-  // l + 16 h works on the rows 8 h .. 8 h + 7 of a block for the part below the diagonal blocks, and on every second row
-  // for the product with the block's inverse.
-  const int half = lane >> 4;
-  auto solve = [&](float* column, bool live_column) {
-#pragma unroll 1
+  __syncthreads();
+
+  // Solves (I + diag(b) A) X = right-hand side for the columns of W (in q's place) and of V' (in k's place) by blocks of 16
+  // rows: X_b = inverse_b (R_b - sum over earlier blocks of (diag(b) A)_bj X_j), as products of two-term operands. The ten
+  // 16 x 16 matrices are laid out as A fragments in the place of the decays, tokens in the order of token_of; a warp takes
+  // 16 columns.
+  uint4* matrices = reinterpret_cast<uint4*>(gs);  // block (b, j) at (b (b + 1) / 2 + j) * 64; (b, b) the inverse
+  if (warp < 10) {
+    const int b = warp < 1 ? 0 : warp < 3 ? 1 : warp < 6 ? 2 : 3, j = warp - b * (b + 1) / 2;
+    float x[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const int row = b * kBlock + g + ((e >> 1) & 1) * 8, col = j * kBlock + token_of(c, e);
+      x[e] = b != j ? -at[col * kPitchA + row] : row == col ? 1.0f : row > col ? at[row * kPitchA + col] : 0.0f;
+    }
+    store_fragment(matrices + warp * 64 + lane, x);
+  }
+  auto solve = [&](float* column, float4* result) {
+    uint32_t xh[3][2][2], xl[3][2][2];  // blocks solved so far, as B operands of two tiles of eight columns
+    auto swap_layout = [&](int b, const float (&acc)[2][4], uint32_t (&h)[2][2], uint32_t (&l)[2][2]) {
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        float* to = column + (b * kBlock + g) * pitch + n * 8 + 2 * c;
+        *reinterpret_cast<float2*>(to) = make_float2(acc[n][0], acc[n][1]);
+        *reinterpret_cast<float2*>(to + 8 * pitch) = make_float2(acc[n][2], acc[n][3]);
+      }
+      __syncwarp();
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        const float* from = column + (b * kBlock + c) * pitch + n * 8 + g;
+        split_pair(from[0], from[4 * pitch], h[n][0], l[n][0]);
+        split_pair(from[8 * pitch], from[12 * pitch], h[n][1], l[n][1]);
+      }
+      __syncwarp();
+    };
+    auto product = [&](int at_matrix, const uint32_t (&h)[2][2], const uint32_t (&l)[2][2], float (&acc)[2][4]) {
+      const uint4 ah = matrices[at_matrix * 64 + lane], al = matrices[at_matrix * 64 + 32 + lane];
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        mma_bf16_16816(acc[n], ah.x, ah.y, ah.z, ah.w, h[n][0], h[n][1]);
+        mma_bf16_16816(acc[n], ah.x, ah.y, ah.z, ah.w, l[n][0], l[n][1]);
+        mma_bf16_16816(acc[n], al.x, al.y, al.z, al.w, h[n][0], h[n][1]);
+      }
+    };
+#pragma unroll
     for (int b = 0; b < kChunk / kBlock; ++b) {
-      float x[8];
-      float* own_rows = column + (b * kBlock + half * 8) * pitch;
-      if (live_column && b) {
+      float acc[2][4];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) x[i] = own_rows[i * pitch];
-#pragma unroll 4
-        for (int j = 0; j < b * kBlock; ++j) {
-          const float known = column[j * pitch];
-          const float* a = at + j * kPitchA + b * kBlock + half * 8;
-          const float4 v = quad_at(a), w = quad_at(a + 4);
-          x[0] = fmaf(-v.x, known, x[0]);
-          x[1] = fmaf(-v.y, known, x[1]);
-          x[2] = fmaf(-v.z, known, x[2]);
-          x[3] = fmaf(-v.w, known, x[3]);
-          x[4] = fmaf(-w.x, known, x[4]);
-          x[5] = fmaf(-w.y, known, x[5]);
-          x[6] = fmaf(-w.z, known, x[6]);
-          x[7] = fmaf(-w.w, known, x[7]);
-        }
-#pragma unroll
-        for (int i = 0; i < 8; ++i) own_rows[i * pitch] = x[i];
+      for (int n = 0; n < 2; ++n) {
+        const float* from = column + (b * kBlock + g) * pitch + n * 8 + 2 * c;
+        const float2 lo = *reinterpret_cast<const float2*>(from), hi = *reinterpret_cast<const float2*>(from + 8 * pitch);
+        acc[n][0] = lo.x;
+        acc[n][1] = lo.y;
+        acc[n][2] = hi.x;
+        acc[n][3] = hi.y;
       }
-      __syncwarp();
-      float r[kBlock];
-      if (live_column) {
 #pragma unroll
-        for (int i = 0; i < kBlock; ++i) r[i] = column[(b * kBlock + i) * pitch];
+      for (int j = 0; j < b; ++j) product(b * (b + 1) / 2 + j, xh[j], xl[j], acc);
+      uint32_t rh[2][2], rl[2][2];
+      swap_layout(b, acc, rh, rl);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const float* t = bm + (b * kBlock + 2 * i + half) * kPitchB + b * kBlock;
-          float sum = 0.0f;
+      for (int n = 0; n < 2; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.0f;
+      product(b * (b + 1) / 2 + b, rh, rl, acc);
+      if (result) {
 #pragma unroll
-          for (int j = 0; j < 2 * i + 2; ++j) sum = fmaf(t[j], r[j], sum);  // row 2 i has a zero at its end
-          x[i] = sum;
+        for (int n = 0; n < 2; ++n)
+          result[(size_t(b) * (o.vdim_pad / 8) + n) * 32 + lane] = make_float4(acc[n][0], acc[n][1], acc[n][2], acc[n][3]);
+      }
+      if (b < 3) {
+        swap_layout(b, acc, xh[b < 3 ? b : 0], xl[b < 3 ? b : 0]);
+      } else if (!result) {
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          float* to = column + (b * kBlock + g) * pitch + n * 8 + 2 * c;
+          *reinterpret_cast<float2*>(to) = make_float2(acc[n][0], acc[n][1]);
+          *reinterpret_cast<float2*>(to + 8 * pitch) = make_float2(acc[n][2], acc[n][3]);
         }
       }
-      __syncwarp();
-      if (live_column)
-#pragma unroll
-        for (int i = 0; i < 8; ++i) column[(b * kBlock + 2 * i + half) * pitch] = x[i];
-      __syncwarp();
     }
   };
-  // The columns of W in place of k, those of V' in place of q, `dim` value columns at a time.
   for (int v0 = 0; v0 < o.vdim_pad; v0 += dim) {
     const int width = min(dim, o.vdim_pad - v0), width_quads = width / 4;
     auto put_value = [&](int i, uint2 raw) {
       const int t = i / width_quads, d = (i - t * width_quads) * 4;
       const float b = beta[t];
-      *reinterpret_cast<float4*>(qs + t * pitch + d) = make_float4(bf16_lo(raw.x) * b, bf16_hi(raw.x) * b, bf16_lo(raw.y) * b, bf16_hi(raw.y) * b);
+      *reinterpret_cast<float4*>(ks + t * pitch + d) = make_float4(bf16_lo(raw.x) * b, bf16_hi(raw.x) * b, bf16_lo(raw.y) * b, bf16_hi(raw.y) * b);
     };
     auto fetch_value = [&](int i) {
       const int t = i / width_quads, d = (i - t * width_quads) * 4;
@@ -389,35 +413,21 @@ __global__ void __launch_bounds__(kPrepareThreads) delta_chunk_kernel(const Delt
         if (i < kChunk * width_quads) put_value(i, ahead[n]);
     }
     for (; i < kChunk * width_quads; i += kPrepareThreads) put_value(i, fetch_value(i));
-    if (v0 == 0) {
-#pragma unroll 4
-      for (int n = threadIdx.x; n < kChunk * quads; n += kPrepareThreads) {
-        const int t = n / quads, d = (n - t * quads) * 4;
-        const float4 e = exp_of(quad_at(gs + t * pitch + d));
-        const float b = beta[t];
-        float4* k = reinterpret_cast<float4*>(ks + t * pitch + d);
-        *k = times(*k, make_float4(e.x * b, e.y * b, e.z * b, e.w * b));
-      }
-    }
     __syncthreads();
     const int unsolved = v0 == 0 ? dim : 0;  // columns of W still to come, ahead of the value columns
     for (int begin = warp * 16; begin < unsolved + width; begin += kWarps * 16) {
-      const int column = begin + (lane & 15);
-      solve(column < unsolved ? ks + column : qs + column - unsolved, column < unsolved + width);
+      const int value = begin - unsolved;
+      if (value < 0)
+        solve(qs + begin, nullptr);
+      else
+        solve(ks + value, v_out + size_t(v0 + value) / 8 * 32);
     }
     __syncthreads();
-    // V' in the order of the accumulators: [row tile][column tile of 8][lane].
-    for (int tile = warp; tile < 4 * (width / 8); tile += kWarps) {
-      const int mt = tile / (width / 8), nt = tile - mt * (width / 8);
-      const float* x = qs + (mt * 16 + g) * pitch + nt * 8 + 2 * c;
-      v_out[(size_t(mt) * (o.vdim_pad / 8) + v0 / 8 + nt) * 32 + lane] = make_float4(x[0], x[1], x[8 * pitch], x[8 * pitch + 1]);
-    }
-    if (v0 + dim < o.vdim_pad) __syncthreads();
   }
   uint4* w_out = reinterpret_cast<uint4*>(own + layout.w);
   for (int tile = warp; tile < 4 * steps; tile += kWarps) {
     const int mt = tile / steps, kk = tile - mt * steps;
-    const float* x = ks + (mt * 16 + g) * pitch + kk * 16 + 4 * c;
+    const float* x = qs + (mt * 16 + g) * pitch + kk * 16 + 4 * c;
     store_fragment(w_out + size_t(tile) * 64 + lane, quad_at(x), quad_at(x + 8 * pitch));
   }
 }
