@@ -2,12 +2,17 @@
 //
 // A step (at most 16 rows: decode, verify, a short portion) runs per layer, with programmatic dependent launch:
 //   parallel mixer   fused projection -> heads prepared, K / V appended -> split attention -> linear attention step ->
-//                    merge + gate -> output projection (FP32 sums) -> join
-//   gated recurrence fused projection -> recurrence step -> output projection (FP32 sums) -> join
-//   feed-forward     gate|up with the gated unit in the epilogue -> down (FP32 sums) -> join
-// where a join finishes one sublayer (norm after, residual add, what a loop pass adds) and starts the next (norm
-// before). A prompt segment runs the same sequence over all its rows on the prompt GEMM, whole-history attention and
-// the chunked forms of the recurrences. A model in true 32-bit runs every token through the step form.
+//                    merge + gate -> output projection (FP32 sums)
+//   gated recurrence fused projection -> recurrence step -> output projection (FP32 sums)
+//   latent attention fused projection -> cache row, queries through the key expansion -> split attention -> merge, value
+//                    expansion, gate -> output projection (FP32 sums)
+//   state space,     fused projection (-> second factors of the low-rank ones) -> convolution and decays -> recurrence
+//   channel delta    step -> norm and gate -> output projection (FP32 sums)
+//   feed-forward     up (gate|up) with the activation in the epilogue -> down (FP32 sums)
+// A sandwich block ends both sublayers with a join, which finishes one (norm after, residual add, what a loop pass adds)
+// and starts the next (norm before); a parallel block has one join behind both. A prompt segment runs the same sequence
+// over all its rows on the prompt GEMM, whole-history attention and the chunked forms of the recurrences. A model in true
+// 32-bit runs every token through the step form.
 #include "layered.cuh"
 
 #include <cmath>

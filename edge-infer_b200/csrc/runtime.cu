@@ -1418,6 +1418,7 @@ static void append_tokens(ei_session& s, const uint32_t* host_tokens, size_t row
         head_over(&last, 1, true);
       }
     }
+    synchronize(s);  // the workspace goes back idle
     return;
   }
   for (size_t first = 0; first < rows; first += kMaxRows) {

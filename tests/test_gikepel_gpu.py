@@ -339,7 +339,7 @@ def test_speculative_rounds_on_the_target(cuda, package):
     assert all(int(np.argmax(row)) == token for row, token, sure in zip(rows, out[1:], decided) if sure)
 
 
-# ---- the contract around it ----
+# ---- refusals and failures ----
 def test_refusals_leave_the_history(cuda, package):
     c = cases.CASES["mixed"]
     model, oracle = build(package, c, "f32")
